@@ -76,11 +76,12 @@ def _stamp(lib: Path, files) -> None:
     lib.with_suffix(".so.srchash").write_text(_source_hash(files))
 
 
-def build_kernels(force: bool = False, verbose_ptxas: bool = False) -> Path:
-    srcs = sorted(CSRC.glob("*.cu"))
+def build_kernels(force: bool = False, verbose_ptxas: bool = False, units=None, lib: Path = KERNEL_LIB) -> Path:
+    """``units``: names of the translation units to build into ``lib`` (default: all of them, the full library)."""
+    srcs = sorted(CSRC.glob("*.cu")) if units is None else [CSRC / f"{u}.cu" for u in units]
     deps = srcs + sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
-    if not force and not verbose_ptxas and _up_to_date(KERNEL_LIB, deps):
-        return KERNEL_LIB
+    if not force and not verbose_ptxas and _up_to_date(lib, deps):
+        return lib
     OBJ.mkdir(exist_ok=True)
     hdr = _newest_header()
     jobs = []
@@ -95,10 +96,24 @@ def build_kernels(force: bool = False, verbose_ptxas: bool = False) -> Path:
         with ThreadPoolExecutor(max_workers=min(8, len(jobs))) as ex:
             list(ex.map(_run, jobs))
     objs = [str(OBJ / (s.stem + ".o")) for s in srcs]
-    if jobs or not KERNEL_LIB.exists():
-        _run([_nvcc(), "-shared", "-o", str(KERNEL_LIB), *objs, "-lcudart"])
-    _stamp(KERNEL_LIB, deps)
-    return KERNEL_LIB
+    if jobs or not _up_to_date(lib, deps):
+        _run([_nvcc(), "-shared", "-o", str(lib), *objs, "-lcudart"])
+    _stamp(lib, deps)
+    return lib
+
+
+def build_family(family: str) -> Path:
+    """The kernel library for one model family: the full one when it is up to date, else a library of the units that the
+    family runs (objects are shared with the full build).  The ops use whichever is returned."""
+    from .models.registry import KERNEL_UNITS
+    from .ops import _lib
+    units = KERNEL_UNITS.get(family)
+    full = sorted(CSRC.glob("*.cu")) + sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
+    if units is None or _up_to_date(KERNEL_LIB, full):
+        return build_kernels()
+    lib = build_kernels(units=units, lib=ROOT / f"libsllm_b200_kernels_{family}.so")
+    _lib.use_kernel_library(lib)
+    return lib
 
 
 def build_host(force: bool = False) -> Path:

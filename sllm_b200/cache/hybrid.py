@@ -16,7 +16,54 @@ from ..models.config import ModelConfig
 from .paged import PagedKVCache
 
 
-class HybridCache(PagedKVCache):
+class StateSlots:
+    """Per-sequence recurrent state in slots.  ``state_planes``: [(tensor, slot dimension)]; a slot is zeroed when a
+    sequence takes it, so slots can be used again in any order."""
+
+    def init_slots(self, max_seqs: int, planes: list) -> None:
+        self.max_seqs = max_seqs
+        self.state_planes = planes
+        self._free = list(range(max_seqs - 1, -1, -1))
+        self.slot_of: dict = {}
+
+    def alloc_slot(self, seq_id: int) -> int:
+        if not self._free:
+            raise RuntimeError("no free recurrent-state slot")
+        s = self._free.pop()
+        self.slot_of[seq_id] = s
+        for t, dim in self.state_planes:
+            t.select(dim, s).zero_()
+        return s
+
+    def free_slot(self, seq_id: int) -> None:
+        s = self.slot_of.pop(seq_id, None)
+        if s is not None:
+            self._free.append(s)
+
+    def copy_slot(self, src_seq: int, dst_seq: int) -> None:
+        a, b = self.slot_of[src_seq], self.slot_of[dst_seq]
+        for t, dim in self.state_planes:
+            t.select(dim, b).copy_(t.select(dim, a))
+
+    def snapshot(self, seq_id: int):
+        s = self.slot_of[seq_id]
+        return tuple(t.select(dim, s).clone() for t, dim in self.state_planes)
+
+    def restore(self, seq_id: int, snap) -> None:
+        s = self.slot_of[seq_id]
+        for (t, dim), v in zip(self.state_planes, snap):
+            t.select(dim, s).copy_(v)
+
+    def save_all(self):
+        """Every slot's state (a graph capture runs the step once more than it counts)."""
+        return tuple(t.clone() for t, _ in self.state_planes)
+
+    def load_all(self, saved) -> None:
+        for (t, _), v in zip(self.state_planes, saved):
+            t.copy_(v)
+
+
+class HybridCache(StateSlots, PagedKVCache):
     def __init__(self, cfg: ModelConfig, num_pages: int, device, max_seqs: int, kv_heads: Optional[int] = None,
                  tp_size: int = 1):
         """``tp_size``: the gated-delta-net heads (and with them the conv and recurrent state) are split over that
@@ -31,13 +78,11 @@ class HybridCache(PagedKVCache):
         hd = cfg.gdn_head_dim
         self.width = (2 * cfg.gdn_qk_heads + cfg.gdn_heads) // tp_size * hd
         n = max(1, len(self.gdn_layers))
-        self.max_seqs = max_seqs
         self.conv_state = torch.zeros((n, max_seqs, cfg.gdn_conv_kernel - 1, self.width), dtype=torch.bfloat16 if
                                       torch.device(device).type == "cuda" or cfg.weight_format != "fp32" else torch.float32,
                                       device=device)
         self.rec_state = torch.zeros((n, max_seqs, cfg.gdn_heads // tp_size, hd, hd), dtype=torch.float32, device=device)
-        self._free = list(range(max_seqs - 1, -1, -1))
-        self.slot_of: dict = {}
+        self.init_slots(max_seqs, [(self.conv_state, 1), (self.rec_state, 1)])
 
     def layer(self, i: int):
         j = self._kv_index.get(i)
@@ -46,35 +91,3 @@ class HybridCache(PagedKVCache):
     def gdn(self, i: int):
         j = self._gdn_index[i]
         return self.conv_state[j], self.rec_state[j]
-
-    # ---------------------------------------------------------------- slots
-    def alloc_slot(self, seq_id: int) -> int:
-        if not self._free:
-            raise RuntimeError("no free recurrent-state slot")
-        s = self._free.pop()
-        self.slot_of[seq_id] = s
-        self.conv_state[:, s].zero_()
-        self.rec_state[:, s].zero_()
-        return s
-
-    def free_slot(self, seq_id: int) -> None:
-        s = self.slot_of.pop(seq_id, None)
-        if s is not None:
-            self._free.append(s)
-
-    def copy_slot(self, src_seq: int, dst_seq: int) -> None:
-        a, b = self.slot_of[src_seq], self.slot_of[dst_seq]
-        self.conv_state[:, b].copy_(self.conv_state[:, a])
-        self.rec_state[:, b].copy_(self.rec_state[:, a])
-
-    def snapshot(self, seq_id: int):
-        s = self.slot_of[seq_id]
-        return self.conv_state[:, s].clone(), self.rec_state[:, s].clone()
-
-    def restore(self, seq_id: int, snap) -> None:
-        s = self.slot_of[seq_id]
-        self.conv_state[:, s].copy_(snap[0])
-        self.rec_state[:, s].copy_(snap[1])
-
-    def bytes_per_token(self) -> int:
-        return super().bytes_per_token()

@@ -368,8 +368,17 @@ __device__ __forceinline__ void argmax_take(float& best, int& bi, float v, int i
   }
 }
 
+__device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&v)[8]) { load8_bf16(p, v); }
+__device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
+  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ float load1(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ float load1(const float* p) { return *p; }
+
+template <typename T>
 __global__ void __launch_bounds__(256)
-argmax_kernel(const __nv_bfloat16* __restrict__ logits, int* __restrict__ out_idx, float* __restrict__ out_val,
+argmax_kernel(const T* __restrict__ logits, int* __restrict__ out_idx, float* __restrict__ out_val,
               int n, int ld, int index_offset, int chunk, ArgmaxPartial* partials, int* counters) {
   pdl_wait();
   pdl_trigger();
@@ -377,7 +386,7 @@ argmax_kernel(const __nv_bfloat16* __restrict__ logits, int* __restrict__ out_id
   const int c0 = blockIdx.y * chunk;
   int c1 = c0 + chunk;
   if (c1 > n) c1 = n;
-  const __nv_bfloat16* row = logits + static_cast<size_t>(r) * ld;
+  const T* row = logits + static_cast<size_t>(r) * ld;
   float best = -INFINITY;
   int bi = 0x7fffffff;
   int nan = 0;
@@ -386,7 +395,7 @@ argmax_kernel(const __nv_bfloat16* __restrict__ logits, int* __restrict__ out_id
   if (vec_ok) {
     for (; i + 8 <= c1; i += blockDim.x * 8) {
       float v[8];
-      load8_bf16(row + i, v);
+      load8(row + i, v);
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
         if (v[j] != v[j]) nan = 1;
@@ -397,14 +406,14 @@ argmax_kernel(const __nv_bfloat16* __restrict__ logits, int* __restrict__ out_id
     const int tail0 = c0 + ((c1 - c0) & ~7);
     if (threadIdx.x == 0) {
       for (int t = tail0; t < c1; ++t) {
-        const float v = __bfloat162float(row[t]);
+        const float v = load1(row + t);
         if (v != v) nan = 1;
         argmax_take(best, bi, v, t);
       }
     }
   } else {
     for (int t = c0 + threadIdx.x; t < c1; t += blockDim.x) {
-      const float v = __bfloat162float(row[t]);
+      const float v = load1(row + t);
       if (v != v) nan = 1;
       argmax_take(best, bi, v, t);
     }
@@ -605,9 +614,8 @@ SLLM_EXPORT int sllm_elementwise(const void* a, const void* b, void* y, long lon
   return check_launch();
 }
 
-SLLM_EXPORT int sllm_argmax(const void* logits, int* out_idx, float* out_val, int rows, int n, int ld,
-                            int index_offset, void* ws, long long ws_bytes, int* counters, int n_counters,
-                            void* stream) {
+static int argmax_impl(const void* logits, int* out_idx, float* out_val, int rows, int n, int ld, int index_offset, void* ws,
+                       long long ws_bytes, int* counters, int n_counters, bool fp32, void* stream) {
   if (!logits || !out_idx || rows <= 0 || n <= 0) return SLLM_ERR_INVALID_ARGUMENT;
   // Enough CTAs to cover the machine, slices a multiple of 8 elements and at least 2048 long.
   int chunks = (2 * 148 + rows - 1) / rows;
@@ -620,10 +628,26 @@ SLLM_EXPORT int sllm_argmax(const void* logits, int* out_idx, float* out_val, in
   chunk = (chunk + 7) & ~7;
   chunks = (n + chunk - 1) / chunk;
   dim3 grid(rows, chunks);
-  launch_kernel(argmax_kernel, dim3(grid), dim3(256), 0, static_cast<cudaStream_t>(stream), 1u, 
-      static_cast<const __nv_bfloat16*>(logits), out_idx, out_val, n, ld, index_offset, chunk,
-      static_cast<ArgmaxPartial*>(ws), counters);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (fp32)
+    launch_kernel(argmax_kernel<float>, grid, dim3(256), 0, st, 1u, static_cast<const float*>(logits), out_idx, out_val, n, ld,
+                  index_offset, chunk, static_cast<ArgmaxPartial*>(ws), counters);
+  else
+    launch_kernel(argmax_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, 1u, static_cast<const __nv_bfloat16*>(logits), out_idx,
+                  out_val, n, ld, index_offset, chunk, static_cast<ArgmaxPartial*>(ws), counters);
   return check_launch();
+}
+
+SLLM_EXPORT int sllm_argmax(const void* logits, int* out_idx, float* out_val, int rows, int n, int ld,
+                            int index_offset, void* ws, long long ws_bytes, int* counters, int n_counters,
+                            void* stream) {
+  return argmax_impl(logits, out_idx, out_val, rows, n, ld, index_offset, ws, ws_bytes, counters, n_counters, false, stream);
+}
+
+// The same over fp32 logits (models that run in 32-bit).
+SLLM_EXPORT int sllm_argmax_f32(const float* logits, int* out_idx, float* out_val, int rows, int n, int ld, int index_offset,
+                                void* ws, long long ws_bytes, int* counters, int n_counters, void* stream) {
+  return argmax_impl(logits, out_idx, out_val, rows, n, ld, index_offset, ws, ws_bytes, counters, n_counters, true, stream);
 }
 
 // ------------------------------------------------------------------------------------------------
@@ -679,7 +703,7 @@ SLLM_EXPORT int sllm_argmax_noalloc(const void* logits, int* out_idx, float* out
   chunk = (chunk + 7) & ~7;
   chunks = (n + chunk - 1) / chunk;
   dim3 grid(rows, chunks);
-  cudaError_t e = launch_kernel(argmax_kernel, grid, dim3(256), 0, st, 1u, static_cast<const __nv_bfloat16*>(logits),
+  cudaError_t e = launch_kernel(argmax_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, 1u, static_cast<const __nv_bfloat16*>(logits),
                                 out_idx, out_val, n, ld, index_offset, chunk, static_cast<ArgmaxPartial*>(base),
                                 reinterpret_cast<int*>(static_cast<unsigned char*>(base) + kNoAllocPartialBytes));
   return e == cudaSuccess ? SLLM_OK : SLLM_ERR_CUDA;

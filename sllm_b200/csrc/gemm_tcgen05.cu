@@ -110,7 +110,7 @@ struct GemmParams {
   int transpose_out;   // 0: Y[a, b]; 1: Y[b, a]
   int ldy;
   int ld_sa, ld_sb;    // leading dimensions of the kb-major scale arrays
-  int epilogue;        // 0 = store, 1 = add residual
+  int epilogue;        // 0 = store, 1 = add residual, 2 = square of relu
   int cluster_split;   // 1: gridDim.z CTAs form one cluster and reduce split-K partials over DSMEM
   int const_operand;   // operand that no kernel writes (weights): 0 none, 1 A, 2 B; loaded before the PDL wait
   int early_trigger;   // 1: dependents may become resident as soon as this CTA holds its resources
@@ -754,6 +754,10 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_const
       return static_cast<long long>(tile_id) * (kTileA * BN) + (tr ? col * kTileA + r0 : r0 * BN + col);
     };
     auto store_unit = [&](int col, int r0, float (&v)[8]) {
+      if (p.epilogue == 2) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[j] = v[j] > 0.f ? v[j] * v[j] : 0.f;
+      }
       if (tr) {
         const int b_row = b_tile * BN + col;
         const int a0 = a_tile * kTileA + r0;
@@ -1127,7 +1131,7 @@ static int gemm_impl(const void* a, const void* b, void* y, const float* scale_a
                      const void* residual, int a_rows, int b_rows, int k, int scaled, int transpose_out, int ldy,
                      int ld_sa, int ld_sb, int bn, int splits, int stages, float* ws, long long ws_floats,
                      int* counters, int n_counters, int* status, void* stream, const SllmCommDesc* comm,
-                     const SllmGatherDesc* gather = nullptr, const FusedEpi* fused = nullptr) {
+                     const SllmGatherDesc* gather = nullptr, const FusedEpi* fused = nullptr, int act = 0) {
   if (gather) b = a;    // the B operand comes from the peers' buffers; keep the argument checks below simple
   if (!a || !b || !y || a_rows <= 0 || b_rows <= 0 || k <= 0 || splits < 1) return SLLM_ERR_INVALID_ARGUMENT;
   if (bn != 16 && bn != 32 && bn != 64 && bn != 128) return SLLM_ERR_UNSUPPORTED_SHAPE;
@@ -1181,7 +1185,8 @@ static int gemm_impl(const void* a, const void* b, void* y, const float* scale_a
 
   p.a_rows = a_rows; p.b_rows = b_rows; p.num_kb = num_kb; p.kb_per_split = kb_per_split; p.stages = stages;
   p.transpose_out = transpose_out; p.ldy = ldy; p.ld_sa = ld_sa; p.ld_sb = ld_sb;
-  p.epilogue = residual ? 1 : 0;
+  if (act < 0 || act > 1 || (act && (residual || comm || fused))) return SLLM_ERR_INVALID_ARGUMENT;
+  p.epilogue = residual ? 1 : act ? 2 : 0;
   // 2..8 splits reduce inside one thread-block cluster over DSMEM; more use the global fix-up.
   // (the output phase needs whole 16-byte units per slice: any slice width when Y is written
   // transposed, at least 8 columns otherwise)
@@ -1264,6 +1269,14 @@ SLLM_EXPORT int sllm_gemm(const void* a, const void* b, void* y, const float* sc
                           long long ws_floats, int* counters, int n_counters, int* status, void* stream) {
   return gemm_impl(a, b, y, scale_a, scale_b, residual, a_rows, b_rows, k, scaled, transpose_out, ldy, ld_sa, ld_sb,
                    bn, splits, stages, ws, ws_floats, counters, n_counters, status, stream, nullptr);
+}
+
+// bf16 GEMM with an activation on the sums (act 1: square of relu).
+SLLM_EXPORT int sllm_gemm_act(const void* a, const void* b, void* y, int a_rows, int b_rows, int k, int transpose_out, int ldy,
+                              int act, int bn, int splits, int stages, float* ws, long long ws_floats, int* counters,
+                              int n_counters, int* status, void* stream) {
+  return gemm_impl(a, b, y, nullptr, nullptr, nullptr, a_rows, b_rows, k, 0, transpose_out, ldy, 0, 0, bn, splits, stages, ws,
+                   ws_floats, counters, n_counters, status, stream, nullptr, nullptr, nullptr, act);
 }
 
 // Same GEMM with the cross-rank sum of the partial products fused into the epilogue (see the file

@@ -33,6 +33,10 @@ class ForwardBatch:
     # slot slots[s] of the state cache.
     row_off: Optional[torch.Tensor] = None     # int32 [S + 1]
     slots: Optional[torch.Tensor] = None       # int32 [S]
+    # Host copies of the same structure, set by eager batches only (a captured decode step has one row per sequence):
+    # row offsets, and the position of every sequence's first row.
+    row_off_host: Optional[list] = None
+    starts_host: Optional[list] = None
 
     @property
     def num_tokens(self) -> int:
@@ -61,4 +65,4 @@ def make_prefill_batch(prompts: list, block_table: torch.Tensor, device, start_p
         block_table=block_table, logit_rows=t(rows, torch.int64) if last_only else None,
         max_kv=max(pos) + 1 if pos else 0, cu_seqlens=t(cu) if fresh else None,
         max_seqlen=max(len(p) for p in prompts) if prompts else 0, cu_seqlens_host=cu if fresh else None,
-        row_off=t(cu))
+        row_off=t(cu), row_off_host=cu, starts_host=list(start_positions) if start_positions is not None else [0] * len(prompts))

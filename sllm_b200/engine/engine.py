@@ -92,6 +92,7 @@ class Engine:
         self.d_rope_delta = torch.zeros(max_batch, dtype=torch.int32, device=self.device)
         self.d_rope3 = torch.zeros(3 * max_batch, dtype=torch.int32, device=self.device)
         self._rope3_on = False
+        self._staged = torch.cuda.Event() if self.is_cuda else None    # last decode step's copies out of the pinned buffers
         self.np_tokens = self.h_tokens.numpy()
         self.np_positions = self.h_positions.numpy()
         self._steps = 0
@@ -216,7 +217,11 @@ class Engine:
             table = torch.zeros((1, self.max_blocks), dtype=torch.int32)
             self.cache.pool.fill_block_table([seq.seq_id], table)
             b = make_prefill_batch([list(ids)], table.to(self.device), self.device, last_only=False)
+            if self.has_state:
+                b.slots = self._slots([seq])
             h = self.model.hidden(b, self.cache)
+            if hasattr(self.model, "final_hidden"):
+                return self.model.final_hidden(h)
             return ops.rmsnorm(h, self.model.w.final_norm, self.cfg.rms_eps, self.cfg.norm_offset_one)
         finally:
             self.free_sequence(seq)
@@ -231,6 +236,9 @@ class Engine:
                 "kv_pool": self.cache.pool.stats() if hasattr(self.cache, "pool") else None}
 
     # ------------------------------------------------------------------ sequences
+    def _slots(self, seqs: list) -> torch.Tensor:
+        return torch.tensor([self.cache.slot_of[s.seq_id] for s in seqs], dtype=torch.int32, device=self.device)
+
     def new_sequence(self, prompt: list, user=None) -> Sequence:
         self._guard()
         s = Sequence(prompt=list(prompt), user=user)
@@ -380,7 +388,7 @@ class Engine:
             elif self.cfg.mrope_sections and any(seqs[i].rope_delta for i in rows):
                 b.rope_pos3 = self._rope3_rows([seqs[i] for i in rows], [len(p) for p in parts], b.positions)
             if self.has_state:
-                b.slots = torch.tensor([self.cache.slot_of[seqs[i].seq_id] for i in rows], dtype=torch.int32, device=self.device)
+                b.slots = self._slots([seqs[i] for i in rows])
             self.h2d_bytes += b.num_tokens * 12
             res = self.model.greedy(b, self.cache) if sample else self.model.forward(b, self.cache)
             if self.keep_hidden:
@@ -426,7 +434,7 @@ class Engine:
         if self.cfg.mrope_sections and any(s.rope_delta for s in seqs):
             b.rope_pos3 = self._rope3_rows(seqs, [len(p) for p in parts], b.positions)
         if self.has_state:
-            b.slots = torch.tensor([self.cache.slot_of[s.seq_id] for s in seqs], dtype=torch.int32, device=self.device)
+            b.slots = self._slots(seqs)
         self.h2d_bytes += table.numel() * 4 + b.num_tokens * 12
         res = self.model.greedy(b, self.cache) if sample else self.model.forward(b, self.cache)
         if self.keep_hidden:
@@ -440,6 +448,50 @@ class Engine:
         for s, p in zip(seqs, parts):
             out.append(flat[r0:r0 + len(p)] if sample else res[r0:r0 + len(p)])
             r0 += len(p)
+            pool.commit(s.seq_id, len(s.tokens))
+            s.num_computed = len(s.tokens)
+        return out
+
+    def step(self, seqs: list, wanted: list) -> torch.Tensor:
+        """One batch over every not-yet-computed token of each sequence - portions of prompts beside single decoded
+        tokens - and the logits [sum of wanted rows, vocab] of the places ``wanted[i]`` among sequence i's new tokens, in
+        that order.  A batch in which every sequence decodes one token is the captured decode step."""
+        self._guard()
+        counts = [len(s.tokens) - s.num_computed for s in seqs]
+        if len(wanted) != len(seqs) or any(n < 1 for n in counts):
+            raise ValueError("step needs at least one uncomputed token and one list of wanted places per sequence")
+        if any(not 0 <= p < n for n, w in zip(counts, wanted) for p in w):
+            raise ValueError("a wanted place lies outside the step's new tokens")
+        if any(len(s.tokens) > self.cfg.max_context for s in seqs):
+            raise ValueError("a sequence is longer than the context")
+        if all(n == 1 and s.num_computed > 0 for n, s in zip(counts, seqs)) and len(seqs) <= self.max_batch:
+            lg = self.decode(seqs, sample=False)
+            rows = [i for i, w in enumerate(wanted) for _ in w]
+            return lg[torch.tensor(rows, dtype=torch.int64, device=lg.device)]
+        pool = self.cache.pool
+        for s in seqs:
+            pool.reserve(s.seq_id, len(s.tokens))
+        table = torch.zeros((len(seqs), self.max_blocks), dtype=torch.int32)
+        pool.fill_block_table([s.seq_id for s in seqs], table)
+        b = make_prefill_batch([s.tokens[s.num_computed:] for s in seqs], table.to(self.device), self.device,
+                               [s.num_computed for s in seqs])
+        rows = [r0 + p for r0, w in zip(b.row_off_host, wanted) for p in w]
+        b.logit_rows = torch.tensor(rows, dtype=torch.int64, device=self.device)
+        if self.cfg.mrope_sections and any(s.rope_delta for s in seqs):
+            b.rope_pos3 = self._rope3_rows(seqs, counts, b.positions)
+        if self.has_state:
+            b.slots = self._slots(seqs)
+        self.h2d_bytes += table.numel() * 4 + b.num_tokens * 12
+        if rows:
+            out = self.model.forward(b, self.cache)
+        else:
+            out = torch.empty((0, self.cfg.vocab), dtype=torch.float32, device=self.device)
+            self.model.last_hidden = self.model.hidden(b, self.cache)
+        if self.keep_hidden:
+            self._log_hidden(seqs, [s.num_computed for s in seqs], counts, self.model.last_hidden)
+        self._table_key = None
+        self._check_status(every=1)
+        for s in seqs:
             pool.commit(s.seq_id, len(s.tokens))
             s.num_computed = len(s.tokens)
         return out
@@ -546,7 +598,7 @@ class Engine:
         if g is None:
             # warm up outside capture (module init, workspace allocation), then capture
             # a recurrent state is advanced by every execution: keep it out of the warm-up run
-            snap = (self.cache.conv_state.clone(), self.cache.rec_state.clone()) if self.has_state else None
+            snap = self.cache.save_all() if self.has_state else None
             s = torch.cuda.Stream(device=self.device)
             s.wait_stream(torch.cuda.current_stream())
             with torch.cuda.stream(s):
@@ -554,8 +606,7 @@ class Engine:
             torch.cuda.current_stream().wait_stream(s)
             torch.cuda.synchronize()
             if snap is not None:
-                self.cache.conv_state.copy_(snap[0])
-                self.cache.rec_state.copy_(snap[1])
+                self.cache.load_all(snap)
                 torch.cuda.synchronize()
             g = torch.cuda.CUDAGraph()
             from ..ops import _lib
@@ -598,6 +649,8 @@ class Engine:
         for s in seqs:
             pool.reserve(s.seq_id, len(s.tokens))
         np_ = self._padded(n)
+        if self._staged is not None:
+            self._staged.synchronize()       # a caller that reads nothing back may be ahead of the device
         self.np_tokens[:n] = [s.tokens[-1] for s in seqs]
         self.np_positions[:n] = [len(s.tokens) - 1 for s in seqs]
         if np_ > n:  # padding rows replay row 0 (same token, same slot, same values: a harmless rewrite)
@@ -632,6 +685,8 @@ class Engine:
             torch.add(self.d_positions[:np_], self.d_rope_delta[:np_], out=r3[0])
             r3[1].copy_(r3[0])
             r3[2].copy_(r3[0])
+        if self._staged is not None:
+            self._staged.record()
         self._run_decode(np_, sample)
         if sample:
             self.h_out[:np_].copy_(self.d_out[:np_], non_blocking=True)
@@ -695,27 +750,27 @@ def build_engine(cfg: ModelConfig, device="cuda", seed: int = 0, num_pages: Opti
     the mixture-of-experts family and to hybrid models with a sparse MLP."""
     device = torch.device(device)
     tp_size, tp_rank = (tp.size, tp.rank) if tp is not None else (1, 0)
-    if cfg.family == "qwen35":
-        from ..cache.hybrid import HybridCache
-        from ..models.qwen35 import Qwen35Model, init_random_qwen35_weights
-        ep_size, ep_rank = (ep.size, ep.rank) if ep is not None else (1, 0)
-        model = Qwen35Model(cfg, init_random_qwen35_weights(cfg, device, seed, tp_size=tp_size, tp_rank=tp_rank,
-                                                            ep_size=ep_size, ep_rank=ep_rank), tp, ep)
-        if num_pages is None:
-            num_pages = max_batch * ((cfg.max_context + cfg.page_size - 1) // cfg.page_size) + 8
-        cache = HybridCache(cfg, num_pages, device, max_seqs=2 * max_batch + 2, kv_heads=model.local_kv_heads,
-                            tp_size=tp_size)
-        return Engine(cfg, model, cache, device, max_batch=max_batch, use_cuda_graphs=use_cuda_graphs, tp=tp)
-    if cfg.family == "moe":
-        from ..models.moe import MoeModel, init_random_moe_weights
-        ep_size, ep_rank = (ep.size, ep.rank) if ep is not None else (1, 0)
-        weights = init_random_moe_weights(cfg, device, seed, tp_size, tp_rank, ep_size, ep_rank)
-        model = MoeModel(cfg, weights, tp, ep)
-    else:
-        from ..models.llama import LlamaModel, init_random_weights
-        weights = init_random_weights(cfg, device, seed, tp_size, tp_rank)
-        model = LlamaModel(cfg, weights, tp)
+    from ..models import registry
+    ep_size, ep_rank = (ep.size, ep.rank) if ep is not None else (1, 0)
+    weights = registry.init_random_weights(cfg, device, seed, tp_size, tp_rank, ep_size, ep_rank)
+    model = registry.make_model(cfg, weights, tp, ep)
     if num_pages is None:
         num_pages = max_batch * ((cfg.max_context + cfg.page_size - 1) // cfg.page_size) + 8
-    cache = PagedKVCache(cfg, num_pages, device, kv_heads=model.local_kv_heads)
+    cache = registry.make_cache(cfg, model, num_pages, device, max_seqs=2 * max_batch + 2)
     return Engine(cfg, model, cache, device, max_batch=max_batch, use_cuda_graphs=use_cuda_graphs, tp=tp)
+
+
+def load_engine(path: str, device="cuda", dtype: str = "bf16", max_tokens: Optional[int] = None, max_batch: int = 8,
+                max_seqs: Optional[int] = None, use_cuda_graphs: bool = True) -> Engine:
+    """Engine of a model folder (config.json + model.safetensors).  ``max_tokens``: tokens that the pages of all live
+    sequences hold together, and the longest context (default: ``max_batch`` sequences of the default context);
+    ``max_seqs``: state slots of recurrent layers."""
+    from ..models import registry
+    device = torch.device(device)
+    cfg = registry.read_folder_config(path, dtype=dtype, max_context=max_tokens)
+    weights = registry.load_folder_weights(path, cfg, device)
+    model = registry.make_model(cfg, weights)
+    blocks = (cfg.max_context + cfg.page_size - 1) // cfg.page_size
+    num_pages = blocks if max_tokens else max_batch * blocks + 8
+    cache = registry.make_cache(cfg, model, num_pages, device, max_seqs=max_seqs or 2 * max_batch + 2)
+    return Engine(cfg, model, cache, device, max_batch=max_batch, use_cuda_graphs=use_cuda_graphs and device.type == "cuda")

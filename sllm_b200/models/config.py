@@ -13,7 +13,7 @@ from typing import Optional
 @dataclass
 class ModelConfig:
     name: str = "tiny-llama"
-    family: str = "llama"            # llama | moe | qwen35 | gemma4
+    family: str = "llama"            # llama | moe | qwen35 | gemma4 | zokuvik
     n_layers: int = 2
     d_model: int = 256
     n_heads: int = 4
@@ -61,6 +61,10 @@ class ModelConfig:
     attn_scale: Optional[float] = None     # softmax scale (None: 1 / sqrt(head_dim)); 1.0 where q / k norms set the scale
     layer_scalar: bool = False       # the residual stream is multiplied by a learned scalar at the end of every layer
     k_equals_v_full: bool = False    # full-attention layers have no value projection: v = the (un-normed) key projection
+    # families whose layers differ in kind and size: one dict per layer, {"type": mixer kind, "mixer": {sizes}, "mlp":
+    # {"kind", "ff"} or None}; the norms split a vector into norm_groups parts
+    layer_specs: Optional[list] = None
+    norm_groups: int = 1
     # vision-language models: rotary pairs [0, t) follow the temporal index, [t, t + h) the height index and the rest
     # the width index of a token's 3-axis position (text tokens carry the same value on all three)
     mrope_sections: Optional[list] = None
@@ -162,7 +166,13 @@ def _qwen35_moe_hybrid():
     return qwen35_moe_hybrid_shape()
 
 
+def _zokuvik():
+    from .zokuvik import zokuvik_shape
+    return zokuvik_shape()
+
+
 NAMED = {
+    "zokuvik": _zokuvik,
     "qwen35-moe": _qwen35_moe,
     "qwen35-moe-hybrid": _qwen35_moe_hybrid,
     "tiny-llama": tiny_llama,

@@ -166,6 +166,9 @@ def check(rc: int, what: str) -> None:
 _KERNEL_SIGNATURES = {
     "sllm_gemm_workspace_floats": (L, [I, I, I, I]),
     "sllm_gemm": (I, [P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, P, L, P, I, P, P]),
+    "sllm_gemm_act": (I, [P, P, P, I, I, I, I, I, I, I, I, I, P, L, P, I, P, P]),
+    "sllm_gemm_simt": (I, [P, P, P, P, I, I, I, I, I, I, I, I, P]),
+    "sllm_group_norm": (I, [P, P, I, P, I, P, P, P, P, P, I, I, I, F, I, P]),
     "sllm_embedding": (I, [P, P, P, I, I, I, F, P]),
     "sllm_rmsnorm": (I, [P, P, P, P, P, I, I, I, F, I, P]),
     "sllm_gated_act": (I, [P, P, P, P, I, I, I, I, P]),
@@ -175,6 +178,7 @@ _KERNEL_SIGNATURES = {
     "sllm_rope_kv_append_mrope": (I, [P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, F, F, P, P, I, I, P]),
     "sllm_elementwise": (I, [P, P, P, L, I, I, F, P]),
     "sllm_argmax": (I, [P, P, P, I, I, I, I, P, L, P, I, P]),
+    "sllm_argmax_f32": (I, [P, P, P, I, I, I, I, P, L, P, I, P]),
     "sllm_gemm_set_cluster_split": (None, [I]),
     "sllm_decode_attention_tc": (I, [P, I, P, P, P, P, F, F, P, I, P, P, I, I, I, I, I, I, F, P, P, P, I, P, I, P, L,
                                       P, I, P, P]),
@@ -233,6 +237,14 @@ def install_fake(fake: Optional[FakeKernelLibrary]) -> None:
 
 def fake_active() -> bool:
     return _fake[0] is not None
+
+
+def use_kernel_library(path) -> None:
+    """Loads the kernels from ``path`` (a build of fewer translation units) instead of the full library."""
+    global _KERNEL_PATH
+    if _kernels is not None and Path(path) != _KERNEL_PATH:
+        raise KernelError("the kernel library is loaded already")
+    _KERNEL_PATH = Path(path)
 
 
 def kernels():

@@ -156,8 +156,24 @@ def gemm_raw(a: torch.Tensor, b: torch.Tensor, y: torch.Tensor, *, scale_a=None,
     _lib.check(rc, "gemm")
 
 
-def linear(x, w: LinearWeight, residual: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """Y = X W^T (+ residual).  x: Tensor [M, K] (bf16 / fp32) or QTensor for FP8 weights."""
+def _linear_simt(x: torch.Tensor, w: torch.Tensor, residual: Optional[torch.Tensor], act: Optional[str]) -> torch.Tensor:
+    """CUDA-core product: fp32 operands, or bf16 rows that a TMA copy cannot address (K not a multiple of 8)."""
+    m, k = x.shape
+    n = w.shape[0]
+    if x.dtype != w.dtype or x.stride(1) != 1:
+        raise ValueError("the CUDA-core product takes operands of one type with contiguous rows")
+    y = torch.empty((m, n), dtype=x.dtype, device=x.device)
+    rc = _lib.kernels().sllm_gemm_simt(_p(x), _p(w), _p(y), _p(residual), m, n, k, x.stride(0), w.stride(0), n,
+                                       1 if act else 0, int(x.dtype == torch.float32), _stream())
+    _lib.check(rc, "gemm_simt")
+    return y
+
+
+def linear(x, w: LinearWeight, residual: Optional[torch.Tensor] = None, act: Optional[str] = None) -> torch.Tensor:
+    """Y = act(X W^T) (+ residual).  x: Tensor [M, K] (bf16 / fp32) or QTensor for FP8 weights.  ``act``: None or
+    "relu_sq" (square of relu; dense weights, without a residual), applied to the fp32 sums."""
+    if act is not None and (act != "relu_sq" or w.kind != "dense" or residual is not None):
+        raise ValueError("the product's activation is relu_sq, on dense weights without a residual")
     xd = x.data if isinstance(x, QTensor) else x
     if w.kind == "w4":
         from .w4 import linear_w4
@@ -170,11 +186,15 @@ def linear(x, w: LinearWeight, residual: Optional[torch.Tensor] = None) -> torch
         if w.kind == "fp8" and not isinstance(x, QTensor):
             xf = ref.dequant_fp8_1x128(*ref.quant_fp8_1x128(x))
         y = xf @ w.dequantized().t()
+        if act:
+            y = torch.relu(y) ** 2
         if residual is not None:
             y = y + residual.to(torch.float32)
         return y.to(residual.dtype if residual is not None else (torch.float32 if w.w.dtype == torch.float32 else torch.bfloat16))
     m = xd.shape[0]
     n = w.out_features
+    if w.kind == "dense" and (w.w.dtype == torch.float32 or w.in_features % 8):
+        return _linear_simt(xd, w.w, residual, act)
     if w.kind == "fp8":
         if not isinstance(x, QTensor):
             x = quant_fp8(x)
@@ -195,7 +215,14 @@ def linear(x, w: LinearWeight, residual: Optional[torch.Tensor] = None) -> torch
             gemm_raw(x.data, w.w, y, scale_a=x.scale, scale_b=w.scale_t, residual=residual, transpose_out=False,
                      bn=bn, splits=splits, stages=stages)
     else:
-        if swap:
+        if act:
+            a, b = (w.w, x) if swap else (x, w.w)
+            wsp = workspace(xd.device)
+            rc = _lib.kernels().sllm_gemm_act(_p(a), _p(b), _p(y), a.shape[0], b.shape[0], w.in_features, int(swap), n, 1, bn, splits,
+                                              stages, _p(wsp.ws), wsp.ws.numel(), _p(wsp.counters), wsp.counters.numel(),
+                                              _p(wsp.status), _stream())
+            _lib.check(rc, "gemm")
+        elif swap:
             gemm_raw(w.w, x, y, residual=residual, transpose_out=True, bn=bn, splits=splits, stages=stages)
         else:
             gemm_raw(x, w.w, y, residual=residual, transpose_out=False, bn=bn, splits=splits, stages=stages)
@@ -239,6 +266,51 @@ def rmsnorm(x: torch.Tensor, w: torch.Tensor, eps: float, offset_one: bool = Fal
     rc = lib.sllm_rmsnorm(_p(x), _p(w), _p(y), None, None, 0, m, d, eps, int(offset_one), _stream())
     _lib.check(rc, "rmsnorm")
     return y
+
+
+# ---- grouped RMSNorm on an fp32 residual stream (csrc/group_norm.cu)
+def _gn_ref(x: torch.Tensor, w: torch.Tensor, eps: float, groups: int) -> torch.Tensor:
+    t, d = x.shape
+    g = x.float().view(t, groups, d // groups)
+    return (g / torch.sqrt((g * g).mean(-1, keepdim=True) + eps)).view(t, d) * w
+
+
+def _group_norm(x, w_out, eps, groups, dtype, *, table=None, ids=None, y=None, w_post=None, rows_idx=None):
+    rows = ids.numel() if table is not None else (rows_idx.numel() if rows_idx is not None else x.shape[0])
+    d = x.shape[1]
+    z = torch.empty((rows, d), dtype=dtype, device=x.device) if w_out is not None else None
+    if rows == 0:
+        return z
+    rc = _lib.kernels().sllm_group_norm(_p(table), _p(ids), table.shape[0] if table is not None else 0, _p(y),
+                                        y.stride(0) if y is not None else 0, _p(w_post), _p(x), _p(rows_idx), _p(w_out), _p(z), rows,
+                                        d, groups, eps, int(dtype == torch.float32), _stream())
+    _lib.check(rc, "group_norm")
+    return z
+
+
+def embed_group_norm(table: torch.Tensor, ids: torch.Tensor, w_out: torch.Tensor, eps: float, groups: int = 1):
+    """(residual fp32 [T, d], its grouped RMSNorm in the table's type): the embedding and the first layer's input norm."""
+    if _lib.on_cpu(table):
+        x = table[ids.long()].float()
+        return x, _gn_ref(x, w_out, eps, groups).to(table.dtype)
+    x = torch.empty((ids.numel(), table.shape[1]), dtype=torch.float32, device=table.device)
+    return x, _group_norm(x, w_out, eps, groups, table.dtype, table=table, ids=ids)
+
+
+def add_group_norm(x: torch.Tensor, y: torch.Tensor, w_post: torch.Tensor, w_out: Optional[torch.Tensor], eps: float,
+                   groups: int = 1):
+    """x += norm(y) * w_post in place (fp32), then norm(x) * w_out in the type of ``y`` (None without ``w_out``)."""
+    if _lib.on_cpu(x):
+        x += _gn_ref(y, w_post, eps, groups)
+        return None if w_out is None else _gn_ref(x, w_out, eps, groups).to(y.dtype)
+    return _group_norm(x, w_out, eps, groups, y.dtype, y=y, w_post=w_post)
+
+
+def group_norm(x: torch.Tensor, w: torch.Tensor, eps: float, groups: int, dtype, rows: Optional[torch.Tensor] = None):
+    """Grouped RMSNorm of an fp32 [T, d] (of the rows listed in ``rows``, int64) in ``dtype``."""
+    if _lib.on_cpu(x):
+        return _gn_ref(x if rows is None else x.index_select(0, rows), w, eps, groups).to(dtype)
+    return _group_norm(x, w, eps, groups, dtype, rows_idx=rows)
 
 
 def gated_act(x: torch.Tensor, act: str = "silu", quant: bool = False):
@@ -312,8 +384,9 @@ def argmax(logits: torch.Tensor, index_offset: int = 0, with_values: bool = Fals
     out = torch.empty(rows, dtype=torch.int32, device=logits.device)
     val = torch.empty(rows, dtype=torch.float32, device=logits.device) if with_values else None
     wsp = workspace(logits.device)
-    rc = _lib.kernels().sllm_argmax(_p(logits), _p(out), _p(val), rows, n, logits.stride(0), index_offset,
-                                    _p(wsp.ws), wsp.ws.numel() * 4, _p(wsp.counters), wsp.counters.numel(), _stream())
+    fn = _lib.kernels().sllm_argmax_f32 if logits.dtype == torch.float32 else _lib.kernels().sllm_argmax
+    rc = fn(_p(logits), _p(out), _p(val), rows, n, logits.stride(0), index_offset, _p(wsp.ws), wsp.ws.numel() * 4, _p(wsp.counters),
+            wsp.counters.numel(), _stream())
     _lib.check(rc, "argmax")
     return (out, val) if with_values else out
 

@@ -1,0 +1,157 @@
+"""Latent attention ops: one cached row [latent | rotated key part] per token serves every head (kernels in
+csrc/latent_attention.cu; PyTorch restatements here for CPU tensors).
+
+A layer runs  append  (norms of the query / key latents, rotation of the shared key part, page write) ->
+absorb  (q_h W_uk[h] and the query's rotated part: queries of the width of a cache row) -> attend  (softmax over the
+visible rows, result in latent space) -> values  (W_uv[h] and the output gate).
+"""
+from __future__ import annotations
+
+import ctypes as C
+from dataclasses import dataclass
+from typing import Optional
+
+import torch
+
+from . import _lib
+
+P, I, F, L = C.c_void_p, C.c_int, C.c_float, C.c_longlong
+_SIGS = {
+    "sllm_latent_append": (I, [P, I, I, I, I, I, I, P, P, F, P, P, I, I, I, P, P, P, P, I, I, I, I, P]),
+    "sllm_head_matmul": (I, [P, L, I, P, P, L, I, I, I, I, I, P, L, I, P, P, I, I, I, P]),
+    "sllm_latent_attention": (I, [P, P, I, I, I, P, P, P, I, I, I, I, I, F, P, I, P]),
+}
+
+
+def _k():
+    for n, s in _SIGS.items():
+        _lib.EXTRA_KERNEL_SIGNATURES.setdefault(n, s)
+    return _lib.kernels()
+
+
+@dataclass
+class LatentSpec:
+    """Sizes and constants of one latent-attention layer."""
+    heads: int
+    dim: int                  # unrotated query / key channels per head
+    rot_dim: int              # rotated channels per head (the key's are shared by all heads)
+    vdim: int
+    kv_rank: int
+    scale: float
+    rot_base: float
+    rot_dims: int             # channels of rot_dim that turn
+    interleaved: bool         # rotary pairs (2i, 2i + 1); else (i, i + rot_dims / 2)
+    q_rank: int = 0           # 0: queries come straight from the layer input
+    window: int = 0           # 0: every earlier position is visible
+    gated: bool = False       # one sigmoid output gate per head
+
+    @property
+    def width(self) -> int:
+        return self.kv_rank + self.rot_dim
+
+    def inv_freq(self, device) -> torch.Tensor:
+        i = torch.arange(self.rot_dims // 2, dtype=torch.float64)
+        return (float(self.rot_base) ** (-2.0 * i / self.rot_dims)).float().to(device)
+
+
+@dataclass
+class LatentPages:
+    """One layer's pages: [num_pages, page, ld], columns [0, kv_rank) the latent, then the rotated key part."""
+    pages: torch.Tensor
+    page_size: int
+
+
+def rotate(x: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tensor, dims: int, interleaved: bool) -> torch.Tensor:
+    """x [T, ..., R] in fp32: the first ``dims`` channels turned by positions * inv_freq."""
+    ang = positions.float().view(-1, *([1] * (x.dim() - 1))) * inv_freq
+    c, s = ang.cos(), ang.sin()
+    out = x.clone()
+    if interleaved:
+        u, v = x[..., 0:dims:2], x[..., 1:dims:2]
+        out[..., 0:dims:2], out[..., 1:dims:2] = u * c - v * s, v * c + u * s
+    else:
+        u, v = x[..., :dims // 2], x[..., dims // 2:dims]
+        out[..., :dims // 2], out[..., dims // 2:dims] = u * c - v * s, v * c + u * s
+    return out
+
+
+def append(proj: torch.Tensor, off_q: int, off_kv: int, spec: LatentSpec, q_norm: Optional[torch.Tensor], kv_norm: torch.Tensor,
+           eps: float, inv_freq: torch.Tensor, kv: LatentPages, positions, seq_index, block_table) -> Optional[torch.Tensor]:
+    """proj [T, *]: columns off_q.. hold the query latent (with ``q_rank``), off_kv.. [key latent | rotated part].  Writes
+    each token's cache row; returns the normed query latent [T, q_rank] or None."""
+    t = proj.shape[0]
+    if _lib.on_cpu(proj):
+        def rms(x, w):
+            x = x.float()
+            return x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps) * w
+        x = proj[:, off_kv:off_kv + spec.width]
+        c = rms(x[:, :spec.kv_rank], kv_norm)
+        kr = rotate(x[:, spec.kv_rank:].float(), positions, inv_freq, spec.rot_dims, spec.interleaved)
+        pos = positions.long()
+        blk = block_table[seq_index.long(), pos // kv.page_size].long()
+        kv.pages[blk, pos % kv.page_size, :spec.width] = torch.cat([c, kr], dim=1).to(kv.pages.dtype)
+        return rms(proj[:, off_q:off_q + spec.q_rank], q_norm).to(proj.dtype) if spec.q_rank else None
+    from .core import _p, _stream
+    cq = torch.empty((t, spec.q_rank), dtype=proj.dtype, device=proj.device) if spec.q_rank else None
+    rc = _k().sllm_latent_append(_p(proj), proj.stride(0), off_q, off_kv, spec.q_rank, spec.kv_rank, spec.rot_dim, _p(q_norm),
+                                 _p(kv_norm), eps, _p(cq), _p(kv.pages), kv.pages.shape[2], kv.page_size, block_table.stride(0),
+                                 _p(positions), _p(seq_index), _p(block_table), _p(inv_freq), spec.rot_dims, int(spec.interleaved),
+                                 t, int(proj.dtype == torch.float32), _stream())
+    _lib.check(rc, "latent_append")
+    return cq
+
+
+def absorb(q: torch.Tensor, spec: LatentSpec, uk: torch.Tensor, inv_freq: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
+    """q [T, heads * (dim + rot_dim)] (row stride allowed), uk [heads, dim, kv_rank] -> [T, heads, kv_rank + rot_dim]."""
+    t, h, hd = q.shape[0], spec.heads, spec.dim + spec.rot_dim
+    if _lib.on_cpu(q):
+        x = q.reshape(t, h, hd).float()
+        a = torch.einsum("thd,hdc->thc", x[..., :spec.dim], uk.float())
+        r = rotate(x[..., spec.dim:], positions, inv_freq, spec.rot_dims, spec.interleaved)
+        return torch.cat([a, r], dim=-1).to(q.dtype)
+    from .core import _p, _stream
+    out = torch.empty((t, h, spec.width), dtype=q.dtype, device=q.device)
+    rc = _k().sllm_head_matmul(_p(q), q.stride(0), hd, _p(uk), _p(out), h * spec.width, spec.width, t, h, spec.dim, spec.kv_rank,
+                               None, 0, spec.rot_dim, _p(positions), _p(inv_freq), spec.rot_dims, int(spec.interleaved),
+                               int(q.dtype == torch.float32), _stream())
+    _lib.check(rc, "latent_absorb")
+    return out
+
+
+def attend(qa: torch.Tensor, spec: LatentSpec, kv: LatentPages, block_table, seq_index, kv_lens) -> torch.Tensor:
+    """Absorbed queries [R, heads, width] over their sequences' pages -> [R, heads, kv_rank]."""
+    r = qa.shape[0]
+    if _lib.on_cpu(qa):
+        out = torch.empty((r, spec.heads, spec.kv_rank), dtype=torch.float32)
+        for i in range(r):
+            n = int(kv_lens[i])
+            blks = block_table[int(seq_index[i]), :(n + kv.page_size - 1) // kv.page_size].long()
+            lo = max(0, n - spec.window) if spec.window else 0
+            rows = kv.pages[blks].flatten(0, 1)[lo:n, :spec.width].float()
+            p = torch.softmax(qa[i].float() @ rows.t() * spec.scale, dim=-1)
+            out[i] = p @ rows[:, :spec.kv_rank]
+        return out.to(qa.dtype)
+    from .core import _p, _stream
+    out = torch.empty((r, spec.heads, spec.kv_rank), dtype=qa.dtype, device=qa.device)
+    rc = _k().sllm_latent_attention(_p(qa), _p(kv.pages), kv.pages.shape[2], kv.page_size, block_table.stride(0), _p(block_table),
+                                    _p(seq_index), _p(kv_lens), r, spec.heads, spec.kv_rank, spec.width, spec.window, spec.scale,
+                                    _p(out), int(qa.dtype == torch.float32), _stream())
+    _lib.check(rc, "latent_attention")
+    return out
+
+
+def values(o: torch.Tensor, spec: LatentSpec, uvt: torch.Tensor, gate: Optional[torch.Tensor]) -> torch.Tensor:
+    """o [T, heads, kv_rank], uvt [heads, kv_rank, vdim], gate [T, heads] logits or None -> [T, heads * vdim]."""
+    t, h = o.shape[0], spec.heads
+    if _lib.on_cpu(o):
+        y = torch.einsum("thc,hcv->thv", o.float(), uvt.float())
+        if gate is not None:
+            y = y * torch.sigmoid(gate.float()).unsqueeze(-1)
+        return y.reshape(t, h * spec.vdim).to(o.dtype)
+    from .core import _p, _stream
+    out = torch.empty((t, h * spec.vdim), dtype=o.dtype, device=o.device)
+    rc = _k().sllm_head_matmul(_p(o), h * spec.kv_rank, spec.kv_rank, _p(uvt), _p(out), h * spec.vdim, spec.vdim, t, h, spec.kv_rank,
+                               spec.vdim, _p(gate), gate.stride(0) if gate is not None else 0, 0, None, None, 0, 0,
+                               int(o.dtype == torch.float32), _stream())
+    _lib.check(rc, "latent_values")
+    return out
