@@ -280,7 +280,7 @@ class ZokuvikModel:
         q = ops.linear(cq, lw.uq) if s.q_rank else proj[:, :q_cols]
         gate = proj[:, q_cols + s.width:q_cols + s.width + s.heads] if s.gated else None
         qa = A.absorb(q, s, lw.uk, lw.inv_freq, b.positions)
-        o = A.attend(qa, s, kv, b.block_table, b.seq_index, b.kv_lens)
+        o = A.attend(qa, s, kv, b.block_table, b.seq_index, b.kv_lens, b.max_kv)
         return ops.linear(A.values(o, s, lw.uvt, gate), lw.o)
 
     def _delta(self, z, lw: ZokuvikLayer, b: ForwardBatch, state):

@@ -19,6 +19,8 @@ P, I, F, L = C.c_void_p, C.c_int, C.c_float, C.c_longlong
 _SIGS = {
     "sllm_latent_append": (I, [P, I, I, I, I, I, I, P, P, F, P, P, I, I, I, P, P, P, P, I, I, I, I, P]),
     "sllm_head_matmul": (I, [P, L, I, P, P, L, I, I, I, I, I, P, L, I, P, P, I, I, I, P]),
+    "sllm_latent_decode_workspace_floats": (L, [I, I, I, I]),
+    "sllm_latent_decode": (I, [P, P, L, I, I, I, P, P, P, I, I, I, I, I, F, P, I, P, L, P, P]),
     "sllm_latent_attention": (I, [P, P, I, I, I, P, P, P, I, I, I, I, I, F, P, I, P]),
 }
 
@@ -118,8 +120,29 @@ def absorb(q: torch.Tensor, spec: LatentSpec, uk: torch.Tensor, inv_freq: torch.
     return out
 
 
-def attend(qa: torch.Tensor, spec: LatentSpec, kv: LatentPages, block_table, seq_index, kv_lens) -> torch.Tensor:
-    """Absorbed queries [R, heads, width] over their sequences' pages -> [R, heads, kv_rank]."""
+def _tensor_core_rows(qa: torch.Tensor, spec: LatentSpec, kv: LatentPages) -> bool:
+    """Whether the page-streaming kernel (csrc/latent_decode.cu) takes this layer."""
+    return (qa.dtype == torch.bfloat16 and spec.width <= 576 and spec.kv_rank <= 512 and spec.kv_rank % 8 == 0
+            and spec.width % 2 == 0 and kv.page_size in (8, 16, 32))
+
+
+def _splits(rows: int, groups: int, keys: int) -> int:
+    """KV splits of the page-streaming kernel: one CTA per SM, so the number of waves times the tiles of a split (and a
+    tile's worth of start-up and merging) is what a launch costs."""
+    tiles = max(1, (keys + 63) // 64)
+    best, cost = 1, None
+    for s in range(1, min(32, tiles) + 1):
+        waves = (rows * groups * s + 147) // 148
+        c = waves * ((tiles + s - 1) // s + 1.5 + (0.5 if s > 1 else 0.0))
+        if cost is None or c < cost - 1e-9:
+            best, cost = s, c
+    return best
+
+
+def attend(qa: torch.Tensor, spec: LatentSpec, kv: LatentPages, block_table, seq_index, kv_lens, max_kv: int = 0,
+           impl: Optional[str] = None) -> torch.Tensor:
+    """Absorbed queries [R, heads, width] over their sequences' pages -> [R, heads, kv_rank].  ``max_kv``: host-side bound
+    on kv_lens (split heuristics); ``impl`` "cuda_core" forces the any-size kernel."""
     r = qa.shape[0]
     if _lib.on_cpu(qa):
         out = torch.empty((r, spec.heads, spec.kv_rank), dtype=torch.float32)
@@ -131,8 +154,26 @@ def attend(qa: torch.Tensor, spec: LatentSpec, kv: LatentPages, block_table, seq
             p = torch.softmax(qa[i].float() @ rows.t() * spec.scale, dim=-1)
             out[i] = p @ rows[:, :spec.kv_rank]
         return out.to(qa.dtype)
-    from .core import _p, _stream
+    from .core import _p, _stream, workspace
     out = torch.empty((r, spec.heads, spec.kv_rank), dtype=qa.dtype, device=qa.device)
+    if impl != "cuda_core" and _tensor_core_rows(qa, spec, kv):
+        wsp = workspace(qa.device)
+        groups = (spec.heads + 31) // 32
+        keys = max_kv if max_kv > 0 else block_table.shape[1] * kv.page_size
+        if spec.window:
+            keys = min(keys, spec.window + kv.page_size)
+        splits = _splits(r, groups, keys)
+        while splits > 1 and r * groups * splits * 32 * (spec.kv_rank + 2) > wsp.ws.numel():
+            splits -= 1
+        if _lib.audit_enabled():
+            _lib.record_dispatch("latent_attention", "latent_decode_kernel", rows=r, heads=spec.heads, width=spec.width,
+                                 window=spec.window, splits=splits, grid=[r, groups, splits])
+        rc = _k().sllm_latent_decode(_p(qa), _p(kv.pages), kv.pages.shape[0] * kv.page_size, kv.pages.shape[2], kv.page_size,
+                                     block_table.stride(0), _p(block_table), _p(seq_index), _p(kv_lens), r, spec.heads, spec.kv_rank,
+                                     spec.width, spec.window, spec.scale, _p(out), splits, _p(wsp.ws), wsp.ws.numel(),
+                                     _p(wsp.status), _stream())
+        _lib.check(rc, "latent_decode")
+        return out
     rc = _k().sllm_latent_attention(_p(qa), _p(kv.pages), kv.pages.shape[2], kv.page_size, block_table.stride(0), _p(block_table),
                                     _p(seq_index), _p(kv_lens), r, spec.heads, spec.kv_rank, spec.width, spec.window, spec.scale,
                                     _p(out), int(qa.dtype == torch.float32), _stream())
