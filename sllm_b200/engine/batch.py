@@ -7,7 +7,7 @@ which is why its batch planner was never connected (docs/plans/main-plan.md:894-
 """
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 from typing import Optional
 
 import torch
@@ -37,6 +37,7 @@ class ForwardBatch:
     # row offsets, and the position of every sequence's first row.
     row_off_host: Optional[list] = None
     starts_host: Optional[list] = None
+    plans: dict = field(default_factory=dict)  # device tables that ops derive from the structure, shared by the layers
 
     @property
     def num_tokens(self) -> int:

@@ -13,7 +13,8 @@ from .config import ModelConfig
 
 # CUDA translation units of a family, for callers that build no more than they run (None: the whole library)
 KERNEL_UNITS = {
-    "zokuvik": ("elementwise", "gemm_tcgen05", "gemm_simt", "group_norm", "latent_attention", "latent_decode", "delta_rule"),
+    "zokuvik": ("elementwise", "gemm_tcgen05", "gemm_simt", "group_norm", "latent_attention", "latent_decode", "latent_prefill",
+                "delta_rule"),
 }
 
 

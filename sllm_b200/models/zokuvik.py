@@ -127,7 +127,8 @@ class ZokuvikLayer:
     uq: Optional[LinearWeight] = None
     q_norm: Optional[torch.Tensor] = None
     kv_norm: Optional[torch.Tensor] = None
-    uk: Optional[torch.Tensor] = None          # [heads, dim, kv_rank]
+    expand: Optional[LinearWeight] = None      # [heads * dim | heads * vdim, kv_rank]: W_uk, then W_uv
+    uk: Optional[torch.Tensor] = None          # [heads, dim, kv_rank], a view of ``expand``
     uvt: Optional[torch.Tensor] = None         # [heads, kv_rank, vdim]
     delta: Optional[D.DeltaSpec] = None
     w2: Optional[LinearWeight] = None          # [heads * dim, rank padded to 8]
@@ -181,8 +182,10 @@ def pack_weights(cfg: ModelConfig, get: Callable, device) -> ZokuvikWeights:
             s = latent_spec(e)
             names = [q + ("dq" if s.q_rank else "q"), q + "dkv"] + ([q + "g"] if s.gated else [])
             kw.update(latent=s, in_proj=mat(*names, pad=True), kv_norm=vec(q + "dkv.norm"), inv_freq=s.inv_freq(device),
-                      uk=mat(q + "uk").w.view(s.heads, s.dim, s.kv_rank),
-                      uvt=mat(q + "uv").w.view(s.heads, s.vdim, s.kv_rank).transpose(1, 2).contiguous())
+                      expand=mat(q + "uk", q + "uv"))
+            nk = s.heads * s.dim
+            kw.update(uk=kw["expand"].w[:nk].view(s.heads, s.dim, s.kv_rank),
+                      uvt=kw["expand"].w[nk:].view(s.heads, s.vdim, s.kv_rank).transpose(1, 2).contiguous())
             if s.q_rank:
                 kw.update(uq=mat(q + "uq"), q_norm=vec(q + "dq.norm"))
         else:
@@ -279,9 +282,7 @@ class ZokuvikModel:
                       b.block_table)
         q = ops.linear(cq, lw.uq) if s.q_rank else proj[:, :q_cols]
         gate = proj[:, q_cols + s.width:q_cols + s.width + s.heads] if s.gated else None
-        qa = A.absorb(q, s, lw.uk, lw.inv_freq, b.positions)
-        o = A.attend(qa, s, kv, b.block_table, b.seq_index, b.kv_lens, b.max_kv)
-        return ops.linear(A.values(o, s, lw.uvt, gate), lw.o)
+        return ops.linear(A.attention(q, gate, s, lw.uk, lw.uvt, lw.expand, lw.inv_freq, kv, b), lw.o)
 
     def _delta(self, z, lw: ZokuvikLayer, b: ForwardBatch, state):
         proj = ops.linear(z, lw.in_proj)

@@ -3,7 +3,8 @@ csrc/latent_attention.cu; PyTorch restatements here for CPU tensors).
 
 A layer runs  append  (norms of the query / key latents, rotation of the shared key part, page write) ->
 absorb  (q_h W_uk[h] and the query's rotated part: queries of the width of a cache row) -> attend  (softmax over the
-visible rows, result in latent space) -> values  (W_uv[h] and the output gate).
+visible rows, result in latent space) -> values  (W_uv[h] and the output gate).  Long prompt portions take the expanded
+form instead (csrc/latent_prefill.cu): keys and values of every head are materialised once for the whole portion.
 """
 from __future__ import annotations
 
@@ -21,6 +22,9 @@ _SIGS = {
     "sllm_head_matmul": (I, [P, L, I, P, P, L, I, I, I, I, I, P, L, I, P, P, I, I, I, P]),
     "sllm_latent_decode_workspace_floats": (L, [I, I, I, I]),
     "sllm_latent_decode": (I, [P, P, L, I, I, I, P, P, P, I, I, I, I, I, F, P, I, P, L, P, P]),
+    "sllm_latent_gather": (I, [P, I, I, P, I, P, I, I, P, P, I, I, I, P]),
+    "sllm_latent_pack_q": (I, [P, L, P, I, I, I, I, I, I, P, P, I, I, P]),
+    "sllm_latent_prefill": (I, [P, I, P, P, I, P, I, I, I, I, I, I, F, P, L, P, P, P]),
     "sllm_latent_attention": (I, [P, P, I, I, I, P, P, P, I, I, I, I, I, F, P, I, P]),
 }
 
@@ -181,8 +185,9 @@ def attend(qa: torch.Tensor, spec: LatentSpec, kv: LatentPages, block_table, seq
     return out
 
 
-def values(o: torch.Tensor, spec: LatentSpec, uvt: torch.Tensor, gate: Optional[torch.Tensor]) -> torch.Tensor:
-    """o [T, heads, kv_rank], uvt [heads, kv_rank, vdim], gate [T, heads] logits or None -> [T, heads * vdim]."""
+def values(o: torch.Tensor, spec: LatentSpec, uvt: torch.Tensor, gate: Optional[torch.Tensor],
+           out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """o [T, heads, kv_rank], uvt [heads, kv_rank, vdim], gate [T, heads] logits or None -> [T, heads * vdim] (``out``)."""
     t, h = o.shape[0], spec.heads
     if _lib.on_cpu(o):
         y = torch.einsum("thc,hcv->thv", o.float(), uvt.float())
@@ -190,9 +195,133 @@ def values(o: torch.Tensor, spec: LatentSpec, uvt: torch.Tensor, gate: Optional[
             y = y * torch.sigmoid(gate.float()).unsqueeze(-1)
         return y.reshape(t, h * spec.vdim).to(o.dtype)
     from .core import _p, _stream
-    out = torch.empty((t, h * spec.vdim), dtype=o.dtype, device=o.device)
+    if out is None:
+        out = torch.empty((t, h * spec.vdim), dtype=o.dtype, device=o.device)
     rc = _k().sllm_head_matmul(_p(o), h * spec.kv_rank, spec.kv_rank, _p(uvt), _p(out), h * spec.vdim, spec.vdim, t, h, spec.kv_rank,
                                spec.vdim, _p(gate), gate.stride(0) if gate is not None else 0, 0, None, None, 0, 0,
                                int(o.dtype == torch.float32), _stream())
     _lib.check(rc, "latent_values")
+    return out
+
+
+# ------------------------------------------------------------------------------------------ expanded form (prompts)
+EXPAND_MIN_ROWS = 64           # a sequence with at least this many rows in the batch takes the expanded form
+EXPAND_MAX_CONTEXT = 1 << 16   # context rows expanded at a time (one sequence may exceed it)
+TILE = 128
+
+
+def expandable(spec: LatentSpec, dtype) -> bool:
+    """Whether csrc/latent_prefill.cu takes this layer's sizes."""
+    nq = (spec.dim + 63) // 64 + (spec.rot_dim + 63) // 64
+    return (dtype == torch.bfloat16 and spec.dim % 8 == 0 and spec.vdim % 8 == 0 and spec.kv_rank % 8 == 0 and nq <= 3
+            and spec.vdim <= 128)
+
+
+@dataclass
+class Portion:
+    """Consecutive rows of a batch that take one form; ``spans`` / ``tiles`` are set for the expanded one."""
+    lo: int
+    hi: int
+    spans: Optional[torch.Tensor] = None     # int32 [sequences, 4]: table row, first position, context rows, gathered row
+    tiles: Optional[torch.Tensor] = None     # int32 [tiles, 8], rows relative to ``lo``
+    context: int = 0
+    longest: int = 0
+
+
+def plan_portions(row_off: list, starts: list, window: int, device) -> list:
+    """Splits a flat batch into runs of sequences with few rows (absorbed form) and with many (expanded form)."""
+    out: list = []
+    run: list = []
+
+    def flush():
+        nonlocal run
+        if not run:
+            return
+        lo, spans, tiles, rows = row_off[run[0]], [], [], 0
+        for s in run:
+            n, st = row_off[s + 1] - row_off[s], starts[s]
+            k_lo = max(0, st - window + 1) if window else 0
+            ctx = st + n - k_lo
+            spans.append((s, k_lo, ctx, rows))
+            for q0 in range(0, n, TILE):
+                tiles.append((row_off[s] - lo + q0, min(TILE, n - q0), st + q0, rows, k_lo, 0, 0, 0))
+            rows += ctx
+        tiles.sort(key=lambda t: -(t[2] - t[4]))         # most keys first
+        out.append(Portion(lo, row_off[run[-1] + 1], torch.tensor(spans, dtype=torch.int32, device=device),
+                           torch.tensor(tiles, dtype=torch.int32, device=device), rows, max(x[2] for x in spans)))
+        run = []
+
+    ctx_run = 0
+    for s in range(len(row_off) - 1):
+        n = row_off[s + 1] - row_off[s]
+        if n >= EXPAND_MIN_ROWS:
+            ctx = starts[s] + n
+            if run and ctx_run + ctx > EXPAND_MAX_CONTEXT:
+                flush()
+            ctx_run = ctx if not run else ctx_run + ctx
+            run.append(s)
+            continue
+        flush()
+        if n == 0:
+            continue
+        if out and out[-1].spans is None and out[-1].hi == row_off[s]:
+            out[-1].hi = row_off[s + 1]
+        else:
+            out.append(Portion(row_off[s], row_off[s + 1]))
+    flush()
+    return out
+
+
+def attend_expanded(q: torch.Tensor, spec: LatentSpec, expand, inv_freq, kv: LatentPages, block_table, positions, gate, pt: Portion,
+                    out: torch.Tensor) -> None:
+    """Rows [pt.lo, pt.hi) of a batch: q [rows, heads * (dim + rot_dim)], ``expand`` LinearWeight [heads * (dim + vdim),
+    kv_rank] (all heads' W_uk, then all heads' W_uv); writes out [rows, heads * vdim]."""
+    from .core import _p, _stream, linear, workspace
+    t, h = q.shape[0], spec.heads
+    dp, rp = (spec.dim + 63) // 64 * 64, (spec.rot_dim + 63) // 64 * 64
+    dev = q.device
+    c = torch.empty((pt.context, spec.kv_rank), dtype=q.dtype, device=dev)
+    r = torch.empty((pt.context, max(rp, 64)), dtype=q.dtype, device=dev)
+    k = _k()
+    rc = k.sllm_latent_gather(_p(kv.pages), kv.pages.shape[2], kv.page_size, _p(block_table), block_table.stride(0), _p(pt.spans),
+                              pt.spans.shape[0], pt.longest, _p(c), _p(r), spec.kv_rank, spec.rot_dim, r.shape[1], _stream())
+    _lib.check(rc, "latent_gather")
+    exp = linear(c, expand)
+    qp = torch.empty((t, h, dp + rp), dtype=q.dtype, device=dev)
+    rc = k.sllm_latent_pack_q(_p(q), q.stride(0), _p(qp), t, h, spec.dim, spec.rot_dim, dp, rp, _p(positions), _p(inv_freq),
+                              spec.rot_dims, int(spec.interleaved), _stream())
+    _lib.check(rc, "latent_pack_q")
+    if _lib.audit_enabled():
+        _lib.record_dispatch("latent_attention", "latent_prefill_kernel", rows=t, heads=h, context=pt.context, window=spec.window,
+                             grid=[pt.tiles.shape[0], h])
+    rc = k.sllm_latent_prefill(_p(qp), t, _p(exp), _p(r), pt.context, _p(pt.tiles), pt.tiles.shape[0], h, spec.dim, spec.rot_dim,
+                               spec.vdim, spec.window, spec.scale, _p(gate), gate.stride(0) if gate is not None else 0, _p(out),
+                               _p(workspace(dev).status), _stream())
+    _lib.check(rc, "latent_prefill")
+
+
+def attention(q: torch.Tensor, gate: Optional[torch.Tensor], spec: LatentSpec, uk, uvt, expand, inv_freq, kv: LatentPages, b):
+    """Attention of a ForwardBatch's rows (already appended to the pages) -> [T, heads * vdim], gated."""
+    def absorbed(lo, hi, out=None):
+        pos = b.positions[lo:hi]
+        qa = absorb(q[lo:hi], spec, uk, inv_freq, pos)
+        o = attend(qa, spec, kv, b.block_table, b.seq_index[lo:hi], b.kv_lens[lo:hi], b.max_kv)
+        return values(o, spec, uvt, None if gate is None else gate[lo:hi], out)
+
+    t = q.shape[0]
+    if b.row_off_host is None or not q.is_cuda or _lib.fake_active() or not expandable(spec, q.dtype):
+        return absorbed(0, t)
+    key = ("latent", spec.window)
+    portions = b.plans.get(key)
+    if portions is None:
+        portions = b.plans[key] = plan_portions(b.row_off_host, b.starts_host, spec.window, q.device)
+    if len(portions) == 1 and portions[0].spans is None:
+        return absorbed(0, t)
+    out = torch.empty((t, spec.heads * spec.vdim), dtype=q.dtype, device=q.device)
+    for pt in portions:
+        if pt.spans is None:
+            absorbed(pt.lo, pt.hi, out[pt.lo:pt.hi])
+        else:
+            attend_expanded(q[pt.lo:pt.hi], spec, expand, inv_freq, kv, b.block_table, b.positions[pt.lo:pt.hi],
+                            None if gate is None else gate[pt.lo:pt.hi], pt, out[pt.lo:pt.hi])
     return out
