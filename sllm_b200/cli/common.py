@@ -67,11 +67,9 @@ _KV_MAP = {"fp16": "bf16", "bf16": "bf16", "fp8": "fp8", "fp8-static": "fp8-stat
 def open_model(args, max_batch: int = 8, tp=None):
     """Returns (engine, tokenizer, gguf_file, lock).  Raises CliError with a user-facing message."""
     import torch
-    from ..cache.paged import PagedKVCache
     from ..engine.engine import Engine
     from ..formats import gguf as G
-    from ..models import loader
-    from ..models.llama import LlamaModel
+    from ..models import loader, registry
     if args.target != TARGET:
         raise CliError(f"unsupported target {args.target!r}: this build runs on {TARGET} only")
     try:
@@ -102,21 +100,13 @@ def open_model(args, max_batch: int = 8, tp=None):
                   "requested": args.context_length, "recommended": cfg.max_context})
         cfg.max_context = args.context_length
     blocks = (cfg.max_context + cfg.page_size - 1) // cfg.page_size
-    if family == "moe":
-        from ..models.moe import MoeModel
-        model = MoeModel(cfg, weights, tp, ep)
-        cache = PagedKVCache(cfg, max_batch * blocks + 8, device, kv_heads=model.local_kv_heads)
-    elif family == "qwen35":
-        from ..cache.hybrid import HybridCache
-        from ..models.qwen35 import Qwen35Model
-        model = Qwen35Model(cfg, weights, tp, ep)
-        cache = HybridCache(cfg, max_batch * blocks + 8, device, max_seqs=2 * max_batch + 2, kv_heads=model.local_kv_heads,
-                            tp_size=tp_size)
-    else:
-        model = LlamaModel(cfg, weights, tp)
-        cache = PagedKVCache(cfg, max_batch * blocks + 8, device, kv_heads=model.local_kv_heads)
+    try:
+        model = registry.make_model(cfg, weights, tp, ep)
+        cache = registry.make_cache(cfg, model, max_batch * blocks + 8, device, max_seqs=2 * max_batch + 2)
+    except ValueError as exc:
+        raise CliError(f"model load failed: {exc}", 3) from None
     eng = Engine(cfg, model, cache, device, max_batch=max_batch, use_cuda_graphs=not use_cpu, tp=tp)
-    dense_family = family not in ("moe", "qwen35")
+    dense_family = family not in ("moe", "qwen35", "zokuvik")
     eng.mtp_weights = loader.load_mtp_gguf(g, cfg, device) if tp_size == 1 and dense_family else None
     vis = loader.load_vision_gguf(g, cfg, device) if dense_family else None
     if vis is not None:

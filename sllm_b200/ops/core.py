@@ -193,7 +193,7 @@ def linear(x, w: LinearWeight, residual: Optional[torch.Tensor] = None, act: Opt
         return y.to(residual.dtype if residual is not None else (torch.float32 if w.w.dtype == torch.float32 else torch.bfloat16))
     m = xd.shape[0]
     n = w.out_features
-    if w.kind == "dense" and (w.w.dtype == torch.float32 or w.in_features % 8):
+    if w.kind == "dense" and (xd.dtype == torch.float32 or w.in_features % 8):
         return _linear_simt(xd, w.w, residual, act)
     if w.kind == "fp8":
         if not isinstance(x, QTensor):
