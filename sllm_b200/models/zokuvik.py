@@ -344,16 +344,16 @@ def shape_from_entries(name: str, entries: list, *, width: int, vocab: int, grou
                                "norm": {"eps": eps, "groups": groups}}, name=name, max_context=max_context)
 
 
-def zokuvik_shape(layers: int = 32) -> ModelConfig:
-    """A size whose layers resemble a served model's (benchmarks, random weights): width 2560, latent attention with 20
-    heads of 128 + 64 channels and a latent of 512, every other latent layer with a 1024-token window, every fourth layer
-    full attention, the others delta rules with 20 heads of 128."""
-    att = dict(heads=20, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5)
-    kinds = [_entry("latent_attention", 9216, q_rank=1024, rot={"base": 1e6, "dims": 64}, **att),
-             _entry("latent_attention_2", 9216, rot={"base": 1e4, "dims": 64}, mask={"size": 1024}, **att)]
-    delta = _entry("general_delta", 9216, heads=20, dim=128)
+def zokuvik_shape(layers: int = 32, width: int = 2560, heads: int = 20, ff: int = 9216, window: int = 1024) -> ModelConfig:
+    """A size whose layers resemble a served model's (benchmarks, random weights): every fourth layer is latent attention
+    with heads of 128 + 64 channels and a latent of 512 - full and windowed ones in turn - the others are delta rules with
+    heads of 128."""
+    att = dict(heads=heads, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5)
+    kinds = [_entry("latent_attention", ff, q_rank=1024, rot={"base": 1e6, "dims": 64}, **att),
+             _entry("latent_attention_2", ff, rot={"base": 1e4, "dims": 64}, mask={"size": window}, **att)]
+    delta = _entry("general_delta", ff, heads=heads, dim=128)
     entries = [kinds[(i // 4) % 2] if i % 4 == 3 else delta for i in range(layers)]
-    return shape_from_entries("zokuvik", entries, width=2560, vocab=151936, groups=1)
+    return shape_from_entries("zokuvik", entries, width=width, vocab=151936, groups=1)
 
 
 def tiny_zokuvik() -> ModelConfig:
