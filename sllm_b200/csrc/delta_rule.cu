@@ -6,7 +6,7 @@
 // The batch is flat (rows of sequence s: row_off[s] .. row_off[s + 1]) and sequence s owns state slot slots[s].
 //
 // Columns of S (value channels) never meet: column j only needs p = u^T S_j, so heads are cut into column tiles.  A
-// thread keeps 16 keys x 2 columns of S in registers; kKL = 1 .. 32 lanes share a column.  Both dot products of a token
+// thread keeps 16 keys x 2 or 4 columns of S in registers; kKL = 1 .. 32 lanes share a column.  Both dot products of a token
 // are taken from the OLD state in one sweep, because
 //   o = S_t^T r = (w r)^T S_{t-1} - p (a u)^T r + v k^T r
 // so a token costs one shuffle reduction and no barrier.
@@ -24,7 +24,6 @@ namespace sllm {
 constexpr int kDrKeys = 16;          // keys per thread
 constexpr int kDrVecs = 6;           // u, w r, w, a u, k, v
 constexpr int kDrChunk = 8;          // tokens staged at a time by the scan
-constexpr int kDrScanWarps = 4;
 constexpr int kDrDecodeThreads = 256;
 constexpr float kDecayRate = 0.60653065971263342f;   // exp(-1/2)
 
@@ -33,6 +32,8 @@ __host__ __device__ constexpr int delta_pad(int dim) {   // padded head size: 16
   while (kl * kDrKeys < dim) kl *= 2;
   return kl * kDrKeys;
 }
+
+__host__ __device__ constexpr int delta_record(int pad) { return kDrVecs * pad + 4; }   // floats per (head, token)
 
 template <typename T>
 struct DeltaParams {
@@ -51,8 +52,7 @@ struct DeltaParams {
   const int* row_off;
   const int* slots;
   int heads, dim, tokens;
-  float* vec;              // [heads][tokens][6][pad]
-  float* sums;             // [heads][tokens][2]: (a u)^T r, k^T r
+  float* vec;              // [heads][tokens][6 pad + 4]: the vectors, then (a u)^T r, k^T r
   float* o_raw;            // [tokens, heads * dim]
   T* out;                  // [tokens, heads * dim]
 };
@@ -68,66 +68,114 @@ __device__ __forceinline__ float block_sum(float v, float* red, int warps) {
 }
 
 // ---------------------------------------------------------------- prompt form
-// grid (tokens, heads), block = padded head size (at least 32).
-template <typename T>
-__global__ void delta_pre_kernel(const DeltaParams<T> p) {
-  pdl_wait();
-  pdl_trigger();
-  __shared__ float red[16];
-  const int t = blockIdx.x, h = blockIdx.y, d = threadIdx.x, D = p.dim, pad = delta_pad(D), warps = blockDim.x >> 5;
-  const bool in = d < D;
-  const int c = h * D + d;
-  float r = 0.f, k = 0.f, v = 0.f, w = 0.f, a = 0.f;
-  if (in) {
-    const T* row = p.proj + static_cast<size_t>(t) * p.ldp;
-    r = ld_f(row + p.off_r + c);
-    k = ld_f(row + p.off_k + c);
-    v = ld_f(row + p.off_v + c);
-    a = sigmoid_f(ld_f(row + p.off_a + c) + p.a_bias[c]);
-    w = expf(-kDecayRate * sigmoid_f(ld_f(p.decay + static_cast<size_t>(t) * p.ld_decay + c) + p.w0[c]));
+// A warp per (token, head), lane l the channels l kN .. l kN + kN - 1 (kN = padded head size / 32, at least 1); vec: heads
+// and offsets allow 4-channel accesses.
+template <typename T, int kN>
+__device__ __forceinline__ void lane_load(const T* src, int d0, int dim, bool vec, float (&v)[kN]) {
+  if constexpr (kN % 4 == 0) {
+    if (vec) {
+#pragma unroll
+      for (int i = 0; i < kN; i += 4) {
+        float x[4] = {0.f, 0.f, 0.f, 0.f};
+        if (d0 + i < dim) ld_vec<4>(src + d0 + i, x);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) v[i + j] = x[j];
+      }
+      return;
+    }
   }
-  const float kk = block_sum(k * k, red, warps);
-  const float u = k / sqrtf(kk + p.eps_u);
-  const float s1 = block_sum(a * u * r, red, warps);
-  const float s2 = block_sum(k * r, red, warps);
-  const size_t ht = static_cast<size_t>(h) * p.tokens + t;
-  if (d < pad) {
-    float* dst = p.vec + ht * kDrVecs * pad + d;
-    dst[0] = u; dst[pad] = w * r; dst[2 * pad] = w; dst[3 * pad] = a * u; dst[4 * pad] = k; dst[5 * pad] = v;
-  }
-  if (d == 0) {
-    p.sums[ht * 2] = s1;
-    p.sums[ht * 2 + 1] = s2;
-  }
+#pragma unroll
+  for (int i = 0; i < kN; ++i) v[i] = d0 + i < dim ? ld_f(src + d0 + i) : 0.f;
 }
 
-// One token on a thread's 16 keys x 2 columns: S is updated, o[2] holds the outputs on every lane of the column.
+constexpr int kDrRowWarps = 8;       // (token, head) pairs per CTA of the row kernels
+
+// No early trigger of the dependent launch here: the scan's few CTAs would become resident while this grid drains, several
+// of them on the first SMs that run empty, and share those SMs' shared-memory bandwidth for their whole run.
+template <typename T, int kN>
+__global__ void __launch_bounds__(kDrRowWarps * 32) delta_pre_kernel(const DeltaParams<T> p, bool vec) {
+  pdl_wait();
+  const int lane = threadIdx.x & 31, D = p.dim, pad = delta_pad(D), d0 = lane * kN;
+  const long long unit = static_cast<long long>(blockIdx.x) * kDrRowWarps + (threadIdx.x >> 5);
+  if (unit >= static_cast<long long>(p.tokens) * p.heads) return;
+  const int t = static_cast<int>(unit / p.heads), h = static_cast<int>(unit % p.heads);
+  const T* row = p.proj + static_cast<size_t>(t) * p.ldp + h * D;
+  float r[kN], k[kN], v[kN], a[kN], w[kN], b0[kN], b1[kN];
+  lane_load<T, kN>(row + p.off_r, d0, D, vec, r);
+  lane_load<T, kN>(row + p.off_k, d0, D, vec, k);
+  lane_load<T, kN>(row + p.off_v, d0, D, vec, v);
+  lane_load<T, kN>(row + p.off_a, d0, D, vec, a);
+  lane_load<T, kN>(p.decay + static_cast<size_t>(t) * p.ld_decay + h * D, d0, D, vec, w);
+  lane_load<float, kN>(p.w0 + h * D, d0, D, vec, b0);
+  lane_load<float, kN>(p.a_bias + h * D, d0, D, vec, b1);
+  float kk = 0.f, s1 = 0.f, s2 = 0.f;
+#pragma unroll
+  for (int i = 0; i < kN; ++i) kk += k[i] * k[i];
+  const float inv = 1.f / sqrtf(warp_sum(kk) + p.eps_u);
+  float u[kN];
+#pragma unroll
+  for (int i = 0; i < kN; ++i) {
+    const bool in = d0 + i < D;
+    w[i] = in ? expf(-kDecayRate * sigmoid_f(w[i] + b0[i])) : 0.f;
+    u[i] = k[i] * inv;
+    a[i] = in ? sigmoid_f(a[i] + b1[i]) * u[i] : 0.f;
+    s1 += a[i] * r[i];
+    s2 += k[i] * r[i];
+    r[i] *= w[i];
+  }
+  s1 = warp_sum(s1);
+  s2 = warp_sum(s2);
+  float* dst = p.vec + (static_cast<size_t>(h) * p.tokens + t) * delta_record(pad) + d0;
+  auto put = [&](int which, const float (&x)[kN]) {
+    if constexpr (kN % 4 == 0) {
+#pragma unroll
+      for (int i = 0; i < kN; i += 4)
+        *reinterpret_cast<float4*>(dst + which * pad + i) = make_float4(x[i], x[i + 1], x[i + 2], x[i + 3]);
+    } else {
+#pragma unroll
+      for (int i = 0; i < kN; ++i)
+        if (d0 + i < pad) dst[which * pad + i] = x[i];
+    }
+  };
+  put(0, u); put(1, r); put(2, w); put(3, a); put(4, k); put(5, v);
+  if (lane == 0) *reinterpret_cast<float2*>(dst + kDrVecs * pad) = make_float2(s1, s2);
+}
+
+// One token on a thread's 16 keys x kC columns: S is updated, o holds the outputs on every lane of the columns.
 // vs: the token's [6][pad] vectors in shared memory.  Key of S[j * 4 + e]: (j * kKL + kl) * 4 + e.
-template <int kKL>
-__device__ __forceinline__ void delta_token(float (&S)[kDrKeys][2], const float* vs, int kl, const float (&v)[2], float s1, float s2,
-                                            float (&o)[2]) {
+template <int kKL, int kC>
+__device__ __forceinline__ void delta_token(float (&S)[kDrKeys][kC], const float* vs, int kl, const float (&v)[kC], float s1, float s2,
+                                            float (&o)[kC]) {
   constexpr int pad = kKL * kDrKeys;
-  float p0 = 0.f, p1 = 0.f, q0 = 0.f, q1 = 0.f;
+  float pc[2][kC], qc[2][kC];                        // two chains per column
+#pragma unroll
+  for (int c = 0; c < kC; ++c) pc[0][c] = pc[1][c] = qc[0][c] = qc[1][c] = 0.f;
 #pragma unroll
   for (int j = 0; j < kDrKeys / 4; ++j) {
     const float4 u = *reinterpret_cast<const float4*>(vs + (j * kKL + kl) * 4);
     const float4 wr = *reinterpret_cast<const float4*>(vs + pad + (j * kKL + kl) * 4);
     const float ua[4] = {u.x, u.y, u.z, u.w}, wa[4] = {wr.x, wr.y, wr.z, wr.w};
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      p0 = fmaf(ua[e], S[j * 4 + e][0], p0);
-      p1 = fmaf(ua[e], S[j * 4 + e][1], p1);
-      q0 = fmaf(wa[e], S[j * 4 + e][0], q0);
-      q1 = fmaf(wa[e], S[j * 4 + e][1], q1);
-    }
+    for (int e = 0; e < 4; ++e)
+#pragma unroll
+      for (int c = 0; c < kC; ++c) {
+        pc[e & 1][c] = fmaf(ua[e], S[j * 4 + e][c], pc[e & 1][c]);
+        qc[e & 1][c] = fmaf(wa[e], S[j * 4 + e][c], qc[e & 1][c]);
+      }
+  }
+  float p[kC], q[kC];
+#pragma unroll
+  for (int c = 0; c < kC; ++c) {
+    p[c] = pc[0][c] + pc[1][c];
+    q[c] = qc[0][c] + qc[1][c];
   }
 #pragma unroll
-  for (int x = kKL / 2; x > 0; x >>= 1) {
-    p0 += __shfl_xor_sync(0xffffffffu, p0, x);
-    p1 += __shfl_xor_sync(0xffffffffu, p1, x);
-    q0 += __shfl_xor_sync(0xffffffffu, q0, x);
-    q1 += __shfl_xor_sync(0xffffffffu, q1, x);
-  }
+  for (int x = kKL / 2; x > 0; x >>= 1)
+#pragma unroll
+    for (int c = 0; c < kC; ++c) {
+      p[c] += __shfl_xor_sync(0xffffffffu, p[c], x);
+      q[c] += __shfl_xor_sync(0xffffffffu, q[c], x);
+    }
 #pragma unroll
   for (int j = 0; j < kDrKeys / 4; ++j) {
     const float4 w = *reinterpret_cast<const float4*>(vs + 2 * pad + (j * kKL + kl) * 4);
@@ -135,45 +183,43 @@ __device__ __forceinline__ void delta_token(float (&S)[kDrKeys][2], const float*
     const float4 k = *reinterpret_cast<const float4*>(vs + 4 * pad + (j * kKL + kl) * 4);
     const float wa[4] = {w.x, w.y, w.z, w.w}, aa[4] = {au.x, au.y, au.z, au.w}, ka[4] = {k.x, k.y, k.z, k.w};
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      S[j * 4 + e][0] = fmaf(ka[e], v[0], fmaf(-aa[e], p0, wa[e] * S[j * 4 + e][0]));
-      S[j * 4 + e][1] = fmaf(ka[e], v[1], fmaf(-aa[e], p1, wa[e] * S[j * 4 + e][1]));
-    }
+    for (int e = 0; e < 4; ++e)
+#pragma unroll
+      for (int c = 0; c < kC; ++c) S[j * 4 + e][c] = fmaf(ka[e], v[c], fmaf(-aa[e], p[c], wa[e] * S[j * 4 + e][c]));
   }
-  o[0] = q0 - p0 * s1 + v[0] * s2;
-  o[1] = q1 - p1 * s1 + v[1] * s2;
+#pragma unroll
+  for (int c = 0; c < kC; ++c) o[c] = q[c] - p[c] * s1 + v[c] * s2;
 }
 
-template <int kKL, bool kStore>
-__device__ __forceinline__ void delta_state_io(float (&S)[kDrKeys][2], float* st, int dim, int kl, int col) {
-  const bool pair = (dim & 1) == 0;                  // col is even: two columns are one aligned 8-byte access
+template <int kKL, int kC, bool kStore>
+__device__ __forceinline__ void delta_state_io(float (&S)[kDrKeys][kC], float* st, int dim, int kl, int col) {
+  const bool whole = dim % kC == 0;                  // col is a multiple of kC: its columns are one aligned access
 #pragma unroll
   for (int j = 0; j < kDrKeys / 4; ++j)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int key = (j * kKL + kl) * 4 + e;
       float* ptr = st + static_cast<size_t>(key) * dim + col;
+      float(&x)[kC] = S[j * 4 + e];
+      const bool in = key < dim && col < dim;
       if constexpr (kStore) {
-        if (key < dim && col < dim) {
-          if (pair) {
-            *reinterpret_cast<float2*>(ptr) = make_float2(S[j * 4 + e][0], S[j * 4 + e][1]);
-          } else {
-            ptr[0] = S[j * 4 + e][0];
-            if (col + 1 < dim) ptr[1] = S[j * 4 + e][1];
-          }
+        if (in && whole) {
+          st_vec<kC>(ptr, x);
+        } else if (in) {
+#pragma unroll
+          for (int c = 0; c < kC; ++c)
+            if (col + c < dim) ptr[c] = x[c];
         }
       } else {
-        float2 x = make_float2(0.f, 0.f);
-        if (key < dim && col < dim) {
-          if (pair) {
-            x = *reinterpret_cast<const float2*>(ptr);
-          } else {
-            x.x = ptr[0];
-            if (col + 1 < dim) x.y = ptr[1];
-          }
+#pragma unroll
+        for (int c = 0; c < kC; ++c) x[c] = 0.f;
+        if (in && whole) {
+          ld_vec<kC>(ptr, x);
+        } else if (in) {
+#pragma unroll
+          for (int c = 0; c < kC; ++c)
+            if (col + c < dim) x[c] = ptr[c];
         }
-        S[j * 4 + e][0] = x.x;
-        S[j * 4 + e][1] = x.y;
       }
     }
 }
@@ -182,24 +228,24 @@ __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
 
-// grid (heads, column tiles, sequences), 4 warps of (32 / kKL) column pairs.
-template <typename T, int kKL>
+constexpr int kDrScanWarps = 4;
+
+// grid (heads, column tiles, sequences), 4 warps of (32 / kKL) groups of kC columns.
+template <typename T, int kKL, int kC>
 __global__ void __launch_bounds__(kDrScanWarps * 32) delta_scan_kernel(const DeltaParams<T> p) {
   pdl_wait();
-  pdl_trigger();
   constexpr int pad = kKL * kDrKeys;
-  constexpr int kTok = kDrVecs * pad;                // floats per token
+  constexpr int kTok = delta_record(pad);
   extern __shared__ __align__(16) float buf[];       // [2][kDrChunk][kTok]
   const int h = blockIdx.x, s = blockIdx.z, D = p.dim;
   const int r0 = p.row_off[s], r1 = p.row_off[s + 1];
   if (r1 <= r0) return;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kl = lane % kKL;
-  const int col = ((blockIdx.y * kDrScanWarps + warp) * (32 / kKL) + lane / kKL) * 2;
+  const int col = ((blockIdx.y * kDrScanWarps + warp) * (32 / kKL) + lane / kKL) * kC;
   float* st = p.state + static_cast<long long>(p.slots[s]) * p.slot_stride + static_cast<size_t>(h) * D * D;
-  float S[kDrKeys][2];
-  delta_state_io<kKL, false>(S, st, D, kl, col);
+  float S[kDrKeys][kC];
+  delta_state_io<kKL, kC, false>(S, st, D, kl, col);
   const float* vec = p.vec + static_cast<size_t>(h) * p.tokens * kTok;
-  const float* sums = p.sums + static_cast<size_t>(h) * p.tokens * 2;
   auto stage = [&](int c0, int b) {
     const int n = min(kDrChunk, r1 - c0) * (kTok / 4);
     for (int e = threadIdx.x; e < n; e += kDrScanWarps * 32)
@@ -215,36 +261,58 @@ __global__ void __launch_bounds__(kDrScanWarps * 32) delta_scan_kernel(const Del
     const int n = min(kDrChunk, r1 - c0);
     for (int i = 0; i < n; ++i) {
       const float* vs = buf + (b * kDrChunk + i) * kTok;
-      const float2 s12 = *reinterpret_cast<const float2*>(sums + static_cast<size_t>(c0 + i) * 2);
-      float v[2] = {0.f, 0.f}, o[2];
-      if (col < pad) { v[0] = vs[5 * pad + col]; v[1] = vs[5 * pad + col + 1]; }
-      delta_token<kKL>(S, vs, kl, v, s12.x, s12.y, o);
+      const float2 s12 = *reinterpret_cast<const float2*>(vs + kDrVecs * pad);
+      float v[kC], o[kC];
+#pragma unroll
+      for (int c = 0; c < kC; ++c) v[c] = col < pad ? vs[5 * pad + col + c] : 0.f;
+      delta_token<kKL, kC>(S, vs, kl, v, s12.x, s12.y, o);
       if (kl == 0) {
         float* dst = p.o_raw + static_cast<size_t>(c0 + i) * p.heads * D + h * D + col;
-        if (col < D) dst[0] = o[0];
-        if (col + 1 < D) dst[1] = o[1];
+#pragma unroll
+        for (int c = 0; c < kC; ++c)
+          if (col + c < D) dst[c] = o[c];
       }
     }
     __syncthreads();                                 // the buffer is refilled by the next iteration's stage()
   }
-  delta_state_io<kKL, true>(S, st, D, kl, col);
+  pdl_trigger();
+  delta_state_io<kKL, kC, true>(S, st, D, kl, col);
 }
 
-// grid (tokens, heads), block = padded head size (at least 32).
-template <typename T>
-__global__ void delta_post_kernel(const DeltaParams<T> p) {
+// A warp per (token, head), as in the first stage.
+template <typename T, int kN>
+__global__ void __launch_bounds__(kDrRowWarps * 32) delta_post_kernel(const DeltaParams<T> p, bool vec) {
   pdl_wait();
   pdl_trigger();
-  __shared__ float red[16];
-  const int t = blockIdx.x, h = blockIdx.y, d = threadIdx.x, D = p.dim, warps = blockDim.x >> 5;
-  const int c = h * D + d;
-  const size_t idx = static_cast<size_t>(t) * p.heads * D + c;
-  const float o = d < D ? p.o_raw[idx] : 0.f;
-  const float ss = block_sum(o * o, red, warps);
-  if (d < D) {
-    const float g = ld_f(p.proj + static_cast<size_t>(t) * p.ldp + p.off_g + c);
-    st_f(p.out + idx, o * (1.f / sqrtf(ss / static_cast<float>(D) + p.eps)) * p.norm_w[c] * sigmoid_f(g));
+  const int lane = threadIdx.x & 31, D = p.dim, d0 = lane * kN;
+  const long long unit = static_cast<long long>(blockIdx.x) * kDrRowWarps + (threadIdx.x >> 5);
+  if (unit >= static_cast<long long>(p.tokens) * p.heads) return;
+  const int t = static_cast<int>(unit / p.heads), h = static_cast<int>(unit % p.heads);
+  const size_t idx = static_cast<size_t>(t) * p.heads * D + h * D;
+  float o[kN], g[kN], w[kN];
+  lane_load<float, kN>(p.o_raw + idx, d0, D, vec, o);
+  lane_load<T, kN>(p.proj + static_cast<size_t>(t) * p.ldp + p.off_g + h * D, d0, D, vec, g);
+  lane_load<float, kN>(p.norm_w + h * D, d0, D, vec, w);
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < kN; ++i) ss += o[i] * o[i];
+  const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(D) + p.eps);
+#pragma unroll
+  for (int i = 0; i < kN; ++i) o[i] = o[i] * inv * w[i] * sigmoid_f(g[i]);
+  T* dst = p.out + idx + d0;
+  if constexpr (kN % 4 == 0) {
+    if (vec) {
+#pragma unroll
+      for (int i = 0; i < kN; i += 4) {
+        const float x[4] = {o[i], o[i + 1], o[i + 2], o[i + 3]};
+        if (d0 + i < D) st_vec<4>(dst + i, x);
+      }
+      return;
+    }
   }
+#pragma unroll
+  for (int i = 0; i < kN; ++i)
+    if (d0 + i < D) st_f(dst + i, o[i]);
 }
 
 // ---------------------------------------------------------------- decode form: exactly one row per sequence
@@ -267,7 +335,7 @@ __global__ void __launch_bounds__(kDrDecodeThreads) delta_decode_kernel(const De
   // the first tile of the state is requested before anything is computed
   int col = (warp * (32 / kKL) + lane / kKL) * 2;
   float S[kDrKeys][2];
-  delta_state_io<kKL, false>(S, st, D, kl, col);
+  delta_state_io<kKL, 2, false>(S, st, D, kl, col);
   for (int i = threadIdx.x; i < p.rank; i += kDrDecodeThreads) low[i] = tanhf(ld_f(row + p.off_w1 + i));
   __syncthreads();
   float kk = 0.f, kr = 0.f;
@@ -313,12 +381,12 @@ __global__ void __launch_bounds__(kDrDecodeThreads) delta_decode_kernel(const De
   for (int base = 0; base < D; base += kSweep) {
     if (base > 0) {
       col += kSweep;
-      delta_state_io<kKL, false>(S, st, D, kl, col);
+      delta_state_io<kKL, 2, false>(S, st, D, kl, col);
     }
     float v[2] = {0.f, 0.f}, o[2];
     if (col < pad) { v[0] = vs[5 * pad + col]; v[1] = vs[5 * pad + col + 1]; }
-    delta_token<kKL>(S, vs, kl, v, s1, s2, o);
-    delta_state_io<kKL, true>(S, st, D, kl, col);
+    delta_token<kKL, 2>(S, vs, kl, v, s1, s2, o);
+    delta_state_io<kKL, 2, true>(S, st, D, kl, col);
     if (kl == 0 && col < pad) { o_s[col] = o[0]; o_s[col + 1] = o[1]; }
   }
   __syncthreads();
@@ -342,24 +410,55 @@ __global__ void tanh_rows_kernel(const T* __restrict__ x, T* __restrict__ y, int
     st_f(y + static_cast<size_t>(t) * n_pad + i, i < n ? tanhf(ld_f(x + static_cast<size_t>(t) * ldx + i)) : 0.f);
 }
 
+template <typename T, int kKL, int kC>
+static int delta_scan_launch_c(const DeltaParams<T>& p, int sequences, cudaStream_t st) {
+  constexpr int cols = kDrScanWarps * (32 / kKL) * kC;
+  const dim3 grid(p.heads, (p.dim + cols - 1) / cols, sequences);
+  size_t smem = sizeof(float) * 2 * kDrChunk * delta_record(kKL * kDrKeys);
+  // a grid that fits one CTA per SM asks for more than half of an SM's shared memory, so that no two share one
+  if (static_cast<long long>(grid.x) * grid.y * grid.z <= 148 && smem < 116 * 1024) smem = 116 * 1024;
+  static size_t configured = 0;
+  if (smem > 48 * 1024 && smem > configured) {
+    if (cudaFuncSetAttribute(delta_scan_kernel<T, kKL, kC>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) !=
+        cudaSuccess)
+      return SLLM_ERR_CUDA;
+    configured = smem;
+  }
+  return launch_kernel(delta_scan_kernel<T, kKL, kC>, grid, dim3(kDrScanWarps * 32), smem, st, 1u, p) == cudaSuccess ? SLLM_OK
+                                                                                                                     : SLLM_ERR_CUDA;
+}
+
+// The scan is bound by its reads of the staged vectors: more columns per thread reuse them more often, fewer spread a small
+// batch over more SMs.
 template <typename T, int kKL>
 static int delta_scan_launch(const DeltaParams<T>& p, int sequences, cudaStream_t st) {
-  constexpr size_t smem = sizeof(float) * 2 * kDrChunk * kDrVecs * kKL * kDrKeys;
-  static bool cfg = false;
-  if (!cfg && smem > 48 * 1024) {
-    if (cudaFuncSetAttribute(delta_scan_kernel<T, kKL>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) != cudaSuccess)
-      return SLLM_ERR_CUDA;
-    cfg = true;
-  }
   constexpr int cols = kDrScanWarps * (32 / kKL) * 2;
-  return launch_kernel(delta_scan_kernel<T, kKL>, dim3(p.heads, (p.dim + cols - 1) / cols, sequences), dim3(kDrScanWarps * 32), smem,
-                       st, 1u, p) == cudaSuccess ? SLLM_OK : SLLM_ERR_CUDA;
+  if (static_cast<long long>(p.heads) * ((p.dim + cols - 1) / cols) * sequences > 148) return delta_scan_launch_c<T, kKL, 4>(p, sequences, st);
+  return delta_scan_launch_c<T, kKL, 2>(p, sequences, st);
+}
+
+template <typename T, int kN>
+static cudaError_t delta_rows_launch(const DeltaParams<T>& p, bool pre, bool vec, cudaStream_t st) {
+  const long long units = static_cast<long long>(p.tokens) * p.heads;
+  const dim3 grid(static_cast<unsigned>((units + kDrRowWarps - 1) / kDrRowWarps));
+  return launch_kernel(pre ? delta_pre_kernel<T, kN> : delta_post_kernel<T, kN>, grid, dim3(kDrRowWarps * 32), 0, st, 1u, p, vec);
+}
+template <typename T>
+static cudaError_t delta_rows(const DeltaParams<T>& p, int pad, bool pre, cudaStream_t st) {
+  const bool vec = ((p.dim | p.ldp | p.off_r | p.off_k | p.off_v | p.off_a | p.off_g | p.ld_decay) & 3) == 0;
+  switch (pad / 32) {
+    case 0: case 1: return delta_rows_launch<T, 1>(p, pre, vec, st);
+    case 2: return delta_rows_launch<T, 2>(p, pre, vec, st);
+    case 4: return delta_rows_launch<T, 4>(p, pre, vec, st);
+    case 8: return delta_rows_launch<T, 8>(p, pre, vec, st);
+    default: return delta_rows_launch<T, 16>(p, pre, vec, st);
+  }
 }
 
 template <typename T>
 static int delta_prompt_launch(DeltaParams<T> p, int sequences, cudaStream_t st) {
-  const int pad = delta_pad(p.dim), block = pad < 32 ? 32 : pad;
-  if (launch_kernel(delta_pre_kernel<T>, dim3(p.tokens, p.heads), dim3(block), 0, st, 1u, p) != cudaSuccess) return SLLM_ERR_CUDA;
+  const int pad = delta_pad(p.dim);
+  if (delta_rows<T>(p, pad, true, st) != cudaSuccess) return SLLM_ERR_CUDA;
   int rc;
   switch (pad / kDrKeys) {
     case 1: rc = delta_scan_launch<T, 1>(p, sequences, st); break;
@@ -370,8 +469,7 @@ static int delta_prompt_launch(DeltaParams<T> p, int sequences, cudaStream_t st)
     default: rc = delta_scan_launch<T, 32>(p, sequences, st); break;
   }
   if (rc != SLLM_OK) return rc;
-  return launch_kernel(delta_post_kernel<T>, dim3(p.tokens, p.heads), dim3(block), 0, st, 1u, p) == cudaSuccess ? SLLM_OK
-                                                                                                              : SLLM_ERR_CUDA;
+  return delta_rows<T>(p, pad, false, st) == cudaSuccess ? SLLM_OK : SLLM_ERR_CUDA;
 }
 
 template <typename T>
@@ -404,7 +502,7 @@ struct SllmDeltaArgs {     // host-side mirror passed by the Python layer (ctype
   float* state;
   const int* row_off;
   const int* slots;
-  float* scratch;          // prompt form: heads * tokens * (6 * pad + 2) + tokens * heads * dim floats, 16-byte aligned
+  float* scratch;          // prompt form: heads * tokens * (6 * pad + 4) + tokens * heads * dim floats, 16-byte aligned
   void* out;
   long long slot_stride, scratch_floats;
   int ldp, off_r, off_k, off_v, off_a, off_g, off_w1, rank, ld_decay, ld_w2, heads, dim, tokens, sequences, fp32, decode;
@@ -418,13 +516,13 @@ SLLM_EXPORT int sllm_general_delta(const SllmDeltaArgs* a, void* stream) {
     return SLLM_ERR_INVALID_ARGUMENT;
   if (a->dim > 512) return SLLM_ERR_UNSUPPORTED_SHAPE;
   const int pad = delta_pad(a->dim);
-  const long long nv = static_cast<long long>(a->heads) * a->tokens * kDrVecs * pad, ns = static_cast<long long>(a->heads) * a->tokens * 2;
+  const long long nv = static_cast<long long>(a->heads) * a->tokens * delta_record(pad);
   const long long no = static_cast<long long>(a->tokens) * a->heads * a->dim;
   if (a->decode) {
     if (!a->w2 || a->rank <= 0 || a->ld_w2 < a->rank || a->rank > 8192) return SLLM_ERR_INVALID_ARGUMENT;
   } else {
     if (!a->decay || !a->scratch) return SLLM_ERR_INVALID_ARGUMENT;
-    if (a->scratch_floats < nv + ns + no) return SLLM_ERR_WORKSPACE_TOO_SMALL;
+    if (a->scratch_floats < nv + no) return SLLM_ERR_WORKSPACE_TOO_SMALL;
     if (reinterpret_cast<uintptr_t>(a->scratch) & 15) return SLLM_ERR_ALIGNMENT;
   }
   cudaStream_t st = static_cast<cudaStream_t>(stream);
@@ -438,7 +536,7 @@ SLLM_EXPORT int sllm_general_delta(const SllmDeltaArgs* a, void* stream) {
     p.eps_u = a->eps_u; p.eps = a->eps; p.state = a->state; p.slot_stride = a->slot_stride; p.row_off = a->row_off; p.slots = a->slots;
     p.heads = a->heads; p.dim = a->dim; p.tokens = a->tokens; p.out = static_cast<T*>(a->out);
     if (a->decode) return delta_decode_launch<T>(p, a->sequences, st);
-    p.vec = a->scratch; p.sums = a->scratch + nv; p.o_raw = p.sums + ns;
+    p.vec = a->scratch; p.o_raw = a->scratch + nv;
     return delta_prompt_launch<T>(p, a->sequences, st);
   };
   return a->fp32 ? run(static_cast<float*>(nullptr)) : run(static_cast<__nv_bfloat16*>(nullptr));

@@ -117,29 +117,31 @@ struct HeadMatmulParams {
   LatentRot rot;
 };
 
-constexpr int kHmRows = 8, kHmLanes = 8, kHmThreads = 256, kHmSlices = kHmThreads / kHmLanes;
+constexpr int kHmRows = 8, kHmThreads = 256;
 
-// grid (ceil(N / (8 * VEC)), heads, ceil(rows / 8)): a CTA covers 8 rows and 8 * VEC columns of one head; 32 K slices
-// of 8 lanes each read 16-byte pieces of the matrix and are summed by shuffles and through shared memory.
+// grid (ceil(N / (kLanes * VEC)), heads, ceil(rows / 8)): a CTA covers 8 rows and kLanes * VEC columns of one head; its
+// 256 / kLanes K slices read 16-byte pieces of the matrix and are summed through shared memory.
 // kAligned: N is a multiple of the 16-byte vector (and so every piece is aligned).
-template <typename T, bool kAligned>
+template <typename T, int kLanes, bool kAligned>
 __global__ void __launch_bounds__(kHmThreads) head_matmul_kernel(const HeadMatmulParams<T> p) {
   pdl_wait();
   pdl_trigger();
   constexpr int V = kVec16<T>;
-  constexpr int kCols = kHmLanes * V;
+  constexpr int kCols = kLanes * V, kSlices = kHmThreads / kLanes;
   extern __shared__ __align__(16) float sm[];
   float* in_s = sm;                                   // [K][kHmRows]
-  float* red = sm + p.k * kHmRows;                    // [8 warps][kHmRows][kCols]
+  float* red = sm + p.k * kHmRows;                    // [kSlices][kHmRows][kCols]
   const int h = blockIdx.y, r0 = blockIdx.z * kHmRows, c0 = blockIdx.x * kCols;
   const int nr = min(kHmRows, p.rows - r0);
-  for (int e = threadIdx.x; e < p.k * kHmRows; e += kHmThreads) {
-    const int r = e / p.k, k = e - r * p.k;
-    in_s[k * kHmRows + r] = r < nr ? ld_f(p.in + (r0 + r) * p.ld_in + static_cast<long long>(h) * p.hs_in + k) : 0.f;
+  {
+    // lane <-> row fastest: the transposed stores are conflict free, and a row's pieces stay in the cache
+    const int r = threadIdx.x & (kHmRows - 1);
+    const T* src = p.in + (r0 + r) * p.ld_in + static_cast<long long>(h) * p.hs_in;
+    for (int k = threadIdx.x / kHmRows; k < p.k; k += kHmThreads / kHmRows) in_s[k * kHmRows + r] = r < nr ? ld_f(src + k) : 0.f;
   }
   __syncthreads();
-  const int lane8 = threadIdx.x & 7, slice = threadIdx.x >> 3;
-  const int col = c0 + lane8 * V;
+  const int lane = threadIdx.x % kLanes, slice = threadIdx.x / kLanes;
+  const int col = c0 + lane * V;
   float acc[kHmRows][V];
 #pragma unroll
   for (int r = 0; r < kHmRows; ++r)
@@ -147,8 +149,8 @@ __global__ void __launch_bounds__(kHmThreads) head_matmul_kernel(const HeadMatmu
     for (int v = 0; v < V; ++v) acc[r][v] = 0.f;
   const T* mh = p.m + static_cast<size_t>(h) * p.k * p.n;
   if (col < p.n) {
-#pragma unroll 4
-    for (int k = slice; k < p.k; k += kHmSlices) {
+#pragma unroll 8
+    for (int k = slice; k < p.k; k += kSlices) {
       float w[V];
       const T* src = mh + static_cast<size_t>(k) * p.n + col;
       if constexpr (kAligned) {
@@ -157,27 +159,21 @@ __global__ void __launch_bounds__(kHmThreads) head_matmul_kernel(const HeadMatmu
 #pragma unroll
         for (int v = 0; v < V; ++v) w[v] = col + v < p.n ? ld_f(src + v) : 0.f;
       }
-      float x[kHmRows];
-      {
-        const float4 a = *reinterpret_cast<const float4*>(in_s + k * kHmRows);
-        const float4 b = *reinterpret_cast<const float4*>(in_s + k * kHmRows + 4);
-        x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w; x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
-      }
+      const float4 a = *reinterpret_cast<const float4*>(in_s + k * kHmRows);
+      const float4 b = *reinterpret_cast<const float4*>(in_s + k * kHmRows + 4);
+      const float x[kHmRows] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
 #pragma unroll
       for (int r = 0; r < kHmRows; ++r)
 #pragma unroll
         for (int v = 0; v < V; ++v) acc[r][v] = fmaf(x[r], w[v], acc[r][v]);
     }
   }
-  const int warp = threadIdx.x >> 5;
 #pragma unroll
   for (int r = 0; r < kHmRows; ++r)
 #pragma unroll
-    for (int v = 0; v < V; ++v) {
-      float a = acc[r][v];
-      a += __shfl_xor_sync(0xffffffffu, a, 8);
-      a += __shfl_xor_sync(0xffffffffu, a, 16);
-      if ((threadIdx.x & 31) < 8) red[(warp * kHmRows + r) * kCols + lane8 * V + v] = a;
+    for (int v = 0; v < V; v += 4) {
+      const float q[4] = {acc[r][v], acc[r][v + 1], acc[r][v + 2], acc[r][v + 3]};
+      st_vec<4>(red + (slice * kHmRows + r) * kCols + lane * V + v, q);
     }
   __syncthreads();
   for (int e = threadIdx.x; e < nr * kCols; e += kHmThreads) {
@@ -185,7 +181,7 @@ __global__ void __launch_bounds__(kHmThreads) head_matmul_kernel(const HeadMatmu
     if (c0 + c >= p.n) continue;
     float a = 0.f;
 #pragma unroll
-    for (int w = 0; w < 8; ++w) a += red[(w * kHmRows + r) * kCols + c];
+    for (int s = 0; s < kSlices; ++s) a += red[(s * kHmRows + r) * kCols + c];
     if (p.gate) a *= sigmoid_f(ld_f(p.gate + (r0 + r) * p.ld_gate + h));
     st_f(p.out + (r0 + r) * p.ld_out + static_cast<long long>(h) * p.hs_out + c0 + c, a);
   }
@@ -350,12 +346,12 @@ static int append_launch(const void* proj, int ldp, int off_q, int off_kv, int q
              ? SLLM_OK : SLLM_ERR_CUDA;
 }
 
-template <typename T>
-static int head_matmul_launch(HeadMatmulParams<T> p, int heads, cudaStream_t st) {
-  constexpr int kCols = kHmLanes * kVec16<T>;
+template <typename T, int kLanes>
+static int head_matmul_launch_l(const HeadMatmulParams<T>& p, int heads, cudaStream_t st) {
+  constexpr int kCols = kLanes * kVec16<T>;
   const bool al = p.n % kVec16<T> == 0 && (reinterpret_cast<uintptr_t>(p.m) & 15) == 0;
-  auto* kernel = al ? head_matmul_kernel<T, true> : head_matmul_kernel<T, false>;
-  size_t red = static_cast<size_t>(8) * kHmRows * kCols;
+  auto* kernel = al ? head_matmul_kernel<T, kLanes, true> : head_matmul_kernel<T, kLanes, false>;
+  size_t red = static_cast<size_t>(kHmThreads / kLanes) * kHmRows * kCols;
   if (static_cast<size_t>(kHmRows) * p.rot_dim > red) red = static_cast<size_t>(kHmRows) * p.rot_dim;
   const size_t smem = sizeof(float) * (static_cast<size_t>(p.k) * kHmRows + red);
   const int rc = opt_in_smem(kernel, smem);
@@ -363,6 +359,14 @@ static int head_matmul_launch(HeadMatmulParams<T> p, int heads, cudaStream_t st)
   const dim3 grid((p.n + kCols - 1) / kCols, heads, (p.rows + kHmRows - 1) / kHmRows);
   if (grid.z > 65535 || grid.y > 65535) return SLLM_ERR_LIMIT;
   return launch_kernel(kernel, grid, dim3(kHmThreads), smem, st, 1u, p) == cudaSuccess ? SLLM_OK : SLLM_ERR_CUDA;
+}
+
+template <typename T>
+static int head_matmul_launch(const HeadMatmulParams<T>& p, int heads, cudaStream_t st) {
+  const int pieces = (p.n + kVec16<T> - 1) / kVec16<T>;
+  if (pieces >= 32) return head_matmul_launch_l<T, 32>(p, heads, st);
+  if (pieces >= 16) return head_matmul_launch_l<T, 16>(p, heads, st);
+  return head_matmul_launch_l<T, 8>(p, heads, st);
 }
 
 template <typename T>

@@ -36,31 +36,66 @@ latent_gather_kernel(const __nv_bfloat16* __restrict__ pages, int ld, int page_s
 }
 
 // ---------------------------------------------------------------- query packing
-// grid (tokens, heads), 64 threads.
-__global__ void __launch_bounds__(64)
-latent_pack_q_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, __nv_bfloat16* __restrict__ out, int dim, int rot_dim,
-                     int dim_pad, int rot_pad, const int* __restrict__ positions, const float* __restrict__ inv_freq, int rot_dims,
-                     int interleaved) {
+// grid (tokens), 256 threads; a token's angles are computed once for all heads.  dim, dim_pad and rot_pad are multiples of 8.
+__global__ void __launch_bounds__(256)
+latent_pack_q_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, __nv_bfloat16* __restrict__ out, int heads, int dim,
+                     int rot_dim, int dim_pad, int rot_pad, const int* __restrict__ positions, const float* __restrict__ inv_freq,
+                     int rot_dims, int interleaved, int vec) {
   pdl_wait();
   pdl_trigger();
-  const int t = blockIdx.x, h = blockIdx.y;
-  const __nv_bfloat16* src = q + t * ldq + static_cast<long long>(h) * (dim + rot_dim);
-  __nv_bfloat16* dst = out + (static_cast<size_t>(t) * gridDim.y + h) * (dim_pad + rot_pad);
-  const __nv_bfloat16 zero = __float2bfloat16_rn(0.f);
-  for (int i = threadIdx.x; i < dim_pad; i += 64) dst[i] = i < dim ? src[i] : zero;
+  extern __shared__ float2 cs[];                     // [rot_dims / 2] = {cos, sin}
+  const int t = blockIdx.x, half = rot_dims >> 1, width = dim_pad + rot_pad;
   const float pos = static_cast<float>(positions[t]);
-  const int half = rot_dims >> 1;
-  for (int i = threadIdx.x; i < rot_pad; i += 64) {
-    if (i >= rot_dims) {
-      dst[dim_pad + i] = i < rot_dim ? src[dim + i] : zero;
-      continue;
+  for (int i = threadIdx.x; i < half; i += 256) {
+    float sn, c;
+    sincosf(pos * inv_freq[i], &sn, &c);
+    cs[i] = make_float2(c, sn);
+  }
+  const __nv_bfloat16* src = q + t * ldq;
+  __nv_bfloat16* dst = out + static_cast<size_t>(t) * heads * width;
+  const __nv_bfloat16 zero = __float2bfloat16_rn(0.f);
+  const int pieces = dim_pad >> 3;
+  for (int e = threadIdx.x; e < heads * pieces; e += 256) {
+    const int h = e / pieces, i = (e - h * pieces) * 8;
+    const __nv_bfloat16* s = src + h * (dim + rot_dim) + i;
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (i < dim) {
+      if (vec) {
+        v = *reinterpret_cast<const uint4*>(s);
+      } else {
+        __nv_bfloat16* x = reinterpret_cast<__nv_bfloat16*>(&v);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) x[j] = s[j];
+      }
     }
-    const int fi = interleaved ? i >> 1 : (i < half ? i : i - half);
-    const int iu = interleaved ? 2 * fi : fi, iv = interleaved ? iu + 1 : fi + half;
-    const float u = __bfloat162float(src[dim + iu]), v = __bfloat162float(src[dim + iv]);
-    float sn, cs;
-    sincosf(pos * inv_freq[fi], &sn, &cs);
-    dst[dim_pad + i] = __float2bfloat16_rn(i == iu ? u * cs - v * sn : v * cs + u * sn);
+    *reinterpret_cast<uint4*>(dst + h * width + i) = v;
+  }
+  __syncthreads();
+  const int pairs = rot_pad >> 1;                    // pairs of neighbouring output channels
+  for (int e = threadIdx.x; e < heads * pairs; e += 256) {
+    const int h = e / pairs, i = (e - h * pairs) * 2;
+    const __nv_bfloat16* s = src + h * (dim + rot_dim) + dim;
+    __nv_bfloat162 o;
+    if (interleaved && i < rot_dims) {
+      const float u = __bfloat162float(s[i]), v = __bfloat162float(s[i + 1]);
+      const float2 c = cs[i >> 1];
+      o = __floats2bfloat162_rn(u * c.x - v * c.y, v * c.x + u * c.y);
+    } else {
+      __nv_bfloat16 x[2];
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        const int k = i + j;
+        if (k >= rot_dims) {
+          x[j] = k < rot_dim ? s[k] : zero;
+        } else {
+          const int fi = k < half ? k : k - half;
+          const float u = __bfloat162float(s[fi]), v = __bfloat162float(s[fi + half]);
+          x[j] = __float2bfloat16_rn(k < half ? u * cs[fi].x - v * cs[fi].y : v * cs[fi].x + u * cs[fi].y);
+        }
+      }
+      o = __halves2bfloat162(x[0], x[1]);
+    }
+    *reinterpret_cast<__nv_bfloat162*>(dst + h * width + dim_pad + i) = o;
   }
 }
 
@@ -385,9 +420,11 @@ SLLM_EXPORT int sllm_latent_pack_q(const void* q, long long ldq, void* out, int 
   if (!q || !out || !positions || tokens <= 0 || heads <= 0 || heads > 65535 || dim <= 0 || rot_dim < 0 || dim_pad < dim ||
       rot_pad < rot_dim || rot_dims > rot_dim || (rot_dims & 1) || (rot_dims > 0 && !inv_freq))
     return SLLM_ERR_INVALID_ARGUMENT;
-  return launch_kernel(latent_pack_q_kernel, dim3(tokens, heads), dim3(64), 0, static_cast<cudaStream_t>(stream), 1u,
-                       static_cast<const __nv_bfloat16*>(q), ldq, static_cast<__nv_bfloat16*>(out), dim, rot_dim, dim_pad, rot_pad,
-                       positions, inv_freq, rot_dims, interleaved) == cudaSuccess ? SLLM_OK : SLLM_ERR_CUDA;
+  if ((dim & 7) || (dim_pad & 7) || (rot_pad & 7) || rot_dims > 4096) return SLLM_ERR_UNSUPPORTED_SHAPE;
+  const int vec = (ldq & 7) == 0 && (rot_dim & 7) == 0 && (reinterpret_cast<uintptr_t>(q) & 15) == 0;
+  return launch_kernel(latent_pack_q_kernel, dim3(tokens), dim3(256), sizeof(float2) * (rot_dims / 2 + 1), static_cast<cudaStream_t>(stream),
+                       1u, static_cast<const __nv_bfloat16*>(q), ldq, static_cast<__nv_bfloat16*>(out), heads, dim, rot_dim, dim_pad,
+                       rot_pad, positions, inv_freq, rot_dims, interleaved, vec) == cudaSuccess ? SLLM_OK : SLLM_ERR_CUDA;
 }
 
 // q: packed [tokens, heads, (dim chunks + rot chunks) * 64]; kv: [context rows, heads * (dim + vdim)] (all heads' keys, then
