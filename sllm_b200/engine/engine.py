@@ -255,8 +255,8 @@ class Engine:
         common = 0
         while common < limit and src.tokens[common] == prompt[common]:
             common += 1
-        if self.has_state and common != src.num_computed:
-            common = 0        # a recurrent state describes the end of the source's computed tokens only
+        if self.has_state and (common != src.num_computed or src.seq_id not in self.cache.slot_of):
+            common = 0        # a recurrent state describes the end of a live source's computed tokens only
         s = Sequence(prompt=list(prompt), user=user)
         if common == 0:
             s.seq_id = self.cache.pool.new_seq()

@@ -284,6 +284,21 @@ def test_fork_copies_pages_and_state(cases):
     assert Z.error(eng.step([a], [[0]]), c.oracle(toks[:22])[-1:]) < Z.TOL["fp32"]
 
 
+def test_fork_without_a_state_starts_over(cases):
+    """A source that holds pages but no state slot (a prefix-cache entry) shares nothing with a recurrent model."""
+    from sllm_b200.engine.engine import Sequence
+    c = cases("mixed")
+    toks = c.prompt(25, 8)
+    eng = c.engine("cpu", "fp32")
+    a = eng.new_sequence([])
+    a.tokens.extend(toks[:20])
+    eng.step([a], [[]])
+    entry = Sequence(prompt=toks[:20], seq_id=eng.fork_kv(a, 20), num_computed=20)
+    b = eng.fork_sequence(entry, toks)
+    assert b.num_computed == 0
+    assert Z.error(eng.step([b], [[24]]), c.oracle(toks)[-1:]) < Z.TOL["fp32"]
+
+
 def test_page_export_round_trip(cases):
     eng = cases("mixed").engine("cpu", "fp32")
     a = eng.new_sequence([])
