@@ -93,7 +93,7 @@ def _rows(kv, table, s, n, width):
 
 
 @pytest.mark.parametrize("heads,rank,rot,lens,window,page", [
-    (4, 128, 32, [1, 65, 700], 0, 16), (20, 512, 64, [2048, 33], 0, 16), (3, 48, 24, [100, 17, 64, 5], 21, 16),
+    (6, 160, 48, [1, 65, 700], 0, 16), (20, 512, 64, [2048, 33], 0, 16), (3, 48, 24, [100, 17, 64, 5], 21, 16),
     (40, 256, 32, [513, 300], 100, 32), (33, 512, 64, [640, 128], 0, 8), (17, 512, 64, [64, 63, 129], 40, 16), (1, 16, 2, [3000], 0, 16)])
 def test_page_streaming_attention(heads, rank, rot, lens, window, page):
     spec, kv, table = _setup(heads, rank, rot, lens, window, page)
@@ -133,7 +133,7 @@ def test_one_loud_key_at_page_and_window_edges(impl, window):
 
 
 @pytest.mark.parametrize("heads,dim,rot,vdim,rank,window,inter,lens,starts", [
-    (4, 32, 32, 32, 128, 0, True, [64], [0]), (4, 32, 32, 48, 128, 72, False, [100, 300], [0, 50]),
+    (6, 48, 32, 40, 160, 0, True, [64], [0]), (7, 24, 40, 56, 144, 90, False, [100, 300], [0, 50]),
     (3, 128, 64, 128, 512, 0, True, [130, 5, 700, 64], [0, 3, 257, 1000]), (2, 40, 24, 104, 96, 300, False, [513, 2, 90], [1000, 7, 0]),
     (5, 64, 2, 64, 64, 1, True, [200], [0]), (2, 128, 64, 128, 256, 128, True, [257, 129], [127, 128])])
 def test_expanded_portions_beside_short_ones(heads, dim, rot, vdim, rank, window, inter, lens, starts):
