@@ -38,7 +38,7 @@ CASES = {
                      windowed(88, heads=5, dim=24, rot=8, vdim=16, rank=64, window=19, scale=0.21, base=7e2)],
                     width=96, vocab=211, groups=3, eps=1e-5),
     "delta-first": config([delta(64, heads=1, dim=33), windowed(None, heads=1, dim=8, rot=16, vdim=8, rank=24, window=1),
-                           delta(40, heads=2, dim=64), latent(56, heads=4, dim=8, rot=2, vdim=24, rank=16, q_rank=24)],
+                           delta(40, heads=2, dim=56), latent(56, heads=4, dim=8, rot=2, vdim=24, rank=16, q_rank=24)],
                           width=80, vocab=96),
     "odd": config([windowed(36, heads=2, dim=10, rot=6, vdim=14, rank=20, window=40), delta(20, heads=3, dim=10),
                    latent(None, heads=2, dim=6, rot=10, vdim=18, rank=28, q_rank=22)], width=60, vocab=77, groups=5),
