@@ -106,7 +106,7 @@ def open_model(args, max_batch: int = 8, tp=None):
     except ValueError as exc:
         raise CliError(f"model load failed: {exc}", 3) from None
     eng = Engine(cfg, model, cache, device, max_batch=max_batch, use_cuda_graphs=not use_cpu, tp=tp)
-    dense_family = family not in ("moe", "qwen35", "zokuvik")
+    dense_family = family not in ("moe", "qwen35", *registry.LAYERED)
     eng.mtp_weights = loader.load_mtp_gguf(g, cfg, device) if tp_size == 1 and dense_family else None
     vis = loader.load_vision_gguf(g, cfg, device) if dense_family else None
     if vis is not None:

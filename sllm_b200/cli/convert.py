@@ -14,8 +14,9 @@ Kinds:
                  `qwen3_5_moe_text` with routed MXFP4 experts stored as packed U8 values plus E8M0 `weight_scale`
                  planes and a gated shared expert); the decoder tensors under `model.language_model.` are consumed,
                  `model.visual.*` and `mtp.*` are recorded as known-unconsumed; same lock verification
-  zokuvik        a Zokuvik folder (config.json with `architecture`, model.safetensors); same lock verification.  The
-                 seeded shapes of that family (`zokuvik`, `tiny-zokuvik`) are written by random-llama
+  zokuvik, sepedra
+                 a folder of that design (config.json with `architecture`, model.safetensors); same lock verification.
+                 The seeded shapes of these families (`zokuvik`, `tiny-zokuvik`, ...) are written by random-llama
 `--weight-format bf16|fp8` selects the resident encoding (fp8 = E4M3FN with FP32 scales per 1x128 block).
 `--dry-run` validates inputs and prints the plan without writing.  (Reference: crates/sllm-server/src/bin/
 sllm-convert-gguf.rs flags --kind --lock --cache --artifact --manifest --output --derived-lock
@@ -29,7 +30,7 @@ import sys
 
 from .common import CliError, StrictParser, emit, run_main
 
-KINDS = ("random-llama", "hf-llama", "hf-qwen35", "mixed-precision", "zokuvik")
+KINDS = ("random-llama", "hf-llama", "hf-qwen35", "mixed-precision", "zokuvik", "sepedra")
 
 
 def _hf_config(raw: dict, weight_format: str):
@@ -294,18 +295,20 @@ def main(argv=None) -> int:
         from ..models import moe as _moe
         from ..models import qwen35 as _q35
         from ..models import registry
+        from ..models import sepedra as _sp
         from ..models import zokuvik as _zk
         named.update({"tiny-moe": _moe.tiny_moe, "tiny-shared-moe": _moe.tiny_shared_moe, "tiny-qwen35": _q35.tiny_qwen35,
-                      "tiny-qwen35-moe": _q35.tiny_qwen35_moe, "tiny-zokuvik": _zk.tiny_zokuvik})
+                      "tiny-qwen35-moe": _q35.tiny_qwen35_moe, "tiny-zokuvik": _zk.tiny_zokuvik, "tiny-sepedra": _sp.tiny_sepedra})
         if a.kind == "random-llama":
             if a.artifact not in named:
                 raise CliError(f"--artifact must be one of {sorted(named)}")
             cfg = named[a.artifact]()
-            if cfg.family in ("moe", "qwen35", "zokuvik"):
+            if cfg.family in ("moe", "qwen35", *registry.LAYERED):
                 ok = ("bf16", "fp32", "fp8") if cfg.family == "qwen35" else ("bf16", "fp32")
                 if a.weight_format not in ok:
                     raise CliError("the mixture-of-experts family keeps bf16 attention (experts are MXFP4); the hybrid "
-                                   "family takes bf16, fp32 or fp8 projections; the zokuvik family bf16 or fp32")
+                                   "family takes bf16, fp32 or fp8 projections; the zokuvik and sepedra families bf16 "
+                                   "or fp32")
                 if a.with_vision or a.with_mtp:
                     raise CliError("--with-vision / --with-mtp apply to the dense decoder family")
             cfg.weight_format = a.weight_format
@@ -336,13 +339,15 @@ def main(argv=None) -> int:
                                    "(routed experts keep their MXFP4 encoding)")
                 cfg = _hf_qwen35_config(raw_cfg)
                 cfg.weight_format = a.weight_format
-            elif a.kind == "zokuvik":
+            elif a.kind in registry.LAYERED:
                 if a.weight_format not in ("bf16", "fp32"):
-                    raise CliError("kind zokuvik writes bf16 or fp32 weights")
+                    raise CliError(f"kind {a.kind} writes bf16 or fp32 weights")
                 try:
                     cfg = registry.read_folder_config(cache.root, dtype=a.weight_format)
                 except registry.ModelFolderError as exc:
                     raise CliError(str(exc), 3) from None
+                if cfg.family != a.kind:
+                    raise CliError(f"kind {a.kind}: the folder holds a {cfg.family} model", 3)
             else:
                 cfg = _hf_config(raw_cfg, a.weight_format)
             if "tokenizer.json" in cache.fds:
@@ -364,7 +369,8 @@ def main(argv=None) -> int:
         if a.dry_run:
             emit({"dry_run": True, **plan})
             return 0
-        if a.kind in ("hf-qwen35", "zokuvik") or (a.kind == "random-llama" and cfg.family in ("moe", "qwen35", "zokuvik")):
+        if a.kind in ("hf-qwen35", *registry.LAYERED) or (a.kind == "random-llama" and
+                                                          cfg.family in ("moe", "qwen35", *registry.LAYERED)):
             from ..models import family_io
             dev = "cuda" if torch.cuda.is_available() else "cpu"
             extra = {}
@@ -373,7 +379,7 @@ def main(argv=None) -> int:
                 cache.close()
                 plan["known_unconsumed_tensors"] = len(unconsumed)
                 extra = {"known_unconsumed": unconsumed, "source_fingerprints": tuple(fps)}
-            elif a.kind == "zokuvik":
+            elif a.kind in registry.LAYERED:
                 try:
                     w = registry.load_folder_weights(cache.root, cfg, "cpu")
                 except registry.ModelFolderError as exc:

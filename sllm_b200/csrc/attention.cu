@@ -314,7 +314,8 @@ SLLM_EXPORT int sllm_paged_attention(const void* q, int q_ld, const void* k_page
                                      const int* seq_index, const int* kv_lens, int rows, int hq, int hkv, int hd,
                                      int page_size, int window, float sm_scale, int kv_fp8, void* out_bf16,
                                      void* out_fp8, float* out_scale, int ld_scale, const float* sinks, int splits,
-                                     float* ws, long long ws_floats, int* counters, int n_counters, void* stream) {
+                                     float* ws, long long ws_floats, int* counters, int n_counters, const void* gate,
+                                     long long ld_gate, void* stream) {
   if (!q || !k_pages || !v_pages || !block_table || !seq_index || !kv_lens || rows <= 0 || hkv <= 0 || hq % hkv)
     return SLLM_ERR_INVALID_ARGUMENT;
   if (!out_bf16 && !out_fp8) return SLLM_ERR_INVALID_ARGUMENT;
@@ -331,6 +332,7 @@ SLLM_EXPORT int sllm_paged_attention(const void* q, int q_ld, const void* k_page
   p.out_bf16 = static_cast<__nv_bfloat16*>(out_bf16); p.out_fp8 = static_cast<uint8_t*>(out_fp8);
   p.out_scale = out_scale; p.ld_scale = ld_scale; p.sinks = sinks;
   p.ws_o = nullptr; p.ws_ml = nullptr; p.counters = counters; p.status_word = nullptr;
+  p.gate = static_cast<const __nv_bfloat16*>(gate); p.ld_gate = ld_gate;
   p.early_trigger = 0;
   if (splits > 1) {
     const long long units = static_cast<long long>(rows) * hkv;

@@ -28,6 +28,8 @@ struct PagedAttnParams {
   float* ws_ml;             // [rows * hkv * splits, G, 2]
   int* counters;            // [rows * hkv]
   const float* sinks;       // optional [hq] attention-sink logits (added to the softmax denominator)
+  const __nv_bfloat16* gate; // optional [rows, ld_gate] logits, one per output channel: out *= sigmoid(gate)
+  long long ld_gate;
   int* status_word;         // device status word for bounded waits (tensor-core kernel)
   int early_trigger;        // tensor-core kernel: let dependent launches start once the CTA holds its TMEM
   STEP_TRACE_FIELD
@@ -130,6 +132,8 @@ __device__ __forceinline__ void attention_tail(const PagedAttnParams& p, int r, 
       }
     }
     float val = (L > 0.f) ? O / L : 0.f;
+    if (p.gate && in)
+      val /= 1.f + __expf(-__bfloat162float(p.gate[static_cast<size_t>(r) * p.ld_gate + (kvh * G + g) * HD + d]));
     val = __bfloat162float(__float2bfloat16_rn(val));
     const size_t oidx = static_cast<size_t>(r) * hq * HD + (kvh * G + g) * HD + d;
     if (p.out_fp8) {

@@ -5,14 +5,16 @@
 #include "typed.cuh"
 #include "api.h"
 
+#include <type_traits>
+
 namespace sllm {
 
 constexpr int kSgTile = 64, kSgK = 16, kSgThreads = 256;
 
-template <typename T>
+template <typename T, typename TY>
 __global__ void __launch_bounds__(kSgThreads)
-gemm_simt_kernel(const T* __restrict__ x, const T* __restrict__ w, T* __restrict__ y, const T* __restrict__ residual, int m, int n,
-                 int k, int ldx, int ldw, int ldy, int act) {
+gemm_simt_kernel(const T* __restrict__ x, const T* __restrict__ w, TY* __restrict__ y, const TY* __restrict__ residual, int m, int n,
+                 int k, int ldx, int ldw, int ldy, int act, float act_arg) {
   pdl_wait();
   pdl_trigger();
   __shared__ float xs[kSgK][kSgTile + 4];
@@ -51,6 +53,7 @@ gemm_simt_kernel(const T* __restrict__ x, const T* __restrict__ w, T* __restrict
       if (c >= n) continue;
       float v = acc[i][j];
       if (act == 1) v = v > 0.f ? v * v : 0.f;
+      else if (act == 2) v = act_arg * tanhf(v / act_arg);
       const size_t idx = static_cast<size_t>(r) * ldy + c;
       if (residual) v += ld_f(residual + idx);
       st_f(y + idx, v);
@@ -62,21 +65,25 @@ gemm_simt_kernel(const T* __restrict__ x, const T* __restrict__ w, T* __restrict
 
 using namespace sllm;
 
-// act: 0 none, 1 square of relu.  fp32: element type of x, w, y and residual (0 bf16, 1 fp32).
+// act: 0 none, 1 square of relu, 2 soft cap act_arg * tanh(y / act_arg).  fp32: element type of x, w, y and residual (0 bf16,
+// 1 fp32); out_fp32: y and residual are fp32 whatever x and w are.
 SLLM_EXPORT int sllm_gemm_simt(const void* x, const void* w, void* y, const void* residual, int m, int n, int k, int ldx, int ldw,
-                               int ldy, int act, int fp32, void* stream) {
-  if (!x || !w || !y || m <= 0 || n <= 0 || k <= 0 || ldx < k || ldw < k || ldy < n || act < 0 || act > 1) return SLLM_ERR_INVALID_ARGUMENT;
+                               int ldy, int act, float act_arg, int fp32, int out_fp32, void* stream) {
+  if (!x || !w || !y || m <= 0 || n <= 0 || k <= 0 || ldx < k || ldw < k || ldy < n || act < 0 || act > 2 || (act == 2 && !(act_arg > 0.f)))
+    return SLLM_ERR_INVALID_ARGUMENT;
   const dim3 grid((n + kSgTile - 1) / kSgTile, (m + kSgTile - 1) / kSgTile);
   if (grid.y > 65535) return SLLM_ERR_LIMIT;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  cudaError_t e;
-  if (fp32)
-    e = launch_kernel(gemm_simt_kernel<float>, grid, dim3(kSgThreads), 0, st, 1u, static_cast<const float*>(x),
-                      static_cast<const float*>(w), static_cast<float*>(y), static_cast<const float*>(residual), m, n, k, ldx, ldw,
-                      ldy, act);
-  else
-    e = launch_kernel(gemm_simt_kernel<__nv_bfloat16>, grid, dim3(kSgThreads), 0, st, 1u, static_cast<const __nv_bfloat16*>(x),
-                      static_cast<const __nv_bfloat16*>(w), static_cast<__nv_bfloat16*>(y),
-                      static_cast<const __nv_bfloat16*>(residual), m, n, k, ldx, ldw, ldy, act);
+  auto go = [&](auto* kernel, auto* xt, auto* yt) {
+    using T = std::remove_pointer_t<decltype(xt)>;
+    using TY = std::remove_pointer_t<decltype(yt)>;
+    return launch_kernel(kernel, grid, dim3(kSgThreads), 0, st, 1u, static_cast<const T*>(x), static_cast<const T*>(w), static_cast<TY*>(y),
+                         static_cast<const TY*>(residual), m, n, k, ldx, ldw, ldy, act, act_arg);
+  };
+  float* f = nullptr;
+  __nv_bfloat16* h = nullptr;
+  const cudaError_t e = fp32 ? go(gemm_simt_kernel<float, float>, f, f)
+                             : out_fp32 ? go(gemm_simt_kernel<__nv_bfloat16, float>, h, f)
+                                        : go(gemm_simt_kernel<__nv_bfloat16, __nv_bfloat16>, h, h);
   return e == cudaSuccess ? SLLM_OK : SLLM_ERR_CUDA;
 }

@@ -110,7 +110,9 @@ struct GemmParams {
   int transpose_out;   // 0: Y[a, b]; 1: Y[b, a]
   int ldy;
   int ld_sa, ld_sb;    // leading dimensions of the kb-major scale arrays
-  int epilogue;        // 0 = store, 1 = add residual, 2 = square of relu
+  int epilogue;        // 0 = store, 1 = add residual, 2 = square of relu, 3 = soft cap
+  int out_fp32;        // y is fp32 (unscaled product, no residual)
+  float act_arg;       // soft cap
   int cluster_split;   // 1: gridDim.z CTAs form one cluster and reduce split-K partials over DSMEM
   int const_operand;   // operand that no kernel writes (weights): 0 none, 1 A, 2 B; loaded before the PDL wait
   int early_trigger;   // 1: dependents may become resident as soon as this CTA holds its resources
@@ -757,6 +759,19 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_const
       if (p.epilogue == 2) {
 #pragma unroll
         for (int j = 0; j < 8; ++j) v[j] = v[j] > 0.f ? v[j] * v[j] : 0.f;
+      } else if (p.epilogue == 3) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[j] = p.act_arg * tanhf(v[j] / p.act_arg);
+      }
+      if (!kScaled && !kComm && p.out_fp32) {
+        float* y = reinterpret_cast<float*>(p.y);
+        const int row = tr ? b_tile * BN + col : a_tile * kTileA + r0, n0 = tr ? a_tile * kTileA + r0 : b_tile * BN + col;
+        const int n = tr ? p.a_rows : p.b_rows;
+        if (row >= (tr ? p.b_rows : p.a_rows)) return;
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+          if (n0 + j < n) y[static_cast<size_t>(row) * p.ldy + n0 + j] = v[j];
+        return;
       }
       if (tr) {
         const int b_row = b_tile * BN + col;
@@ -1131,7 +1146,8 @@ static int gemm_impl(const void* a, const void* b, void* y, const float* scale_a
                      const void* residual, int a_rows, int b_rows, int k, int scaled, int transpose_out, int ldy,
                      int ld_sa, int ld_sb, int bn, int splits, int stages, float* ws, long long ws_floats,
                      int* counters, int n_counters, int* status, void* stream, const SllmCommDesc* comm,
-                     const SllmGatherDesc* gather = nullptr, const FusedEpi* fused = nullptr, int act = 0) {
+                     const SllmGatherDesc* gather = nullptr, const FusedEpi* fused = nullptr, int act = 0, float act_arg = 0.f,
+                     int out_fp32 = 0) {
   if (gather) b = a;    // the B operand comes from the peers' buffers; keep the argument checks below simple
   if (!a || !b || !y || a_rows <= 0 || b_rows <= 0 || k <= 0 || splits < 1) return SLLM_ERR_INVALID_ARGUMENT;
   if (bn != 16 && bn != 32 && bn != 64 && bn != 128) return SLLM_ERR_UNSUPPORTED_SHAPE;
@@ -1185,8 +1201,11 @@ static int gemm_impl(const void* a, const void* b, void* y, const float* scale_a
 
   p.a_rows = a_rows; p.b_rows = b_rows; p.num_kb = num_kb; p.kb_per_split = kb_per_split; p.stages = stages;
   p.transpose_out = transpose_out; p.ldy = ldy; p.ld_sa = ld_sa; p.ld_sb = ld_sb;
-  if (act < 0 || act > 1 || (act && (residual || comm || fused))) return SLLM_ERR_INVALID_ARGUMENT;
-  p.epilogue = residual ? 1 : act ? 2 : 0;
+  if (act < 0 || act > 2 || (act && (residual || comm || fused)) || (act == 2 && !(act_arg > 0.f)) ||
+      (out_fp32 && (residual || comm || fused || scaled)))
+    return SLLM_ERR_INVALID_ARGUMENT;
+  p.epilogue = residual ? 1 : act ? act + 1 : 0;
+  p.act_arg = act_arg; p.out_fp32 = out_fp32;
   // 2..8 splits reduce inside one thread-block cluster over DSMEM; more use the global fix-up.
   // (the output phase needs whole 16-byte units per slice: any slice width when Y is written
   // transposed, at least 8 columns otherwise)
@@ -1271,12 +1290,13 @@ SLLM_EXPORT int sllm_gemm(const void* a, const void* b, void* y, const float* sc
                    bn, splits, stages, ws, ws_floats, counters, n_counters, status, stream, nullptr);
 }
 
-// bf16 GEMM with an activation on the sums (act 1: square of relu).
+// bf16 GEMM with an activation on the sums (act 1: square of relu, 2: soft cap act_arg * tanh(y / act_arg)), stored as bf16 or
+// (out_fp32) as they are.
 SLLM_EXPORT int sllm_gemm_act(const void* a, const void* b, void* y, int a_rows, int b_rows, int k, int transpose_out, int ldy,
-                              int act, int bn, int splits, int stages, float* ws, long long ws_floats, int* counters,
-                              int n_counters, int* status, void* stream) {
+                              int act, float act_arg, int out_fp32, int bn, int splits, int stages, float* ws, long long ws_floats,
+                              int* counters, int n_counters, int* status, void* stream) {
   return gemm_impl(a, b, y, nullptr, nullptr, nullptr, a_rows, b_rows, k, 0, transpose_out, ldy, 0, 0, bn, splits, stages, ws,
-                   ws_floats, counters, n_counters, status, stream, nullptr, nullptr, nullptr, act);
+                   ws_floats, counters, n_counters, status, stream, nullptr, nullptr, nullptr, act, act_arg, out_fp32);
 }
 
 // Same GEMM with the cross-rank sum of the partial products fused into the epilogue (see the file

@@ -5,9 +5,10 @@
 //
 // One launch does, per row:
 //   1. x  = table[id]                (embedding),  or
-//      x += norm(y) * w_post         (sandwich: the sublayer's output is normalised before it joins the residual), or
+//      x += norm(y) * w_post         (sandwich: the sublayer's output is normalised before it joins the residual; y may be
+//                                     the sum of several listed rows, the routed experts of a token), or
 //      x  as it is, optionally of a gathered row
-//   2. z  = norm(x) * w_out          (the next sublayer's input, in the activation type)
+//   2. z  = norm(x) * w_out          (the next sublayer's input, in the activation type), or z = x without w_out
 // so a decoder layer with norms before and after each sublayer costs one such launch per sublayer.
 #include "typed.cuh"
 #include "api.h"
@@ -24,11 +25,13 @@ struct GroupNormParams {
   int vocab;
   const T* y;                // sandwich mode: [rows, ldy]
   int ldy;
+  const int* y_rows;         // sandwich mode: y is the sum of the rows y_rows[r * y_terms ..] >= 0 (null: row r)
+  int y_terms;
   const float* w_post;       // [d]
   float* x;                  // residual [*, d]: written in the embedding and sandwich modes
   const long long* row_idx;  // read-only mode: z row r comes from x row row_idx[r] (null: row r)
-  const float* w_out;        // [d], null: no z
-  T* z;                      // [rows, d]
+  const float* w_out;        // [d], null: z is x itself
+  T* z;                      // [rows, d], null: none
   int d, groups, parts;
   float eps;
 };
@@ -86,11 +89,28 @@ __global__ void __launch_bounds__(kGnThreads) group_norm_kernel(const GroupNormP
     }
   } else if (p.y) {
     xr += static_cast<size_t>(r) * d;
-    const T* src = p.y + static_cast<size_t>(r) * p.ldy;
-    for (int i = threadIdx.x * kV; i < d; i += kGnThreads * kV) {
-      float v[kV];
-      load(src + i, v);
-      store(row + i, v);
+    if (p.y_rows) {
+      const int* rows = p.y_rows + static_cast<size_t>(r) * p.y_terms;
+      for (int i = threadIdx.x * kV; i < d; i += kGnThreads * kV) {
+        float v[kV] = {};
+#pragma unroll 4
+        for (int t = 0; t < p.y_terms; ++t) {
+          const int src = rows[t];
+          if (src < 0) continue;
+          float a[kV];
+          load(p.y + static_cast<size_t>(src) * p.ldy + i, a);
+#pragma unroll
+          for (int j = 0; j < kV; ++j) v[j] += a[j];
+        }
+        store(row + i, v);
+      }
+    } else {
+      const T* src = p.y + static_cast<size_t>(r) * p.ldy;
+      for (int i = threadIdx.x * kV; i < d; i += kGnThreads * kV) {
+        float v[kV];
+        load(src + i, v);
+        store(row + i, v);
+      }
     }
     __syncthreads();
     group_inv_rms(row, gs, p.groups, p.parts, p.eps, part, inv);
@@ -115,9 +135,17 @@ __global__ void __launch_bounds__(kGnThreads) group_norm_kernel(const GroupNormP
     }
   }
   if (!p.z) return;
+  T* zr = p.z + static_cast<size_t>(r) * d;
+  if (!p.w_out) {                                    // every thread reads back what it wrote
+    for (int i = threadIdx.x * kV; i < d; i += kGnThreads * kV) {
+      float v[kV];
+      load(row + i, v);
+      store(zr + i, v);
+    }
+    return;
+  }
   __syncthreads();
   group_inv_rms(row, gs, p.groups, p.parts, p.eps, part, inv);
-  T* zr = p.z + static_cast<size_t>(r) * d;
   for (int i = threadIdx.x * kV; i < d; i += kGnThreads * kV) {
     float v[kV], w[kV];
     load(row + i, v);
@@ -130,12 +158,12 @@ __global__ void __launch_bounds__(kGnThreads) group_norm_kernel(const GroupNormP
 }
 
 template <typename T>
-static int group_norm_launch(const void* table, const int* ids, int vocab, const void* y, int ldy, const float* w_post, float* x,
-                             const long long* row_idx, const float* w_out, void* z, int rows, int d, int groups, float eps,
+static int group_norm_launch(const void* table, const int* ids, int vocab, const void* y, int ldy, const int* y_rows, int y_terms,
+                             const float* w_post, float* x, const long long* row_idx, const float* w_out, void* z, int rows, int d, int groups, float eps,
                              cudaStream_t st) {
   GroupNormParams<T> p = {};
   p.table = static_cast<const T*>(table); p.ids = ids; p.vocab = vocab;
-  p.y = static_cast<const T*>(y); p.ldy = ldy; p.w_post = w_post; p.x = x; p.row_idx = row_idx;
+  p.y = static_cast<const T*>(y); p.ldy = ldy; p.y_rows = y_rows; p.y_terms = y_terms; p.w_post = w_post; p.x = x; p.row_idx = row_idx;
   p.w_out = w_out; p.z = static_cast<T*>(z); p.d = d; p.groups = groups; p.eps = eps;
   p.parts = groups >= kGnWarps ? 1 : (kGnWarps + groups - 1) / groups;
   const size_t smem = sizeof(float) * (((d + 3) & ~3) + groups + static_cast<size_t>(groups) * p.parts);
@@ -153,14 +181,15 @@ static int group_norm_launch(const void* table, const int* ids, int vocab, const
 using namespace sllm;
 
 // table + ids: embedding mode; y + w_post: sandwich mode; neither: x is read only (rows picked by row_idx when given).
-// z / w_out may both be null (residual update alone).  fp32: element type of table, y and z (0 bf16, 1 fp32).
-SLLM_EXPORT int sllm_group_norm(const void* table, const int* ids, int vocab, const void* y, int ldy, const float* w_post,
-                                float* x, const long long* row_idx, const float* w_out, void* z, int rows, int d, int groups,
+// y_rows [rows, y_terms]: y is the sum of those rows of it.  z may be null (residual update alone), z without w_out is x in
+// the element type.  fp32: element type of table, y and z (0 bf16, 1 fp32).
+SLLM_EXPORT int sllm_group_norm(const void* table, const int* ids, int vocab, const void* y, int ldy, const int* y_rows,
+                                int y_terms, const float* w_post, float* x, const long long* row_idx, const float* w_out, void* z, int rows, int d, int groups,
                                 float eps, int fp32, void* stream) {
   if (!x || rows <= 0 || d <= 0 || groups <= 0 || d % groups) return SLLM_ERR_INVALID_ARGUMENT;
-  if ((table && (!ids || vocab <= 0 || y)) || (y && !w_post) || (!z != !w_out) || (!z && !y && !table)) return SLLM_ERR_INVALID_ARGUMENT;
+  if ((table && (!ids || vocab <= 0 || y)) || (y && !w_post) || (!z && w_out) || (y_rows && (!y || y_terms <= 0)) || (!z && !y && !table)) return SLLM_ERR_INVALID_ARGUMENT;
   if (row_idx && (table || y)) return SLLM_ERR_INVALID_ARGUMENT;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  return fp32 ? group_norm_launch<float>(table, ids, vocab, y, ldy, w_post, x, row_idx, w_out, z, rows, d, groups, eps, st)
-              : group_norm_launch<__nv_bfloat16>(table, ids, vocab, y, ldy, w_post, x, row_idx, w_out, z, rows, d, groups, eps, st);
+  return fp32 ? group_norm_launch<float>(table, ids, vocab, y, ldy, y_rows, y_terms, w_post, x, row_idx, w_out, z, rows, d, groups, eps, st)
+              : group_norm_launch<__nv_bfloat16>(table, ids, vocab, y, ldy, y_rows, y_terms, w_post, x, row_idx, w_out, z, rows, d, groups, eps, st);
 }

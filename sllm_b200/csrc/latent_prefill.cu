@@ -8,7 +8,8 @@
 //   latent_gather_kernel   pages -> [context rows, kv_rank] and [context rows, rotated part padded to 64]
 //   latent_pack_q_kernel   q -> [tokens, heads, unrotated padded to 64 | rotated padded to 64], rotation applied; the
 //                          padding is zero, so key columns that a 64-wide box reads beyond a head's own do not count
-//   latent_prefill_kernel  see below
+//   latent_prefill_kernel  see below; it also serves ordinary keys and values gathered from their pages (kv_attention.cu),
+//                          with fewer key / value heads than query heads, attention sinks and a gate per output channel
 #include "typed.cuh"
 #include "api.h"
 #include "tmap.h"
@@ -115,10 +116,12 @@ constexpr int kLpChunk = kLpTile * 128;
 
 struct LatentPrefillParams {
   const int* tiles;          // [tiles][8]: query row, rows, position of the first row, context row, its position, -, -, -
-  int heads, dim, vdim, dim_chunks, v_stages, window;
+  int heads, kv_heads, dim, vdim, dim_chunks, v_stages, window;
   float scale_log2;
-  const __nv_bfloat16* gate; // optional [tokens, ld_gate]
+  const float* sinks;        // optional [heads]: scores that join the denominator only
+  const __nv_bfloat16* gate; // optional logits [tokens, ld_gate], one per head or (gate_channels) per output channel
   long long ld_gate;
+  int gate_channels;
   __nv_bfloat16* out;        // [tokens, heads * vdim]
   int* status;
 };
@@ -169,7 +172,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   LatentPrefillShared* sh = reinterpret_cast<LatentPrefillShared*>(v_s + p.v_stages * kNV * kLpChunk);
   constexpr uint32_t kTmemCols = 512;                // S at columns 0 and 128, PV at 256
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int head = blockIdx.y;
+  const int head = blockIdx.y, kvh = head / (p.heads / p.kv_heads);
   const int* tile = p.tiles + 8 * blockIdx.x;
   const int q_row = tile[0], rows = tile[1], q0 = tile[2], k_lo = tile[4];
   const int first = p.window > 0 ? max(k_lo, q0 - p.window + 1) : k_lo;   // first visible position of the tile's rows
@@ -214,14 +217,14 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
         mbar_expect_tx(&sh->k_full[st], kNQ * kLpChunk);
         for (int c = 0; c < kNQ; ++c) {
           uint8_t* dst = k_s + (st * kNQ + c) * kLpChunk;
-          if (c < p.dim_chunks) tma_load_2d(dst, &tm_kv, &sh->k_full[st], head * p.dim + c * 64, y);
+          if (c < p.dim_chunks) tma_load_2d(dst, &tm_kv, &sh->k_full[st], kvh * p.dim + c * 64, y);
           else tma_load_2d(dst, &tm_r, &sh->k_full[st], (c - p.dim_chunks) * 64, y);
         }
         ks = j + 1;
         if (!mbar_wait(&sh->v_empty[sv], ((j / p.v_stages) & 1) ^ 1, abort_flag, p.status, SLLM_DEV_TIMEOUT_SMEM_EMPTY)) break;
         mbar_expect_tx(&sh->v_full[sv], kNV * kLpChunk);
         for (int c = 0; c < kNV; ++c)
-          tma_load_2d(v_s + (sv * kNV + c) * kLpChunk, &tm_kv, &sh->v_full[sv], p.heads * p.dim + head * p.vdim + c * 64, y);
+          tma_load_2d(v_s + (sv * kNV + c) * kLpChunk, &tm_kv, &sh->v_full[sv], p.kv_heads * p.dim + kvh * p.vdim + c * 64, y);
         vs = j + 1;
       }
       // every copy has landed before the CTA may leave
@@ -352,19 +355,26 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
     fold(nt - 1);
     sh->red[nt & 1][half][r] = l;                    // the other parity's buffer was last read before tile nt - 1's barrier
     lp_bar_softmax();
-    const float total = l + sh->red[nt & 1][half ^ 1][r];
+    float total = l + sh->red[nt & 1][half ^ 1][r];
+    if (p.sinks) total += lp_ex2(p.sinks[head] * 1.4426950408889634f - m);
     if (ok && r < rows) {
       float inv = total > 0.f ? 1.f / total : 0.f;
       const long long t = q_row + r;
-      if (p.gate) inv *= sigmoid_f(__bfloat162float(p.gate[t * p.ld_gate + head]));
+      const bool per_channel = p.gate && p.gate_channels;
+      if (p.gate && !p.gate_channels) inv *= sigmoid_f(__bfloat162float(p.gate[t * p.ld_gate + head]));
+      const __nv_bfloat16* gate = p.gate + t * p.ld_gate + head * p.vdim;
       __nv_bfloat16* dst = p.out + (t * p.heads + head) * p.vdim;
 #pragma unroll
       for (int i = 0; i < kO; i += 8) {
         if (half * kO + i < p.vdim) {
           uint4 w;
           __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&w);
+          float g[8];
+          if (per_channel) ld16(gate + half * kO + i, g);
 #pragma unroll
-          for (int k = 0; k < 4; ++k) h[k] = __floats2bfloat162_rn(o[i + 2 * k] * inv, o[i + 2 * k + 1] * inv);
+          for (int k = 0; k < 8; ++k) g[k] = per_channel ? inv / (1.f + __expf(-g[k])) : inv;
+#pragma unroll
+          for (int k = 0; k < 4; ++k) h[k] = __floats2bfloat162_rn(o[i + 2 * k] * g[2 * k], o[i + 2 * k + 1] * g[2 * k + 1]);
           *reinterpret_cast<uint4*>(dst + half * kO + i) = w;
         }
       }
@@ -427,28 +437,19 @@ SLLM_EXPORT int sllm_latent_pack_q(const void* q, long long ldq, void* out, int 
                        rot_pad, positions, inv_freq, rot_dims, interleaved, vec) == cudaSuccess ? SLLM_OK : SLLM_ERR_CUDA;
 }
 
-// q: packed [tokens, heads, (dim chunks + rot chunks) * 64]; kv: [context rows, heads * (dim + vdim)] (all heads' keys, then
-// all heads' values); r: [context rows, rot chunks * 64]; tiles: [num_tiles][8], see LatentPrefillParams.
-SLLM_EXPORT int sllm_latent_prefill(const void* q, int tokens, const void* kv, const void* r, int context, const int* tiles,
-                                    int num_tiles, int heads, int dim, int rot_dim, int vdim, int window, float scale,
-                                    const void* gate, long long ld_gate, void* out, int* status, void* stream) {
-  if (!q || !kv || !r || !tiles || !out || tokens <= 0 || context <= 0 || num_tiles <= 0 || heads <= 0 || heads > 65535 || dim <= 0 ||
-      rot_dim < 0 || vdim <= 0 || window < 0)
-    return SLLM_ERR_INVALID_ARGUMENT;
+static int latent_prefill_impl(const void* q, int tokens, const void* kv, const void* r, int context, const int* tiles, int num_tiles,
+                               int rot_dim, LatentPrefillParams p, cudaStream_t st) {
+  const int dim = p.dim, vdim = p.vdim;
   const int nd = (dim + 63) / 64, nr = (rot_dim + 63) / 64, nq = nd + nr, nv = (vdim + 63) / 64;
   if (nq < 1 || nq > 3 || nv > 2 || (dim & 7) || (vdim & 7)) return SLLM_ERR_UNSUPPORTED_SHAPE;
-  if (reinterpret_cast<uintptr_t>(out) & 15) return SLLM_ERR_ALIGNMENT;
-  const long long wq = static_cast<long long>(heads) * nq * 64, wkv = static_cast<long long>(heads) * (dim + vdim);
+  if (reinterpret_cast<uintptr_t>(p.out) & 15) return SLLM_ERR_ALIGNMENT;
+  const long long wq = static_cast<long long>(p.heads) * nq * 64, wkv = static_cast<long long>(p.kv_heads) * (dim + vdim);
   CUtensorMap tq, tkv, tr;
   int rc = cached_kmajor_tmap(&tq, q, 2, tokens, wq, wq * 2, kLpTile);
   if (rc == SLLM_OK) rc = cached_kmajor_tmap(&tkv, kv, 2, context, wkv, wkv * 2, kLpTile);
   if (rc == SLLM_OK) rc = nr > 0 ? cached_kmajor_tmap(&tr, r, 2, context, nr * 64, nr * 128, kLpTile) : (tr = tkv, SLLM_OK);
   if (rc != SLLM_OK) return rc;
-  LatentPrefillParams p = {};
-  p.tiles = tiles; p.heads = heads; p.dim = dim; p.vdim = vdim; p.dim_chunks = nd; p.window = window;
-  p.scale_log2 = scale * 1.4426950408889634f;
-  p.gate = static_cast<const __nv_bfloat16*>(gate); p.ld_gate = ld_gate; p.out = static_cast<__nv_bfloat16*>(out); p.status = status;
-  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  p.tiles = tiles; p.dim_chunks = nd;
   switch (nq * 2 + nv - 1) {
     case 2: return latent_prefill_launch<1, 1>(tq, tkv, tr, p, num_tiles, st);
     case 3: return latent_prefill_launch<1, 2>(tq, tkv, tr, p, num_tiles, st);
@@ -457,4 +458,34 @@ SLLM_EXPORT int sllm_latent_prefill(const void* q, int tokens, const void* kv, c
     case 6: return latent_prefill_launch<3, 1>(tq, tkv, tr, p, num_tiles, st);
     default: return latent_prefill_launch<3, 2>(tq, tkv, tr, p, num_tiles, st);
   }
+}
+
+// q: packed [tokens, heads, (dim chunks + rot chunks) * 64]; kv: [context rows, heads * (dim + vdim)] (all heads' keys, then
+// all heads' values); r: [context rows, rot chunks * 64]; tiles: [num_tiles][8], see LatentPrefillParams; gate per head.
+SLLM_EXPORT int sllm_latent_prefill(const void* q, int tokens, const void* kv, const void* r, int context, const int* tiles,
+                                    int num_tiles, int heads, int dim, int rot_dim, int vdim, int window, float scale,
+                                    const void* gate, long long ld_gate, void* out, int* status, void* stream) {
+  if (!q || !kv || !r || !tiles || !out || tokens <= 0 || context <= 0 || num_tiles <= 0 || heads <= 0 || heads > 65535 || dim <= 0 ||
+      rot_dim < 0 || vdim <= 0 || window < 0)
+    return SLLM_ERR_INVALID_ARGUMENT;
+  LatentPrefillParams p = {};
+  p.heads = p.kv_heads = heads; p.dim = dim; p.vdim = vdim; p.window = window; p.scale_log2 = scale * 1.4426950408889634f;
+  p.gate = static_cast<const __nv_bfloat16*>(gate); p.ld_gate = ld_gate; p.out = static_cast<__nv_bfloat16*>(out); p.status = status;
+  return latent_prefill_impl(q, tokens, kv, r, context, tiles, num_tiles, rot_dim, p, static_cast<cudaStream_t>(stream));
+}
+
+// The same kernel over ordinary keys and values: q [tokens, heads, dim padded to 64 with zeros]; kv [context rows, kv_heads *
+// (dim + vdim)]; sinks: optional [heads]; gate: optional logits [tokens, ld_gate], one per output channel.
+SLLM_EXPORT int sllm_kv_prefill(const void* q, int tokens, const void* kv, int context, const int* tiles, int num_tiles, int heads,
+                                int kv_heads, int dim, int vdim, int window, float scale, const float* sinks, const void* gate,
+                                long long ld_gate, void* out, int* status, void* stream) {
+  if (!q || !kv || !tiles || !out || tokens <= 0 || context <= 0 || num_tiles <= 0 || heads <= 0 || heads > 65535 || kv_heads <= 0 ||
+      heads % kv_heads || dim <= 0 || vdim <= 0 || window < 0)
+    return SLLM_ERR_INVALID_ARGUMENT;
+  if (gate && ((ld_gate & 7) || (reinterpret_cast<uintptr_t>(gate) & 15))) return SLLM_ERR_ALIGNMENT;
+  LatentPrefillParams p = {};
+  p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim; p.window = window; p.scale_log2 = scale * 1.4426950408889634f;
+  p.sinks = sinks; p.gate = static_cast<const __nv_bfloat16*>(gate); p.ld_gate = ld_gate; p.gate_channels = 1;
+  p.out = static_cast<__nv_bfloat16*>(out); p.status = status;
+  return latent_prefill_impl(q, tokens, kv, nullptr, context, tiles, num_tiles, 0, p, static_cast<cudaStream_t>(stream));
 }

@@ -1,7 +1,8 @@
 // Mixture-of-experts routing and token movement.
 //
 //   moe_route        router logits [T, E] -> top-k experts per token and their weights (softmax over the k
-//                    selected logits, or the selected entries of the softmax over all experts);
+//                    selected logits, or the selected entries of the softmax over all experts), optionally from the
+//                    best groups of experts only; moe_router computes the logits as well;
 //   moe_permute      groups the T x k assignments by expert: tok_off[E_local + 1], perm_src[P] (source token of
 //                    each permuted row), perm_dst[T, k] (row of each assignment, -1 when the expert is not local),
 //                    perm_w[P] (routing weight of each permuted row);
@@ -18,80 +19,161 @@
 //
 // Reference counterparts: reference_sparse_moe_route (crates/sllm-core/src/moe.rs:229), the routing / expert
 // kernels of native/hip/src/moe_expert_kernel.hip.cpp (one request at a time, no expert parallelism).
-#include "common.cuh"
+#include "typed.cuh"
 #include "api.h"
 
 namespace sllm {
 
-constexpr int kMaxTopK = 8;
+constexpr int kMaxTopK = 32;
 constexpr int kMaxExperts = 256;
+constexpr int kRouteSlots = kMaxExperts / 32;
+
+struct RouteRule {
+  int experts, top_k, softmax_all;
+  int group_size, keep;      // only experts of the `keep` groups with the largest scores are eligible (keep 0: all)
+};
+
+// Largest of the eligible v over a warp, ties to the lower index; index 0x7fffffff when there is none.
+__device__ __forceinline__ void route_best(const float (&v)[kRouteSlots], unsigned eligible, int lane, float& best, int& bi) {
+  best = -INFINITY;
+  bi = 0x7fffffff;
+#pragma unroll
+  for (int i = 0; i < kRouteSlots; ++i) {
+    const int e = i * 32 + lane;
+    if (((eligible >> i) & 1u) && v[i] != -INFINITY && (v[i] > best || (v[i] == best && e < bi))) {
+      best = v[i];
+      bi = e;
+    }
+  }
+  for (int off = 16; off > 0; off >>= 1) {
+    const float ob = __shfl_xor_sync(0xffffffffu, best, off);
+    const int oi = __shfl_xor_sync(0xffffffffu, bi, off);
+    if (ob > best || (ob == best && oi < bi)) {
+      best = ob;
+      bi = oi;
+    }
+  }
+}
+
+// One warp routes one token: v[i] is the logit of expert i * 32 + lane (-inf past the experts and for NaN).
+template <bool kExact>
+__device__ __forceinline__ void route_warp(const float (&v)[kRouteSlots], int lane, const RouteRule& rule, int* __restrict__ out_idx,
+                                           float* __restrict__ out_w) {
+  auto ex = [](float x) { return kExact ? expf(x) : __expf(x); };
+  float denom_all = 0.f, mx_all = -INFINITY;
+  if (rule.softmax_all) {
+#pragma unroll
+    for (int i = 0; i < kRouteSlots; ++i) mx_all = fmaxf(mx_all, v[i]);
+    mx_all = warp_max(mx_all);
+#pragma unroll
+    for (int i = 0; i < kRouteSlots; ++i) denom_all += (v[i] == -INFINITY) ? 0.f : ex(v[i] - mx_all);
+    denom_all = warp_sum(denom_all);
+  }
+  unsigned eligible = 0xffffffffu;
+  float best;
+  int bi;
+  if (rule.keep > 0) {
+    unsigned kept = 0u;
+    for (int g = 0; g < rule.keep; ++g) {
+      route_best(v, ~kept, lane, best, bi);
+      if (bi == 0x7fffffff) break;
+#pragma unroll
+      for (int i = 0; i < kRouteSlots; ++i)
+        if ((i * 32 + lane) / rule.group_size == bi / rule.group_size) kept |= 1u << i;
+    }
+    eligible = kept;
+  }
+  float my_v = -INFINITY;
+  int my_i = lane;
+  for (int j = 0; j < rule.top_k; ++j) {
+    route_best(v, eligible, lane, best, bi);
+    if (bi == 0x7fffffff) bi = j;     // fewer finite logits than k: fall back to distinct low indices
+    if (lane == j) {
+      my_v = best;
+      my_i = bi;
+    }
+    if ((bi & 31) == lane) eligible &= ~(1u << (bi >> 5));
+  }
+  // mode 0: softmax over the selected logits; mode 1: probabilities of the softmax over all experts
+  const float m0 = rule.softmax_all ? mx_all : __shfl_sync(0xffffffffu, my_v, 0);
+  const float w = lane >= rule.top_k || my_v == -INFINITY ? 0.f : ex(my_v - m0);
+  const float sum = warp_sum(w);
+  const float total = rule.softmax_all ? denom_all : sum;
+  if (lane < rule.top_k) {
+    out_idx[lane] = my_i;
+    out_w[lane] = sum > 0.f && total > 0.f ? w / total : 1.f / rule.top_k;
+  }
+}
 
 // One warp per token.  Ties go to the lower expert index; NaN logits count as -inf.
-__global__ void moe_route_kernel(const __nv_bfloat16* __restrict__ logits, int ld, int tokens, int experts, int top_k,
-                                 int softmax_all, int* __restrict__ out_idx, float* __restrict__ out_w) {
+template <typename T>
+__global__ void moe_route_kernel(const T* __restrict__ logits, int ld, int tokens, RouteRule rule, int* __restrict__ out_idx,
+                                 float* __restrict__ out_w) {
   pdl_wait();
   pdl_trigger();
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   if (warp >= tokens) return;
-  float v[kMaxExperts / 32];
+  float v[kRouteSlots];
 #pragma unroll
-  for (int i = 0; i < kMaxExperts / 32; ++i) {
+  for (int i = 0; i < kRouteSlots; ++i) {
     const int e = i * 32 + lane;
-    float x = e < experts ? __bfloat162float(logits[static_cast<size_t>(warp) * ld + e]) : -INFINITY;
+    const float x = e < rule.experts ? ld_f(logits + static_cast<size_t>(warp) * ld + e) : -INFINITY;
     v[i] = (x == x) ? x : -INFINITY;
   }
-  float denom_all = 0.f, mx_all = -INFINITY;
-  if (softmax_all) {
+  route_warp<sizeof(T) == 4>(v, lane, rule, out_idx + static_cast<size_t>(warp) * rule.top_k, out_w + static_cast<size_t>(warp) * rule.top_k);
+}
+
+// Router product (fp32 sums, never rounded) and selection of one token per CTA: decode batches and 32-bit models.
+template <typename T>
+__global__ void __launch_bounds__(256)
+moe_router_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ w, int d, RouteRule rule, int vec, int* __restrict__ out_idx,
+                  float* __restrict__ out_w) {
+  pdl_wait();
+  pdl_trigger();
+  extern __shared__ __align__(16) float row[];          // [d]
+  __shared__ float z[kMaxExperts];
+  constexpr int V = kVec16<T>;
+  const T* src = x + static_cast<size_t>(blockIdx.x) * ldx;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int c = threadIdx.x; c < d; c += 256) row[c] = ld_f(src + c);
+  __syncthreads();
+  for (int e0 = warp * 4; e0 < rule.experts; e0 += 32) {
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    if (vec) {
+      for (int c = lane * V; c < d; c += 32 * V) {
+        float v[4][V];
 #pragma unroll
-    for (int i = 0; i < kMaxExperts / 32; ++i) mx_all = fmaxf(mx_all, v[i]);
-    mx_all = warp_max(mx_all);
+        for (int j = 0; j < 4; ++j)
+          if (e0 + j < rule.experts) ld16(w + static_cast<size_t>(e0 + j) * d + c, v[j]);
 #pragma unroll
-    for (int i = 0; i < kMaxExperts / 32; ++i) denom_all += (v[i] == -INFINITY) ? 0.f : __expf(v[i] - mx_all);
-    denom_all = warp_sum(denom_all);
-  }
-  float sel_v[kMaxTopK];
-  int sel_i[kMaxTopK];
-  for (int j = 0; j < top_k; ++j) {
-    float best = -INFINITY;
-    int bi = 0x7fffffff;
+        for (int j = 0; j < 4; ++j)
+          if (e0 + j < rule.experts) {
 #pragma unroll
-    for (int i = 0; i < kMaxExperts / 32; ++i) {
-      const int e = i * 32 + lane;
-      if (v[i] > best || (v[i] == best && e < bi && v[i] != -INFINITY)) {
-        best = v[i];
-        bi = e;
+            for (int i = 0; i < V; ++i) acc[j] = fmaf(v[j][i], row[c + i], acc[j]);
+          }
       }
-    }
-    for (int off = 16; off > 0; off >>= 1) {
-      const float ob = __shfl_xor_sync(0xffffffffu, best, off);
-      const int oi = __shfl_xor_sync(0xffffffffu, bi, off);
-      if (ob > best || (ob == best && oi < bi)) {
-        best = ob;
-        bi = oi;
-      }
-    }
-    if (bi == 0x7fffffff) bi = j;     // fewer finite logits than k: fall back to distinct low indices
-    sel_v[j] = best;
-    sel_i[j] = bi;
+    } else {
+      for (int c = lane; c < d; c += 32)
 #pragma unroll
-    for (int i = 0; i < kMaxExperts / 32; ++i)
-      if (i * 32 + lane == bi) v[i] = -INFINITY;
-  }
-  if (lane == 0) {
-    float w[kMaxTopK];
-    float sum = 0.f;
-    const float m0 = softmax_all ? mx_all : sel_v[0];
-    for (int j = 0; j < top_k; ++j) {
-      w[j] = sel_v[j] == -INFINITY ? 0.f : __expf(sel_v[j] - m0);
-      sum += w[j];
+        for (int j = 0; j < 4; ++j)
+          if (e0 + j < rule.experts) acc[j] = fmaf(ld_f(w + static_cast<size_t>(e0 + j) * d + c), row[c], acc[j]);
     }
-    // mode 0: softmax over the selected logits; mode 1: probabilities of the softmax over all experts
-    const float inv = softmax_all ? (denom_all > 0.f ? 1.f / denom_all : 0.f) : (sum > 0.f ? 1.f / sum : 0.f);
-    for (int j = 0; j < top_k; ++j) {
-      out_idx[warp * top_k + j] = sel_i[j];
-      out_w[warp * top_k + j] = sum > 0.f ? w[j] * inv : 1.f / top_k;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      acc[j] = warp_sum(acc[j]);
+      if (lane == 0 && e0 + j < rule.experts) z[e0 + j] = acc[j];
     }
   }
+  __syncthreads();
+  if (warp != 0) return;
+  float v[kRouteSlots];
+#pragma unroll
+  for (int i = 0; i < kRouteSlots; ++i) {
+    const int e = i * 32 + lane;
+    const float t = e < rule.experts ? z[e] : -INFINITY;
+    v[i] = (t == t) ? t : -INFINITY;
+  }
+  route_warp<true>(v, lane, rule, out_idx + static_cast<size_t>(blockIdx.x) * rule.top_k, out_w + static_cast<size_t>(blockIdx.x) * rule.top_k);
 }
 
 // Single CTA of kPermuteThreads threads.  Counts per local expert in shared memory, exclusive scan, then a stable
@@ -511,14 +593,50 @@ SLLM_EXPORT int sllm_moe_owner_combine(void* const* recv, void* const* gath, voi
   return SLLM_OK;
 }
 
-SLLM_EXPORT int sllm_moe_route(const void* logits, int ld, int tokens, int experts, int top_k, int softmax_all,
-                               int* out_idx, float* out_w, void* stream) {
-  if (!logits || !out_idx || !out_w || tokens <= 0 || experts <= 0 || experts > kMaxExperts || top_k <= 0 ||
-      top_k > kMaxTopK || top_k > experts)
+static int route_rule(RouteRule* r, int experts, int top_k, int softmax_all, int groups, int keep) {
+  if (experts <= 0 || experts > kMaxExperts || top_k <= 0 || top_k > kMaxTopK || top_k > experts || groups < 0 || keep < 0)
     return SLLM_ERR_INVALID_ARGUMENT;
-  cudaError_t e = launch_kernel(moe_route_kernel, dim3((tokens + 3) / 4), dim3(128), 0, static_cast<cudaStream_t>(stream),
-                                1u, static_cast<const __nv_bfloat16*>(logits), ld, tokens, experts, top_k, softmax_all,
-                                out_idx, out_w);
+  r->experts = experts; r->top_k = top_k; r->softmax_all = softmax_all; r->group_size = experts; r->keep = 0;
+  if (groups > 1) {
+    if (experts % groups || keep < 1 || keep > groups || keep * (experts / groups) < top_k) return SLLM_ERR_INVALID_ARGUMENT;
+    r->group_size = experts / groups;
+    r->keep = keep == groups ? 0 : keep;
+  }
+  return SLLM_OK;
+}
+
+// groups > 1: neighbouring experts form that many equal groups, a group's score is its largest, and only experts of the
+// `keep` best groups are selected.  fp32: element type of the logits (0 bf16, 1 fp32).
+SLLM_EXPORT int sllm_moe_route(const void* logits, int ld, int tokens, int experts, int top_k, int softmax_all, int groups, int keep,
+                               int fp32, int* out_idx, float* out_w, void* stream) {
+  RouteRule rule;
+  if (!logits || !out_idx || !out_w || tokens <= 0 || ld < experts) return SLLM_ERR_INVALID_ARGUMENT;
+  const int rc = route_rule(&rule, experts, top_k, softmax_all, groups, keep);
+  if (rc != SLLM_OK) return rc;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const cudaError_t e = fp32 ? launch_kernel(moe_route_kernel<float>, dim3((tokens + 3) / 4), dim3(128), 0, st, 1u,
+                                             static_cast<const float*>(logits), ld, tokens, rule, out_idx, out_w)
+                             : launch_kernel(moe_route_kernel<__nv_bfloat16>, dim3((tokens + 3) / 4), dim3(128), 0, st, 1u,
+                                             static_cast<const __nv_bfloat16*>(logits), ld, tokens, rule, out_idx, out_w);
+  return e == cudaSuccess ? SLLM_OK : SLLM_ERR_CUDA;
+}
+
+// Router product x w^T (x [tokens, d], w [experts, d], both bf16 or both fp32) and the selection in one launch.
+SLLM_EXPORT int sllm_moe_router(const void* x, int ldx, const void* w, int tokens, int d, int experts, int top_k, int softmax_all,
+                                int groups, int keep, int fp32, int* out_idx, float* out_w, void* stream) {
+  RouteRule rule;
+  if (!x || !w || !out_idx || !out_w || tokens <= 0 || d <= 0 || ldx < d) return SLLM_ERR_INVALID_ARGUMENT;
+  const int rc = route_rule(&rule, experts, top_k, softmax_all, groups, keep);
+  if (rc != SLLM_OK) return rc;
+  const size_t smem = sizeof(float) * d;
+  if (smem > 40 * 1024) return SLLM_ERR_UNSUPPORTED_SHAPE;
+  const int vec = d % (fp32 ? 4 : 8) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const cudaError_t e = fp32 ? launch_kernel(moe_router_kernel<float>, dim3(tokens), dim3(256), smem, st, 1u,
+                                             static_cast<const float*>(x), ldx, static_cast<const float*>(w), d, rule, vec, out_idx, out_w)
+                             : launch_kernel(moe_router_kernel<__nv_bfloat16>, dim3(tokens), dim3(256), smem, st, 1u,
+                                             static_cast<const __nv_bfloat16*>(x), ldx, static_cast<const __nv_bfloat16*>(w), d, rule,
+                                             vec, out_idx, out_w);
   return e == cudaSuccess ? SLLM_OK : SLLM_ERR_CUDA;
 }
 

@@ -13,7 +13,7 @@ from typing import Optional
 @dataclass
 class ModelConfig:
     name: str = "tiny-llama"
-    family: str = "llama"            # llama | moe | qwen35 | gemma4 | zokuvik
+    family: str = "llama"            # llama | moe | qwen35 | gemma4 | zokuvik | sepedra
     n_layers: int = 2
     d_model: int = 256
     n_heads: int = 4
@@ -62,7 +62,7 @@ class ModelConfig:
     layer_scalar: bool = False       # the residual stream is multiplied by a learned scalar at the end of every layer
     k_equals_v_full: bool = False    # full-attention layers have no value projection: v = the (un-normed) key projection
     # families whose layers differ in kind and size: one dict per layer, {"type": mixer kind, "mixer": {sizes}, "mlp":
-    # {"kind", "ff"} or None}; the norms split a vector into norm_groups parts
+    # {"kind", ...} or None}; the norms split a vector into norm_groups parts
     layer_specs: Optional[list] = None
     norm_groups: int = 1
     # vision-language models: rotary pairs [0, t) follow the temporal index, [t, t + h) the height index and the rest
@@ -171,7 +171,13 @@ def _zokuvik():
     return zokuvik_shape()
 
 
+def _sepedra():
+    from .sepedra import sepedra_shape
+    return sepedra_shape()
+
+
 NAMED = {
+    "sepedra": _sepedra,
     "zokuvik": _zokuvik,
     "qwen35-moe": _qwen35_moe,
     "qwen35-moe-hybrid": _qwen35_moe_hybrid,

@@ -11,8 +11,8 @@ ffn_gate_inp (router; rows past n_experts: the shared-expert gate and zero paddi
 ffn_gate_up_shexp | ffn_down_shexp.  Hybrid layer i: blk.i.attn_norm | ffn_norm | ffn_gate | ffn_up | ffn_down (or, with
 a sparse MLP, the ffn_gate_inp / ffn_*_exps / ffn_*_shexp tensors of the MoE layer) and either
 attn_q | attn_k | attn_v | attn_gate | attn_output | attn_q_norm | attn_k_norm (full attention) or ssm_in | ssm_conv1d |
-ssm_a | ssm_dt | ssm_norm | ssm_out (gated delta net).  A `zokuvik` file keeps the design's own names (models/zokuvik.py,
-source_shapes): its layers differ in kind and size, and the configuration in the metadata lists them.
+ssm_a | ssm_dt | ssm_norm | ssm_out (gated delta net).  A `zokuvik` or `sepedra` file keeps the design's own names
+(source_shapes of its module): its layers differ in kind and size, and the configuration in the metadata lists them.
 
 Reference: the per-family conversion plans of crates/sllm-core/src/gguf_convert.rs:145-704 (Qwen3.5 BF16 / FP8 /
 MoE-MXFP4 plans) and the expert tensor contract of crates/sllm-core/src/qwen35_moe.rs:1277-1600.
@@ -31,8 +31,9 @@ from ..ops.core import LinearWeight
 from ..ops.w4 import W4Weight
 from .config import ModelConfig
 from .loader import CONVERTER_ID, FP8_ENCODING, MXFP4_ENCODING, NVFP4_ENCODING, config_from_gguf
+from .registry import LAYERED, layered
 
-FAMILIES = ("moe", "qwen35", "zokuvik")
+FAMILIES = ("moe", "qwen35", *LAYERED)
 
 
 def _bytes(t: torch.Tensor) -> tuple:
@@ -146,15 +147,14 @@ def _sink_blocks(s: _Sink, cfg: ModelConfig, w) -> None:
 def export_family_gguf(cfg: ModelConfig, w, path: str, tokenizer_json: Optional[str] = None,
                        chat_template: Optional[str] = None, converter_args: Optional[dict] = None,
                        known_unconsumed: Optional[list] = None, source_fingerprints: tuple = ()) -> dict:
-    """Writes unsharded weights of a `moe`, `qwen35` or `zokuvik` model; returns the derived lock document.  `known_unconsumed`
+    """Writes unsharded weights of a model of FAMILIES; returns the derived lock document.  `known_unconsumed`
     names source tensors the converter left out on purpose (vision tower, multi-token-prediction head); they are
     recorded in the tensor recipe."""
     if cfg.family not in FAMILIES:
         raise G.GgufError(f"family {cfg.family!r} is written by models.loader.export_llama_gguf")
     s = _Sink()
-    if cfg.family == "zokuvik":
-        from .zokuvik import named_tensors
-        for name, t in named_tensors(cfg, w):
+    if cfg.family in LAYERED:
+        for name, t in layered(cfg.family).named_tensors(cfg, w):
             s.dense(name, t)
     else:
         _sink_blocks(s, cfg, w)
@@ -306,21 +306,20 @@ class _Source:
 
 def load_family_gguf(g: G.GgufFile, device, tp_size: int = 1, tp_rank: int = 0, ep_size: int = 1, ep_rank: int = 0,
                      kv_format: Optional[str] = None):
-    """(cfg, weights) of this rank for a `moe`, `qwen35` or `zokuvik` file."""
+    """(cfg, weights) of this rank for a file of FAMILIES."""
     cfg = config_from_gguf(g)
     if cfg.family not in FAMILIES:
         raise G.GgufError(f"family {cfg.family!r} is read by models.loader.load_llama_gguf")
     if kv_format:
         cfg.kv_format = kv_format
     src = _Source(g, cfg, device)
-    if cfg.family == "zokuvik":
+    if cfg.family in LAYERED:
         if tp_size != 1 or ep_size != 1:
-            raise G.GgufError("the zokuvik family runs on one GPU")
-        from .zokuvik import pack_weights
+            raise G.GgufError(f"the {cfg.family} family runs on one GPU")
         try:
-            return cfg, pack_weights(cfg, lambda n: src.dense(n, keep_f32=True), device)
+            return cfg, layered(cfg.family).pack_weights(cfg, lambda n: src.dense(n, keep_f32=True), device)
         except (KeyError, ValueError) as exc:
-            raise G.GgufError(f"unusable zokuvik file: {exc}") from None
+            raise G.GgufError(f"unusable {cfg.family} file: {exc}") from None
     L = src.to_linear
     d, hd, hq, hkv, f = cfg.d_model, cfg.head_dim, cfg.n_heads, cfg.n_kv_heads, cfg.ffn
     if hq % tp_size or (hkv % tp_size and tp_size % hkv):

@@ -20,6 +20,7 @@ from ..formats import gguf as G
 from ..ops.core import LinearWeight
 from .config import ModelConfig
 from .llama import LayerWeights, LlamaWeights
+from .registry import LAYERED
 
 CONVERTER_ID = "sllm-b200-convert-gguf-v1"
 FP8_ENCODING = "fp8-e4m3fn-kblock128-f32-scale"
@@ -299,9 +300,9 @@ def load_llama_gguf(g: G.GgufFile, device, tp_size: int = 1, tp_rank: int = 0, k
 def load_model_gguf(g: G.GgufFile, device, tp_size: int = 1, tp_rank: int = 0, ep_size: int = 1, ep_rank: int = 0,
                     kv_format: Optional[str] = None):
     """(cfg, weights, family) of this rank for any model family a file can carry: the dense decoder (`llama`,
-    `gemma4`) through load_llama_gguf, `moe`, `qwen35` and `zokuvik` through models.family_io."""
+    `gemma4`) through load_llama_gguf, `moe`, `qwen35`, `zokuvik` and `sepedra` through models.family_io."""
     cfg = config_from_gguf(g)
-    if cfg.family in ("moe", "qwen35", "zokuvik"):
+    if cfg.family in ("moe", "qwen35", *LAYERED):
         from . import family_io
         cfg, w = family_io.load_family_gguf(g, device, tp_size, tp_rank, ep_size, ep_rank, kv_format=kv_format)
         return cfg, w, cfg.family

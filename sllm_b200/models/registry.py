@@ -15,7 +15,19 @@ from .config import ModelConfig
 KERNEL_UNITS = {
     "zokuvik": ("elementwise", "gemm_tcgen05", "gemm_simt", "group_norm", "latent_attention", "latent_decode", "latent_prefill",
                 "delta_rule"),
+    "sepedra": ("elementwise", "gemm_tcgen05", "gemm_simt", "group_norm", "attention", "kv_attention", "latent_prefill", "rglru", "moe",
+                "moe_dense"),
 }
+
+# families whose configuration lists its layers (ModelConfig.layer_specs): modules with ARCHITECTURE, config_from_source,
+# pack_weights, named_tensors and make_cache.  They run on one GPU, in bf16 or fp32
+LAYERED = ("zokuvik", "sepedra")
+
+
+def layered(family: str):
+    """The module of a family in LAYERED."""
+    import importlib
+    return importlib.import_module(f".{family}", __package__)
 
 
 def make_model(cfg: ModelConfig, weights, tp=None, ep=None):
@@ -28,6 +40,9 @@ def make_model(cfg: ModelConfig, weights, tp=None, ep=None):
     if cfg.family == "zokuvik":
         from .zokuvik import ZokuvikModel
         return ZokuvikModel(cfg, weights, tp)
+    if cfg.family == "sepedra":
+        from .sepedra import SepedraModel
+        return SepedraModel(cfg, weights, tp)
     from .llama import LlamaModel
     return LlamaModel(cfg, weights, tp)
 
@@ -37,9 +52,8 @@ def make_cache(cfg: ModelConfig, model, num_pages: int, device, max_seqs: int):
     if cfg.family == "qwen35":
         from ..cache.hybrid import HybridCache
         return HybridCache(cfg, num_pages, device, max_seqs=max_seqs, kv_heads=model.local_kv_heads, tp_size=model.tp.size)
-    if cfg.family == "zokuvik":
-        from .zokuvik import make_cache as make
-        return make(cfg, model, num_pages, device, max_seqs)
+    if cfg.family in LAYERED:
+        return layered(cfg.family).make_cache(cfg, model, num_pages, device, max_seqs)
     from ..cache.paged import PagedKVCache
     return PagedKVCache(cfg, num_pages, device, kv_heads=model.local_kv_heads)
 
@@ -55,6 +69,9 @@ def init_random_weights(cfg: ModelConfig, device, seed: int = 0, tp_size: int = 
     if cfg.family == "zokuvik":
         from .zokuvik import init_random_zokuvik_weights
         return init_random_zokuvik_weights(cfg, device, seed)
+    if cfg.family == "sepedra":
+        from .sepedra import init_random_sepedra_weights
+        return init_random_sepedra_weights(cfg, device, seed)
     from .llama import init_random_weights as init
     return init(cfg, device, seed, tp_size, tp_rank)
 
@@ -66,8 +83,7 @@ class ModelFolderError(RuntimeError):
 
 def read_folder_config(path: str, dtype: str = "bf16", max_context: Optional[int] = None) -> ModelConfig:
     """ModelConfig of a folder with config.json, chosen by its ``architecture``."""
-    from . import zokuvik
-    readers = {zokuvik.ARCHITECTURE: zokuvik.config_from_source}
+    readers = {m.ARCHITECTURE: m.config_from_source for m in map(layered, LAYERED)}
     try:
         with open(os.path.join(path, "config.json"), "r", encoding="utf-8") as f:
             d = json.load(f)
@@ -83,9 +99,8 @@ def read_folder_config(path: str, dtype: str = "bf16", max_context: Optional[int
 def load_folder_weights(path: str, cfg: ModelConfig, device):
     """Resident weights of a folder with model.safetensors."""
     from ..formats.safetensors import SafetensorsError, SafetensorsFile
-    from .zokuvik import pack_weights
     try:
         with SafetensorsFile(os.path.join(path, "model.safetensors")) as f:
-            return pack_weights(cfg, f.tensor, torch.device(device))
+            return layered(cfg.family).pack_weights(cfg, f.tensor, torch.device(device))
     except (OSError, ValueError, SafetensorsError) as exc:
         raise ModelFolderError(f"{path}: unusable model.safetensors: {exc}") from None

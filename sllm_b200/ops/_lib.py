@@ -166,9 +166,9 @@ def check(rc: int, what: str) -> None:
 _KERNEL_SIGNATURES = {
     "sllm_gemm_workspace_floats": (L, [I, I, I, I]),
     "sllm_gemm": (I, [P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, P, L, P, I, P, P]),
-    "sllm_gemm_act": (I, [P, P, P, I, I, I, I, I, I, I, I, I, P, L, P, I, P, P]),
-    "sllm_gemm_simt": (I, [P, P, P, P, I, I, I, I, I, I, I, I, P]),
-    "sllm_group_norm": (I, [P, P, I, P, I, P, P, P, P, P, I, I, I, F, I, P]),
+    "sllm_gemm_act": (I, [P, P, P, I, I, I, I, I, I, F, I, I, I, I, P, L, P, I, P, P]),
+    "sllm_gemm_simt": (I, [P, P, P, P, I, I, I, I, I, I, I, F, I, I, P]),
+    "sllm_group_norm": (I, [P, P, I, P, I, P, I, P, P, P, P, P, I, I, I, F, I, P]),
     "sllm_embedding": (I, [P, P, P, I, I, I, F, P]),
     "sllm_rmsnorm": (I, [P, P, P, P, P, I, I, I, F, I, P]),
     "sllm_gated_act": (I, [P, P, P, P, I, I, I, I, P]),
@@ -185,7 +185,7 @@ _KERNEL_SIGNATURES = {
     "sllm_prefill_attention": (I, [P, I, I, P, I, I, I, I, F, P, P, P, I, P, P]),
     "sllm_paged_attention_workspace_floats": (L, [I, I, I, I, I]),
     "sllm_paged_attention": (I, [P, I, P, P, P, P, F, F, P, I, P, P, I, I, I, I, I, I, F, I, P, P, P, I, P, I, P, L,
-                                  P, I, P]),
+                                  P, I, P, L, P]),
 }
 
 # Entry points added by later translation units register themselves here (name -> (restype, argtypes)).

@@ -156,24 +156,30 @@ def gemm_raw(a: torch.Tensor, b: torch.Tensor, y: torch.Tensor, *, scale_a=None,
     _lib.check(rc, "gemm")
 
 
-def _linear_simt(x: torch.Tensor, w: torch.Tensor, residual: Optional[torch.Tensor], act: Optional[str]) -> torch.Tensor:
+_ACTS = {None: 0, "relu_sq": 1, "softcap": 2}
+
+
+def _linear_simt(x: torch.Tensor, w: torch.Tensor, residual: Optional[torch.Tensor], act: Optional[str], act_arg: float,
+                 out_fp32: bool) -> torch.Tensor:
     """CUDA-core product: fp32 operands, or bf16 rows that a TMA copy cannot address (K not a multiple of 8)."""
     m, k = x.shape
     n = w.shape[0]
     if x.dtype != w.dtype or x.stride(1) != 1:
         raise ValueError("the CUDA-core product takes operands of one type with contiguous rows")
-    y = torch.empty((m, n), dtype=x.dtype, device=x.device)
-    rc = _lib.kernels().sllm_gemm_simt(_p(x), _p(w), _p(y), _p(residual), m, n, k, x.stride(0), w.stride(0), n,
-                                       1 if act else 0, int(x.dtype == torch.float32), _stream())
+    y = torch.empty((m, n), dtype=torch.float32 if out_fp32 else x.dtype, device=x.device)
+    rc = _lib.kernels().sllm_gemm_simt(_p(x), _p(w), _p(y), _p(residual), m, n, k, x.stride(0), w.stride(0), n, _ACTS[act], act_arg,
+                                       int(x.dtype == torch.float32), int(out_fp32), _stream())
     _lib.check(rc, "gemm_simt")
     return y
 
 
-def linear(x, w: LinearWeight, residual: Optional[torch.Tensor] = None, act: Optional[str] = None) -> torch.Tensor:
-    """Y = act(X W^T) (+ residual).  x: Tensor [M, K] (bf16 / fp32) or QTensor for FP8 weights.  ``act``: None or
-    "relu_sq" (square of relu; dense weights, without a residual), applied to the fp32 sums."""
-    if act is not None and (act != "relu_sq" or w.kind != "dense" or residual is not None):
-        raise ValueError("the product's activation is relu_sq, on dense weights without a residual")
+def linear(x, w: LinearWeight, residual: Optional[torch.Tensor] = None, act: Optional[str] = None, act_arg: float = 0.0,
+           out_fp32: bool = False) -> torch.Tensor:
+    """Y = act(X W^T) (+ residual).  x: Tensor [M, K] (bf16 / fp32) or QTensor for FP8 weights.  ``act``: None, "relu_sq"
+    (square of relu) or "softcap" (act_arg * tanh(y / act_arg)), applied to the fp32 sums; ``out_fp32`` stores the sums
+    unrounded.  Both take dense weights without a residual."""
+    if act not in _ACTS or ((act or out_fp32) and (w.kind != "dense" or residual is not None)):
+        raise ValueError("the product's activation is relu_sq or softcap, on dense weights without a residual")
     xd = x.data if isinstance(x, QTensor) else x
     if w.kind == "w4":
         from .w4 import linear_w4
@@ -186,22 +192,26 @@ def linear(x, w: LinearWeight, residual: Optional[torch.Tensor] = None, act: Opt
         if w.kind == "fp8" and not isinstance(x, QTensor):
             xf = ref.dequant_fp8_1x128(*ref.quant_fp8_1x128(x))
         y = xf @ w.dequantized().t()
-        if act:
+        if act == "relu_sq":
             y = torch.relu(y) ** 2
+        elif act == "softcap":
+            y = act_arg * torch.tanh(y / act_arg)
+        if out_fp32:
+            return y
         if residual is not None:
             y = y + residual.to(torch.float32)
         return y.to(residual.dtype if residual is not None else (torch.float32 if w.w.dtype == torch.float32 else torch.bfloat16))
     m = xd.shape[0]
     n = w.out_features
     if w.kind == "dense" and (xd.dtype == torch.float32 or w.in_features % 8):
-        return _linear_simt(xd, w.w, residual, act)
+        return _linear_simt(xd, w.w, residual, act, act_arg, out_fp32)
     if w.kind == "fp8":
         if not isinstance(x, QTensor):
             x = quant_fp8(x)
         k_blocks = (w.in_features + 127) // 128
     else:
         k_blocks = (w.in_features + 63) // 64
-    y = torch.empty((m, n), dtype=torch.bfloat16, device=xd.device)
+    y = torch.empty((m, n), dtype=torch.float32 if out_fp32 else torch.bfloat16, device=xd.device)
     swap, bn, splits, stages = _gemm_plan(m, n, k_blocks)
     if _lib.audit_enabled():
         _lib.record_dispatch("linear", "gemm_tcgen05_kernel", m=m, n=n, k=w.in_features, kind=w.kind, swap_ab=swap, bn=bn,
@@ -215,11 +225,11 @@ def linear(x, w: LinearWeight, residual: Optional[torch.Tensor] = None, act: Opt
             gemm_raw(x.data, w.w, y, scale_a=x.scale, scale_b=w.scale_t, residual=residual, transpose_out=False,
                      bn=bn, splits=splits, stages=stages)
     else:
-        if act:
+        if act or out_fp32:
             a, b = (w.w, x) if swap else (x, w.w)
             wsp = workspace(xd.device)
-            rc = _lib.kernels().sllm_gemm_act(_p(a), _p(b), _p(y), a.shape[0], b.shape[0], w.in_features, int(swap), n, 1, bn, splits,
-                                              stages, _p(wsp.ws), wsp.ws.numel(), _p(wsp.counters), wsp.counters.numel(),
+            rc = _lib.kernels().sllm_gemm_act(_p(a), _p(b), _p(y), a.shape[0], b.shape[0], w.in_features, int(swap), n, _ACTS[act],
+                                              act_arg, int(out_fp32), bn, splits, stages, _p(wsp.ws), wsp.ws.numel(), _p(wsp.counters), wsp.counters.numel(),
                                               _p(wsp.status), _stream())
             _lib.check(rc, "gemm")
         elif swap:
@@ -275,35 +285,46 @@ def _gn_ref(x: torch.Tensor, w: torch.Tensor, eps: float, groups: int) -> torch.
     return (g / torch.sqrt((g * g).mean(-1, keepdim=True) + eps)).view(t, d) * w
 
 
-def _group_norm(x, w_out, eps, groups, dtype, *, table=None, ids=None, y=None, w_post=None, rows_idx=None):
+def _group_norm(x, w_out, eps, groups, dtype, *, table=None, ids=None, y=None, w_post=None, rows_idx=None, terms=None, raw=False):
     rows = ids.numel() if table is not None else (rows_idx.numel() if rows_idx is not None else x.shape[0])
     d = x.shape[1]
-    z = torch.empty((rows, d), dtype=dtype, device=x.device) if w_out is not None else None
+    z = torch.empty((rows, d), dtype=dtype, device=x.device) if w_out is not None or raw else None
     if rows == 0:
         return z
     rc = _lib.kernels().sllm_group_norm(_p(table), _p(ids), table.shape[0] if table is not None else 0, _p(y),
-                                        y.stride(0) if y is not None else 0, _p(w_post), _p(x), _p(rows_idx), _p(w_out), _p(z), rows,
-                                        d, groups, eps, int(dtype == torch.float32), _stream())
+                                        y.stride(0) if y is not None else 0, _p(terms), terms.shape[1] if terms is not None else 0,
+                                        _p(w_post), _p(x), _p(rows_idx), _p(w_out), _p(z), rows, d, groups, eps,
+                                        int(dtype == torch.float32), _stream())
     _lib.check(rc, "group_norm")
     return z
 
 
-def embed_group_norm(table: torch.Tensor, ids: torch.Tensor, w_out: torch.Tensor, eps: float, groups: int = 1):
-    """(residual fp32 [T, d], its grouped RMSNorm in the table's type): the embedding and the first layer's input norm."""
+def embed_group_norm(table: torch.Tensor, ids: torch.Tensor, w_out: Optional[torch.Tensor], eps: float, groups: int = 1):
+    """(residual fp32 [T, d], its grouped RMSNorm in the table's type): the embedding and the first layer's input norm.
+    Without ``w_out`` the second is the residual itself in the table's type."""
     if _lib.on_cpu(table):
         x = table[ids.long()].float()
-        return x, _gn_ref(x, w_out, eps, groups).to(table.dtype)
+        return x, (x if w_out is None else _gn_ref(x, w_out, eps, groups)).to(table.dtype, copy=True)
     x = torch.empty((ids.numel(), table.shape[1]), dtype=torch.float32, device=table.device)
-    return x, _group_norm(x, w_out, eps, groups, table.dtype, table=table, ids=ids)
+    return x, _group_norm(x, w_out, eps, groups, table.dtype, table=table, ids=ids, raw=True)
 
 
 def add_group_norm(x: torch.Tensor, y: torch.Tensor, w_post: torch.Tensor, w_out: Optional[torch.Tensor], eps: float,
-                   groups: int = 1):
-    """x += norm(y) * w_post in place (fp32), then norm(x) * w_out in the type of ``y`` (None without ``w_out``)."""
+                   groups: int = 1, terms: Optional[torch.Tensor] = None, raw: bool = False):
+    """x += norm(y) * w_post in place (fp32), then norm(x) * w_out in the type of ``y`` (without ``w_out``: x in that type with
+    ``raw``, else None).  ``terms`` (int32 [T, n]): row t of the summand is the sum of the rows terms[t] >= 0 of ``y``."""
     if _lib.on_cpu(x):
-        x += _gn_ref(y, w_post, eps, groups)
-        return None if w_out is None else _gn_ref(x, w_out, eps, groups).to(y.dtype)
-    return _group_norm(x, w_out, eps, groups, y.dtype, y=y, w_post=w_post)
+        s = y
+        if terms is not None:
+            s = torch.zeros_like(x)
+            for j in range(terms.shape[1]):
+                p = terms[:, j].long()
+                s[p >= 0] += y[p[p >= 0]].float()
+        x += _gn_ref(s, w_post, eps, groups)
+        if w_out is None:
+            return x.to(y.dtype, copy=True) if raw else None
+        return _gn_ref(x, w_out, eps, groups).to(y.dtype)
+    return _group_norm(x, w_out, eps, groups, y.dtype, y=y, w_post=w_post, terms=terms, raw=raw)
 
 
 def group_norm(x: torch.Tensor, w: torch.Tensor, eps: float, groups: int, dtype, rows: Optional[torch.Tensor] = None):
@@ -493,10 +514,12 @@ def _attn_splits(rows: int, hkv: int, max_kv: int) -> int:
 def paged_attention(q: torch.Tensor, kv: KVLayer, block_table: torch.Tensor, seq_index: torch.Tensor,
                     kv_lens: torch.Tensor, hq: int, hkv: int, hd: int, *, window: int = 0,
                     sm_scale: Optional[float] = None, max_kv: int = 0, quant_out: bool = False,
-                    sinks: Optional[torch.Tensor] = None, impl: Optional[str] = None, out: Optional[QTensor] = None):
+                    sinks: Optional[torch.Tensor] = None, impl: Optional[str] = None, out: Optional[QTensor] = None,
+                    gate: Optional[torch.Tensor] = None):
     """Attention of each query row over its sequence's pages. q: [R, hq*hd] (row stride allowed).
     Returns [R, hq*hd] (bf16) or a QTensor when quant_out (head_dim 128); ``out`` supplies the QTensor to fill
-    (its scale plane may have a leading dimension larger than R)."""
+    (its scale plane may have a leading dimension larger than R), or the bf16 rows.  ``gate``: logits [R, hq*hd] (row stride
+    allowed) whose sigmoid multiplies the output; not on the tensor-core kernel."""
     scale = sm_scale if sm_scale is not None else 1.0 / math.sqrt(hd)
     r = q.shape[0]
     if _lib.on_cpu(q):
@@ -522,6 +545,8 @@ def paged_attention(q: torch.Tensor, kv: KVLayer, block_table: torch.Tensor, seq
                 vv = kv.v[blks].transpose(1, 2).reshape(-1, hkv, hd).to(torch.float32)
             out[i] = ref.attention_rows(q[i].view(hq, hd), kk, vv, n, window, scale, sinks)
         out = out.view(r, hq * hd)
+        if gate is not None:
+            out = out * torch.sigmoid(gate.float())
         if q.dtype == torch.float32 and not quant_out:
             return out
         out = ref.round_bf16(out)
@@ -535,10 +560,10 @@ def paged_attention(q: torch.Tensor, kv: KVLayer, block_table: torch.Tensor, seq
         oq = out if out is not None else _alloc_q(r, hq * hd, q.device)
         out_b, out_q, out_s, ld = None, oq.data, oq.scale, max(oq.scale.stride(0), oq.scale.shape[1])
     else:
-        ob = torch.empty((r, hq * hd), dtype=torch.bfloat16, device=q.device)
+        ob = out if out is not None else torch.empty((r, hq * hd), dtype=torch.bfloat16, device=q.device)
         out_b, out_q, out_s, ld = ob, None, None, 0
     use_tc = (kv.fp8 and hd == 128 and (hq // hkv) in (1, 2, 4, 8, 16) and 128 % kv.page_size == 0
-              and kv.page_size >= 8 and impl != "cuda_core")
+              and kv.page_size >= 8 and impl != "cuda_core" and gate is None)
     if impl == "tensor_core" and not use_tc:
         raise ValueError("tensor-core decode attention needs FP8 pages, head_dim 128 and a GQA group <= 16")
     if use_tc:
@@ -565,6 +590,6 @@ def paged_attention(q: torch.Tensor, kv: KVLayer, block_table: torch.Tensor, seq
         _p(q), q.stride(0), _p(kv.k), _p(kv.v), _p(kv.k_scale), _p(kv.v_scale), kv.k_static, kv.v_static,
         _p(block_table), block_table.stride(0), _p(seq_index), _p(kv_lens), r, hq, hkv, hd, kv.page_size, window,
         scale, kv.mode, _p(out_b), _p(out_q), _p(out_s), ld, _p(sinks), splits, _p(wsp.ws), wsp.ws.numel(),
-        _p(wsp.counters), wsp.counters.numel(), _stream())
+        _p(wsp.counters), wsp.counters.numel(), _p(gate), gate.stride(0) if gate is not None else 0, _stream())
     _lib.check(rc, "paged_attention")
     return oq if quant_out else ob

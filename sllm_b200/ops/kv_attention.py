@@ -1,0 +1,232 @@
+"""Attention with keys and values of different widths: short convolutions on q, k and v, rotation in neighbouring pairs with
+scaled frequencies, unweighted query / key norms, a sink in the softmax and an output gate per channel, each optional
+(kernels in csrc/kv_attention.cu; PyTorch restatements here for CPU tensors).
+
+A layer runs  prepare  (everything between the projection and the scores, page write) -> attention.  Decoded tokens and short
+portions read the pages row by row; long portions gather them once and run on the tensor cores (csrc/latent_prefill.cu).  A
+layer that takes its keys and values from another one prepares queries only and is handed that layer's pages."""
+from __future__ import annotations
+
+import ctypes as C
+import math
+from dataclasses import dataclass
+from typing import Optional
+
+import torch
+
+from . import _lib
+from .latent import plan_portions, rotate
+from .short_conv import causal_conv
+
+P, I, F, L = C.c_void_p, C.c_int, C.c_float, C.c_longlong
+
+
+class KvPrepareArgs(C.Structure):
+    _fields_ = [(n, P) for n in ("proj", "conv_w", "ring", "inv_freq", "row_off", "slots", "positions", "seq_index", "block_table", "q",
+                                 "k_pages", "v_pages")] + [("ring_stride", L)] + \
+        [(n, I) for n in ("ldp", "max_blocks", "heads", "kv_heads", "dim", "vdim", "q_pad", "ld_k", "ld_v", "rot_dims", "taps",
+                          "page_size", "tokens", "sequences", "norm", "decode", "fp32")] + [("eps", F)]
+
+
+_SIGS = {
+    "sllm_kv_prepare": (I, [P, P]),
+    "sllm_kv_abi": (I, [P, I]),
+    "sllm_kv_gather": (I, [P, P, I, P, I, P, I, I, P, I, I, I, P]),
+    "sllm_kv_attention": (I, [P, P, P, P, L, P, P, I, P, P, I, I, I, I, I, I, I, I, I, I, F, P, I, P]),
+    "sllm_kv_prefill": (I, [P, I, P, I, P, I, I, I, I, I, I, F, P, P, L, P, P, P]),
+}
+
+
+def _k():
+    for n, s in _SIGS.items():
+        _lib.EXTRA_KERNEL_SIGNATURES.setdefault(n, s)
+    return _lib.kernels()
+
+
+def rope_frequencies(base: float, dims: int, scaling: Optional[dict] = None) -> torch.Tensor:
+    """fp64 [dims / 2].  ``scaling`` {factor, low, high, original} stretches long wavelengths: pairs that turn more than `high`
+    times within `original` positions stay, those that turn less than `low` times are slowed down by `factor`, and between
+    the two the rates are blended."""
+    f = float(base) ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / dims)
+    if not scaling:
+        return f
+    turns = float(scaling["original"]) * f / (2 * math.pi)
+    low, high, slow = float(scaling["low"]), float(scaling["high"]), f / float(scaling["factor"])
+    s = (turns - low) / (high - low) if high != low else torch.zeros_like(f)
+    return torch.where(turns > high, f, torch.where(turns < low, slow, (1 - s) * slow + s * f))
+
+
+@dataclass
+class KVSpec:
+    """Sizes and constants of one layer; its packed input projection is q | k | v | g (q | g without keys of its own)."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot_base: float
+    rot_dims: int
+    taps: int = 1
+    rot_scaling: Optional[dict] = None
+    qk_norm: bool = True
+    window: int = 0
+    own_kv: bool = True
+
+    @property
+    def q_cols(self) -> int:
+        return self.heads * self.dim
+
+    @property
+    def channels(self) -> int:
+        """Columns that the short convolution covers."""
+        return self.q_cols + (self.kv_heads * (self.dim + self.vdim) if self.own_kv else 0)
+
+    @property
+    def out_cols(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def q_pad(self) -> int:
+        return (self.dim + 63) // 64 * 64
+
+    def inv_freq(self, device) -> torch.Tensor:
+        return rope_frequencies(self.rot_base, self.rot_dims, self.rot_scaling).float().to(device)
+
+
+@dataclass
+class KVPages:
+    """One layer's pages: k [num_pages, kv_heads, page, >= dim], v [num_pages, kv_heads, page, >= vdim]."""
+    k: torch.Tensor
+    v: torch.Tensor
+    page_size: int
+
+    # what ops.paged_attention reads of a layer
+    k_scale = v_scale = None
+    fp8 = nvfp4 = False
+    k_static = v_static = 0.0
+    mode = 0
+
+
+def prepare(proj: torch.Tensor, spec: KVSpec, conv_w: torch.Tensor, inv_freq: torch.Tensor, eps: float, kv: Optional[KVPages],
+            ring: torch.Tensor, b) -> torch.Tensor:
+    """proj [T, >= channels]; conv_w [taps, channels]; ring [slots, taps, channels]; ``kv`` the layer's own pages (None: the
+    layer has no keys of its own).  Returns q [T, heads, q_pad], zero past ``dim``."""
+    t, H, G, D, V = proj.shape[0], spec.heads, spec.kv_heads, spec.dim, spec.vdim
+    if _lib.on_cpu(proj):
+        x = causal_conv(proj[:, :spec.channels].float(), conv_w, ring, b.row_off, b.slots, b.positions)
+
+        def turned(y):
+            y = rotate(y, b.positions, inv_freq, spec.rot_dims, True)
+            return y / torch.sqrt((y * y).mean(-1, keepdim=True) + eps) if spec.qk_norm else y
+        q = torch.zeros((t, H, spec.q_pad), dtype=proj.dtype)
+        q[..., :D] = turned(x[:, :spec.q_cols].reshape(t, H, D)).to(proj.dtype)
+        if kv is not None:
+            k = turned(x[:, spec.q_cols:spec.q_cols + G * D].reshape(t, G, D))
+            v = x[:, spec.q_cols + G * D:].reshape(t, G, V)
+            pos = b.positions.long()
+            blk = b.block_table[b.seq_index.long(), pos // kv.page_size].long()
+            kv.k[blk, :, pos % kv.page_size, :D] = k.to(kv.k.dtype)
+            kv.v[blk, :, pos % kv.page_size, :V] = v.to(kv.v.dtype)
+        return q
+    from .core import _stream
+    q = torch.empty((t, H, spec.q_pad), dtype=proj.dtype, device=proj.device)
+    p = lambda x: None if x is None else x.data_ptr()
+    decode = b.row_off_host is None and t == b.slots.numel()
+    own = kv is not None
+    args = KvPrepareArgs(p(proj), p(conv_w), p(ring), p(inv_freq), p(b.row_off), p(b.slots), p(b.positions), p(b.seq_index),
+                         p(b.block_table), p(q), p(kv.k) if own else None, p(kv.v) if own else None, ring.stride(0), proj.stride(0),
+                         b.block_table.stride(0), H, G if own else 0, D, V, spec.q_pad, kv.k.shape[3] if own else 0,
+                         kv.v.shape[3] if own else 0, spec.rot_dims, spec.taps, kv.page_size if own else 1, t, b.slots.numel(),
+                         int(spec.qk_norm), int(decode), int(proj.dtype == torch.float32), eps)
+    _lib.check(_k().sllm_kv_prepare(C.byref(args), _stream()), "kv_prepare")
+    return q
+
+
+def paged_rows(q: torch.Tensor, gate: Optional[torch.Tensor], spec: KVSpec, kv: KVPages, sinks: Optional[torch.Tensor], block_table,
+               seq_index, kv_lens, max_kv: int = 0, out: Optional[torch.Tensor] = None, impl: Optional[str] = None) -> torch.Tensor:
+    """Rows q [R, heads, q_pad] over their sequences' pages -> [R, heads * vdim].  ``impl`` "cuda_core_any" forces the any-size
+    kernel."""
+    from . import core
+    r, H, G, D, V = q.shape[0], spec.heads, spec.kv_heads, spec.dim, spec.vdim
+    if _lib.on_cpu(q):
+        res = torch.empty((r, H, V))
+        for i in range(r):
+            n = int(kv_lens[i])
+            blks = block_table[int(seq_index[i]), :(n + kv.page_size - 1) // kv.page_size].long()
+            lo = max(0, n - spec.window) if spec.window else 0
+            k = kv.k[blks].transpose(1, 2).reshape(-1, G, kv.k.shape[3])[lo:n, :, :D].float().repeat_interleave(H // G, dim=1)
+            v = kv.v[blks].transpose(1, 2).reshape(-1, G, kv.v.shape[3])[lo:n, :, :V].float().repeat_interleave(H // G, dim=1)
+            s = torch.einsum("hd,jhd->hj", q[i, :, :D].float(), k) * spec.scale
+            if sinks is not None:
+                s = torch.cat([s, sinks[:, None]], dim=1)
+            p = torch.softmax(s, dim=-1)[:, :n - lo]
+            res[i] = torch.einsum("hj,jhv->hv", p, v)
+        res = res.view(r, H * V)
+        if gate is not None:
+            res = res * torch.sigmoid(gate.float())
+        res = res.to(q.dtype)
+        if out is not None:
+            out.copy_(res)
+        return res
+    g = H // G
+    if q.dtype == torch.bfloat16 and D == V and D in (64, 128, 256) and g in (1, 2, 4, 8) and impl != "cuda_core_any":
+        return core.paged_attention(q.view(r, H * D), kv, block_table, seq_index, kv_lens, H, G, D, window=spec.window,
+                                    sm_scale=spec.scale, max_kv=max_kv, sinks=sinks, gate=gate, out=out)
+    out = torch.empty((r, H * V), dtype=q.dtype, device=q.device) if out is None else out
+    rc = _k().sllm_kv_attention(core._p(q), core._p(kv.k), core._p(kv.v), core._p(gate), gate.stride(0) if gate is not None else 0,
+                                core._p(sinks), core._p(block_table), block_table.stride(0), core._p(seq_index), core._p(kv_lens), r, H,
+                                G, D, V, spec.q_pad, kv.k.shape[3], kv.v.shape[3], kv.page_size, spec.window, spec.scale, core._p(out),
+                                int(q.dtype == torch.float32), core._stream())
+    _lib.check(rc, "kv_attention")
+    return out
+
+
+def gatherable(spec: KVSpec, dtype, gate: Optional[torch.Tensor]) -> bool:
+    """Whether long portions of this layer run on the tensor cores."""
+    return (dtype == torch.bfloat16 and spec.dim % 8 == 0 and spec.vdim % 8 == 0 and spec.dim <= 192 and spec.vdim <= 128
+            and (gate is None or (gate.stride(0) % 8 == 0 and gate.data_ptr() % 16 == 0)))
+
+
+def attend_gathered(q, gate, spec: KVSpec, kv: KVPages, sinks, b, pt, out) -> None:
+    """Rows [pt.lo, pt.hi) of a batch (q, gate and out are those rows)."""
+    from .core import _p, _stream, workspace
+    key = ("gathered", pt.lo)
+    held = b.plans.get(key)
+    if held is None or held[0] is not kv:             # layers that share keys and values share the gathered rows
+        rows = torch.empty((pt.context, spec.kv_heads * (spec.dim + spec.vdim)), dtype=q.dtype, device=q.device)
+        rc = _k().sllm_kv_gather(_p(kv.k), _p(kv.v), kv.page_size, _p(b.block_table), b.block_table.stride(0), _p(pt.spans),
+                                 pt.spans.shape[0], pt.longest, _p(rows), spec.kv_heads, spec.dim, spec.vdim, _stream())
+        _lib.check(rc, "kv_gather")
+        held = b.plans[key] = (kv, rows)
+    if _lib.audit_enabled():
+        _lib.record_dispatch("kv_attention", "latent_prefill_kernel", rows=q.shape[0], heads=spec.heads, context=pt.context,
+                             window=spec.window, grid=[pt.tiles.shape[0], spec.heads])
+    rc = _k().sllm_kv_prefill(_p(q), q.shape[0], _p(held[1]), pt.context, _p(pt.tiles), pt.tiles.shape[0], spec.heads, spec.kv_heads,
+                              spec.dim, spec.vdim, spec.window, spec.scale, _p(sinks), _p(gate), gate.stride(0) if gate is not None else 0,
+                              _p(out), _p(workspace(q.device).status), _stream())
+    _lib.check(rc, "kv_prefill")
+
+
+def attention(q: torch.Tensor, gate: Optional[torch.Tensor], spec: KVSpec, kv: KVPages, sinks: Optional[torch.Tensor], b) -> torch.Tensor:
+    """Attention of a ForwardBatch's rows over ``kv`` (already appended to) -> [T, heads * vdim], gated."""
+    t = q.shape[0]
+
+    def rows(lo, hi, out=None):
+        return paged_rows(q[lo:hi], None if gate is None else gate[lo:hi], spec, kv, sinks, b.block_table, b.seq_index[lo:hi],
+                          b.kv_lens[lo:hi], b.max_kv, out)
+
+    if b.row_off_host is None or not q.is_cuda or _lib.fake_active() or not gatherable(spec, q.dtype, gate):
+        return rows(0, t)
+    key = ("portions", spec.window)
+    portions = b.plans.get(key)
+    if portions is None:
+        portions = b.plans[key] = plan_portions(b.row_off_host, b.starts_host, spec.window, q.device)
+    if len(portions) == 1 and portions[0].spans is None:
+        return rows(0, t)
+    out = torch.empty((t, spec.out_cols), dtype=q.dtype, device=q.device)
+    for pt in portions:
+        if pt.spans is None:
+            rows(pt.lo, pt.hi, out[pt.lo:pt.hi])
+        else:
+            attend_gathered(q[pt.lo:pt.hi], None if gate is None else gate[pt.lo:pt.hi], spec, kv, sinks, b, pt, out[pt.lo:pt.hi])
+    return out

@@ -6,6 +6,7 @@ crates/sllm-core/src/moe.rs:229: top-k by logit, ties to the lower index, softma
 from __future__ import annotations
 
 import ctypes as C
+from dataclasses import dataclass
 from typing import Optional
 
 import torch
@@ -13,9 +14,12 @@ import torch
 from . import _lib
 from .w4 import W4Weight, linear_w4
 
-P, I, L = C.c_void_p, C.c_int, C.c_longlong
+P, I, L, F = C.c_void_p, C.c_int, C.c_longlong, C.c_float
 _SIGS = {
-    "sllm_moe_route": (I, [P, I, I, I, I, I, P, P, P]),
+    "sllm_moe_route": (I, [P, I, I, I, I, I, I, I, I, P, P, P]),
+    "sllm_moe_router": (I, [P, I, P, I, I, I, I, I, I, I, I, P, P, P]),
+    "sllm_moe_grouped": (I, [P, P, P, I, I, I, I, P, F, F, F, P, I, I, I, I, I, P, P]),
+    "sllm_moe_grouped_simt": (I, [P, I, P, P, P, I, I, I, I, P, F, F, F, P, I, I, I, I, P]),
     "sllm_moe_permute": (I, [P, P, I, I, I, I, P, P, P, P, P]),
     "sllm_moe_gather": (I, [P, I, P, P, I, P, I, I, P]),
     "sllm_moe_combine": (I, [P, P, I, P, P, I, I, P]),
@@ -32,13 +36,20 @@ def _k():
     return _lib.kernels()
 
 
-def route(logits: torch.Tensor, top_k: int, softmax_all: bool = False):
-    """[T, E] -> (idx int32 [T, k], weights fp32 [T, k])."""
+def route(logits: torch.Tensor, top_k: int, softmax_all: bool = False, groups: int = 1, keep: int = 1):
+    """[T, E] (bf16 or fp32) -> (idx int32 [T, k], weights fp32 [T, k]).  ``groups`` > 1: neighbouring experts form equal
+    groups, a group's score is the largest in it, and only experts of the ``keep`` best groups are selected."""
     t, e = logits.shape
     if _lib.on_cpu(logits):
         lf = torch.nan_to_num(logits.float(), nan=float("-inf"))
+        pick = lf
+        if groups > 1 and keep < groups:
+            top = lf.view(t, groups, e // groups).max(-1).values
+            best = torch.sort(-top, dim=1, stable=True).indices[:, :keep]
+            shut = torch.ones((t, groups), dtype=torch.bool).scatter(1, best, False)
+            pick = lf.masked_fill(shut.repeat_interleave(e // groups, dim=1), float("-inf"))
         # stable ordering: larger logit first, ties to the lower index
-        order = torch.sort(-lf, dim=1, stable=True).indices[:, :top_k]
+        order = torch.sort(-pick, dim=1, stable=True).indices[:, :top_k]
         sel = torch.gather(lf, 1, order)
         if softmax_all:
             w = torch.softmax(lf, dim=1).gather(1, order)
@@ -48,9 +59,27 @@ def route(logits: torch.Tensor, top_k: int, softmax_all: bool = False):
     from .core import _p, _stream
     idx = torch.empty((t, top_k), dtype=torch.int32, device=logits.device)
     w = torch.empty((t, top_k), dtype=torch.float32, device=logits.device)
-    rc = _k().sllm_moe_route(_p(logits), logits.stride(0), t, e, top_k, int(softmax_all), _p(idx), _p(w), _stream())
+    rc = _k().sllm_moe_route(_p(logits), logits.stride(0), t, e, top_k, int(softmax_all), groups, keep,
+                             int(logits.dtype == torch.float32), _p(idx), _p(w), _stream())
     _lib.check(rc, "moe_route")
     return idx, w
+
+
+ROUTER_FUSED_ROWS = 64         # up to this many tokens the product and the selection are one launch
+
+
+def router(x: torch.Tensor, w, top_k: int, softmax_all: bool = False, groups: int = 1, keep: int = 1):
+    """Routing from fp32 router logits: x [T, d], w LinearWeight [E, d] of the type of x.  Returns (idx, weights) as `route`."""
+    from . import core
+    t, e = x.shape[0], w.out_features
+    if _lib.on_cpu(x) or (t > ROUTER_FUSED_ROWS and x.dtype == torch.bfloat16 and w.in_features % 8 == 0):
+        return route(core.linear(x, w, out_fp32=True), top_k, softmax_all, groups, keep)
+    idx = torch.empty((t, top_k), dtype=torch.int32, device=x.device)
+    wt = torch.empty((t, top_k), dtype=torch.float32, device=x.device)
+    rc = _k().sllm_moe_router(core._p(x), x.stride(0), core._p(w.w), t, w.in_features, e, top_k, int(softmax_all), groups, keep,
+                              int(x.dtype == torch.float32), core._p(idx), core._p(wt), core._stream())
+    _lib.check(rc, "moe_router")
+    return idx, wt
 
 
 def permute(idx: torch.Tensor, w: torch.Tensor, e_lo: int, e_hi: int):
@@ -165,3 +194,99 @@ def experts_forward(x: torch.Tensor, idx: torch.Tensor, w: torch.Tensor, gate_up
     weights applied, perm_dst [T, k])."""
     tok_off, perm_src, perm_dst, perm_w = permute(idx, w, e_lo, e_hi)
     return expert_mlp(x, tok_off, perm_src, perm_w, gate_up, down, act), perm_dst
+
+
+# ------------------------------------------------------------------------------------------ experts with dense weights
+@dataclass
+class GatedAct:
+    """g sigmoid(alpha g) (u + shift) with g = min(gate, limit), u = clamp(up, -limit, limit).  alpha 1, shift 0 and an
+    infinite limit give SiLU(gate) * up."""
+    limit: float = float("inf")
+    alpha: float = 1.0
+    shift: float = 0.0
+
+
+GATE_BLOCK = 64                # gate rows, then the up rows of the same features, in blocks of this many
+
+
+@dataclass
+class ExpertBank:
+    """bf16 / fp32 experts of one layer.  gate_up [E, 2 * padded, d]: blocks of 64 gate rows and the 64 up rows of the same
+    features; down [E, d, padded]; ``ff`` real features, the rest is zero."""
+    gate_up: torch.Tensor
+    down: torch.Tensor
+    ff: int
+    act: GatedAct
+
+    @property
+    def experts(self) -> int:
+        return self.gate_up.shape[0]
+
+    @property
+    def padded(self) -> int:
+        return self.down.shape[2]
+
+    @staticmethod
+    def pack(gates: list, ups: list, downs: list, act: GatedAct) -> "ExpertBank":
+        """Per-expert [ff, d], [ff, d] and [d, ff] matrices."""
+        ff, d = gates[0].shape
+        n = (ff + GATE_BLOCK - 1) // GATE_BLOCK * GATE_BLOCK
+        gate_up = gates[0].new_zeros((len(gates), n // GATE_BLOCK, 2, GATE_BLOCK, d))
+        down = gates[0].new_zeros((len(gates), d, n))
+        for e, (g, u, w) in enumerate(zip(gates, ups, downs)):
+            for part, m in enumerate((g, u)):
+                rows = m.new_zeros((n, d))
+                rows[:ff] = m
+                gate_up[e, :, part] = rows.view(-1, GATE_BLOCK, d)
+            down[e, :, :ff] = w
+        return ExpertBank(gate_up.view(len(gates), 2 * n, d), down, ff, act)
+
+    def matrices(self, e: int) -> tuple:
+        """(gate, up, down) of expert ``e``: the inverse of `pack`."""
+        d = self.gate_up.shape[2]
+        g = self.gate_up[e].view(-1, 2, GATE_BLOCK, d)
+        return (g[:, 0].reshape(-1, d)[:self.ff], g[:, 1].reshape(-1, d)[:self.ff], self.down[e, :, :self.ff])
+
+
+def _grouped(x, src, w, tok_off, mode, row_w, act, features, rows, tile_rows, bn):
+    from .core import _p, _stream, workspace
+    e, n, k = w.shape
+    y = torch.empty((rows, features), dtype=x.dtype, device=x.device)
+    if tile_rows:
+        rc = _k().sllm_moe_grouped(_p(x), _p(w), _p(tok_off), e, n, k, mode, _p(row_w), act.limit, act.alpha, act.shift, _p(y), features,
+                                   features, rows, tile_rows, bn, _p(workspace(x.device).status), _stream())
+    else:
+        rc = _k().sllm_moe_grouped_simt(_p(x), x.stride(0), _p(src), _p(w), _p(tok_off), e, n, k, mode, _p(row_w), act.limit, act.alpha,
+                                        act.shift, _p(y), features, features, rows, int(x.dtype == torch.float32), _stream())
+    _lib.check(rc, "moe_grouped")
+    return y
+
+
+def bank_forward(x: torch.Tensor, idx: torch.Tensor, w: torch.Tensor, bank: ExpertBank):
+    """The experts' outputs with routing weights applied: (y_perm [T * k, d], perm_dst [T, k]); row perm_dst[t, j] belongs to
+    the j-th expert of token t (`combine` or `add_group_norm(terms=)` sum them)."""
+    tok_off, perm_src, perm_dst, perm_w = permute(idx, w, 0, bank.experts)
+    d, act = x.shape[1], bank.act
+    if _lib.on_cpu(x):
+        y = torch.zeros((perm_src.numel(), d), dtype=x.dtype)
+        offs = tok_off.tolist()
+        for e in range(bank.experts):
+            lo, hi = offs[e], offs[e + 1]
+            if lo == hi:
+                continue
+            gate, up, down = (m.float() for m in bank.matrices(e))
+            h = x[perm_src[lo:hi].long()].float()
+            g, u = torch.clamp(h @ gate.t(), max=act.limit), torch.clamp(h @ up.t(), min=-act.limit, max=act.limit)
+            a = (g * torch.sigmoid(act.alpha * g) * (u + act.shift)).to(x.dtype).float()
+            y[lo:hi] = ((a @ down.t()) * perm_w[lo:hi, None]).to(x.dtype)
+        return y, perm_dst
+    rows = perm_src.numel()
+    if x.dtype == torch.float32 or d % 8:
+        a = _grouped(x, perm_src, bank.gate_up, tok_off, 0, None, act, bank.padded, rows, 0, 0)
+        return _grouped(a, None, bank.down, tok_off, 1, perm_w, act, d, rows, 0, 0), perm_dst
+    tile_rows, bn = (32, 128) if rows <= 24 * bank.experts else (128, 256)
+    if _lib.audit_enabled():
+        _lib.record_dispatch("moe_experts", "grouped_gemm_kernel", rows=rows, experts=bank.experts, d=d, ff=bank.ff, tile_rows=tile_rows,
+                             bn=bn)
+    a = _grouped(gather(x, perm_src, tok_off), None, bank.gate_up, tok_off, 0, None, act, bank.padded, rows, tile_rows, bn)
+    return _grouped(a, None, bank.down, tok_off, 1, perm_w, act, d, rows, tile_rows, bn), perm_dst
