@@ -192,7 +192,7 @@ def attend_gathered(q, gate, spec: KVSpec, kv: KVPages, sinks, b, pt, out) -> No
     from .core import _p, _stream, workspace
     key = ("gathered", pt.lo)
     held = b.plans.get(key)
-    if held is None or held[0] is not kv:             # layers that share keys and values share the gathered rows
+    if spec.own_kv or held is None or held[0] is not kv:      # a layer that borrows its keys finds them gathered already
         rows = torch.empty((pt.context, spec.kv_heads * (spec.dim + spec.vdim)), dtype=q.dtype, device=q.device)
         rc = _k().sllm_kv_gather(_p(kv.k), _p(kv.v), kv.page_size, _p(b.block_table), b.block_table.stride(0), _p(pt.spans),
                                  pt.spans.shape[0], pt.longest, _p(rows), spec.kv_heads, spec.dim, spec.vdim, _stream())
