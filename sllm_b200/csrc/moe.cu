@@ -124,8 +124,10 @@ __global__ void moe_route_kernel(const T* __restrict__ logits, int ld, int token
 }
 
 // Router product (fp32 sums, never rounded) and selection of one token per CTA: decode batches and 32-bit models.
+constexpr int kRouterThreads = 1024, kRouterWarps = kRouterThreads / 32;
+
 template <typename T>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(kRouterThreads)
 moe_router_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ w, int d, RouteRule rule, int vec, int* __restrict__ out_idx,
                   float* __restrict__ out_w) {
   pdl_wait();
@@ -135,33 +137,36 @@ moe_router_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ w, int
   constexpr int V = kVec16<T>;
   const T* src = x + static_cast<size_t>(blockIdx.x) * ldx;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int c = threadIdx.x; c < d; c += 256) row[c] = ld_f(src + c);
+  for (int c = threadIdx.x; c < d; c += kRouterThreads) row[c] = ld_f(src + c);
   __syncthreads();
-  for (int e0 = warp * 4; e0 < rule.experts; e0 += 32) {
-    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+  // a warp works on two experts at a time, with several pieces of both rows in flight
+  for (int e0 = warp; e0 < rule.experts; e0 += 2 * kRouterWarps) {
+    const int e1 = e0 + kRouterWarps < rule.experts ? e0 + kRouterWarps : e0;
+    const T *w0 = w + static_cast<size_t>(e0) * d, *w1 = w + static_cast<size_t>(e1) * d;
+    float a0 = 0.f, a1 = 0.f;
     if (vec) {
+#pragma unroll 4
       for (int c = lane * V; c < d; c += 32 * V) {
-        float v[4][V];
+        float v0[V], v1[V];
+        ld16(w0 + c, v0);
+        ld16(w1 + c, v1);
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
-          if (e0 + j < rule.experts) ld16(w + static_cast<size_t>(e0 + j) * d + c, v[j]);
-#pragma unroll
-        for (int j = 0; j < 4; ++j)
-          if (e0 + j < rule.experts) {
-#pragma unroll
-            for (int i = 0; i < V; ++i) acc[j] = fmaf(v[j][i], row[c + i], acc[j]);
-          }
+        for (int i = 0; i < V; ++i) {
+          a0 = fmaf(v0[i], row[c + i], a0);
+          a1 = fmaf(v1[i], row[c + i], a1);
+        }
       }
     } else {
-      for (int c = lane; c < d; c += 32)
-#pragma unroll
-        for (int j = 0; j < 4; ++j)
-          if (e0 + j < rule.experts) acc[j] = fmaf(ld_f(w + static_cast<size_t>(e0 + j) * d + c), row[c], acc[j]);
+      for (int c = lane; c < d; c += 32) {
+        a0 = fmaf(ld_f(w0 + c), row[c], a0);
+        a1 = fmaf(ld_f(w1 + c), row[c], a1);
+      }
     }
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      acc[j] = warp_sum(acc[j]);
-      if (lane == 0 && e0 + j < rule.experts) z[e0 + j] = acc[j];
+    a0 = warp_sum(a0);
+    a1 = warp_sum(a1);
+    if (lane == 0) {
+      z[e0] = a0;
+      z[e1] = e1 != e0 ? a1 : a0;
     }
   }
   __syncthreads();
@@ -247,6 +252,83 @@ moe_permute_kernel(const int* __restrict__ idx, const float* __restrict__ w, int
       perm_dst[a] = -1;
     }
     __syncthreads();
+  }
+}
+
+// The same for prompts, a CTA per chunk of kPermuteThreads assignments: the first kernel counts each chunk's experts
+// (counts [chunks][experts]), the second derives its cursors from all chunks' counts and places its own chunk.
+__global__ void __launch_bounds__(kPermuteThreads)
+moe_permute_count_kernel(const int* __restrict__ idx, int total, int e_lo, int n_local, int* __restrict__ counts) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ int n[kMaxExperts];
+  for (int i = threadIdx.x; i < n_local; i += kPermuteThreads) n[i] = 0;
+  __syncthreads();
+  const int a = blockIdx.x * kPermuteThreads + threadIdx.x;
+  const int e = a < total ? idx[a] - e_lo : -1;
+  if (e >= 0 && e < n_local) atomicAdd(&n[e], 1);
+  __syncthreads();
+  for (int i = threadIdx.x; i < n_local; i += kPermuteThreads) counts[static_cast<size_t>(blockIdx.x) * n_local + i] = n[i];
+}
+
+__global__ void __launch_bounds__(kPermuteThreads)
+moe_permute_place_kernel(const int* __restrict__ idx, const float* __restrict__ w, int total, int top_k, int e_lo, int n_local,
+                         const int* __restrict__ counts, int* __restrict__ tok_off, int* __restrict__ perm_src,
+                         int* __restrict__ perm_dst, float* __restrict__ perm_w) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ int before[kMaxExperts], sum[kMaxExperts], base[kMaxExperts + 1];
+  __shared__ int wcount[kPermuteWarps * kMaxExperts];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, chunks = gridDim.x, mine = blockIdx.x;
+  for (int i = threadIdx.x; i < n_local; i += kPermuteThreads) before[i] = sum[i] = 0;
+  for (int i = threadIdx.x; i < kPermuteWarps * n_local; i += kPermuteThreads) wcount[i] = 0;
+  __syncthreads();
+  for (int i = threadIdx.x; i < chunks * n_local; i += kPermuteThreads) {
+    const int c = counts[i], e = i % n_local;
+    if (c == 0) continue;
+    atomicAdd(&sum[e], c);
+    if (i / n_local < mine) atomicAdd(&before[e], c);
+  }
+  const int a = mine * kPermuteThreads + threadIdx.x;
+  int e = a < total ? idx[a] - e_lo : -1;
+  if (e < 0 || e >= n_local) e = -1;
+  const unsigned peers = __match_any_sync(0xffffffffu, e >= 0 ? e : (0x40000000 | lane));
+  const int rank = __popc(peers & ((1u << lane) - 1u));
+  if (e >= 0 && rank == 0) wcount[warp * n_local + e] = __popc(peers);
+  __syncthreads();
+  if (warp == 0) {                                    // exclusive scan of the experts' totals
+    int run = 0;
+    for (int e0 = 0; e0 < n_local; e0 += 32) {
+      const int v = e0 + lane < n_local ? sum[e0 + lane] : 0;
+      int s = v;
+      for (int o = 1; o < 32; o <<= 1) {
+        const int u = __shfl_up_sync(0xffffffffu, s, o);
+        if (lane >= o) s += u;
+      }
+      if (e0 + lane < n_local) base[e0 + lane] = run + s - v;
+      run += __shfl_sync(0xffffffffu, s, 31);
+    }
+    if (lane == 0) base[n_local] = run;
+  }
+  __syncthreads();
+  for (int x = threadIdx.x; x < n_local; x += kPermuteThreads) {
+    int run = base[x] + before[x];
+    for (int wv = 0; wv < kPermuteWarps; ++wv) {
+      const int c = wcount[wv * n_local + x];
+      wcount[wv * n_local + x] = run;
+      run += c;
+    }
+  }
+  if (mine == 0)
+    for (int x = threadIdx.x; x <= n_local; x += kPermuteThreads) tok_off[x] = base[x];
+  __syncthreads();
+  if (e >= 0) {
+    const int pos = wcount[warp * n_local + e] + rank;
+    perm_src[pos] = a / top_k;
+    perm_w[pos] = w[a];
+    perm_dst[a] = pos;
+  } else if (a < total) {
+    perm_dst[a] = -1;
   }
 }
 
@@ -632,22 +714,34 @@ SLLM_EXPORT int sllm_moe_router(const void* x, int ldx, const void* w, int token
   if (smem > 40 * 1024) return SLLM_ERR_UNSUPPORTED_SHAPE;
   const int vec = d % (fp32 ? 4 : 8) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const cudaError_t e = fp32 ? launch_kernel(moe_router_kernel<float>, dim3(tokens), dim3(256), smem, st, 1u,
+  const cudaError_t e = fp32 ? launch_kernel(moe_router_kernel<float>, dim3(tokens), dim3(kRouterThreads), smem, st, 1u,
                                              static_cast<const float*>(x), ldx, static_cast<const float*>(w), d, rule, vec, out_idx, out_w)
-                             : launch_kernel(moe_router_kernel<__nv_bfloat16>, dim3(tokens), dim3(256), smem, st, 1u,
+                             : launch_kernel(moe_router_kernel<__nv_bfloat16>, dim3(tokens), dim3(kRouterThreads), smem, st, 1u,
                                              static_cast<const __nv_bfloat16*>(x), ldx, static_cast<const __nv_bfloat16*>(w), d, rule,
                                              vec, out_idx, out_w);
   return e == cudaSuccess ? SLLM_OK : SLLM_ERR_CUDA;
 }
 
+// counts: optional scratch of ceil(tokens * top_k / 1024) * (e_hi - e_lo) ints; with it, batches of more than one chunk take
+// a CTA per chunk.
 SLLM_EXPORT int sllm_moe_permute(const int* idx, const float* w, int tokens, int top_k, int e_lo, int e_hi, int* tok_off,
-                                 int* perm_src, int* perm_dst, float* perm_w, void* stream) {
+                                 int* perm_src, int* perm_dst, float* perm_w, int* counts, void* stream) {
   if (!idx || !w || !tok_off || !perm_src || !perm_dst || !perm_w || tokens <= 0 || top_k <= 0 || e_lo < 0 ||
       e_hi <= e_lo || e_hi - e_lo > kMaxExperts)
     return SLLM_ERR_INVALID_ARGUMENT;
   if (static_cast<long long>(tokens) * top_k > (1LL << 30)) return SLLM_ERR_UNSUPPORTED_SHAPE;
-  cudaError_t e = launch_kernel(moe_permute_kernel, dim3(1), dim3(kPermuteThreads), 0, static_cast<cudaStream_t>(stream), 1u,
-                                idx, w, tokens, top_k, e_lo, e_hi, tok_off, perm_src, perm_dst, perm_w);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int total = tokens * top_k, chunks = (total + kPermuteThreads - 1) / kPermuteThreads;
+  cudaError_t e;
+  if (counts && chunks > 1) {
+    e = launch_kernel(moe_permute_count_kernel, dim3(chunks), dim3(kPermuteThreads), 0, st, 1u, idx, total, e_lo, e_hi - e_lo, counts);
+    if (e == cudaSuccess)
+      e = launch_kernel(moe_permute_place_kernel, dim3(chunks), dim3(kPermuteThreads), 0, st, 1u, idx, w, total, top_k, e_lo, e_hi - e_lo,
+                        counts, tok_off, perm_src, perm_dst, perm_w);
+  } else {
+    e = launch_kernel(moe_permute_kernel, dim3(1), dim3(kPermuteThreads), 0, st, 1u, idx, w, tokens, top_k, e_lo, e_hi, tok_off, perm_src,
+                      perm_dst, perm_w);
+  }
   return e == cudaSuccess ? SLLM_OK : SLLM_ERR_CUDA;
 }
 

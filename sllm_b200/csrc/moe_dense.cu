@@ -76,7 +76,7 @@ __device__ __forceinline__ void grouped_find(const int* tok_off, int experts, in
 __device__ __forceinline__ float gated_clamp(float g, float u, float limit, float alpha, float shift) {
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
-  return g / (1.f + __expf(-alpha * g)) * (u + shift);
+  return __fdividef(g, 1.f + __expf(-alpha * g)) * (u + shift);      // 0 where the exponential overflows
 }
 
 template <int BN, int kRows>

@@ -25,7 +25,8 @@
 
 namespace sllm {
 
-constexpr int kRgTokens = 64;            // tokens of a tile
+constexpr int kRgTokens = 64;            // tokens of a tile (prompt form)
+constexpr int kRgDecodeRows = 16;        // tokens of a tile (decode form)
 constexpr int kRgChannels = 128;         // channels of a tile
 constexpr int kRgTaps = 4;               // taps of the tile kernel (shorter filters are padded)
 constexpr int kRgMaxChunks = 4;          // 64-channel chunks of a block
@@ -99,12 +100,14 @@ struct __align__(16) RglruShared {
 };
 
 // grid (blocks * ct, CTAs per channel tile), 256 threads: warps 0-3 build u and issue the products, warps 4-7 finish.
+// TMEM columns of buffer b: gate r at 128 b, gate i 64 further.
 template <bool kDecode>
 __global__ void __launch_bounds__(256, 1)
 rglru_tile_kernel(const __grid_constant__ CUtensorMap tm_w, const RglruParams p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  constexpr int kWChunk = kRgChannels * 128, kUChunk = kRgTokens * 128;
+  constexpr int kN = kDecode ? kRgDecodeRows : kRgTokens;
+  constexpr int kWChunk = kRgChannels * 128, kUChunk = kN * 128;
   uint8_t* w_s = smem;                                  // [2 gates][kc] chunks
   uint8_t* u_s = smem + 2 * p.kc * kWChunk;             // [2 buffers][kc] chunks
   RglruShared* sh = reinterpret_cast<RglruShared*>(u_s + 2 * p.kc * kUChunk);
@@ -137,7 +140,7 @@ rglru_tile_kernel(const __grid_constant__ CUtensorMap tm_w, const RglruParams p)
   const int W = p.width;
 
   if (warp < 4) {
-    const int tid = threadIdx.x, cgs = p.kc * 8, tgs = 128 / cgs, per = (kRgTokens + tgs - 1) / tgs;
+    const int tid = threadIdx.x, cgs = p.kc * 8, tgs = 128 / cgs, per = (kN + tgs - 1) / tgs;
     const int k0 = (tid % cgs) * 8, tg = tid / cgs;
     const bool active = tg < tgs, real = active && k0 < p.bs;
     const int ch = blk * p.bs + k0;                     // first of this thread's eight channels
@@ -160,8 +163,8 @@ rglru_tile_kernel(const __grid_constant__ CUtensorMap tm_w, const RglruParams p)
       const int buf = it & 1;
       int row0, rows, seq = 0, pos0 = 0, first = 0;
       if (kDecode) {
-        row0 = tile * kRgTokens;
-        rows = min(kRgTokens, p.tokens - row0);
+        row0 = tile * kN;
+        rows = min(kN, p.tokens - row0);
       } else {
         const int4 tl = reinterpret_cast<const int4*>(p.tiles)[tile];
         row0 = tl.x; rows = tl.y; seq = tl.z;
@@ -172,50 +175,89 @@ rglru_tile_kernel(const __grid_constant__ CUtensorMap tm_w, const RglruParams p)
       if (active) {
         uint8_t* dst = u_s + (buf * p.kc + (k0 >> 6)) * kUChunk;
         const int unit = (k0 & 63) >> 3;
-        const int t_lo = tg * per, t_hi = min(kRgTokens, t_lo + per);
-        float win[kRgTaps - 1][8];                      // win[b - 1]: the input b positions back
-        if (!kDecode && real && t_lo < rows) {
-          const float* ring = p.ring + p.slots[seq] * p.ring_stride;
+        const int t_lo = tg * per, t_hi = min(kN, t_lo + per);
+        auto put = [&](int t, const float (&x)[8], const float (&win)[kRgTaps - 1][8]) {   // win[b - 1]: b positions back
+          float acc[8];
 #pragma unroll
-          for (int b = 1; b < kRgTaps; ++b) {
-            const int row = row0 + t_lo - b, pos = pos0 + t_lo - b;
+          for (int j = 0; j < 8; ++j) acc[j] = fmaf(cw[kRgTaps - 1][j], x[j], cb[j]);
 #pragma unroll
-            for (int j = 0; j < 8; ++j) win[b - 1][j] = 0.f;
-            if (b < p.taps && pos >= 0) {
-              if (row >= first) rg_row8(proj + static_cast<size_t>(row) * p.ldp + p.off_x + ch, bx, win[b - 1]);
-              else rg_ld8(ring + static_cast<size_t>(pos % p.taps) * W + ch, win[b - 1]);
+          for (int b = 1; b < kRgTaps; ++b)
+#pragma unroll
+            for (int j = 0; j < 8; ++j) acc[j] = fmaf(cw[kRgTaps - 1 - b][j], win[b - 1][j], acc[j]);
+          uint4 o;
+          __nv_bfloat162* h2 = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) h2[j] = __floats2bfloat162_rn(acc[2 * j], acc[2 * j + 1]);
+          *reinterpret_cast<uint4*>(dst + t * 128 + ((unit ^ (t & 7)) << 4)) = o;
+        };
+        auto zero = [&](int t) { *reinterpret_cast<uint4*>(dst + t * 128 + ((unit ^ (t & 7)) << 4)) = make_uint4(0, 0, 0, 0); };
+        constexpr int kBatch = kDecode ? 4 : 8;         // rows whose loads are in flight together
+        if constexpr (kDecode) {
+          for (int t0 = t_lo; t0 < t_hi; t0 += kBatch) {
+            int pos[kBatch], slot[kBatch];
+            uint4 raw[kBatch];
+            float win[kBatch][kRgTaps - 1][8];
+#pragma unroll
+            for (int i = 0; i < kBatch; ++i) {
+              const bool in = real && t0 + i < t_hi && t0 + i < rows;
+              pos[i] = in ? p.positions[row0 + t0 + i] : -1;
+              slot[i] = in ? p.slots[row0 + t0 + i] : 0;
+              raw[i] = in ? *reinterpret_cast<const uint4*>(proj + static_cast<size_t>(row0 + t0 + i) * p.ldp + p.off_x + ch) : make_uint4(0, 0, 0, 0);
             }
-          }
-        }
-#pragma unroll 2
-        for (int t = t_lo; t < t_hi; ++t) {
-          uint4 o = make_uint4(0, 0, 0, 0);
-          if (real && t < rows) {
-            const int row = row0 + t;
-            float x[8], acc[8];
-            rg_row8(proj + static_cast<size_t>(row) * p.ldp + p.off_x + ch, bx, x);
-            if (kDecode) {
-              const int pos = p.positions[row];
-              float* ring = p.ring + p.slots[row] * p.ring_stride;
+#pragma unroll
+            for (int i = 0; i < kBatch; ++i)
 #pragma unroll
               for (int b = 1; b < kRgTaps; ++b) {
 #pragma unroll
-                for (int j = 0; j < 8; ++j) win[b - 1][j] = 0.f;
-                if (b < p.taps && pos - b >= 0) rg_ld8(ring + static_cast<size_t>((pos - b) % p.taps) * W + ch, win[b - 1]);
+                for (int j = 0; j < 8; ++j) win[i][b - 1][j] = 0.f;
+                if (b < p.taps && pos[i] - b >= 0)
+                  rg_ld8(p.ring + slot[i] * p.ring_stride + static_cast<size_t>((pos[i] - b) % p.taps) * W + ch, win[i][b - 1]);
               }
+#pragma unroll
+            for (int i = 0; i < kBatch; ++i) {
+              if (t0 + i >= t_hi) break;
+              if (pos[i] < 0) {
+                zero(t0 + i);
+                continue;
+              }
+              float x[8];
+              rg_row8(reinterpret_cast<const __nv_bfloat16*>(&raw[i]), bx, x);
               if (owner) {
-                float* d = ring + static_cast<size_t>(pos % p.taps) * W + ch;
+                float* d = p.ring + slot[i] * p.ring_stride + static_cast<size_t>(pos[i] % p.taps) * W + ch;
                 *reinterpret_cast<float4*>(d) = make_float4(x[0], x[1], x[2], x[3]);
                 *reinterpret_cast<float4*>(d + 4) = make_float4(x[4], x[5], x[6], x[7]);
               }
+              put(t0 + i, x, win[i]);
             }
+          }
+        } else {
+          const int n = real ? min(t_hi, rows) : t_lo;  // rows [t_lo, n) are real
+          const __nv_bfloat16* src = proj + static_cast<size_t>(row0) * p.ldp + p.off_x + ch;
+          float win[kRgTaps - 1][8];
+          if (t_lo < n) {
+            const float* ring = p.ring + p.slots[seq] * p.ring_stride;
 #pragma unroll
-            for (int j = 0; j < 8; ++j) acc[j] = fmaf(cw[kRgTaps - 1][j], x[j], cb[j]);
+            for (int b = 1; b < kRgTaps; ++b) {
+              const int t = t_lo - b, pos = pos0 + t;
 #pragma unroll
-            for (int b = 1; b < kRgTaps; ++b)
+              for (int j = 0; j < 8; ++j) win[b - 1][j] = 0.f;
+              if (b < p.taps && pos >= 0) {
+                if (row0 + t >= first) rg_row8(src + static_cast<long long>(t) * p.ldp, bx, win[b - 1]);
+                else rg_ld8(ring + static_cast<size_t>(pos % p.taps) * W + ch, win[b - 1]);
+              }
+            }
+          }
+          for (int t0 = t_lo; t0 < n; t0 += kBatch) {
+            uint4 raw[kBatch];
 #pragma unroll
-              for (int j = 0; j < 8; ++j) acc[j] = fmaf(cw[kRgTaps - 1 - b][j], win[b - 1][j], acc[j]);
-            if (!kDecode) {
+            for (int i = 0; i < kBatch; ++i)
+              raw[i] = t0 + i < n ? *reinterpret_cast<const uint4*>(src + static_cast<size_t>(t0 + i) * p.ldp) : make_uint4(0, 0, 0, 0);
+#pragma unroll
+            for (int i = 0; i < kBatch; ++i) {
+              if (t0 + i >= n) break;
+              float x[8];
+              rg_row8(reinterpret_cast<const __nv_bfloat16*>(&raw[i]), bx, x);
+              put(t0 + i, x, win);
 #pragma unroll
               for (int b = kRgTaps - 1; b > 1; --b)
 #pragma unroll
@@ -223,11 +265,8 @@ rglru_tile_kernel(const __grid_constant__ CUtensorMap tm_w, const RglruParams p)
 #pragma unroll
               for (int j = 0; j < 8; ++j) win[0][j] = x[j];
             }
-            __nv_bfloat162* h2 = reinterpret_cast<__nv_bfloat162*>(&o);
-#pragma unroll
-            for (int j = 0; j < 4; ++j) h2[j] = __floats2bfloat162_rn(acc[2 * j], acc[2 * j + 1]);
           }
-          *reinterpret_cast<uint4*>(dst + t * 128 + ((unit ^ (t & 7)) << 4)) = o;
+          for (int t = max(n, t_lo); t < t_hi; ++t) zero(t);
         }
       }
       fence_proxy_async_smem();
@@ -236,7 +275,7 @@ rglru_tile_kernel(const __grid_constant__ CUtensorMap tm_w, const RglruParams p)
         if (ok && it == 0) ok = mbar_wait(&sh->w_full, 0, abort_flag, p.status, SLLM_DEV_TIMEOUT_TMA_FULL);
         if (ok) {
           tc_fence_after();
-          constexpr uint32_t idesc = make_idesc(kFmtBf16, kRgChannels, kRgTokens, 0, 0);
+          constexpr uint32_t idesc = make_idesc(kFmtBf16, kRgChannels, kN, 0, 0);
           for (int g = 0; g < 2; ++g)
             for (int c = 0; c < p.kc; ++c) {
               const uint64_t da = make_smem_desc_sw128(smem_u32(w_s + (g * p.kc + c) * kWChunk));
@@ -268,15 +307,15 @@ rglru_tile_kernel(const __grid_constant__ CUtensorMap tm_w, const RglruParams p)
       const uint8_t* u_t = u_s + (buf * p.kc + ((valid ? kch : 0) >> 6)) * kUChunk + u_byte;
       int row0, rows, slot = 0, chunk = 0;
       if (kDecode) {
-        row0 = tile * kRgTokens;
-        rows = min(kRgTokens, p.tokens - row0);
+        row0 = tile * kN;
+        rows = min(kN, p.tokens - row0);
       } else {
         const int4 tl = reinterpret_cast<const int4*>(p.tiles)[tile];
         row0 = tl.x; rows = tl.y; slot = p.slots[tl.z]; chunk = tl.w & 0xffffff;
       }
       float S = 0.f, A = 1.f;
       if (!kDecode && chunk == 0 && valid) S = p.state[slot * p.state_stride + ch];
-      for (int c = 0; c < kRgTokens / 16; ++c) {
+      for (int c = 0; c < kN / 16; ++c) {
         float st[16], yv[16];
         int sl[16];
         if (kDecode) {
@@ -512,7 +551,7 @@ SLLM_EXPORT int sllm_rglru(const SllmRglru* a, void* stream) {
     return SLLM_ERR_ALIGNMENT;
   if (a->decode) {
     if (a->tokens != a->sequences) return SLLM_ERR_INVALID_ARGUMENT;
-    p.n_tiles = (a->tokens + kRgTokens - 1) / kRgTokens;
+    p.n_tiles = (a->tokens + kRgDecodeRows - 1) / kRgDecodeRows;
   } else if (!a->tiles || a->n_tiles <= 0 || !a->h || !a->prod || !a->row_off) {
     return SLLM_ERR_INVALID_ARGUMENT;
   }
@@ -522,7 +561,7 @@ SLLM_EXPORT int sllm_rglru(const SllmRglru* a, void* stream) {
   CUtensorMap tm;
   rc = cached_kmajor_tmap(&tm, a->gate_tiles, 2, static_cast<long long>(units) * 2 * kRgChannels, p.kc * 64, p.kc * 128, kRgChannels);
   if (rc != SLLM_OK) return rc;
-  const size_t smem = static_cast<size_t>(p.kc) * (2 * kRgChannels + 2 * kRgTokens) * 128 + sizeof(RglruShared) + 1024;
+  const size_t smem = static_cast<size_t>(p.kc) * (2 * kRgChannels + 2 * (a->decode ? kRgDecodeRows : kRgTokens)) * 128 + sizeof(RglruShared) + 1024;
   static size_t cfg[2] = {0, 0};
   auto* kernel = a->decode ? rglru_tile_kernel<true> : rglru_tile_kernel<false>;
   if (smem > cfg[a->decode ? 1 : 0]) {
@@ -530,8 +569,8 @@ SLLM_EXPORT int sllm_rglru(const SllmRglru* a, void* stream) {
       return SLLM_ERR_CUDA;
     cfg[a->decode ? 1 : 0] = smem;
   }
-  const int per_sm = smem <= 110 * 1024 ? 2 : 1;
-  int gy = (148 * per_sm + units - 1) / units;
+  int gy = 148 / units;                              // one CTA per SM, each with its share of the tiles
+  if (gy < 1) gy = 1;
   if (gy > p.n_tiles) gy = p.n_tiles;
   if (gy > 65535 || p.n_tiles > 65535) return SLLM_ERR_LIMIT;
   cudaStream_t st = static_cast<cudaStream_t>(stream);

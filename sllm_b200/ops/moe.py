@@ -20,7 +20,7 @@ _SIGS = {
     "sllm_moe_router": (I, [P, I, P, I, I, I, I, I, I, I, I, P, P, P]),
     "sllm_moe_grouped": (I, [P, P, P, I, I, I, I, P, F, F, F, P, I, I, I, I, I, P, P]),
     "sllm_moe_grouped_simt": (I, [P, I, P, P, P, I, I, I, I, P, F, F, F, P, I, I, I, I, P]),
-    "sllm_moe_permute": (I, [P, P, I, I, I, I, P, P, P, P, P]),
+    "sllm_moe_permute": (I, [P, P, I, I, I, I, P, P, P, P, P, P]),
     "sllm_moe_gather": (I, [P, I, P, P, I, P, I, I, P]),
     "sllm_moe_combine": (I, [P, P, I, P, P, I, I, P]),
     "sllm_moe_shared_add": (I, [P, P, P, I, P, I, I, P]),
@@ -82,6 +82,9 @@ def router(x: torch.Tensor, w, top_k: int, softmax_all: bool = False, groups: in
     return idx, wt
 
 
+PERMUTE_CHUNK = 1024           # assignments of one CTA of the chunked permutation
+
+
 def permute(idx: torch.Tensor, w: torch.Tensor, e_lo: int, e_hi: int):
     """Groups assignments by local expert.  Returns (tok_off [n_local + 1], perm_src [T*k], perm_dst [T, k],
     perm_w [T*k]); rows beyond tok_off[-1] are unused."""
@@ -107,7 +110,9 @@ def permute(idx: torch.Tensor, w: torch.Tensor, e_lo: int, e_hi: int):
         tok_off[n_local] = cur
         return tok_off, perm_src, perm_dst, perm_w
     from .core import _p, _stream
-    rc = _k().sllm_moe_permute(_p(idx), _p(w), t, k, e_lo, e_hi, _p(tok_off), _p(perm_src), _p(perm_dst), _p(perm_w), _stream())
+    chunks = (t * k + PERMUTE_CHUNK - 1) // PERMUTE_CHUNK
+    counts = torch.empty(chunks * n_local, dtype=torch.int32, device=dev) if chunks > 1 else None
+    rc = _k().sllm_moe_permute(_p(idx), _p(w), t, k, e_lo, e_hi, _p(tok_off), _p(perm_src), _p(perm_dst), _p(perm_w), _p(counts), _stream())
     _lib.check(rc, "moe_permute")
     return tok_off, perm_src, perm_dst, perm_w
 

@@ -137,7 +137,7 @@ def recurrence(tab: _Table, width: int, batch: int, seqs: int, n: int) -> None:
 
 def experts(tab: _Table, d: int, E: int, top: int, ff: int, rows: dict) -> None:
     act = M.GatedAct(7.0, 1.702, 1.0)
-    gu, dn = _bf(E, 2 * ff, d), _bf(E, d, ff)
+    gu, dn = _bf(E, 2 * ff, d).mul_(d ** -0.5), _bf(E, d, ff).mul_(ff ** -0.5)
     g4, d4 = (W4Weight.quantize_device("mxfp4", w.float()) for w in (gu, dn))
     wr = LinearWeight("dense", _bf(E, d))
     bank = M.ExpertBank(gu, dn, ff, act)
