@@ -57,6 +57,9 @@ CASES = {
                        rglru(None, width=64, blocks=8, conv=3), attention(None, kv_from=0, **_EIGHT),
                        attention(moe(experts=7, top=7, ff=64), heads=3, kv_heads=1, dim=72, vdim=40, rot=8, conv=2)],
                       width=96, vocab=100, cap=40.0),
+    # no attention at all; a filter and a block beyond the tensor-core form of the recurrence; no soft cap
+    "states": config([rglru(None, width=64, blocks=1, conv=6), rglru(moe(experts=6, top=2, ff=80, count=2, keep=1), width=264, blocks=1)],
+                     width=72, vocab=90, cap=None),
 }
 
 

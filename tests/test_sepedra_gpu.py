@@ -62,7 +62,7 @@ def test_residual_rows_without_an_input_norm(dtype, d):
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("t", [1, 33, 200])
-@pytest.mark.parametrize("d,E,top,count,keep", [(192, 12, 4, 3, 2), (61, 5, 2, 1, 1), (1024, 256, 32, 8, 4), (72, 1, 1, 1, 1)])
+@pytest.mark.parametrize("d,E,top,count,keep", [(176, 10, 4, 5, 3), (61, 5, 2, 1, 1), (1024, 256, 32, 8, 4), (72, 1, 1, 1, 1)])
 def test_router_from_unrounded_logits(dtype, t, d, E, top, count, keep):
     torch.manual_seed(d + t)
     x, w = torch.randn(t, d, device=DEV).to(dtype), torch.randn(E, d, device=DEV).to(dtype)
@@ -76,7 +76,7 @@ def test_router_from_unrounded_logits(dtype, t, d, E, top, count, keep):
 
 
 # ------------------------------------------------------------------------------------------ experts
-@pytest.mark.parametrize("T,d,ff,E,top", [(3, 192, 96, 12, 4), (40, 128, 136, 5, 2), (300, 256, 64, 3, 2), (700, 200, 200, 4, 3), (64, 64, 24, 40, 8),
+@pytest.mark.parametrize("T,d,ff,E,top", [(3, 184, 80, 11, 3), (40, 128, 136, 5, 2), (300, 256, 64, 3, 2), (700, 200, 200, 4, 3), (64, 64, 24, 40, 8),
                                            (9, 61, 30, 4, 2), (1, 512, 512, 1, 1)])
 def test_grouped_experts(T, d, ff, E, top):
     torch.manual_seed(T)
@@ -140,7 +140,7 @@ def _rec_want(proj, spec, w, past):
 
 
 @pytest.mark.parametrize("impl", [None, "cuda_core"])
-@pytest.mark.parametrize("width,blocks,taps", [(256, 4, 4), (512, 2, 4), (320, 2, 3), (72, 9, 2), (160, 1, 1), (768, 3, 4), (96, 4, 4)])
+@pytest.mark.parametrize("width,blocks,taps", [(384, 6, 4), (512, 2, 4), (320, 2, 3), (72, 9, 2), (160, 1, 1), (768, 3, 4), (96, 4, 4)])
 def test_recurrence_over_portions_and_steps(impl, width, blocks, taps):
     """Portions around the tile's edges, then single tokens of all sequences, each slot going on where it was."""
     spec, w = _rec(width, blocks, taps)
