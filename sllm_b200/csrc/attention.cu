@@ -45,14 +45,12 @@ __global__ void __launch_bounds__(128) paged_attention_kernel(const PagedAttnPar
   const int hq = p.hkv * G;
   const int seq = p.seq_index[r];
   const int kv_len = p.kv_lens[r];
-  int first = 0;
-  if (p.window > 0 && kv_len > p.window) first = kv_len - p.window;
-  const int n = kv_len - first;
-  int chunk = (n + splits - 1) / splits;
+  const VisibleKeys keys(kv_len, p.window, p.keep_first, p.chunk);
+  int chunk = (keys.n + splits - 1) / splits;
   chunk = (chunk + 31) & ~31;
-  const int begin = first + split * chunk;
+  const int begin = split * chunk;
   int end = begin + chunk;
-  if (end > kv_len) end = kv_len;
+  if (end > keys.n) end = keys.n;
 
   for (int e = threadIdx.x; e < G * HD; e += blockDim.x) {
     const int g = e / HD, d = e % HD;
@@ -74,8 +72,8 @@ __global__ void __launch_bounds__(128) paged_attention_kernel(const PagedAttnPar
   float* my_p = p_s + warp * 32 * G;
 
   for (int base = begin + warp * 32; base < end; base += 4 * 32) {
-    const int tok = base + lane;
-    const bool valid = tok < end;
+    const bool valid = base + lane < end;
+    const int tok = keys.position(base + lane);
     size_t slot = 0;
     float s[G];
 #pragma unroll
@@ -169,6 +167,10 @@ __global__ void __launch_bounds__(128) paged_attention_kernel(const PagedAttnPar
       } else {
         vsc = 1.f;
       }
+    }
+    if (p.slopes) {
+#pragma unroll
+      for (int g = 0; g < G; ++g) s[g] = fmaf(-p.slopes[kvh * G + g], static_cast<float>(kv_len - 1 - tok), s[g]);
     }
 #pragma unroll
     for (int g = 0; g < G; ++g) {
@@ -315,7 +317,9 @@ SLLM_EXPORT int sllm_paged_attention(const void* q, int q_ld, const void* k_page
                                      int page_size, int window, float sm_scale, int kv_fp8, void* out_bf16,
                                      void* out_fp8, float* out_scale, int ld_scale, const float* sinks, int splits,
                                      float* ws, long long ws_floats, int* counters, int n_counters, const void* gate,
-                                     long long ld_gate, void* stream) {
+                                     long long ld_gate, int gate_heads, int keep_first, int chunk, const float* slopes,
+                                     void* stream) {
+  if (keep_first < 0 || chunk < 0 || (keep_first > 0 && window <= 0) || (chunk > 0 && window > 0)) return SLLM_ERR_INVALID_ARGUMENT;
   if (!q || !k_pages || !v_pages || !block_table || !seq_index || !kv_lens || rows <= 0 || hkv <= 0 || hq % hkv)
     return SLLM_ERR_INVALID_ARGUMENT;
   if (!out_bf16 && !out_fp8) return SLLM_ERR_INVALID_ARGUMENT;
@@ -333,6 +337,7 @@ SLLM_EXPORT int sllm_paged_attention(const void* q, int q_ld, const void* k_page
   p.out_scale = out_scale; p.ld_scale = ld_scale; p.sinks = sinks;
   p.ws_o = nullptr; p.ws_ml = nullptr; p.counters = counters; p.status_word = nullptr;
   p.gate = static_cast<const __nv_bfloat16*>(gate); p.ld_gate = ld_gate;
+  p.gate_heads = gate_heads; p.keep_first = keep_first; p.chunk = chunk; p.slopes = slopes;
   p.early_trigger = 0;
   if (splits > 1) {
     const long long units = static_cast<long long>(rows) * hkv;

@@ -6,6 +6,23 @@
 
 namespace sllm {
 
+// The keys that the last of `len` positions sees: all of them, the last `window`, or those of its own chunk (chunks of
+// `chunk` positions counted from 0), with a window also the first `keep_first`.  They are numbered 0 .. n - 1: the kept
+// ones, then the rest.
+struct VisibleKeys {
+  int keep, first, n;
+  __device__ __forceinline__ VisibleKeys(int len, int window, int keep_first, int chunk) {
+    first = window > 0 && len > window ? len - window : chunk > 0 ? (len - 1) / chunk * chunk : 0;
+    keep = 0;
+    if (keep_first > 0 && first > 0) {
+      if (first > keep_first) keep = keep_first;
+      else first = 0;
+    }
+    n = keep + len - first;
+  }
+  __device__ __forceinline__ int position(int i) const { return i < keep ? i : i - keep + first; }
+};
+
 struct PagedAttnParams {
   const __nv_bfloat16* q;  // [rows, hq * hd] (row stride q_ld)
   int q_ld;
@@ -28,8 +45,12 @@ struct PagedAttnParams {
   float* ws_ml;             // [rows * hkv * splits, G, 2]
   int* counters;            // [rows * hkv]
   const float* sinks;       // optional [hq] attention-sink logits (added to the softmax denominator)
-  const __nv_bfloat16* gate; // optional [rows, ld_gate] logits, one per output channel: out *= sigmoid(gate)
+  const __nv_bfloat16* gate; // optional [rows, ld_gate] logits, one per output channel (gate_heads: per head): out *= sigmoid(gate)
   long long ld_gate;
+  int gate_heads;
+  // CUDA-core kernel only: see VisibleKeys; slopes (optional [hq]) are taken off a score per position of distance
+  int keep_first, chunk;
+  const float* slopes;
   int* status_word;         // device status word for bounded waits (tensor-core kernel)
   int early_trigger;        // tensor-core kernel: let dependent launches start once the CTA holds its TMEM
   STEP_TRACE_FIELD
@@ -133,7 +154,7 @@ __device__ __forceinline__ void attention_tail(const PagedAttnParams& p, int r, 
     }
     float val = (L > 0.f) ? O / L : 0.f;
     if (p.gate && in)
-      val /= 1.f + __expf(-__bfloat162float(p.gate[static_cast<size_t>(r) * p.ld_gate + (kvh * G + g) * HD + d]));
+      val /= 1.f + __expf(-__bfloat162float(p.gate[static_cast<size_t>(r) * p.ld_gate + (p.gate_heads ? kvh * G + g : (kvh * G + g) * HD + d)]));
     val = __bfloat162float(__float2bfloat16_rn(val));
     const size_t oidx = static_cast<size_t>(r) * hq * HD + (kvh * G + g) * HD + d;
     if (p.out_fp8) {

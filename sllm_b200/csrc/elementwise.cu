@@ -9,7 +9,7 @@
 // Counterparts in the reference: rmsnorm_kernel.hip.cpp:67, elementwise_kernel.hip.cpp:40-147,
 // embedding_kernel.hip.cpp:4, rotary_kernel.hip.cpp:40, kv_state_kernel.hip.cpp:161-335,
 // matmul_kernel.hip.cpp:210-247 (activation quantisation), argmax_kernel.hip.cpp:37.
-#include "common.cuh"
+#include "typed.cuh"
 #include "api.h"
 #include "noalloc.h"
 #include <mutex>
@@ -178,6 +178,19 @@ gated_act_kernel(const __nv_bfloat16* __restrict__ in, __nv_bfloat16* __restrict
   } else if (in_range) {
     store8_bf16(y_bf16 + static_cast<size_t>(r) * inter + i, v);
   }
+}
+
+// The same for any sizes and row strides in bf16 or fp32; the activation is not rounded before the product.
+template <typename T>
+__global__ void __launch_bounds__(256)
+gated_act_any_kernel(const T* __restrict__ in, T* __restrict__ y, int inter, int ld, int act) {
+  pdl_wait();
+  pdl_trigger();
+  const int i = blockIdx.y * 256 + threadIdx.x;
+  if (i >= inter) return;
+  const T* row = in + static_cast<size_t>(blockIdx.x) * ld;
+  const float g = ld_f(row + i), u = ld_f(row + inter + i);
+  st_f(y + static_cast<size_t>(blockIdx.x) * inter + i, (act == 0 ? g * sigmoid_f(g) : gelu_tanh(g)) * u);
 }
 
 // ---------------------------------------------------------------- stand-alone 1x128 quantisation
@@ -531,6 +544,19 @@ SLLM_EXPORT int sllm_gated_act(const void* in, void* y_bf16, void* y_fp8, float*
     launch_kernel(gated_act_kernel<false>, dim3(grid), dim3(256), 0, st, 1u, static_cast<const __nv_bfloat16*>(in),
                                                   static_cast<__nv_bfloat16*>(y_bf16), nullptr, nullptr, 0, inter, act);
   }
+  return check_launch();
+}
+
+// in [rows, ld]: gate | up, inter columns each; act 0 SiLU, 1 GELU (tanh form); fp32: element type (0 bf16, 1 fp32).
+SLLM_EXPORT int sllm_gated_act_any(const void* in, void* y, int rows, int inter, int ld, int act, int fp32, void* stream) {
+  if (!in || !y || rows <= 0 || inter <= 0 || ld < 2 * inter) return SLLM_ERR_INVALID_ARGUMENT;
+  const dim3 grid(rows, (inter + 255) / 256);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (fp32)
+    launch_kernel(gated_act_any_kernel<float>, grid, dim3(256), 0, st, 1u, static_cast<const float*>(in), static_cast<float*>(y), inter, ld, act);
+  else
+    launch_kernel(gated_act_any_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, 1u, static_cast<const __nv_bfloat16*>(in),
+                  static_cast<__nv_bfloat16*>(y), inter, ld, act);
   return check_launch();
 }
 

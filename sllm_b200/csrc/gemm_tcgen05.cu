@@ -1147,7 +1147,7 @@ static int gemm_impl(const void* a, const void* b, void* y, const float* scale_a
                      int ld_sa, int ld_sb, int bn, int splits, int stages, float* ws, long long ws_floats,
                      int* counters, int n_counters, int* status, void* stream, const SllmCommDesc* comm,
                      const SllmGatherDesc* gather = nullptr, const FusedEpi* fused = nullptr, int act = 0, float act_arg = 0.f,
-                     int out_fp32 = 0) {
+                     int out_fp32 = 0, int ld_x = 0) {
   if (gather) b = a;    // the B operand comes from the peers' buffers; keep the argument checks below simple
   if (!a || !b || !y || a_rows <= 0 || b_rows <= 0 || k <= 0 || splits < 1) return SLLM_ERR_INVALID_ARGUMENT;
   if (bn != 16 && bn != 32 && bn != 64 && bn != 128) return SLLM_ERR_UNSUPPORTED_SHAPE;
@@ -1194,9 +1194,11 @@ static int gemm_impl(const void* a, const void* b, void* y, const float* scale_a
   }
 
   CUtensorMap ta, tb;
-  int rc = cached_kmajor_tmap(&ta, a, elem, a_rows, k, static_cast<long long>(k) * elem, kTileA);
+  if (ld_x && (ld_x < k || (static_cast<long long>(ld_x) * elem) % 16)) return SLLM_ERR_ALIGNMENT;
+  const long long stride_x = static_cast<long long>(ld_x ? ld_x : k) * elem, stride_w = static_cast<long long>(k) * elem;
+  int rc = cached_kmajor_tmap(&ta, a, elem, a_rows, k, transpose_out ? stride_w : stride_x, kTileA);
   if (rc != SLLM_OK) return rc;
-  rc = cached_kmajor_tmap(&tb, b, elem, b_rows, k, static_cast<long long>(k) * elem, bn);
+  rc = cached_kmajor_tmap(&tb, b, elem, b_rows, k, transpose_out ? stride_x : stride_w, bn);
   if (rc != SLLM_OK) return rc;
 
   p.a_rows = a_rows; p.b_rows = b_rows; p.num_kb = num_kb; p.kb_per_split = kb_per_split; p.stages = stages;
@@ -1291,12 +1293,13 @@ SLLM_EXPORT int sllm_gemm(const void* a, const void* b, void* y, const float* sc
 }
 
 // bf16 GEMM with an activation on the sums (act 1: square of relu, 2: soft cap act_arg * tanh(y / act_arg)), stored as bf16 or
-// (out_fp32) as they are.
-SLLM_EXPORT int sllm_gemm_act(const void* a, const void* b, void* y, int a_rows, int b_rows, int k, int transpose_out, int ldy,
+// (out_fp32) as they are.  ld_x: row stride of the activation operand (b with transpose_out, else a) in elements, a multiple
+// of 8 (0: k); its base is 16-byte aligned.
+SLLM_EXPORT int sllm_gemm_act(const void* a, const void* b, void* y, int a_rows, int b_rows, int k, int ld_x, int transpose_out, int ldy,
                               int act, float act_arg, int out_fp32, int bn, int splits, int stages, float* ws, long long ws_floats,
                               int* counters, int n_counters, int* status, void* stream) {
   return gemm_impl(a, b, y, nullptr, nullptr, nullptr, a_rows, b_rows, k, 0, transpose_out, ldy, 0, 0, bn, splits, stages, ws,
-                   ws_floats, counters, n_counters, status, stream, nullptr, nullptr, nullptr, act, act_arg, out_fp32);
+                   ws_floats, counters, n_counters, status, stream, nullptr, nullptr, nullptr, act, act_arg, out_fp32, ld_x);
 }
 
 // Same GEMM with the cross-rank sum of the partial products fused into the epilogue (see the file

@@ -1,17 +1,20 @@
 // Attention over paged keys and values whose widths differ (dim, vdim), with the work between the input projection and the
 // scores in one launch.
 //
-//   kv_prepare_kernel   per (token, head): short causal convolution of the q / k / v columns, rotation of the first
-//                       channels in pairs (2i, 2i+1), optional unweighted RMS norm of q and k, page write of k and v;
-//                       q goes to [T, heads, q_pad].  In a decode step the kernel also stores the conv inputs.
-//   conv_ring_kernel    prompt form of that store: the last `taps` conv inputs of every sequence, ring row position mod taps
+//   kv_prepare_kernel   per (token, head): bias or short causal convolution of the q / k / v columns, optional RMS norm of
+//                       q and k (weighted or not), rotation of the first channels in pairs (2i, 2i+1) or (i, i + half),
+//                       page write of k and v; q goes to [T, heads, q_pad].  In a decode step the kernel also stores the
+//                       conv inputs; short_conv.cu has the prompt form of that store
 //   kv_gather_kernel    pages -> contiguous [context rows, all heads' keys | all heads' values] for the tensor-core prompt
 //                       kernel (latent_prefill.cu)
-//   kv_attention_kernel any sizes, bf16 or fp32: one warp per (row, query head); sinks, window and output gate
+//   kv_attention_kernel any sizes, bf16 or fp32: one warp per (row, query head); sinks, windows with kept first tokens,
+//                       chunks, distance slopes and output gate
 //
 // Pages of a layer: keys [num_pages, kv_heads, page, ld_k], values [num_pages, kv_heads, page, ld_v].
 #include "typed.cuh"
 #include "api.h"
+#include "attention_common.cuh"
+#include "short_conv.h"
 
 #include <cstddef>
 #include <type_traits>
@@ -23,13 +26,16 @@ constexpr int kKpThreads = 256, kKpRun = 8;
 template <typename T>
 struct KvPrepareParams {
   const T* proj;             // [T, ldp]: q | k | v columns from 0
-  const float* conv_w;       // [taps, channels]
+  const float* conv_w;       // [taps, channels], null: no convolution
+  const float* bias;         // optional [channels], joins the columns first
+  const float *q_norm, *k_norm;   // optional [dim] weights of the norms
   float* ring;               // [slots (ring_stride)][taps][channels]
   const float* inv_freq;     // [rot_dims / 2]
   const int *row_off, *slots, *positions, *seq_index, *block_table;
   T *q, *k_pages, *v_pages;
   long long ring_stride;
-  int ldp, max_blocks, heads, kv_heads, dim, vdim, q_pad, ld_k, ld_v, rot_dims, taps, page_size, tokens, run, norm, decode, vec;
+  int ldp, max_blocks, heads, kv_heads, dim, vdim, q_pad, ld_k, ld_v, rot_dims, taps, page_size, tokens, run, norm, decode, vec,
+      interleaved;
   float eps;
 };
 
@@ -39,6 +45,7 @@ __global__ void __launch_bounds__(kKpThreads) kv_prepare_kernel(const KvPrepareP
   pdl_wait();
   pdl_trigger();
   extern __shared__ float2 cs[];                        // [run][rot_dims / 2]
+  __shared__ __align__(8) float swap_s[8][kNP * 64];    // a warp's head, where rotary pairs lie in different lanes
   __shared__ int m_pos[kKpRun], m_seq[kKpRun], m_first[kKpRun], m_slot[kKpRun], m_page[kKpRun];
   const int r0 = blockIdx.x * p.run, n = min(p.run, p.tokens - r0), half = p.rot_dims >> 1;
   if (threadIdx.x < n) {
@@ -86,9 +93,19 @@ __global__ void __launch_bounds__(kKpThreads) kv_prepare_kernel(const KvPrepareP
 #pragma unroll
     for (int s = 0; s < kNP; ++s) {
       w[t][s][0] = w[t][s][1] = 0.f;
-      if (t >= kTaps - p.taps)
+      if (!p.conv_w) w[t][s][0] = w[t][s][1] = t == kTaps - 1 ? 1.f : 0.f;
+      else if (t >= kTaps - p.taps)
         ld2(p.conv_w + static_cast<size_t>(t - (kTaps - p.taps)) * channels + col, 2 * (lane + 32 * s), w[t][s]);
     }
+  float nw[kNP][2], bias[kNP][2];                       // norm weight and bias of the lane's channels
+#pragma unroll
+  for (int s = 0; s < kNP; ++s) {
+    nw[s][0] = nw[s][1] = 1.f;
+    bias[s][0] = bias[s][1] = 0.f;
+    const float* src = is_v ? nullptr : is_q ? p.q_norm : p.k_norm;
+    if (src) ld2(src, 2 * (lane + 32 * s), nw[s]);
+    if (p.bias) ld2(p.bias + col, 2 * (lane + 32 * s), bias[s]);
+  }
   float win[kTaps > 1 ? kTaps - 1 : 1][kNP][2];         // win[b - 1]: the input b positions back
   int prev = -1;
   for (int i = 0; i < n; ++i) {
@@ -115,7 +132,9 @@ __global__ void __launch_bounds__(kKpThreads) kv_prepare_kernel(const KvPrepareP
       const int c = 2 * (lane + 32 * s);
       float x[2];
       ld2(src, c, x);
-      if (p.decode) st2(ring + static_cast<size_t>(pos % p.taps) * channels, c, width, x);
+      x[0] += bias[s][0];
+      x[1] += bias[s][1];
+      if (p.decode && p.ring) st2(ring + static_cast<size_t>(pos % p.taps) * channels, c, width, x);
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         float a = w[kTaps - 1][s][j] * x[j];
@@ -131,23 +150,46 @@ __global__ void __launch_bounds__(kKpThreads) kv_prepare_kernel(const KvPrepareP
 #pragma unroll
         for (int j = 0; j < 2; ++j) win[0][s][j] = x[j];
       }
-      if (!is_v) {
+      ss += y[s][0] * y[s][0] + y[s][1] * y[s][1];
+    }
+    if (!is_v && p.norm) {                              // (an unweighted norm and the rotation commute)
+      const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(p.dim) + p.eps);
+#pragma unroll
+      for (int s = 0; s < kNP; ++s) {
+        y[s][0] *= inv * nw[s][0];
+        y[s][1] *= inv * nw[s][1];
+      }
+    }
+    if (!is_v && p.interleaved) {
+#pragma unroll
+      for (int s = 0; s < kNP; ++s) {
+        const int c = 2 * (lane + 32 * s);
         if (c < p.rot_dims) {
           const float2 a = cs[i * half + (c >> 1)];
           const float u = y[s][0], v = y[s][1];
           y[s][0] = u * a.x - v * a.y;
           y[s][1] = v * a.x + u * a.y;
         }
-        ss += y[s][0] * y[s][0] + y[s][1] * y[s][1];
       }
-    }
-    if (!is_v && p.norm) {
-      const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(p.dim) + p.eps);
+    } else if (!is_v && half > 0) {
+      float* sw = swap_s[warp];
 #pragma unroll
-      for (int s = 0; s < kNP; ++s) {
-        y[s][0] *= inv;
-        y[s][1] *= inv;
-      }
+      for (int s = 0; s < kNP; ++s) *reinterpret_cast<float2*>(sw + 2 * (lane + 32 * s)) = make_float2(y[s][0], y[s][1]);
+      __syncwarp();
+#pragma unroll
+      for (int s = 0; s < kNP; ++s)
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          const int c = 2 * (lane + 32 * s) + j;
+          if (c < half) {
+            const float2 a = cs[i * half + c];
+            y[s][j] = y[s][j] * a.x - sw[c + half] * a.y;
+          } else if (c < p.rot_dims) {
+            const float2 a = cs[i * half + c - half];
+            y[s][j] = y[s][j] * a.x + sw[c - half] * a.y;
+          }
+        }
+      __syncwarp();
     }
     T* dst;
     int w_out;
@@ -162,20 +204,6 @@ __global__ void __launch_bounds__(kKpThreads) kv_prepare_kernel(const KvPrepareP
 #pragma unroll
     for (int s = 0; s < kNP; ++s) st2(dst, 2 * (lane + 32 * s), w_out, y[s]);
   }
-}
-
-// grid (ceil(channels / 256), sequences).
-template <typename T>
-__global__ void __launch_bounds__(256)
-conv_ring_kernel(const T* __restrict__ x, int ldx, float* __restrict__ ring, long long ring_stride, const int* __restrict__ row_off,
-                 const int* __restrict__ slots, const int* __restrict__ positions, int channels, int taps) {
-  pdl_wait();
-  pdl_trigger();
-  const int c = blockIdx.x * 256 + threadIdx.x, seq = blockIdx.y;
-  if (c >= channels) return;
-  const int r1 = row_off[seq + 1];
-  for (int row = max(row_off[seq], r1 - taps); row < r1; ++row)
-    ring[slots[seq] * ring_stride + static_cast<size_t>(positions[row] % taps) * channels + c] = ld_f(x + static_cast<size_t>(row) * ldx + c);
 }
 
 // spans: [sequences][4] = {row of the block table, first context position, context rows, first gathered row}.
@@ -208,8 +236,9 @@ struct KvAttentionParams {
   const float* sinks;
   const int *block_table, *seq_index, *kv_lens;
   T* out;
+  const float* slopes;
   long long ld_gate;
-  int max_blocks, heads, kv_heads, dim, vdim, q_pad, ld_k, ld_v, page_size, window;
+  int max_blocks, heads, kv_heads, dim, vdim, q_pad, ld_k, ld_v, page_size, window, keep_first, chunk, gate_heads;
   float scale;
 };
 
@@ -222,32 +251,35 @@ __global__ void __launch_bounds__(128) kv_attention_kernel(const KvAttentionPara
   const int r = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, head = blockIdx.y * 4 + warp;
   if (head >= p.heads) return;
   float* q = q_all + warp * p.dim;
-  const int kvh = head / (p.heads / p.kv_heads), n = p.kv_lens[r];
-  const int first = p.window > 0 && n > p.window ? n - p.window : 0;
+  const int kvh = head / (p.heads / p.kv_heads), len = p.kv_lens[r];
+  const VisibleKeys keys(len, p.window, p.keep_first, p.chunk);
+  const float slope = p.slopes ? p.slopes[head] : 0.f;
   const int* bt = p.block_table + static_cast<size_t>(p.seq_index[r]) * p.max_blocks;
   for (int c = lane; c < p.dim; c += 32) q[c] = ld_f(p.q + (static_cast<size_t>(r) * p.heads + head) * p.q_pad + c) * p.scale;
   __syncwarp();
   float m = -INFINITY, l = 0.f, o[kNV];
 #pragma unroll
   for (int j = 0; j < kNV; ++j) o[j] = 0.f;
-  for (int base = first; base < n; base += 32) {
-    const int tok = base + lane;
+  for (int base = 0; base < keys.n; base += 32) {
+    const bool live = base + lane < keys.n;
     long long slot = 0;
     float s = -INFINITY;
-    if (tok < n) {
+    if (live) {
+      const int tok = keys.position(base + lane);
       slot = (static_cast<long long>(bt[tok / p.page_size]) * p.kv_heads + kvh) * p.page_size + tok % p.page_size;
       const T* k = p.k_pages + slot * p.ld_k;
       s = 0.f;
       for (int c = 0; c < p.dim; ++c) s = fmaf(q[c], ld_f(k + c), s);
+      s = fmaf(-slope, static_cast<float>(len - 1 - tok), s);
     }
     const float m_new = fmaxf(m, warp_max(s));
-    const float pr = tok < n ? expf(s - m_new) : 0.f;
+    const float pr = live ? expf(s - m_new) : 0.f;
     const float alpha = m == -INFINITY ? 0.f : expf(m - m_new);
     l = l * alpha + warp_sum(pr);
     m = m_new;
 #pragma unroll
     for (int j = 0; j < kNV; ++j) o[j] *= alpha;
-    const int cnt = min(32, n - base);
+    const int cnt = min(32, keys.n - base);
     for (int i = 0; i < cnt; ++i) {
       const float pi = __shfl_sync(0xffffffffu, pr, i);
       const T* v = p.v_pages + __shfl_sync(0xffffffffu, slot, i) * p.ld_v;
@@ -268,7 +300,7 @@ __global__ void __launch_bounds__(128) kv_attention_kernel(const KvAttentionPara
     const int c = lane + 32 * j;
     if (c < p.vdim) {
       float v = o[j] * inv;
-      if (p.gate) v *= sigmoid_f(ld_f(p.gate + r * p.ld_gate + head * p.vdim + c));
+      if (p.gate) v *= sigmoid_f(ld_f(p.gate + r * p.ld_gate + (p.gate_heads ? head : head * p.vdim + c)));
       st_f(p.out + (static_cast<size_t>(r) * p.heads + head) * p.vdim + c, v);
     }
   }
@@ -280,9 +312,11 @@ using namespace sllm;
 
 // Mirrored by ops/kv_attention.py (ctypes.Structure); checked by sllm_kv_abi.
 struct SllmKvPrepare {
-  const void *proj, *conv_w, *ring, *inv_freq, *row_off, *slots, *positions, *seq_index, *block_table, *q, *k_pages, *v_pages;
+  const void *proj, *conv_w, *bias, *q_norm, *k_norm, *ring, *inv_freq, *row_off, *slots, *positions, *seq_index, *block_table, *q,
+      *k_pages, *v_pages;
   long long ring_stride;
-  int ldp, max_blocks, heads, kv_heads, dim, vdim, q_pad, ld_k, ld_v, rot_dims, taps, page_size, tokens, sequences, norm, decode, fp32;
+  int ldp, max_blocks, heads, kv_heads, dim, vdim, q_pad, ld_k, ld_v, rot_dims, taps, page_size, tokens, sequences, norm, decode, fp32,
+      interleaved;
   float eps;
 };
 
@@ -304,6 +338,8 @@ static int kv_prepare_launch(const SllmKvPrepare* a, cudaStream_t st) {
   KvPrepareParams<T> p = {};
   auto n = [](const void* x) { return static_cast<const int*>(x); };
   auto t = [](const void* x) { return static_cast<T*>(const_cast<void*>(x)); };
+  p.bias = static_cast<const float*>(a->bias); p.q_norm = static_cast<const float*>(a->q_norm);
+  p.k_norm = static_cast<const float*>(a->k_norm); p.interleaved = a->interleaved;
   p.proj = t(a->proj); p.conv_w = static_cast<const float*>(a->conv_w); p.ring = static_cast<float*>(const_cast<void*>(a->ring));
   p.inv_freq = static_cast<const float*>(a->inv_freq); p.row_off = n(a->row_off); p.slots = n(a->slots);
   p.positions = n(a->positions); p.seq_index = n(a->seq_index); p.block_table = n(a->block_table);
@@ -319,7 +355,10 @@ static int kv_prepare_launch(const SllmKvPrepare* a, cudaStream_t st) {
   const size_t smem = sizeof(float2) * p.run * (p.rot_dims / 2 + 1);
   const int wide = p.q_pad > p.vdim ? p.q_pad : p.vdim;
   cudaError_t e;
-  if (p.taps <= 4) {
+  if (p.taps == 1) {
+    e = wide <= 64 ? kv_prepare_go<T, 1, 1>(p, smem, st) : wide <= 128 ? kv_prepare_go<T, 2, 1>(p, smem, st)
+                                                                        : kv_prepare_go<T, 4, 1>(p, smem, st);
+  } else if (p.taps <= 4) {
     e = wide <= 64 ? kv_prepare_go<T, 1, 4>(p, smem, st) : wide <= 128 ? kv_prepare_go<T, 2, 4>(p, smem, st)
                                                                         : kv_prepare_go<T, 4, 4>(p, smem, st);
   } else {
@@ -327,15 +366,15 @@ static int kv_prepare_launch(const SllmKvPrepare* a, cudaStream_t st) {
                                                                         : kv_prepare_go<T, 4, 8>(p, smem, st);
   }
   if (e != cudaSuccess) return SLLM_ERR_CUDA;
-  if (p.decode || p.taps < 2) return SLLM_OK;
+  if (p.decode || p.taps < 2 || !p.conv_w) return SLLM_OK;
   const int channels = (p.heads + p.kv_heads) * p.dim + p.kv_heads * p.vdim;
-  return launch_kernel(conv_ring_kernel<T>, dim3((channels + 255) / 256, a->sequences), dim3(256), 0, st, 1u, p.proj, p.ldp, p.ring,
-                       p.ring_stride, p.row_off, p.slots, p.positions, channels, p.taps) == cudaSuccess ? SLLM_OK : SLLM_ERR_CUDA;
+  return conv_ring_launch(p.proj, p.ldp, std::is_same_v<T, float>, p.ring, p.ring_stride, p.row_off, p.slots, p.positions, channels,
+                          p.taps, a->sequences, st) == cudaSuccess ? SLLM_OK : SLLM_ERR_CUDA;
 }
 
 // kv_heads 0: a layer without keys and values of its own (queries only).
 SLLM_EXPORT int sllm_kv_prepare(const SllmKvPrepare* a, void* stream) {
-  if (!a || !a->proj || !a->conv_w || !a->ring || !a->slots || !a->positions || !a->seq_index || !a->q || a->heads <= 0 ||
+  if (!a || !a->proj || (a->conv_w && !a->ring) || (!a->conv_w && a->taps != 1) || (a->bias && a->conv_w) || !a->slots || !a->positions || !a->seq_index || !a->q || a->heads <= 0 ||
       a->kv_heads < 0 || a->dim <= 0 || a->vdim <= 0 || a->q_pad < a->dim || a->taps <= 0 || a->tokens <= 0 || a->sequences <= 0 ||
       a->rot_dims < 0 || a->rot_dims > a->dim || (a->rot_dims & 1) || (a->rot_dims > 0 && !a->inv_freq) || (!a->decode && !a->row_off) ||
       (a->decode && a->tokens != a->sequences))
@@ -372,13 +411,16 @@ static int kv_attention_launch(const KvAttentionParams<T>& p, int rows, cudaStre
   return e == cudaSuccess ? SLLM_OK : SLLM_ERR_CUDA;
 }
 
-// q [rows, heads, q_pad]; gate: optional logits [rows, ld_gate], one per output channel; out [rows, heads * vdim].
+// q [rows, heads, q_pad]; gate: optional logits [rows, ld_gate], one per output channel (gate_heads: per head); keep_first,
+// chunk: see VisibleKeys; slopes: optional [heads]; out [rows, heads * vdim].
 SLLM_EXPORT int sllm_kv_attention(const void* q, const void* k_pages, const void* v_pages, const void* gate, long long ld_gate,
                                   const float* sinks, const int* block_table, int max_blocks, const int* seq_index, const int* kv_lens,
                                   int rows, int heads, int kv_heads, int dim, int vdim, int q_pad, int ld_k, int ld_v, int page_size,
-                                  int window, float scale, void* out, int fp32, void* stream) {
+                                  int window, int keep_first, int chunk, const float* slopes, int gate_heads, float scale, void* out,
+                                  int fp32, void* stream) {
   if (!q || !k_pages || !v_pages || !block_table || !seq_index || !kv_lens || !out || rows <= 0 || heads <= 0 || kv_heads <= 0 ||
-      heads % kv_heads || dim <= 0 || vdim <= 0 || q_pad < dim || ld_k < dim || ld_v < vdim || page_size <= 0 || window < 0)
+      heads % kv_heads || dim <= 0 || vdim <= 0 || q_pad < dim || ld_k < dim || ld_v < vdim || page_size <= 0 || window < 0 || keep_first < 0 ||
+      chunk < 0 || (keep_first > 0 && window == 0) || (chunk > 0 && window > 0))
     return SLLM_ERR_INVALID_ARGUMENT;
   if (vdim > 256 || dim > 2048) return SLLM_ERR_UNSUPPORTED_SHAPE;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
@@ -388,7 +430,7 @@ SLLM_EXPORT int sllm_kv_attention(const void* q, const void* k_pages, const void
     p->gate = static_cast<const T*>(gate); p->ld_gate = ld_gate; p->sinks = sinks; p->block_table = block_table;
     p->max_blocks = max_blocks; p->seq_index = seq_index; p->kv_lens = kv_lens; p->out = static_cast<T*>(out);
     p->heads = heads; p->kv_heads = kv_heads; p->dim = dim; p->vdim = vdim; p->q_pad = q_pad; p->ld_k = ld_k; p->ld_v = ld_v;
-    p->page_size = page_size; p->window = window; p->scale = scale;
+    p->page_size = page_size; p->window = window; p->keep_first = keep_first; p->chunk = chunk; p->slopes = slopes; p->gate_heads = gate_heads; p->scale = scale;
   };
   if (fp32) {
     KvAttentionParams<float> p = {};

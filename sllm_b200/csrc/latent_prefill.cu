@@ -110,14 +110,18 @@ latent_pack_q_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, __nv_bf
 //   warps 4-11  softmax: two threads per query row, 64 keys each; row maxima meet in shared memory, P goes to shared
 //               memory as the bf16 K-major operand, each thread folds half of the value columns into registers
 // Causal with any offset between queries and context, optional sliding window (key tiles outside it are not visited).
+// kRich adds chunks of positions, distance slopes, and windows whose first `keep_first` positions stay visible: a tile that
+// lies past those walks two runs of key tiles, the kept positions and the window.
 constexpr int kLpThreads = 384;
 constexpr int kLpTile = 128;
 constexpr int kLpChunk = kLpTile * 128;
 
 struct LatentPrefillParams {
-  const int* tiles;          // [tiles][8]: query row, rows, position of the first row, context row, its position, -, -, -
-  int heads, kv_heads, dim, vdim, dim_chunks, v_stages, window;
+  const int* tiles;          // [tiles][8]: query row, rows, position of the first row, context row, its position, context row
+                             // of position 0 (with kept positions), -, -
+  int heads, kv_heads, dim, vdim, dim_chunks, v_stages, window, keep_first, chunk;
   float scale_log2;
+  const float* slopes;       // optional [heads]: taken off a score per position of distance
   const float* sinks;        // optional [heads]: scores that join the denominator only
   const __nv_bfloat16* gate; // optional logits [tokens, ld_gate], one per head or (gate_channels) per output channel
   long long ld_gate;
@@ -158,7 +162,7 @@ __device__ __forceinline__ float lp_ex2(float x) {
 __device__ __forceinline__ void lp_bar_softmax() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 
 // kNQ: 64-channel chunks of a query / key row; kNV: of a value row.
-template <int kNQ, int kNV>
+template <int kNQ, int kNV, bool kRich>
 __global__ void __launch_bounds__(kLpThreads, 1)
 latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_kv,
                       const __grid_constant__ CUtensorMap tm_r, const LatentPrefillParams p) {
@@ -175,9 +179,16 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   const int head = blockIdx.y, kvh = head / (p.heads / p.kv_heads);
   const int* tile = p.tiles + 8 * blockIdx.x;
   const int q_row = tile[0], rows = tile[1], q0 = tile[2], k_lo = tile[4];
-  const int first = p.window > 0 ? max(k_lo, q0 - p.window + 1) : k_lo;   // first visible position of the tile's rows
-  const int c_row = tile[3] + first - k_lo;
-  const int nt = (q0 + rows - first + kLpTile - 1) / kLpTile;
+  // first visible position of the tile's rows; with kept positions, those below `kept` take `kept_tiles` key tiles of their own
+  int first = p.window > 0 ? max(k_lo, q0 - p.window + 1) : kRich && p.chunk > 0 ? max(k_lo, q0 / p.chunk * p.chunk) : k_lo;
+  int kept = 0;
+  if (kRich && p.keep_first > 0) {
+    if (first > p.keep_first) kept = p.keep_first;
+    else first = k_lo;                               // 0: the rows are gathered from the start
+  }
+  const int kept_tiles = kRich ? (kept + kLpTile - 1) / kLpTile : 0, kept_row = tile[5];
+  const int c_row = tile[3] + first - k_lo - kept_tiles * kLpTile;
+  const int nt = kept_tiles + (q0 + rows - first + kLpTile - 1) / kLpTile;
   volatile int* abort_flag = &sh->abort_flag;
   if (threadIdx.x == 0) {
     mbar_init(&sh->q_full, 1);
@@ -212,7 +223,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
         tma_load_2d(q_s + c * kLpChunk, &tm_q, &sh->q_full, (head * kNQ + c) * 64, q_row);
       int ks = 0, vs = 0;
       for (int j = 0; j < nt; ++j) {
-        const int y = c_row + j * kLpTile, st = j & 1, sv = j % p.v_stages;
+        const int y = (j < kept_tiles ? kept_row : c_row) + j * kLpTile, st = j & 1, sv = j % p.v_stages;
         if (!mbar_wait(&sh->k_empty[st], ((j >> 1) & 1) ^ 1, abort_flag, p.status, SLLM_DEV_TIMEOUT_SMEM_EMPTY)) break;
         mbar_expect_tx(&sh->k_full[st], kNQ * kLpChunk);
         for (int c = 0; c < kNQ; ++c) {
@@ -286,6 +297,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
     for (int i = 0; i < kO; ++i) o[i] = 0.f;
     float m = -INFINITY, l = 0.f, alpha_prev = 0.f;
     bool ok = true;
+    const float slope = kRich && p.slopes ? p.slopes[head] * 1.4426950408889634f : 0.f;
+    const float mul = kRich && p.slopes ? 1.f : p.scale_log2;   // with slopes the scores are scaled before the mask
     auto fold = [&](int j) {                         // o <- o * alpha(j) + PV(j)
       if (ok) ok = mbar_wait(&sh->o_full[j & 1], (j >> 1) & 1, abort_flag, p.status, SLLM_DEV_TIMEOUT_TMEM_FULL);
       tc_fence_after();
@@ -312,8 +325,27 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
 #pragma unroll
         for (int i = 0; i < 16; ++i) s[c * 16 + i] = __uint_as_float(v[i]);
       }
-      const int k0 = first + j * kLpTile;
-      if (k0 + kLpTile - 1 > q0 || (p.window > 0 && k0 <= q0 + kLpTile - 1 - p.window)) {
+      const int k0 = (j < kept_tiles ? 0 : first - kept_tiles * kLpTile) + j * kLpTile;
+      if constexpr (kRich) {
+        if (p.slopes) {
+          const float d0 = static_cast<float>(k0 + half * 64 - qpos);
+#pragma unroll
+          for (int i = 0; i < 64; ++i) s[i] = fmaf(s[i], p.scale_log2, slope * (d0 + static_cast<float>(i)));
+        }
+        // keys [lo, hi] of this thread's 64 are visible, and those before `head_keys`
+        int hi = 64, lo = 0, head_keys = 0;
+        if (j < kept_tiles) {
+          hi = kept - 1 - half * 64;                 // all kept positions precede the tile's rows
+        } else {
+          hi = qpos - (k0 + half * 64);
+          lo = p.window > 0 ? hi - p.window + 1 : p.chunk > 0 ? hi - qpos % p.chunk : 0;
+          if (kept == 0) head_keys = p.keep_first - (k0 + half * 64);
+        }
+        if (hi < 63 || lo > 0) {
+#pragma unroll
+          for (int i = 0; i < 64; ++i) s[i] = i > hi || (i < lo && i >= head_keys) ? -INFINITY : s[i];
+        }
+      } else if (k0 + kLpTile - 1 > q0 || (p.window > 0 && k0 <= q0 + kLpTile - 1 - p.window)) {
         const int hi = qpos - (k0 + half * 64);      // keys [lo, hi] of this thread's 64 are visible
         const int lo = p.window > 0 ? hi - p.window + 1 : 0;
 #pragma unroll
@@ -325,7 +357,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
       const float tmax = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
       sh->red[j & 1][half][r] = tmax;
       lp_bar_softmax();
-      const float m_new = fmaxf(m, fmaxf(tmax, sh->red[j & 1][half ^ 1][r]) * p.scale_log2);
+      const float m_new = fmaxf(m, fmaxf(tmax, sh->red[j & 1][half ^ 1][r]) * mul);
       const float m_use = m_new == -INFINITY ? 0.f : m_new;
       const float alpha = m == -INFINITY ? 0.f : lp_ex2(m - m_use);
       if (j > 0) fold(j - 1);                        // P(j - 1) has been consumed: its buffer is free
@@ -336,8 +368,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
         uint32_t w[4];
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
-          const __nv_bfloat162 h = __floats2bfloat162_rn(lp_ex2(fmaf(s[u * 8 + 2 * i], p.scale_log2, -m_use)),
-                                                         lp_ex2(fmaf(s[u * 8 + 2 * i + 1], p.scale_log2, -m_use)));
+          const __nv_bfloat162 h = __floats2bfloat162_rn(lp_ex2(fmaf(s[u * 8 + 2 * i], mul, -m_use)),
+                                                         lp_ex2(fmaf(s[u * 8 + 2 * i + 1], mul, -m_use)));
           // the normaliser sums the rounded values, which are what the product multiplies
           sum[0] += __bfloat162float(h.x);
           sum[1] += __bfloat162float(h.y);
@@ -388,8 +420,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   }
 }
 
-template <int kNQ, int kNV>
-static int latent_prefill_launch(const CUtensorMap& tq, const CUtensorMap& tkv, const CUtensorMap& tr, LatentPrefillParams p,
+template <int kNQ, int kNV, bool kRich>
+static int latent_prefill_go(const CUtensorMap& tq, const CUtensorMap& tkv, const CUtensorMap& tr, LatentPrefillParams p,
                                  int tiles, cudaStream_t st) {
   // two V stages where they fit; at least 120 KB, so that one CTA (which takes the whole TMEM) is on an SM at a time
   p.v_stages = (3 * kNQ + 2 + 2 * kNV) * kLpChunk <= 208 * 1024 ? 2 : 1;
@@ -397,13 +429,20 @@ static int latent_prefill_launch(const CUtensorMap& tq, const CUtensorMap& tkv, 
   if (smem < 120 * 1024) smem = 120 * 1024;
   static bool cfg = false;
   if (!cfg) {
-    if (cudaFuncSetAttribute(latent_prefill_kernel<kNQ, kNV>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) !=
+    if (cudaFuncSetAttribute(latent_prefill_kernel<kNQ, kNV, kRich>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) !=
         cudaSuccess)
       return SLLM_ERR_CUDA;
     cfg = true;
   }
-  return launch_kernel(latent_prefill_kernel<kNQ, kNV>, dim3(tiles, p.heads), dim3(kLpThreads), smem, st, 1u, tq, tkv, tr, p) ==
+  return launch_kernel(latent_prefill_kernel<kNQ, kNV, kRich>, dim3(tiles, p.heads), dim3(kLpThreads), smem, st, 1u, tq, tkv, tr, p) ==
                  cudaSuccess ? SLLM_OK : SLLM_ERR_CUDA;
+}
+
+template <int kNQ, int kNV>
+static int latent_prefill_launch(const CUtensorMap& tq, const CUtensorMap& tkv, const CUtensorMap& tr, const LatentPrefillParams& p,
+                                 int tiles, cudaStream_t st) {
+  return p.keep_first > 0 || p.chunk > 0 || p.slopes ? latent_prefill_go<kNQ, kNV, true>(tq, tkv, tr, p, tiles, st)
+                                                     : latent_prefill_go<kNQ, kNV, false>(tq, tkv, tr, p, tiles, st);
 }
 
 }  // namespace sllm
@@ -475,17 +514,21 @@ SLLM_EXPORT int sllm_latent_prefill(const void* q, int tokens, const void* kv, c
 }
 
 // The same kernel over ordinary keys and values: q [tokens, heads, dim padded to 64 with zeros]; kv [context rows, kv_heads *
-// (dim + vdim)]; sinks: optional [heads]; gate: optional logits [tokens, ld_gate], one per output channel.
+// (dim + vdim)]; sinks, slopes: optional [heads]; gate: optional logits [tokens, ld_gate], one per output channel
+// (gate_heads: per head).
 SLLM_EXPORT int sllm_kv_prefill(const void* q, int tokens, const void* kv, int context, const int* tiles, int num_tiles, int heads,
-                                int kv_heads, int dim, int vdim, int window, float scale, const float* sinks, const void* gate,
-                                long long ld_gate, void* out, int* status, void* stream) {
+                                int kv_heads, int dim, int vdim, int window, int keep_first, int chunk, const float* slopes, float scale,
+                                const float* sinks, const void* gate, long long ld_gate, int gate_heads, void* out, int* status,
+                                void* stream) {
   if (!q || !kv || !tiles || !out || tokens <= 0 || context <= 0 || num_tiles <= 0 || heads <= 0 || heads > 65535 || kv_heads <= 0 ||
-      heads % kv_heads || dim <= 0 || vdim <= 0 || window < 0)
+      heads % kv_heads || dim <= 0 || vdim <= 0 || window < 0 || keep_first < 0 || chunk < 0 || (keep_first > 0 && window == 0) ||
+      (chunk > 0 && window > 0))
     return SLLM_ERR_INVALID_ARGUMENT;
-  if (gate && ((ld_gate & 7) || (reinterpret_cast<uintptr_t>(gate) & 15))) return SLLM_ERR_ALIGNMENT;
+  if (gate && !gate_heads && ((ld_gate & 7) || (reinterpret_cast<uintptr_t>(gate) & 15))) return SLLM_ERR_ALIGNMENT;
   LatentPrefillParams p = {};
   p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim; p.window = window; p.scale_log2 = scale * 1.4426950408889634f;
-  p.sinks = sinks; p.gate = static_cast<const __nv_bfloat16*>(gate); p.ld_gate = ld_gate; p.gate_channels = 1;
+  p.sinks = sinks; p.gate = static_cast<const __nv_bfloat16*>(gate); p.ld_gate = ld_gate; p.gate_channels = !gate_heads;
+  p.keep_first = keep_first; p.chunk = chunk; p.slopes = slopes;
   p.out = static_cast<__nv_bfloat16*>(out); p.status = status;
   return latent_prefill_impl(q, tokens, kv, nullptr, context, tiles, num_tiles, 0, p, static_cast<cudaStream_t>(stream));
 }

@@ -1,8 +1,9 @@
 // Mixture-of-experts routing and token movement.
 //
 //   moe_route        router logits [T, E] -> top-k experts per token and their weights (softmax over the k
-//                    selected logits, or the selected entries of the softmax over all experts), optionally from the
-//                    best groups of experts only; moe_router computes the logits as well;
+//                    selected logits, the selected entries of the softmax over all experts, or sigmoid scores with a
+//                    correction that only takes part in the choice), optionally from the best groups of experts only;
+//                    moe_router computes the logits as well;
 //   moe_permute      groups the T x k assignments by expert: tok_off[E_local + 1], perm_src[P] (source token of
 //                    each permuted row), perm_dst[T, k] (row of each assignment, -1 when the expert is not local),
 //                    perm_w[P] (routing weight of each permuted row);
@@ -22,15 +23,22 @@
 #include "typed.cuh"
 #include "api.h"
 
+#include <cstddef>
+
 namespace sllm {
 
 constexpr int kMaxTopK = 32;
 constexpr int kMaxExperts = 256;
 constexpr int kRouteSlots = kMaxExperts / 32;
 
+enum RouteMode { kRouteSoftmaxTop = 0, kRouteSoftmaxAll = 1, kRouteSigmoid = 2 };
+
 struct RouteRule {
-  int experts, top_k, softmax_all;
+  int experts, top_k, mode;
   int group_size, keep;      // only experts of the `keep` groups with the largest scores are eligible (keep 0: all)
+  int group_top;             // a group's score is the sum of this many of its largest (1 or 2)
+  const float* correction;   // optional [experts]: joins the scores for the choice, not for the weights
+  float scale;               // of the weights
 };
 
 // Largest of the eligible v over a warp, ties to the lower index; index 0x7fffffff when there is none.
@@ -55,13 +63,22 @@ __device__ __forceinline__ void route_best(const float (&v)[kRouteSlots], unsign
   }
 }
 
-// One warp routes one token: v[i] is the logit of expert i * 32 + lane (-inf past the experts and for NaN).
+// One warp routes one token: v[i] is the logit of expert i * 32 + lane (-inf past the experts and for NaN); `scratch`:
+// kMaxExperts floats of shared memory of this warp.
 template <bool kExact>
-__device__ __forceinline__ void route_warp(const float (&v)[kRouteSlots], int lane, const RouteRule& rule, int* __restrict__ out_idx,
-                                           float* __restrict__ out_w) {
+__device__ __forceinline__ void route_warp(float (&v)[kRouteSlots], int lane, const RouteRule& rule, float* scratch,
+                                           int* __restrict__ out_idx, float* __restrict__ out_w) {
   auto ex = [](float x) { return kExact ? expf(x) : __expf(x); };
   float denom_all = 0.f, mx_all = -INFINITY;
-  if (rule.softmax_all) {
+  float score[kRouteSlots];
+  if (rule.mode == kRouteSigmoid) {                     // v becomes the choice scores
+#pragma unroll
+    for (int i = 0; i < kRouteSlots; ++i) {
+      score[i] = v[i] == -INFINITY ? 0.f : 1.f / (1.f + ex(-v[i]));
+      if (v[i] != -INFINITY) v[i] = score[i] + (rule.correction ? rule.correction[i * 32 + lane] : 0.f);
+    }
+  }
+  if (rule.mode == kRouteSoftmaxAll) {
 #pragma unroll
     for (int i = 0; i < kRouteSlots; ++i) mx_all = fmaxf(mx_all, v[i]);
     mx_all = warp_max(mx_all);
@@ -74,12 +91,43 @@ __device__ __forceinline__ void route_warp(const float (&v)[kRouteSlots], int la
   int bi;
   if (rule.keep > 0) {
     unsigned kept = 0u;
-    for (int g = 0; g < rule.keep; ++g) {
-      route_best(v, ~kept, lane, best, bi);
-      if (bi == 0x7fffffff) break;
+    if (rule.group_top == 2) {                          // lane g scores groups g, g + 32, ..
 #pragma unroll
       for (int i = 0; i < kRouteSlots; ++i)
-        if ((i * 32 + lane) / rule.group_size == bi / rule.group_size) kept |= 1u << i;
+        if (i * 32 + lane < rule.experts) scratch[i * 32 + lane] = v[i];
+      __syncwarp();
+      const int groups = rule.experts / rule.group_size;
+      float gs[kRouteSlots];
+#pragma unroll
+      for (int i = 0; i < kRouteSlots; ++i) {
+        gs[i] = -INFINITY;
+        if (i * 32 + lane < groups) {
+          const float* m = scratch + (i * 32 + lane) * rule.group_size;
+          float a = -INFINITY, b = -INFINITY;
+          for (int e = 0; e < rule.group_size; ++e) {
+            b = fmaxf(b, fminf(a, m[e]));
+            a = fmaxf(a, m[e]);
+          }
+          gs[i] = b == -INFINITY ? a : a + b;
+        }
+      }
+      unsigned open = 0xffffffffu;
+      for (int g = 0; g < rule.keep; ++g) {
+        route_best(gs, open, lane, best, bi);
+        if (bi == 0x7fffffff) break;
+        if ((bi & 31) == lane) open &= ~(1u << (bi >> 5));
+#pragma unroll
+        for (int i = 0; i < kRouteSlots; ++i)
+          if ((i * 32 + lane) / rule.group_size == bi) kept |= 1u << i;
+      }
+    } else {
+      for (int g = 0; g < rule.keep; ++g) {
+        route_best(v, ~kept, lane, best, bi);
+        if (bi == 0x7fffffff) break;
+#pragma unroll
+        for (int i = 0; i < kRouteSlots; ++i)
+          if ((i * 32 + lane) / rule.group_size == bi / rule.group_size) kept |= 1u << i;
+      }
     }
     eligible = kept;
   }
@@ -88,20 +136,34 @@ __device__ __forceinline__ void route_warp(const float (&v)[kRouteSlots], int la
   for (int j = 0; j < rule.top_k; ++j) {
     route_best(v, eligible, lane, best, bi);
     if (bi == 0x7fffffff) bi = j;     // fewer finite logits than k: fall back to distinct low indices
+    if (rule.mode == kRouteSigmoid) {                   // the weight is the score without the correction
+      float s = 0.f;
+#pragma unroll
+      for (int i = 0; i < kRouteSlots; ++i) s = bi >> 5 == i ? score[i] : s;
+      s = __shfl_sync(0xffffffffu, s, bi & 31);
+      best = best == -INFINITY ? best : s;
+    }
     if (lane == j) {
       my_v = best;
       my_i = bi;
     }
     if ((bi & 31) == lane) eligible &= ~(1u << (bi >> 5));
   }
-  // mode 0: softmax over the selected logits; mode 1: probabilities of the softmax over all experts
-  const float m0 = rule.softmax_all ? mx_all : __shfl_sync(0xffffffffu, my_v, 0);
+  if (rule.mode == kRouteSigmoid) {
+    if (lane < rule.top_k) {
+      out_idx[lane] = my_i;
+      out_w[lane] = my_v == -INFINITY ? 0.f : my_v * rule.scale;
+    }
+    return;
+  }
+  // softmax over the selected logits, or probabilities of the softmax over all experts
+  const float m0 = rule.mode == kRouteSoftmaxAll ? mx_all : __shfl_sync(0xffffffffu, my_v, 0);
   const float w = lane >= rule.top_k || my_v == -INFINITY ? 0.f : ex(my_v - m0);
   const float sum = warp_sum(w);
-  const float total = rule.softmax_all ? denom_all : sum;
+  const float total = rule.mode == kRouteSoftmaxAll ? denom_all : sum;
   if (lane < rule.top_k) {
     out_idx[lane] = my_i;
-    out_w[lane] = sum > 0.f && total > 0.f ? w / total : 1.f / rule.top_k;
+    out_w[lane] = rule.scale * (sum > 0.f && total > 0.f ? w / total : 1.f / rule.top_k);
   }
 }
 
@@ -113,6 +175,7 @@ __global__ void moe_route_kernel(const T* __restrict__ logits, int ld, int token
   pdl_trigger();
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   if (warp >= tokens) return;
+  __shared__ float scratch[4 * kMaxExperts];
   float v[kRouteSlots];
 #pragma unroll
   for (int i = 0; i < kRouteSlots; ++i) {
@@ -120,7 +183,7 @@ __global__ void moe_route_kernel(const T* __restrict__ logits, int ld, int token
     const float x = e < rule.experts ? ld_f(logits + static_cast<size_t>(warp) * ld + e) : -INFINITY;
     v[i] = (x == x) ? x : -INFINITY;
   }
-  route_warp<sizeof(T) == 4>(v, lane, rule, out_idx + static_cast<size_t>(warp) * rule.top_k, out_w + static_cast<size_t>(warp) * rule.top_k);
+  route_warp<sizeof(T) == 4>(v, lane, rule, scratch + (threadIdx.x >> 5) * kMaxExperts, out_idx + static_cast<size_t>(warp) * rule.top_k, out_w + static_cast<size_t>(warp) * rule.top_k);
 }
 
 // Router product (fp32 sums, never rounded) and selection of one token per CTA: decode batches and 32-bit models.
@@ -178,7 +241,7 @@ moe_router_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ w, int
     const float t = e < rule.experts ? z[e] : -INFINITY;
     v[i] = (t == t) ? t : -INFINITY;
   }
-  route_warp<true>(v, lane, rule, out_idx + static_cast<size_t>(blockIdx.x) * rule.top_k, out_w + static_cast<size_t>(blockIdx.x) * rule.top_k);
+  route_warp<true>(v, lane, rule, z, out_idx + static_cast<size_t>(blockIdx.x) * rule.top_k, out_w + static_cast<size_t>(blockIdx.x) * rule.top_k);
 }
 
 // Single CTA of kPermuteThreads threads.  Counts per local expert in shared memory, exclusive scan, then a stable
@@ -675,26 +738,36 @@ SLLM_EXPORT int sllm_moe_owner_combine(void* const* recv, void* const* gath, voi
   return SLLM_OK;
 }
 
-static int route_rule(RouteRule* r, int experts, int top_k, int softmax_all, int groups, int keep) {
-  if (experts <= 0 || experts > kMaxExperts || top_k <= 0 || top_k > kMaxTopK || top_k > experts || groups < 0 || keep < 0)
+struct SllmRouteRule {     // host-side mirror passed by the Python layer (ctypes.Structure)
+  const float* correction;
+  int experts, top_k, mode, groups, keep, group_top;
+  float scale;
+};
+
+static int route_rule(RouteRule* r, const SllmRouteRule* a) {
+  if (!a || a->experts <= 0 || a->experts > kMaxExperts || a->top_k <= 0 || a->top_k > kMaxTopK || a->top_k > a->experts || a->groups < 0 ||
+      a->keep < 0 || a->mode < kRouteSoftmaxTop || a->mode > kRouteSigmoid || a->group_top < 1 || a->group_top > 2 ||
+      (a->correction && a->mode != kRouteSigmoid))
     return SLLM_ERR_INVALID_ARGUMENT;
-  r->experts = experts; r->top_k = top_k; r->softmax_all = softmax_all; r->group_size = experts; r->keep = 0;
-  if (groups > 1) {
-    if (experts % groups || keep < 1 || keep > groups || keep * (experts / groups) < top_k) return SLLM_ERR_INVALID_ARGUMENT;
-    r->group_size = experts / groups;
-    r->keep = keep == groups ? 0 : keep;
+  r->experts = a->experts; r->top_k = a->top_k; r->mode = a->mode; r->group_size = a->experts; r->keep = 0;
+  r->group_top = a->group_top; r->correction = a->correction; r->scale = a->scale;
+  if (a->groups > 1) {
+    if (a->experts % a->groups || a->keep < 1 || a->keep > a->groups || a->keep * (a->experts / a->groups) < a->top_k)
+      return SLLM_ERR_INVALID_ARGUMENT;
+    r->group_size = a->experts / a->groups;
+    r->keep = a->keep == a->groups ? 0 : a->keep;
   }
   return SLLM_OK;
 }
 
-// groups > 1: neighbouring experts form that many equal groups, a group's score is its largest, and only experts of the
-// `keep` best groups are selected.  fp32: element type of the logits (0 bf16, 1 fp32).
-SLLM_EXPORT int sllm_moe_route(const void* logits, int ld, int tokens, int experts, int top_k, int softmax_all, int groups, int keep,
-                               int fp32, int* out_idx, float* out_w, void* stream) {
+// route->groups > 1: neighbouring experts form that many equal groups, a group's score is the sum of its group_top largest,
+// and only experts of the `keep` best groups are selected.  fp32: element type of the logits (0 bf16, 1 fp32).
+SLLM_EXPORT int sllm_moe_route(const void* logits, int ld, int tokens, const SllmRouteRule* route, int fp32, int* out_idx, float* out_w,
+                               void* stream) {
   RouteRule rule;
-  if (!logits || !out_idx || !out_w || tokens <= 0 || ld < experts) return SLLM_ERR_INVALID_ARGUMENT;
-  const int rc = route_rule(&rule, experts, top_k, softmax_all, groups, keep);
+  const int rc = route_rule(&rule, route);
   if (rc != SLLM_OK) return rc;
+  if (!logits || !out_idx || !out_w || tokens <= 0 || ld < rule.experts) return SLLM_ERR_INVALID_ARGUMENT;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const cudaError_t e = fp32 ? launch_kernel(moe_route_kernel<float>, dim3((tokens + 3) / 4), dim3(128), 0, st, 1u,
                                              static_cast<const float*>(logits), ld, tokens, rule, out_idx, out_w)
@@ -704,12 +777,12 @@ SLLM_EXPORT int sllm_moe_route(const void* logits, int ld, int tokens, int exper
 }
 
 // Router product x w^T (x [tokens, d], w [experts, d], both bf16 or both fp32) and the selection in one launch.
-SLLM_EXPORT int sllm_moe_router(const void* x, int ldx, const void* w, int tokens, int d, int experts, int top_k, int softmax_all,
-                                int groups, int keep, int fp32, int* out_idx, float* out_w, void* stream) {
+SLLM_EXPORT int sllm_moe_router(const void* x, int ldx, const void* w, int tokens, int d, const SllmRouteRule* route, int fp32, int* out_idx,
+                                float* out_w, void* stream) {
   RouteRule rule;
-  if (!x || !w || !out_idx || !out_w || tokens <= 0 || d <= 0 || ldx < d) return SLLM_ERR_INVALID_ARGUMENT;
-  const int rc = route_rule(&rule, experts, top_k, softmax_all, groups, keep);
+  const int rc = route_rule(&rule, route);
   if (rc != SLLM_OK) return rc;
+  if (!x || !w || !out_idx || !out_w || tokens <= 0 || d <= 0 || ldx < d) return SLLM_ERR_INVALID_ARGUMENT;
   const size_t smem = sizeof(float) * d;
   if (smem > 40 * 1024) return SLLM_ERR_UNSUPPORTED_SHAPE;
   const int vec = d % (fp32 ? 4 : 8) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0;
@@ -720,6 +793,12 @@ SLLM_EXPORT int sllm_moe_router(const void* x, int ldx, const void* w, int token
                                              static_cast<const __nv_bfloat16*>(x), ldx, static_cast<const __nv_bfloat16*>(w), d, rule,
                                              vec, out_idx, out_w);
   return e == cudaSuccess ? SLLM_OK : SLLM_ERR_CUDA;
+}
+
+SLLM_EXPORT int sllm_moe_route_abi(int* out, int n) {
+  const int v[2] = {static_cast<int>(sizeof(SllmRouteRule)), static_cast<int>(offsetof(SllmRouteRule, scale))};
+  for (int i = 0; i < n && i < 2; ++i) out[i] = v[i];
+  return 2;
 }
 
 // counts: optional scratch of ceil(tokens * top_k / 1024) * (e_hi - e_lo) ints; with it, batches of more than one chunk take

@@ -15,7 +15,7 @@ from .config import ModelConfig
 KERNEL_UNITS = {
     "zokuvik": ("elementwise", "gemm_tcgen05", "gemm_simt", "group_norm", "latent_attention", "latent_decode", "latent_prefill",
                 "delta_rule"),
-    "sepedra": ("elementwise", "gemm_tcgen05", "gemm_simt", "group_norm", "attention", "kv_attention", "latent_prefill", "rglru", "moe",
+    "sepedra": ("elementwise", "gemm_tcgen05", "gemm_simt", "group_norm", "attention", "kv_attention", "short_conv", "latent_prefill", "rglru", "moe",
                 "moe_dense"),
 }
 

@@ -166,12 +166,14 @@ def check(rc: int, what: str) -> None:
 _KERNEL_SIGNATURES = {
     "sllm_gemm_workspace_floats": (L, [I, I, I, I]),
     "sllm_gemm": (I, [P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, P, L, P, I, P, P]),
-    "sllm_gemm_act": (I, [P, P, P, I, I, I, I, I, I, F, I, I, I, I, P, L, P, I, P, P]),
+    "sllm_gemm_act": (I, [P, P, P, I, I, I, I, I, I, I, F, I, I, I, I, P, L, P, I, P, P]),
     "sllm_gemm_simt": (I, [P, P, P, P, I, I, I, I, I, I, I, F, I, I, P]),
-    "sllm_group_norm": (I, [P, P, I, P, I, P, I, P, P, P, P, P, I, I, I, F, I, P]),
+    "sllm_group_norm": (I, [P, P]),
+    "sllm_group_norm_abi": (I, [P, I]),
     "sllm_embedding": (I, [P, P, P, I, I, I, F, P]),
     "sllm_rmsnorm": (I, [P, P, P, P, P, I, I, I, F, I, P]),
     "sllm_gated_act": (I, [P, P, P, P, I, I, I, I, P]),
+    "sllm_gated_act_any": (I, [P, P, I, I, I, I, I, P]),
     "sllm_quant_fp8_1x128": (I, [P, P, P, I, I, I, P]),
     "sllm_rope_kv_append": (I, [P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, F, F, P, P]),
     "sllm_rope_kv_append_paired": (I, [P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, F, F, P, I, P]),
@@ -185,7 +187,7 @@ _KERNEL_SIGNATURES = {
     "sllm_prefill_attention": (I, [P, I, I, P, I, I, I, I, F, P, P, P, I, P, P]),
     "sllm_paged_attention_workspace_floats": (L, [I, I, I, I, I]),
     "sllm_paged_attention": (I, [P, I, P, P, P, P, F, F, P, I, P, P, I, I, I, I, I, I, F, I, P, P, P, I, P, I, P, L,
-                                  P, I, P, L, P]),
+                                  P, I, P, L, I, I, I, P, P]),
 }
 
 # Entry points added by later translation units register themselves here (name -> (restype, argtypes)).

@@ -177,7 +177,8 @@ def linear(x, w: LinearWeight, residual: Optional[torch.Tensor] = None, act: Opt
            out_fp32: bool = False) -> torch.Tensor:
     """Y = act(X W^T) (+ residual).  x: Tensor [M, K] (bf16 / fp32) or QTensor for FP8 weights.  ``act``: None, "relu_sq"
     (square of relu) or "softcap" (act_arg * tanh(y / act_arg)), applied to the fp32 sums; ``out_fp32`` stores the sums
-    unrounded.  Both take dense weights without a residual."""
+    unrounded.  Both take dense weights without a residual, and so does an ``x`` of columns of a wider matrix (row stride a multiple
+    of 8, 16-byte aligned)."""
     if act not in _ACTS or ((act or out_fp32) and (w.kind != "dense" or residual is not None)):
         raise ValueError("the product's activation is relu_sq or softcap, on dense weights without a residual")
     xd = x.data if isinstance(x, QTensor) else x
@@ -225,12 +226,15 @@ def linear(x, w: LinearWeight, residual: Optional[torch.Tensor] = None, act: Opt
             gemm_raw(x.data, w.w, y, scale_a=x.scale, scale_b=w.scale_t, residual=residual, transpose_out=False,
                      bn=bn, splits=splits, stages=stages)
     else:
-        if act or out_fp32:
+        strided = m > 1 and x.stride(0) != x.shape[1]
+        if strided and residual is not None:
+            raise ValueError("a product with a residual takes contiguous rows")
+        if act or out_fp32 or strided:
             a, b = (w.w, x) if swap else (x, w.w)
             wsp = workspace(xd.device)
-            rc = _lib.kernels().sllm_gemm_act(_p(a), _p(b), _p(y), a.shape[0], b.shape[0], w.in_features, int(swap), n, _ACTS[act],
-                                              act_arg, int(out_fp32), bn, splits, stages, _p(wsp.ws), wsp.ws.numel(), _p(wsp.counters), wsp.counters.numel(),
-                                              _p(wsp.status), _stream())
+            rc = _lib.kernels().sllm_gemm_act(_p(a), _p(b), _p(y), a.shape[0], b.shape[0], w.in_features, x.stride(0) if strided else 0,
+                                              int(swap), n, _ACTS[act], act_arg, int(out_fp32), bn, splits, stages, _p(wsp.ws),
+                                              wsp.ws.numel(), _p(wsp.counters), wsp.counters.numel(), _p(wsp.status), _stream())
             _lib.check(rc, "gemm")
         elif swap:
             gemm_raw(w.w, x, y, residual=residual, transpose_out=True, bn=bn, splits=splits, stages=stages)
@@ -279,40 +283,66 @@ def rmsnorm(x: torch.Tensor, w: torch.Tensor, eps: float, offset_one: bool = Fal
 
 
 # ---- grouped RMSNorm on an fp32 residual stream (csrc/group_norm.cu)
+class GroupNormArgs(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("table", "ids", "step", "y", "y_rows", "w_post", "y2", "w_post2", "x", "row_idx", "w_out", "z")] + \
+        [(n, C.c_int) for n in ("vocab", "ldy", "y_terms", "ldy2", "rows", "d", "groups", "fp32")] + \
+        [(n, C.c_float) for n in ("table_scale", "coef", "coef2", "eps")]
+
+
+class Again(NamedTuple):
+    """What joins the residual before a pass of a looped block: ``scale`` table[ids] (without ``table``: nothing) and the fp32
+    vector ``step`` (or None)."""
+    table: Optional[torch.Tensor] = None
+    ids: Optional[torch.Tensor] = None
+    scale: float = 1.0
+    step: Optional[torch.Tensor] = None
+
+
 def _gn_ref(x: torch.Tensor, w: torch.Tensor, eps: float, groups: int) -> torch.Tensor:
     t, d = x.shape
     g = x.float().view(t, groups, d // groups)
     return (g / torch.sqrt((g * g).mean(-1, keepdim=True) + eps)).view(t, d) * w
 
 
-def _group_norm(x, w_out, eps, groups, dtype, *, table=None, ids=None, y=None, w_post=None, rows_idx=None, terms=None, raw=False):
-    rows = ids.numel() if table is not None else (rows_idx.numel() if rows_idx is not None else x.shape[0])
+def _group_norm(x, w_out, eps, groups, dtype, *, again=Again(), y=None, w_post=None, coef=1.0, second=None, rows_idx=None, terms=None,
+                raw=False):
+    rows = again.ids.numel() if y is None and again.ids is not None else (rows_idx.numel() if rows_idx is not None else x.shape[0])
     d = x.shape[1]
     z = torch.empty((rows, d), dtype=dtype, device=x.device) if w_out is not None or raw else None
     if rows == 0:
         return z
-    rc = _lib.kernels().sllm_group_norm(_p(table), _p(ids), table.shape[0] if table is not None else 0, _p(y),
-                                        y.stride(0) if y is not None else 0, _p(terms), terms.shape[1] if terms is not None else 0,
-                                        _p(w_post), _p(x), _p(rows_idx), _p(w_out), _p(z), rows, d, groups, eps,
-                                        int(dtype == torch.float32), _stream())
-    _lib.check(rc, "group_norm")
+    v = lambda t: None if t is None else t.data_ptr()
+    y2, w2, c2 = second or (None, None, 0.0)
+    a = GroupNormArgs(v(again.table), v(again.ids) if again.table is not None else None, v(again.step), v(y), v(terms), v(w_post), v(y2), v(w2),
+                      v(x), v(rows_idx), v(w_out), v(z), again.table.shape[0] if again.table is not None else 0,
+                      y.stride(0) if y is not None else 0, terms.shape[1] if terms is not None else 0, y2.stride(0) if y2 is not None else 0,
+                      rows, d, groups, int(dtype == torch.float32), again.scale, coef, c2, eps)
+    _lib.check(_lib.kernels().sllm_group_norm(C.byref(a), _stream()), "group_norm")
     return z
 
 
-def embed_group_norm(table: torch.Tensor, ids: torch.Tensor, w_out: Optional[torch.Tensor], eps: float, groups: int = 1):
-    """(residual fp32 [T, d], its grouped RMSNorm in the table's type): the embedding and the first layer's input norm.
-    Without ``w_out`` the second is the residual itself in the table's type."""
+def embed_group_norm(table: torch.Tensor, ids: torch.Tensor, w_out: Optional[torch.Tensor], eps: float, groups: int = 1,
+                     scale: float = 1.0, step: Optional[torch.Tensor] = None):
+    """(residual fp32 [T, d], its grouped RMSNorm in the table's type): the embedding times ``scale`` (plus the vector ``step``)
+    and the first layer's input norm.  Without ``w_out`` the second is the residual itself in the table's type."""
     if _lib.on_cpu(table):
         x = table[ids.long()].float()
+        if scale != 1.0:
+            x = x * scale
+        if step is not None:
+            x = x + step
         return x, (x if w_out is None else _gn_ref(x, w_out, eps, groups)).to(table.dtype, copy=True)
     x = torch.empty((ids.numel(), table.shape[1]), dtype=torch.float32, device=table.device)
-    return x, _group_norm(x, w_out, eps, groups, table.dtype, table=table, ids=ids, raw=True)
+    return x, _group_norm(x, w_out, eps, groups, table.dtype, again=Again(table, ids, scale, step), raw=True)
 
 
-def add_group_norm(x: torch.Tensor, y: torch.Tensor, w_post: torch.Tensor, w_out: Optional[torch.Tensor], eps: float,
-                   groups: int = 1, terms: Optional[torch.Tensor] = None, raw: bool = False):
-    """x += norm(y) * w_post in place (fp32), then norm(x) * w_out in the type of ``y`` (without ``w_out``: x in that type with
-    ``raw``, else None).  ``terms`` (int32 [T, n]): row t of the summand is the sum of the rows terms[t] >= 0 of ``y``."""
+def add_group_norm(x: torch.Tensor, y: torch.Tensor, w_post: Optional[torch.Tensor], w_out: Optional[torch.Tensor], eps: float,
+                   groups: int = 1, terms: Optional[torch.Tensor] = None, raw: bool = False, coef: float = 1.0,
+                   second: Optional[tuple] = None, again: Optional[Again] = None):
+    """x += coef norm(y) * w_post in place (fp32; without ``w_post`` x += coef y), then norm(x) * w_out in the type of ``y``
+    (without ``w_out``: x in that type with ``raw``, else None).  ``terms`` (int32 [T, n]): row t of the summand is the sum of
+    the rows terms[t] >= 0 of ``y``.  ``second``: (y2, its w_post or None, its coef), a further summand.  ``again`` joins x
+    before the output norm."""
     if _lib.on_cpu(x):
         s = y
         if terms is not None:
@@ -320,11 +350,19 @@ def add_group_norm(x: torch.Tensor, y: torch.Tensor, w_post: torch.Tensor, w_out
             for j in range(terms.shape[1]):
                 p = terms[:, j].long()
                 s[p >= 0] += y[p[p >= 0]].float()
-        x += _gn_ref(s, w_post, eps, groups)
+        for v, w, c in ((s, w_post, coef),) + (() if second is None else (second,)):
+            v = v.float() if w is None else _gn_ref(v, w, eps, groups)
+            x += v if c == 1.0 else v * c
+        if again is not None:
+            if again.table is not None:
+                x += again.table[again.ids.long()].float() * again.scale
+            if again.step is not None:
+                x += again.step
         if w_out is None:
             return x.to(y.dtype, copy=True) if raw else None
         return _gn_ref(x, w_out, eps, groups).to(y.dtype)
-    return _group_norm(x, w_out, eps, groups, y.dtype, y=y, w_post=w_post, terms=terms, raw=raw)
+    return _group_norm(x, w_out, eps, groups, y.dtype, y=y, w_post=w_post, coef=coef, second=second, terms=terms, raw=raw,
+                       again=again or Again())
 
 
 def group_norm(x: torch.Tensor, w: torch.Tensor, eps: float, groups: int, dtype, rows: Optional[torch.Tensor] = None):
@@ -346,6 +384,11 @@ def gated_act(x: torch.Tensor, act: str = "silu", quant: bool = False):
     inter = two_i // 2
     lib = _lib.kernels()
     a = 0 if act == "silu" else 1
+    if not quant and (x.dtype == torch.float32 or inter % 8 or x.stride(0) != two_i):
+        y = torch.empty((m, inter), dtype=x.dtype, device=x.device)
+        rc = lib.sllm_gated_act_any(_p(x), _p(y), m, inter, x.stride(0), a, int(x.dtype == torch.float32), _stream())
+        _lib.check(rc, "gated_act")
+        return y
     if quant:
         q = _alloc_q(m, inter, x.device)
         rc = lib.sllm_gated_act(_p(x), None, _p(q.data), _p(q.scale), m, m, inter, a, _stream())
@@ -515,11 +558,15 @@ def paged_attention(q: torch.Tensor, kv: KVLayer, block_table: torch.Tensor, seq
                     kv_lens: torch.Tensor, hq: int, hkv: int, hd: int, *, window: int = 0,
                     sm_scale: Optional[float] = None, max_kv: int = 0, quant_out: bool = False,
                     sinks: Optional[torch.Tensor] = None, impl: Optional[str] = None, out: Optional[QTensor] = None,
-                    gate: Optional[torch.Tensor] = None):
+                    gate: Optional[torch.Tensor] = None, gate_heads: bool = False, keep_first: int = 0, chunk: int = 0,
+                    slopes: Optional[torch.Tensor] = None):
     """Attention of each query row over its sequence's pages. q: [R, hq*hd] (row stride allowed).
     Returns [R, hq*hd] (bf16) or a QTensor when quant_out (head_dim 128); ``out`` supplies the QTensor to fill
     (its scale plane may have a leading dimension larger than R), or the bf16 rows.  ``gate``: logits [R, hq*hd] (row stride
-    allowed) whose sigmoid multiplies the output; not on the tensor-core kernel."""
+    allowed) whose sigmoid multiplies the output, with ``gate_heads`` one per head.  ``keep_first`` positions stay visible
+    behind a window; ``chunk`` limits a row to the keys of its own chunk of positions; ``slopes`` (fp32 [hq]) are taken off
+    the scores per position of distance.  None of these five is on the tensor-core kernel, and the CPU form has ``gate``
+    only (ops.kv_attention states the others)."""
     scale = sm_scale if sm_scale is not None else 1.0 / math.sqrt(hd)
     r = q.shape[0]
     if _lib.on_cpu(q):
@@ -545,6 +592,8 @@ def paged_attention(q: torch.Tensor, kv: KVLayer, block_table: torch.Tensor, seq
                 vv = kv.v[blks].transpose(1, 2).reshape(-1, hkv, hd).to(torch.float32)
             out[i] = ref.attention_rows(q[i].view(hq, hd), kk, vv, n, window, scale, sinks)
         out = out.view(r, hq * hd)
+        if keep_first or chunk or slopes is not None or gate_heads:
+            raise ValueError("ops.kv_attention states these masks for CPU tensors")
         if gate is not None:
             out = out * torch.sigmoid(gate.float())
         if q.dtype == torch.float32 and not quant_out:
@@ -553,7 +602,8 @@ def paged_attention(q: torch.Tensor, kv: KVLayer, block_table: torch.Tensor, seq
         return QTensor(*ref.quant_fp8_1x128(out)) if quant_out else out.to(q.dtype)
     lib = _lib.kernels()
     wsp = workspace(q.device)
-    splits = _attn_splits(r, hkv, max_kv if max_kv > 0 else block_table.shape[1] * kv.page_size)
+    mk = max_kv if max_kv > 0 else block_table.shape[1] * kv.page_size
+    splits = _attn_splits(r, hkv, min(mk, window + keep_first) if window else min(mk, chunk) if chunk else mk)
     if quant_out:
         if hd != 128:
             raise ValueError("quantised attention output needs head_dim 128")
@@ -563,7 +613,8 @@ def paged_attention(q: torch.Tensor, kv: KVLayer, block_table: torch.Tensor, seq
         ob = out if out is not None else torch.empty((r, hq * hd), dtype=torch.bfloat16, device=q.device)
         out_b, out_q, out_s, ld = ob, None, None, 0
     use_tc = (kv.fp8 and hd == 128 and (hq // hkv) in (1, 2, 4, 8, 16) and 128 % kv.page_size == 0
-              and kv.page_size >= 8 and impl != "cuda_core" and gate is None)
+              and kv.page_size >= 8 and impl != "cuda_core" and gate is None
+              and not (keep_first or chunk or slopes is not None))
     if impl == "tensor_core" and not use_tc:
         raise ValueError("tensor-core decode attention needs FP8 pages, head_dim 128 and a GQA group <= 16")
     if use_tc:
@@ -590,6 +641,7 @@ def paged_attention(q: torch.Tensor, kv: KVLayer, block_table: torch.Tensor, seq
         _p(q), q.stride(0), _p(kv.k), _p(kv.v), _p(kv.k_scale), _p(kv.v_scale), kv.k_static, kv.v_static,
         _p(block_table), block_table.stride(0), _p(seq_index), _p(kv_lens), r, hq, hkv, hd, kv.page_size, window,
         scale, kv.mode, _p(out_b), _p(out_q), _p(out_s), ld, _p(sinks), splits, _p(wsp.ws), wsp.ws.numel(),
-        _p(wsp.counters), wsp.counters.numel(), _p(gate), gate.stride(0) if gate is not None else 0, _stream())
+        _p(wsp.counters), wsp.counters.numel(), _p(gate), gate.stride(0) if gate is not None else 0,
+        int(gate_heads), keep_first, chunk, _p(slopes), _stream())
     _lib.check(rc, "paged_attention")
     return oq if quant_out else ob

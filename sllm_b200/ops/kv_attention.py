@@ -1,6 +1,6 @@
-"""Attention with keys and values of different widths: short convolutions on q, k and v, rotation in neighbouring pairs with
-scaled frequencies, unweighted query / key norms, a sink in the softmax and an output gate per channel, each optional
-(kernels in csrc/kv_attention.cu; PyTorch restatements here for CPU tensors).
+"""Attention with keys and values of different widths: biases or short convolutions on q, k and v, rotation in neighbouring or
+half-split pairs with scaled frequencies, query / key norms, a sink in the softmax, a window with kept first positions or
+chunks of positions, slopes over the distance, and an output gate per channel or head, each optional (kernels in csrc/kv_attention.cu; PyTorch restatements here for CPU tensors).
 
 A layer runs  prepare  (everything between the projection and the scores, page write) -> attention.  Decoded tokens and short
 portions read the pages row by row; long portions gather them once and run on the tensor cores (csrc/latent_prefill.cu).  A
@@ -22,18 +22,18 @@ P, I, F, L = C.c_void_p, C.c_int, C.c_float, C.c_longlong
 
 
 class KvPrepareArgs(C.Structure):
-    _fields_ = [(n, P) for n in ("proj", "conv_w", "ring", "inv_freq", "row_off", "slots", "positions", "seq_index", "block_table", "q",
+    _fields_ = [(n, P) for n in ("proj", "conv_w", "bias", "q_norm", "k_norm", "ring", "inv_freq", "row_off", "slots", "positions", "seq_index", "block_table", "q",
                                  "k_pages", "v_pages")] + [("ring_stride", L)] + \
         [(n, I) for n in ("ldp", "max_blocks", "heads", "kv_heads", "dim", "vdim", "q_pad", "ld_k", "ld_v", "rot_dims", "taps",
-                          "page_size", "tokens", "sequences", "norm", "decode", "fp32")] + [("eps", F)]
+                          "page_size", "tokens", "sequences", "norm", "decode", "fp32", "interleaved")] + [("eps", F)]
 
 
 _SIGS = {
     "sllm_kv_prepare": (I, [P, P]),
     "sllm_kv_abi": (I, [P, I]),
     "sllm_kv_gather": (I, [P, P, I, P, I, P, I, I, P, I, I, I, P]),
-    "sllm_kv_attention": (I, [P, P, P, P, L, P, P, I, P, P, I, I, I, I, I, I, I, I, I, I, F, P, I, P]),
-    "sllm_kv_prefill": (I, [P, I, P, I, P, I, I, I, I, I, I, F, P, P, L, P, P, P]),
+    "sllm_kv_attention": (I, [P, P, P, P, L, P, P, I, P, P, I, I, I, I, I, I, I, I, I, I, I, I, P, I, F, P, I, P]),
+    "sllm_kv_prefill": (I, [P, I, P, I, P, I, I, I, I, I, I, I, I, P, F, P, P, L, I, P, P, P]),
 }
 
 
@@ -58,7 +58,8 @@ def rope_frequencies(base: float, dims: int, scaling: Optional[dict] = None) -> 
 
 @dataclass
 class KVSpec:
-    """Sizes and constants of one layer; its packed input projection is q | k | v | g (q | g without keys of its own)."""
+    """Sizes and constants of one layer; its packed input projection is q | k | v | g (q | g without keys of its own).  A row sees
+    all earlier positions, the last ``window`` and the first ``keep_first`` ones, or those of its own ``chunk``."""
     heads: int
     kv_heads: int
     dim: int
@@ -71,6 +72,10 @@ class KVSpec:
     qk_norm: bool = True
     window: int = 0
     own_kv: bool = True
+    keep_first: int = 0
+    chunk: int = 0
+    interleaved: bool = True         # rotary pairs (2i, 2i + 1); else (i, i + rot_dims / 2)
+    gate_heads: bool = False         # the output gate has one logit per head; else one per channel
 
     @property
     def q_cols(self) -> int:
@@ -89,8 +94,19 @@ class KVSpec:
     def q_pad(self) -> int:
         return (self.dim + 63) // 64 * 64
 
+    def sees(self, i: int, j: torch.Tensor) -> torch.Tensor:
+        """Which of the positions ``j`` <= i position i sees."""
+        if self.chunk:
+            return j // self.chunk == i // self.chunk
+        return (i - j < self.window) | (j < self.keep_first) if self.window else torch.ones_like(j, dtype=torch.bool)
+
     def inv_freq(self, device) -> torch.Tensor:
         return rope_frequencies(self.rot_base, self.rot_dims, self.rot_scaling).float().to(device)
+
+
+def distance_slopes(heads: int, device) -> torch.Tensor:
+    """fp32 [heads]: 2^(-8 (h + 1) / heads), the geometric slopes of linear distance biases."""
+    return torch.exp2(-8.0 * torch.arange(1, heads + 1, dtype=torch.float64) / heads).float().to(device)
 
 
 @dataclass
@@ -107,21 +123,29 @@ class KVPages:
     mode = 0
 
 
-def prepare(proj: torch.Tensor, spec: KVSpec, conv_w: torch.Tensor, inv_freq: torch.Tensor, eps: float, kv: Optional[KVPages],
-            ring: torch.Tensor, b) -> torch.Tensor:
-    """proj [T, >= channels]; conv_w [taps, channels]; ring [slots, taps, channels]; ``kv`` the layer's own pages (None: the
-    layer has no keys of its own).  Returns q [T, heads, q_pad], zero past ``dim``."""
+def prepare(proj: torch.Tensor, spec: KVSpec, conv_w: Optional[torch.Tensor], inv_freq: Optional[torch.Tensor], eps: float,
+            kv: Optional[KVPages], ring: Optional[torch.Tensor], b, bias: Optional[torch.Tensor] = None,
+            q_norm: Optional[torch.Tensor] = None, k_norm: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """proj [T, >= channels]; conv_w [taps, channels] and ring [slots, taps, channels], or neither; bias fp32 [channels]; q_norm,
+    k_norm fp32 [dim] weights of the norms; ``kv`` the layer's own pages (None: the layer has no keys of its own).  Returns q
+    [T, heads, q_pad], zero past ``dim``."""
     t, H, G, D, V = proj.shape[0], spec.heads, spec.kv_heads, spec.dim, spec.vdim
     if _lib.on_cpu(proj):
-        x = causal_conv(proj[:, :spec.channels].float(), conv_w, ring, b.row_off, b.slots, b.positions)
+        x = proj[:, :spec.channels].float()
+        if bias is not None:
+            x = x + bias
+        if conv_w is not None:
+            x = causal_conv(x, conv_w, ring, b.row_off, b.slots, b.positions)
 
-        def turned(y):
-            y = rotate(y, b.positions, inv_freq, spec.rot_dims, True)
-            return y / torch.sqrt((y * y).mean(-1, keepdim=True) + eps) if spec.qk_norm else y
+        def turned(y, w):
+            if spec.qk_norm:
+                y = y / torch.sqrt((y * y).mean(-1, keepdim=True) + eps)
+                y = y if w is None else y * w
+            return rotate(y, b.positions, inv_freq, spec.rot_dims, spec.interleaved) if spec.rot_dims else y
         q = torch.zeros((t, H, spec.q_pad), dtype=proj.dtype)
-        q[..., :D] = turned(x[:, :spec.q_cols].reshape(t, H, D)).to(proj.dtype)
+        q[..., :D] = turned(x[:, :spec.q_cols].reshape(t, H, D), q_norm).to(proj.dtype)
         if kv is not None:
-            k = turned(x[:, spec.q_cols:spec.q_cols + G * D].reshape(t, G, D))
+            k = turned(x[:, spec.q_cols:spec.q_cols + G * D].reshape(t, G, D), k_norm)
             v = x[:, spec.q_cols + G * D:].reshape(t, G, V)
             pos = b.positions.long()
             blk = b.block_table[b.seq_index.long(), pos // kv.page_size].long()
@@ -133,17 +157,18 @@ def prepare(proj: torch.Tensor, spec: KVSpec, conv_w: torch.Tensor, inv_freq: to
     p = lambda x: None if x is None else x.data_ptr()
     decode = b.row_off_host is None and t == b.slots.numel()
     own = kv is not None
-    args = KvPrepareArgs(p(proj), p(conv_w), p(ring), p(inv_freq), p(b.row_off), p(b.slots), p(b.positions), p(b.seq_index),
-                         p(b.block_table), p(q), p(kv.k) if own else None, p(kv.v) if own else None, ring.stride(0), proj.stride(0),
+    args = KvPrepareArgs(p(proj), p(conv_w), p(bias), p(q_norm), p(k_norm), p(ring), p(inv_freq), p(b.row_off), p(b.slots), p(b.positions), p(b.seq_index),
+                         p(b.block_table), p(q), p(kv.k) if own else None, p(kv.v) if own else None, 0 if ring is None else ring.stride(0), proj.stride(0),
                          b.block_table.stride(0), H, G if own else 0, D, V, spec.q_pad, kv.k.shape[3] if own else 0,
                          kv.v.shape[3] if own else 0, spec.rot_dims, spec.taps, kv.page_size if own else 1, t, b.slots.numel(),
-                         int(spec.qk_norm), int(decode), int(proj.dtype == torch.float32), eps)
+                         int(spec.qk_norm), int(decode), int(proj.dtype == torch.float32), int(spec.interleaved), eps)
     _lib.check(_k().sllm_kv_prepare(C.byref(args), _stream()), "kv_prepare")
     return q
 
 
 def paged_rows(q: torch.Tensor, gate: Optional[torch.Tensor], spec: KVSpec, kv: KVPages, sinks: Optional[torch.Tensor], block_table,
-               seq_index, kv_lens, max_kv: int = 0, out: Optional[torch.Tensor] = None, impl: Optional[str] = None) -> torch.Tensor:
+               seq_index, kv_lens, max_kv: int = 0, out: Optional[torch.Tensor] = None, impl: Optional[str] = None,
+               slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Rows q [R, heads, q_pad] over their sequences' pages -> [R, heads * vdim].  ``impl`` "cuda_core_any" forces the any-size
     kernel."""
     from . import core
@@ -153,17 +178,20 @@ def paged_rows(q: torch.Tensor, gate: Optional[torch.Tensor], spec: KVSpec, kv: 
         for i in range(r):
             n = int(kv_lens[i])
             blks = block_table[int(seq_index[i]), :(n + kv.page_size - 1) // kv.page_size].long()
-            lo = max(0, n - spec.window) if spec.window else 0
-            k = kv.k[blks].transpose(1, 2).reshape(-1, G, kv.k.shape[3])[lo:n, :, :D].float().repeat_interleave(H // G, dim=1)
-            v = kv.v[blks].transpose(1, 2).reshape(-1, G, kv.v.shape[3])[lo:n, :, :V].float().repeat_interleave(H // G, dim=1)
+            j = torch.arange(n)
+            j = j[spec.sees(n - 1, j)]
+            k = kv.k[blks].transpose(1, 2).reshape(-1, G, kv.k.shape[3])[j, :, :D].float().repeat_interleave(H // G, dim=1)
+            v = kv.v[blks].transpose(1, 2).reshape(-1, G, kv.v.shape[3])[j, :, :V].float().repeat_interleave(H // G, dim=1)
             s = torch.einsum("hd,jhd->hj", q[i, :, :D].float(), k) * spec.scale
+            if slopes is not None:
+                s = s - slopes[:, None] * (n - 1 - j).float()
             if sinks is not None:
                 s = torch.cat([s, sinks[:, None]], dim=1)
-            p = torch.softmax(s, dim=-1)[:, :n - lo]
+            p = torch.softmax(s, dim=-1)[:, :j.numel()]
             res[i] = torch.einsum("hj,jhv->hv", p, v)
-        res = res.view(r, H * V)
         if gate is not None:
-            res = res * torch.sigmoid(gate.float())
+            res = res * torch.sigmoid(gate.float()).reshape(r, H, -1)
+        res = res.reshape(r, H * V)
         res = res.to(q.dtype)
         if out is not None:
             out.copy_(res)
@@ -171,11 +199,13 @@ def paged_rows(q: torch.Tensor, gate: Optional[torch.Tensor], spec: KVSpec, kv: 
     g = H // G
     if q.dtype == torch.bfloat16 and D == V and D in (64, 128, 256) and g in (1, 2, 4, 8) and impl != "cuda_core_any":
         return core.paged_attention(q.view(r, H * D), kv, block_table, seq_index, kv_lens, H, G, D, window=spec.window,
-                                    sm_scale=spec.scale, max_kv=max_kv, sinks=sinks, gate=gate, out=out)
+                                    sm_scale=spec.scale, max_kv=max_kv, sinks=sinks, gate=gate, out=out, gate_heads=spec.gate_heads,
+                                    keep_first=spec.keep_first, chunk=spec.chunk, slopes=slopes)
     out = torch.empty((r, H * V), dtype=q.dtype, device=q.device) if out is None else out
     rc = _k().sllm_kv_attention(core._p(q), core._p(kv.k), core._p(kv.v), core._p(gate), gate.stride(0) if gate is not None else 0,
                                 core._p(sinks), core._p(block_table), block_table.stride(0), core._p(seq_index), core._p(kv_lens), r, H,
-                                G, D, V, spec.q_pad, kv.k.shape[3], kv.v.shape[3], kv.page_size, spec.window, spec.scale, core._p(out),
+                                G, D, V, spec.q_pad, kv.k.shape[3], kv.v.shape[3], kv.page_size, spec.window, spec.keep_first, spec.chunk,
+                                core._p(slopes), int(spec.gate_heads), spec.scale, core._p(out),
                                 int(q.dtype == torch.float32), core._stream())
     _lib.check(rc, "kv_attention")
     return out
@@ -184,10 +214,10 @@ def paged_rows(q: torch.Tensor, gate: Optional[torch.Tensor], spec: KVSpec, kv: 
 def gatherable(spec: KVSpec, dtype, gate: Optional[torch.Tensor]) -> bool:
     """Whether long portions of this layer run on the tensor cores."""
     return (dtype == torch.bfloat16 and spec.dim % 8 == 0 and spec.vdim % 8 == 0 and spec.dim <= 192 and spec.vdim <= 128
-            and (gate is None or (gate.stride(0) % 8 == 0 and gate.data_ptr() % 16 == 0)))
+            and (gate is None or spec.gate_heads or (gate.stride(0) % 8 == 0 and gate.data_ptr() % 16 == 0)))
 
 
-def attend_gathered(q, gate, spec: KVSpec, kv: KVPages, sinks, b, pt, out) -> None:
+def attend_gathered(q, gate, spec: KVSpec, kv: KVPages, sinks, b, pt, out, slopes=None) -> None:
     """Rows [pt.lo, pt.hi) of a batch (q, gate and out are those rows)."""
     from .core import _p, _stream, workspace
     key = ("gathered", pt.lo)
@@ -202,25 +232,26 @@ def attend_gathered(q, gate, spec: KVSpec, kv: KVPages, sinks, b, pt, out) -> No
         _lib.record_dispatch("kv_attention", "latent_prefill_kernel", rows=q.shape[0], heads=spec.heads, context=pt.context,
                              window=spec.window, grid=[pt.tiles.shape[0], spec.heads])
     rc = _k().sllm_kv_prefill(_p(q), q.shape[0], _p(held[1]), pt.context, _p(pt.tiles), pt.tiles.shape[0], spec.heads, spec.kv_heads,
-                              spec.dim, spec.vdim, spec.window, spec.scale, _p(sinks), _p(gate), gate.stride(0) if gate is not None else 0,
-                              _p(out), _p(workspace(q.device).status), _stream())
+                              spec.dim, spec.vdim, spec.window, spec.keep_first, spec.chunk, _p(slopes), spec.scale, _p(sinks), _p(gate),
+                              gate.stride(0) if gate is not None else 0, int(spec.gate_heads), _p(out), _p(workspace(q.device).status), _stream())
     _lib.check(rc, "kv_prefill")
 
 
-def attention(q: torch.Tensor, gate: Optional[torch.Tensor], spec: KVSpec, kv: KVPages, sinks: Optional[torch.Tensor], b) -> torch.Tensor:
+def attention(q: torch.Tensor, gate: Optional[torch.Tensor], spec: KVSpec, kv: KVPages, sinks: Optional[torch.Tensor], b,
+              slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of a ForwardBatch's rows over ``kv`` (already appended to) -> [T, heads * vdim], gated."""
     t = q.shape[0]
 
     def rows(lo, hi, out=None):
         return paged_rows(q[lo:hi], None if gate is None else gate[lo:hi], spec, kv, sinks, b.block_table, b.seq_index[lo:hi],
-                          b.kv_lens[lo:hi], b.max_kv, out)
+                          b.kv_lens[lo:hi], b.max_kv, out, slopes=slopes)
 
     if b.row_off_host is None or not q.is_cuda or _lib.fake_active() or not gatherable(spec, q.dtype, gate):
         return rows(0, t)
-    key = ("portions", spec.window)
+    key = ("portions", spec.window, spec.keep_first, spec.chunk)
     portions = b.plans.get(key)
     if portions is None:
-        portions = b.plans[key] = plan_portions(b.row_off_host, b.starts_host, spec.window, q.device)
+        portions = b.plans[key] = plan_portions(b.row_off_host, b.starts_host, spec.window, q.device, spec.keep_first, spec.chunk)
     if len(portions) == 1 and portions[0].spans is None:
         return rows(0, t)
     out = torch.empty((t, spec.out_cols), dtype=q.dtype, device=q.device)
@@ -228,5 +259,6 @@ def attention(q: torch.Tensor, gate: Optional[torch.Tensor], spec: KVSpec, kv: K
         if pt.spans is None:
             rows(pt.lo, pt.hi, out[pt.lo:pt.hi])
         else:
-            attend_gathered(q[pt.lo:pt.hi], None if gate is None else gate[pt.lo:pt.hi], spec, kv, sinks, b, pt, out[pt.lo:pt.hi])
+            attend_gathered(q[pt.lo:pt.hi], None if gate is None else gate[pt.lo:pt.hi], spec, kv, sinks, b, pt, out[pt.lo:pt.hi],
+                            slopes)
     return out

@@ -228,8 +228,10 @@ class Portion:
     longest: int = 0
 
 
-def plan_portions(row_off: list, starts: list, window: int, device) -> list:
-    """Splits a flat batch into runs of sequences with few rows (absorbed form) and with many (expanded form)."""
+def plan_portions(row_off: list, starts: list, window: int, device, keep_first: int = 0, chunk: int = 0) -> list:
+    """Splits a flat batch into runs of sequences with few rows (absorbed form) and with many (expanded form).  The context of
+    a portion starts where its first row's window, or chunk of positions, does; ``keep_first`` positions that a window does not
+    reach are gathered ahead of it."""
     out: list = []
     run: list = []
 
@@ -240,11 +242,17 @@ def plan_portions(row_off: list, starts: list, window: int, device) -> list:
         lo, spans, tiles, rows = row_off[run[0]], [], [], 0
         for s in run:
             n, st = row_off[s + 1] - row_off[s], starts[s]
-            k_lo = max(0, st - window + 1) if window else 0
+            k_lo = max(0, st - window + 1) if window else st // chunk * chunk if chunk else 0
+            if k_lo <= keep_first and not chunk:
+                k_lo = 0
+            start = rows
+            if keep_first and k_lo:
+                spans.append((s, 0, keep_first, rows))
+                rows += keep_first
             ctx = st + n - k_lo
             spans.append((s, k_lo, ctx, rows))
             for q0 in range(0, n, TILE):
-                tiles.append((row_off[s] - lo + q0, min(TILE, n - q0), st + q0, rows, k_lo, 0, 0, 0))
+                tiles.append((row_off[s] - lo + q0, min(TILE, n - q0), st + q0, rows, k_lo, start, 0, 0))
             rows += ctx
         tiles.sort(key=lambda t: -(t[2] - t[4]))         # most keys first
         out.append(Portion(lo, row_off[run[-1] + 1], torch.tensor(spans, dtype=torch.int32, device=device),

@@ -16,8 +16,9 @@ from .w4 import W4Weight, linear_w4
 
 P, I, L, F = C.c_void_p, C.c_int, C.c_longlong, C.c_float
 _SIGS = {
-    "sllm_moe_route": (I, [P, I, I, I, I, I, I, I, I, P, P, P]),
-    "sllm_moe_router": (I, [P, I, P, I, I, I, I, I, I, I, I, P, P, P]),
+    "sllm_moe_route": (I, [P, I, I, P, I, P, P, P]),
+    "sllm_moe_router": (I, [P, I, P, I, I, P, I, P, P, P]),
+    "sllm_moe_route_abi": (I, [P, I]),
     "sllm_moe_grouped": (I, [P, P, P, I, I, I, I, P, F, F, F, P, I, I, I, I, I, P, P]),
     "sllm_moe_grouped_simt": (I, [P, I, P, P, P, I, I, I, I, P, F, F, F, P, I, I, I, I, P]),
     "sllm_moe_permute": (I, [P, P, I, I, I, I, P, P, P, P, P, P]),
@@ -36,22 +37,46 @@ def _k():
     return _lib.kernels()
 
 
-def route(logits: torch.Tensor, top_k: int, softmax_all: bool = False, groups: int = 1, keep: int = 1):
+class RouteArgs(C.Structure):
+    _fields_ = [("correction", P)] + [(n, I) for n in ("experts", "top_k", "mode", "groups", "keep", "group_top")] + [("scale", F)]
+
+
+@dataclass
+class SigmoidScores:
+    """Experts are chosen by sigmoid(logit) + correction; their weights are scale * sigmoid(logit), not renormalised."""
+    correction: Optional[torch.Tensor] = None      # fp32 [E]
+    scale: float = 1.0
+
+
+def _route_args(e: int, top_k: int, softmax_all: bool, groups: int, keep: int, group_top: int, sigmoid: Optional[SigmoidScores]):
+    c = None if sigmoid is None or sigmoid.correction is None else sigmoid.correction.data_ptr()
+    return C.byref(RouteArgs(c, e, top_k, 2 if sigmoid is not None else int(softmax_all), groups, keep, group_top,
+                             1.0 if sigmoid is None else sigmoid.scale))
+
+
+def route(logits: torch.Tensor, top_k: int, softmax_all: bool = False, groups: int = 1, keep: int = 1, group_top: int = 1,
+          sigmoid: Optional[SigmoidScores] = None):
     """[T, E] (bf16 or fp32) -> (idx int32 [T, k], weights fp32 [T, k]).  ``groups`` > 1: neighbouring experts form equal
-    groups, a group's score is the largest in it, and only experts of the ``keep`` best groups are selected."""
+    groups, a group's score is the sum of its ``group_top`` (1 or 2) largest, and only experts of the ``keep`` best groups are
+    selected.  ``sigmoid`` replaces the softmax."""
     t, e = logits.shape
     if _lib.on_cpu(logits):
         lf = torch.nan_to_num(logits.float(), nan=float("-inf"))
+        if sigmoid is not None:
+            score = torch.sigmoid(lf)
+            lf = score if sigmoid.correction is None else score + sigmoid.correction
         pick = lf
         if groups > 1 and keep < groups:
-            top = lf.view(t, groups, e // groups).max(-1).values
+            top = lf.view(t, groups, e // groups).topk(min(group_top, e // groups), -1).values.sum(-1)
             best = torch.sort(-top, dim=1, stable=True).indices[:, :keep]
             shut = torch.ones((t, groups), dtype=torch.bool).scatter(1, best, False)
             pick = lf.masked_fill(shut.repeat_interleave(e // groups, dim=1), float("-inf"))
         # stable ordering: larger logit first, ties to the lower index
         order = torch.sort(-pick, dim=1, stable=True).indices[:, :top_k]
         sel = torch.gather(lf, 1, order)
-        if softmax_all:
+        if sigmoid is not None:
+            w = score.gather(1, order) * sigmoid.scale
+        elif softmax_all:
             w = torch.softmax(lf, dim=1).gather(1, order)
         else:
             w = torch.softmax(sel, dim=1)
@@ -59,7 +84,7 @@ def route(logits: torch.Tensor, top_k: int, softmax_all: bool = False, groups: i
     from .core import _p, _stream
     idx = torch.empty((t, top_k), dtype=torch.int32, device=logits.device)
     w = torch.empty((t, top_k), dtype=torch.float32, device=logits.device)
-    rc = _k().sllm_moe_route(_p(logits), logits.stride(0), t, e, top_k, int(softmax_all), groups, keep,
+    rc = _k().sllm_moe_route(_p(logits), logits.stride(0), t, _route_args(e, top_k, softmax_all, groups, keep, group_top, sigmoid),
                              int(logits.dtype == torch.float32), _p(idx), _p(w), _stream())
     _lib.check(rc, "moe_route")
     return idx, w
@@ -68,16 +93,18 @@ def route(logits: torch.Tensor, top_k: int, softmax_all: bool = False, groups: i
 ROUTER_FUSED_ROWS = 64         # up to this many tokens the product and the selection are one launch
 
 
-def router(x: torch.Tensor, w, top_k: int, softmax_all: bool = False, groups: int = 1, keep: int = 1):
+def router(x: torch.Tensor, w, top_k: int, softmax_all: bool = False, groups: int = 1, keep: int = 1, group_top: int = 1,
+           sigmoid: Optional[SigmoidScores] = None):
     """Routing from fp32 router logits: x [T, d], w LinearWeight [E, d] of the type of x.  Returns (idx, weights) as `route`."""
     from . import core
     t, e = x.shape[0], w.out_features
     if _lib.on_cpu(x) or (t > ROUTER_FUSED_ROWS and x.dtype == torch.bfloat16 and w.in_features % 8 == 0):
-        return route(core.linear(x, w, out_fp32=True), top_k, softmax_all, groups, keep)
+        return route(core.linear(x, w, out_fp32=True), top_k, softmax_all, groups, keep, group_top, sigmoid)
     idx = torch.empty((t, top_k), dtype=torch.int32, device=x.device)
     wt = torch.empty((t, top_k), dtype=torch.float32, device=x.device)
-    rc = _k().sllm_moe_router(core._p(x), x.stride(0), core._p(w.w), t, w.in_features, e, top_k, int(softmax_all), groups, keep,
-                              int(x.dtype == torch.float32), core._p(idx), core._p(wt), core._stream())
+    rc = _k().sllm_moe_router(core._p(x), x.stride(0), core._p(w.w), t, w.in_features,
+                              _route_args(e, top_k, softmax_all, groups, keep, group_top, sigmoid), int(x.dtype == torch.float32),
+                              core._p(idx), core._p(wt), core._stream())
     _lib.check(rc, "moe_router")
     return idx, wt
 

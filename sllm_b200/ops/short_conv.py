@@ -1,5 +1,5 @@
 """Short causal convolution with its inputs in a ring per state slot (PyTorch form; the CUDA kernels that consume the
-convolution's result compute it themselves: csrc/kv_attention.cu, csrc/rglru.cu).
+convolution's result compute it themselves: csrc/kv_attention.cu, csrc/rglru.cu, csrc/linear_state.cu).
 
 ring [slots, taps, channels], fp32: row (position mod taps) holds the conv input of that position, for the last ``taps``
 positions of the slot's sequence.  A decoded token reads the rows of the taps - 1 positions before it and writes its own."""
