@@ -5,35 +5,19 @@
 //   y = o / rms(o) * norm_w * sigmoid(g).
 // The batch is flat (rows of sequence s: row_off[s] .. row_off[s + 1]) and sequence s owns state slot slots[s].
 //
-// Columns of S (value channels) never meet: column j only needs p = u^T S_j, so heads are cut into column tiles.  A
-// thread keeps 16 keys x 2 or 4 columns of S in registers; kKL = 1 .. 32 lanes share a column.  Both dot products of a token
-// are taken from the OLD state in one sweep, because
-//   o = S_t^T r = (w r)^T S_{t-1} - p (a u)^T r + v k^T r
-// so a token costs one shuffle reduction and no barrier.
-//
-// Prompts: delta_pre_kernel computes everything that does not depend on the state in parallel over the tokens,
-// delta_scan_kernel runs the recurrence, delta_post_kernel normalises and gates.  One-token batches (decode) take
+// Prompts: delta_pre_kernel computes everything that does not depend on the state in parallel over the tokens, the scan of
+// state_scan.cu runs the recurrence, delta_post_kernel normalises and gates.  One-token batches (decode) take
 // delta_decode_kernel, which does all of it, the low-rank decay projection included, in one launch.
 #include <cstddef>
 #include <type_traits>
-#include "typed.cuh"
+#include "state_scan.cuh"
+#include "state_scan.h"
 #include "api.h"
 
 namespace sllm {
 
-constexpr int kDrKeys = 16;          // keys per thread
-constexpr int kDrVecs = 6;           // u, w r, w, a u, k, v
-constexpr int kDrChunk = 8;          // tokens staged at a time by the scan
 constexpr int kDrDecodeThreads = 256;
 constexpr float kDecayRate = 0.60653065971263342f;   // exp(-1/2)
-
-__host__ __device__ constexpr int delta_pad(int dim) {   // padded head size: 16 x a power of two
-  int kl = 1;
-  while (kl * kDrKeys < dim) kl *= 2;
-  return kl * kDrKeys;
-}
-
-__host__ __device__ constexpr int delta_record(int pad) { return kDrVecs * pad + 4; }   // floats per (head, token)
 
 template <typename T>
 struct DeltaParams {
@@ -52,42 +36,14 @@ struct DeltaParams {
   const int* row_off;
   const int* slots;
   int heads, dim, tokens;
-  float* vec;              // [heads][tokens][6 pad + 4]: the vectors, then (a u)^T r, k^T r
+  float* vec;              // [heads][tokens] records of the scan
   float* o_raw;            // [tokens, heads * dim]
   T* out;                  // [tokens, heads * dim]
 };
 
-__device__ __forceinline__ float block_sum(float v, float* red, int warps) {
-  v = warp_sum(v);
-  __syncthreads();                                   // red may still be read from the previous sum
-  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
-  __syncthreads();
-  float s = 0.f;
-  for (int i = 0; i < warps; ++i) s += red[i];
-  return s;
-}
-
 // ---------------------------------------------------------------- prompt form
 // A warp per (token, head), lane l the channels l kN .. l kN + kN - 1 (kN = padded head size / 32, at least 1); vec: heads
 // and offsets allow 4-channel accesses.
-template <typename T, int kN>
-__device__ __forceinline__ void lane_load(const T* src, int d0, int dim, bool vec, float (&v)[kN]) {
-  if constexpr (kN % 4 == 0) {
-    if (vec) {
-#pragma unroll
-      for (int i = 0; i < kN; i += 4) {
-        float x[4] = {0.f, 0.f, 0.f, 0.f};
-        if (d0 + i < dim) ld_vec<4>(src + d0 + i, x);
-#pragma unroll
-        for (int j = 0; j < 4; ++j) v[i + j] = x[j];
-      }
-      return;
-    }
-  }
-#pragma unroll
-  for (int i = 0; i < kN; ++i) v[i] = d0 + i < dim ? ld_f(src + d0 + i) : 0.f;
-}
-
 constexpr int kDrRowWarps = 8;       // (token, head) pairs per CTA of the row kernels
 
 // No early trigger of the dependent launch here: the scan's few CTAs would become resident while this grid drains, several
@@ -95,7 +51,7 @@ constexpr int kDrRowWarps = 8;       // (token, head) pairs per CTA of the row k
 template <typename T, int kN>
 __global__ void __launch_bounds__(kDrRowWarps * 32) delta_pre_kernel(const DeltaParams<T> p, bool vec) {
   pdl_wait();
-  const int lane = threadIdx.x & 31, D = p.dim, pad = delta_pad(D), d0 = lane * kN;
+  const int lane = threadIdx.x & 31, D = p.dim, pad = state_pad(D), d0 = lane * kN;
   const long long unit = static_cast<long long>(blockIdx.x) * kDrRowWarps + (threadIdx.x >> 5);
   if (unit >= static_cast<long long>(p.tokens) * p.heads) return;
   const int t = static_cast<int>(unit / p.heads), h = static_cast<int>(unit % p.heads);
@@ -125,158 +81,15 @@ __global__ void __launch_bounds__(kDrRowWarps * 32) delta_pre_kernel(const Delta
   }
   s1 = warp_sum(s1);
   s2 = warp_sum(s2);
-  float* dst = p.vec + (static_cast<size_t>(h) * p.tokens + t) * delta_record(pad) + d0;
-  auto put = [&](int which, const float (&x)[kN]) {
-    if constexpr (kN % 4 == 0) {
-#pragma unroll
-      for (int i = 0; i < kN; i += 4)
-        *reinterpret_cast<float4*>(dst + which * pad + i) = make_float4(x[i], x[i + 1], x[i + 2], x[i + 3]);
-    } else {
-#pragma unroll
-      for (int i = 0; i < kN; ++i)
-        if (d0 + i < pad) dst[which * pad + i] = x[i];
-    }
-  };
-  put(0, u); put(1, r); put(2, w); put(3, a); put(4, k); put(5, v);
-  if (lane == 0) *reinterpret_cast<float2*>(dst + kDrVecs * pad) = make_float2(s1, s2);
-}
-
-// One token on a thread's 16 keys x kC columns: S is updated, o holds the outputs on every lane of the columns.
-// vs: the token's [6][pad] vectors in shared memory.  Key of S[j * 4 + e]: (j * kKL + kl) * 4 + e.
-template <int kKL, int kC>
-__device__ __forceinline__ void delta_token(float (&S)[kDrKeys][kC], const float* vs, int kl, const float (&v)[kC], float s1, float s2,
-                                            float (&o)[kC]) {
-  constexpr int pad = kKL * kDrKeys;
-  float pc[2][kC], qc[2][kC];                        // two chains per column
-#pragma unroll
-  for (int c = 0; c < kC; ++c) pc[0][c] = pc[1][c] = qc[0][c] = qc[1][c] = 0.f;
-#pragma unroll
-  for (int j = 0; j < kDrKeys / 4; ++j) {
-    const float4 u = *reinterpret_cast<const float4*>(vs + (j * kKL + kl) * 4);
-    const float4 wr = *reinterpret_cast<const float4*>(vs + pad + (j * kKL + kl) * 4);
-    const float ua[4] = {u.x, u.y, u.z, u.w}, wa[4] = {wr.x, wr.y, wr.z, wr.w};
-#pragma unroll
-    for (int e = 0; e < 4; ++e)
-#pragma unroll
-      for (int c = 0; c < kC; ++c) {
-        pc[e & 1][c] = fmaf(ua[e], S[j * 4 + e][c], pc[e & 1][c]);
-        qc[e & 1][c] = fmaf(wa[e], S[j * 4 + e][c], qc[e & 1][c]);
-      }
-  }
-  float p[kC], q[kC];
-#pragma unroll
-  for (int c = 0; c < kC; ++c) {
-    p[c] = pc[0][c] + pc[1][c];
-    q[c] = qc[0][c] + qc[1][c];
-  }
-#pragma unroll
-  for (int x = kKL / 2; x > 0; x >>= 1)
-#pragma unroll
-    for (int c = 0; c < kC; ++c) {
-      p[c] += __shfl_xor_sync(0xffffffffu, p[c], x);
-      q[c] += __shfl_xor_sync(0xffffffffu, q[c], x);
-    }
-#pragma unroll
-  for (int j = 0; j < kDrKeys / 4; ++j) {
-    const float4 w = *reinterpret_cast<const float4*>(vs + 2 * pad + (j * kKL + kl) * 4);
-    const float4 au = *reinterpret_cast<const float4*>(vs + 3 * pad + (j * kKL + kl) * 4);
-    const float4 k = *reinterpret_cast<const float4*>(vs + 4 * pad + (j * kKL + kl) * 4);
-    const float wa[4] = {w.x, w.y, w.z, w.w}, aa[4] = {au.x, au.y, au.z, au.w}, ka[4] = {k.x, k.y, k.z, k.w};
-#pragma unroll
-    for (int e = 0; e < 4; ++e)
-#pragma unroll
-      for (int c = 0; c < kC; ++c) S[j * 4 + e][c] = fmaf(ka[e], v[c], fmaf(-aa[e], p[c], wa[e] * S[j * 4 + e][c]));
-  }
-#pragma unroll
-  for (int c = 0; c < kC; ++c) o[c] = q[c] - p[c] * s1 + v[c] * s2;
-}
-
-template <int kKL, int kC, bool kStore>
-__device__ __forceinline__ void delta_state_io(float (&S)[kDrKeys][kC], float* st, int dim, int kl, int col) {
-  const bool whole = dim % kC == 0;                  // col is a multiple of kC: its columns are one aligned access
-#pragma unroll
-  for (int j = 0; j < kDrKeys / 4; ++j)
-#pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int key = (j * kKL + kl) * 4 + e;
-      float* ptr = st + static_cast<size_t>(key) * dim + col;
-      float(&x)[kC] = S[j * 4 + e];
-      const bool in = key < dim && col < dim;
-      if constexpr (kStore) {
-        if (in && whole) {
-          st_vec<kC>(ptr, x);
-        } else if (in) {
-#pragma unroll
-          for (int c = 0; c < kC; ++c)
-            if (col + c < dim) ptr[c] = x[c];
-        }
-      } else {
-#pragma unroll
-        for (int c = 0; c < kC; ++c) x[c] = 0.f;
-        if (in && whole) {
-          ld_vec<kC>(ptr, x);
-        } else if (in) {
-#pragma unroll
-          for (int c = 0; c < kC; ++c)
-            if (col + c < dim) x[c] = ptr[c];
-        }
-      }
-    }
-}
-
-__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-}
-
-constexpr int kDrScanWarps = 4;
-
-// grid (heads, column tiles, sequences), 4 warps of (32 / kKL) groups of kC columns.
-template <typename T, int kKL, int kC>
-__global__ void __launch_bounds__(kDrScanWarps * 32) delta_scan_kernel(const DeltaParams<T> p) {
-  pdl_wait();
-  constexpr int pad = kKL * kDrKeys;
-  constexpr int kTok = delta_record(pad);
-  extern __shared__ __align__(16) float buf[];       // [2][kDrChunk][kTok]
-  const int h = blockIdx.x, s = blockIdx.z, D = p.dim;
-  const int r0 = p.row_off[s], r1 = p.row_off[s + 1];
-  if (r1 <= r0) return;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kl = lane % kKL;
-  const int col = ((blockIdx.y * kDrScanWarps + warp) * (32 / kKL) + lane / kKL) * kC;
-  float* st = p.state + static_cast<long long>(p.slots[s]) * p.slot_stride + static_cast<size_t>(h) * D * D;
-  float S[kDrKeys][kC];
-  delta_state_io<kKL, kC, false>(S, st, D, kl, col);
-  const float* vec = p.vec + static_cast<size_t>(h) * p.tokens * kTok;
-  auto stage = [&](int c0, int b) {
-    const int n = min(kDrChunk, r1 - c0) * (kTok / 4);
-    for (int e = threadIdx.x; e < n; e += kDrScanWarps * 32)
-      cp_async16(buf + b * kDrChunk * kTok + e * 4, vec + static_cast<size_t>(c0) * kTok + e * 4);
-  };
-  stage(r0, 0);
-  asm volatile("cp.async.commit_group;" ::: "memory");
-  int b = 0;
-  for (int c0 = r0; c0 < r1; c0 += kDrChunk, b ^= 1) {
-    if (c0 + kDrChunk < r1) stage(c0 + kDrChunk, b ^ 1);
-    asm volatile("cp.async.commit_group;\n\tcp.async.wait_group 1;" ::: "memory");
-    __syncthreads();
-    const int n = min(kDrChunk, r1 - c0);
-    for (int i = 0; i < n; ++i) {
-      const float* vs = buf + (b * kDrChunk + i) * kTok;
-      const float2 s12 = *reinterpret_cast<const float2*>(vs + kDrVecs * pad);
-      float v[kC], o[kC];
-#pragma unroll
-      for (int c = 0; c < kC; ++c) v[c] = col < pad ? vs[5 * pad + col + c] : 0.f;
-      delta_token<kKL, kC>(S, vs, kl, v, s12.x, s12.y, o);
-      if (kl == 0) {
-        float* dst = p.o_raw + static_cast<size_t>(c0 + i) * p.heads * D + h * D + col;
-#pragma unroll
-        for (int c = 0; c < kC; ++c)
-          if (col + c < D) dst[c] = o[c];
-      }
-    }
-    __syncthreads();                                 // the buffer is refilled by the next iteration's stage()
-  }
-  pdl_trigger();
-  delta_state_io<kKL, kC, true>(S, st, D, kl, col);
+  float* dst = p.vec + (static_cast<size_t>(h) * p.tokens + t) * state_record(true, pad, D);
+  lane_store(dst + kVecWR * pad, d0, pad, r);
+  lane_store(dst + kVecW * pad, d0, pad, w);
+  lane_store(dst + kVecK * pad, d0, pad, k);
+  lane_store(dst + kVecU * pad, d0, pad, u);
+  lane_store(dst + kVecAU * pad, d0, pad, a);
+  dst += state_vecs(true) * pad;
+  lane_store(dst, d0, state_vpad(D), v);
+  if (lane == 0) *reinterpret_cast<float2*>(dst + state_vpad(D)) = make_float2(s1, s2);
 }
 
 // A warp per (token, head), as in the first stage.
@@ -323,7 +136,7 @@ __global__ void __launch_bounds__(kDrDecodeThreads) delta_decode_kernel(const De
   pdl_trigger();
   constexpr int pad = kKL * kDrKeys;
   constexpr int kWarps = kDrDecodeThreads / 32;
-  __shared__ __align__(16) float vs[kDrVecs * pad];
+  __shared__ __align__(16) float vs[(state_vecs(true) + 1) * pad];
   __shared__ float o_s[pad];
   __shared__ float red[kWarps];
   extern __shared__ float low[];                     // [rank] tanh of the low-rank decay input
@@ -335,7 +148,7 @@ __global__ void __launch_bounds__(kDrDecodeThreads) delta_decode_kernel(const De
   // the first tile of the state is requested before anything is computed
   int col = (warp * (32 / kKL) + lane / kKL) * 2;
   float S[kDrKeys][2];
-  delta_state_io<kKL, 2, false>(S, st, D, kl, col);
+  state_io<kKL, 2, false>(S, st, D, D, kl, col);
   for (int i = threadIdx.x; i < p.rank; i += kDrDecodeThreads) low[i] = tanhf(ld_f(row + p.off_w1 + i));
   __syncthreads();
   float kk = 0.f, kr = 0.f;
@@ -361,8 +174,8 @@ __global__ void __launch_bounds__(kDrDecodeThreads) delta_decode_kernel(const De
       }
       w = expf(-kDecayRate * sigmoid_f(x));
     }
-    vs[pad + d] = w * r; vs[2 * pad + d] = w; vs[3 * pad + d] = a; vs[4 * pad + d] = k; vs[5 * pad + d] = v;
-    vs[d] = r;
+    vs[kVecWR * pad + d] = w * r; vs[kVecW * pad + d] = w; vs[kVecAU * pad + d] = a; vs[kVecK * pad + d] = k; vs[5 * pad + d] = v;
+    vs[kVecU * pad + d] = r;
     kk += k * k;
     kr += k * r;
   }
@@ -371,22 +184,22 @@ __global__ void __launch_bounds__(kDrDecodeThreads) delta_decode_kernel(const De
   const float inv_u = 1.f / sqrtf(kk + p.eps_u);
   float s1 = 0.f;
   for (int d = threadIdx.x; d < pad; d += kDrDecodeThreads) {   // each thread rewrites only what it wrote above
-    const float r = vs[d], u = vs[4 * pad + d] * inv_u, au = vs[3 * pad + d] * u;
+    const float r = vs[kVecU * pad + d], u = vs[kVecK * pad + d] * inv_u, au = vs[kVecAU * pad + d] * u;
     s1 += au * r;
-    vs[d] = u;
-    vs[3 * pad + d] = au;
+    vs[kVecU * pad + d] = u;
+    vs[kVecAU * pad + d] = au;
   }
   s1 = block_sum(s1, red, kWarps);                   // its barriers also publish vs
   constexpr int kSweep = kWarps * (32 / kKL) * 2;    // columns per sweep of the CTA
   for (int base = 0; base < D; base += kSweep) {
     if (base > 0) {
       col += kSweep;
-      delta_state_io<kKL, 2, false>(S, st, D, kl, col);
+      state_io<kKL, 2, false>(S, st, D, D, kl, col);
     }
     float v[2] = {0.f, 0.f}, o[2];
     if (col < pad) { v[0] = vs[5 * pad + col]; v[1] = vs[5 * pad + col + 1]; }
-    delta_token<kKL, 2>(S, vs, kl, v, s1, s2, o);
-    delta_state_io<kKL, 2, true>(S, st, D, kl, col);
+    state_token<kKL, 2, true>(S, vs, kl, v, s1, s2, o);
+    state_io<kKL, 2, true>(S, st, D, D, kl, col);
     if (kl == 0 && col < pad) { o_s[col] = o[0]; o_s[col + 1] = o[1]; }
   }
   __syncthreads();
@@ -410,33 +223,6 @@ __global__ void tanh_rows_kernel(const T* __restrict__ x, T* __restrict__ y, int
     st_f(y + static_cast<size_t>(t) * n_pad + i, i < n ? tanhf(ld_f(x + static_cast<size_t>(t) * ldx + i)) : 0.f);
 }
 
-template <typename T, int kKL, int kC>
-static int delta_scan_launch_c(const DeltaParams<T>& p, int sequences, cudaStream_t st) {
-  constexpr int cols = kDrScanWarps * (32 / kKL) * kC;
-  const dim3 grid(p.heads, (p.dim + cols - 1) / cols, sequences);
-  size_t smem = sizeof(float) * 2 * kDrChunk * delta_record(kKL * kDrKeys);
-  // a grid that fits one CTA per SM asks for more than half of an SM's shared memory, so that no two share one
-  if (static_cast<long long>(grid.x) * grid.y * grid.z <= 148 && smem < 116 * 1024) smem = 116 * 1024;
-  static size_t configured = 0;
-  if (smem > 48 * 1024 && smem > configured) {
-    if (cudaFuncSetAttribute(delta_scan_kernel<T, kKL, kC>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) !=
-        cudaSuccess)
-      return SLLM_ERR_CUDA;
-    configured = smem;
-  }
-  return launch_kernel(delta_scan_kernel<T, kKL, kC>, grid, dim3(kDrScanWarps * 32), smem, st, 1u, p) == cudaSuccess ? SLLM_OK
-                                                                                                                     : SLLM_ERR_CUDA;
-}
-
-// The scan is bound by its reads of the staged vectors: more columns per thread reuse them more often, fewer spread a small
-// batch over more SMs.
-template <typename T, int kKL>
-static int delta_scan_launch(const DeltaParams<T>& p, int sequences, cudaStream_t st) {
-  constexpr int cols = kDrScanWarps * (32 / kKL) * 2;
-  if (static_cast<long long>(p.heads) * ((p.dim + cols - 1) / cols) * sequences > 148) return delta_scan_launch_c<T, kKL, 4>(p, sequences, st);
-  return delta_scan_launch_c<T, kKL, 2>(p, sequences, st);
-}
-
 template <typename T, int kN>
 static cudaError_t delta_rows_launch(const DeltaParams<T>& p, bool pre, bool vec, cudaStream_t st) {
   const long long units = static_cast<long long>(p.tokens) * p.heads;
@@ -457,17 +243,10 @@ static cudaError_t delta_rows(const DeltaParams<T>& p, int pad, bool pre, cudaSt
 
 template <typename T>
 static int delta_prompt_launch(DeltaParams<T> p, int sequences, cudaStream_t st) {
-  const int pad = delta_pad(p.dim);
+  const int pad = state_pad(p.dim);
   if (delta_rows<T>(p, pad, true, st) != cudaSuccess) return SLLM_ERR_CUDA;
-  int rc;
-  switch (pad / kDrKeys) {
-    case 1: rc = delta_scan_launch<T, 1>(p, sequences, st); break;
-    case 2: rc = delta_scan_launch<T, 2>(p, sequences, st); break;
-    case 4: rc = delta_scan_launch<T, 4>(p, sequences, st); break;
-    case 8: rc = delta_scan_launch<T, 8>(p, sequences, st); break;
-    case 16: rc = delta_scan_launch<T, 16>(p, sequences, st); break;
-    default: rc = delta_scan_launch<T, 32>(p, sequences, st); break;
-  }
+  const ScanParams sp{p.vec, p.state, p.slot_stride, p.row_off, p.slots, p.o_raw, p.heads, p.dim, p.dim, p.tokens};
+  const int rc = state_scan_launch(sp, true, sequences, st);
   if (rc != SLLM_OK) return rc;
   return delta_rows<T>(p, pad, false, st) == cudaSuccess ? SLLM_OK : SLLM_ERR_CUDA;
 }
@@ -477,7 +256,7 @@ static int delta_decode_launch(const DeltaParams<T>& p, int sequences, cudaStrea
   const dim3 grid(p.heads, sequences), block(kDrDecodeThreads);
   const size_t smem = sizeof(float) * p.rank;
   cudaError_t e;
-  switch (delta_pad(p.dim) / kDrKeys) {
+  switch (state_pad(p.dim) / kDrKeys) {
     case 1: e = launch_kernel(delta_decode_kernel<T, 1>, grid, block, smem, st, 1u, p); break;
     case 2: e = launch_kernel(delta_decode_kernel<T, 2>, grid, block, smem, st, 1u, p); break;
     case 4: e = launch_kernel(delta_decode_kernel<T, 4>, grid, block, smem, st, 1u, p); break;
@@ -502,7 +281,7 @@ struct SllmDeltaArgs {     // host-side mirror passed by the Python layer (ctype
   float* state;
   const int* row_off;
   const int* slots;
-  float* scratch;          // prompt form: heads * tokens * (6 * pad + 4) + tokens * heads * dim floats, 16-byte aligned
+  float* scratch;          // prompt form: heads * tokens * (5 * pad + dim padded to 4 + 4) + tokens * heads * dim floats, 16-byte aligned
   void* out;
   long long slot_stride, scratch_floats;
   int ldp, off_r, off_k, off_v, off_a, off_g, off_w1, rank, ld_decay, ld_w2, heads, dim, tokens, sequences, fp32, decode;
@@ -515,8 +294,8 @@ SLLM_EXPORT int sllm_general_delta(const SllmDeltaArgs* a, void* stream) {
       a->dim <= 0 || a->tokens <= 0 || a->sequences <= 0 || a->heads > 65535 || a->sequences > 65535)
     return SLLM_ERR_INVALID_ARGUMENT;
   if (a->dim > 512) return SLLM_ERR_UNSUPPORTED_SHAPE;
-  const int pad = delta_pad(a->dim);
-  const long long nv = static_cast<long long>(a->heads) * a->tokens * delta_record(pad);
+  const int pad = state_pad(a->dim);
+  const long long nv = static_cast<long long>(a->heads) * a->tokens * state_record(true, pad, a->dim);
   const long long no = static_cast<long long>(a->tokens) * a->heads * a->dim;
   if (a->decode) {
     if (!a->w2 || a->rank <= 0 || a->ld_w2 < a->rank || a->rank > 8192) return SLLM_ERR_INVALID_ARGUMENT;

@@ -13,7 +13,7 @@ from typing import Optional
 @dataclass
 class ModelConfig:
     name: str = "tiny-llama"
-    family: str = "llama"            # llama | moe | qwen35 | gemma4 | zokuvik | sepedra
+    family: str = "llama"            # llama | moe | qwen35 | gemma4 | zokuvik | sepedra | kegorax
     n_layers: int = 2
     d_model: int = 256
     n_heads: int = 4
@@ -64,6 +64,7 @@ class ModelConfig:
     # families whose layers differ in kind and size: one dict per layer, {"type": mixer kind, "mixer": {sizes}, "mlp":
     # {"kind", ...} or None}; the norms split a vector into norm_groups parts
     layer_specs: Optional[list] = None
+    layer_loop: Optional[dict] = None        # {"start", "stop", "times"}: layers that run several times in a row, same weights
     norm_groups: int = 1
     # vision-language models: rotary pairs [0, t) follow the temporal index, [t, t + h) the height index and the rest
     # the width index of a token's 3-axis position (text tokens carry the same value on all three)
@@ -176,7 +177,13 @@ def _sepedra():
     return sepedra_shape()
 
 
+def _kegorax():
+    from .kegorax import kegorax_shape
+    return kegorax_shape()
+
+
 NAMED = {
+    "kegorax": _kegorax,
     "sepedra": _sepedra,
     "zokuvik": _zokuvik,
     "qwen35-moe": _qwen35_moe,

@@ -14,14 +14,16 @@ from .config import ModelConfig
 # CUDA translation units of a family, for callers that build no more than they run (None: the whole library)
 KERNEL_UNITS = {
     "zokuvik": ("elementwise", "gemm_tcgen05", "gemm_simt", "group_norm", "latent_attention", "latent_decode", "latent_prefill",
-                "delta_rule"),
+                "delta_rule", "state_scan"),
     "sepedra": ("elementwise", "gemm_tcgen05", "gemm_simt", "group_norm", "attention", "kv_attention", "short_conv", "latent_prefill", "rglru", "moe",
                 "moe_dense"),
+    "kegorax": ("elementwise", "gemm_tcgen05", "gemm_simt", "group_norm", "attention", "kv_attention", "short_conv", "latent_prefill",
+                "linear_state", "state_scan", "moe", "moe_dense"),
 }
 
 # families whose configuration lists its layers (ModelConfig.layer_specs): modules with ARCHITECTURE, config_from_source,
 # pack_weights, named_tensors and make_cache.  They run on one GPU, in bf16 or fp32
-LAYERED = ("zokuvik", "sepedra")
+LAYERED = ("zokuvik", "sepedra", "kegorax")
 
 
 def layered(family: str):
@@ -43,6 +45,9 @@ def make_model(cfg: ModelConfig, weights, tp=None, ep=None):
     if cfg.family == "sepedra":
         from .sepedra import SepedraModel
         return SepedraModel(cfg, weights, tp)
+    if cfg.family == "kegorax":
+        from .kegorax import KegoraxModel
+        return KegoraxModel(cfg, weights, tp)
     from .llama import LlamaModel
     return LlamaModel(cfg, weights, tp)
 
@@ -72,6 +77,9 @@ def init_random_weights(cfg: ModelConfig, device, seed: int = 0, tp_size: int = 
     if cfg.family == "sepedra":
         from .sepedra import init_random_sepedra_weights
         return init_random_sepedra_weights(cfg, device, seed)
+    if cfg.family == "kegorax":
+        from .kegorax import init_random_kegorax_weights
+        return init_random_kegorax_weights(cfg, device, seed)
     from .llama import init_random_weights as init
     return init(cfg, device, seed, tp_size, tp_rank)
 

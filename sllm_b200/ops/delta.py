@@ -103,7 +103,7 @@ def general_delta(proj: torch.Tensor, spec: DeltaSpec, w2, w0: torch.Tensor, a_b
     scratch: Optional[torch.Tensor] = None
     if not one_row_each:
         decay = linear(tanh_rows(proj[:, col["w1"]:col["w1"] + spec.rank], w2.in_features), w2)
-        scratch = torch.empty(H * t * (6 * _pad(D) + 4) + t * H * D, dtype=torch.float32, device=proj.device)
+        scratch = torch.empty(H * t * (5 * _pad(D) + (D + 3) // 4 * 4 + 4) + t * H * D, dtype=torch.float32, device=proj.device)
     v = lambda x: None if x is None else x.data_ptr()
     args = DeltaArgs(v(proj), v(decay), v(w2.w), v(w0), v(a_bias), v(norm_w), v(state), v(row_off), v(slots), v(scratch), v(out),
                      state.stride(0), 0 if scratch is None else scratch.numel(), proj.stride(0), col["r"], col["k"], col["v"],
