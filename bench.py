@@ -59,7 +59,7 @@ def parse_args():
                     help="4-bit-weight models: quantise activations to the weights' 4-bit format and run the GEMMs on the "
                          "block-scaled tensor-core kernel (W4A4) instead of W4A16")
     ap.add_argument("--layers", type=int, default=0, help="profiling only: override the layer count")
-    ap.add_argument("--compare", default=None, choices=["zokuvik", "sepedra"],
+    ap.add_argument("--compare", default=None, choices=["zokuvik", "sepedra", "kegorax"],
                     help="instead of the headline workload: prompt and decode throughput and per-kernel roofline fractions of "
                          "a design beside the framework's closest model at equal sizes (one GPU)")
     ap.add_argument("--no-batch1", action="store_true", help="skip the extra batch-1 measurement")
@@ -336,8 +336,9 @@ def main():
     from sllm_b200.ops import _lib
 
     if args.compare:
-        from sllm_b200.utils import family_bench, sepedra_bench
-        return (sepedra_bench if args.compare == "sepedra" else family_bench).main(args)
+        import importlib
+        module = {"zokuvik": "family_bench", "sepedra": "sepedra_bench", "kegorax": "kegorax_bench"}[args.compare]
+        return importlib.import_module(f"sllm_b200.utils.{module}").main(args)
     if args.act4:
         from sllm_b200.ops import w4 as _w4
         _w4.set_w4a4(True)

@@ -335,7 +335,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
         // keys [lo, hi] of this thread's 64 are visible, and those before `head_keys`
         int hi = 64, lo = 0, head_keys = 0;
         if (j < kept_tiles) {
-          hi = kept - 1 - half * 64;                 // all kept positions precede the tile's rows
+          hi = kept - 1 - (k0 + half * 64);          // all kept positions precede the tile's rows
         } else {
           hi = qpos - (k0 + half * 64);
           lo = p.window > 0 ? hi - p.window + 1 : p.chunk > 0 ? hi - qpos % p.chunk : 0;

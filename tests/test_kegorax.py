@@ -495,7 +495,7 @@ def test_planted_mistakes_show(tmp_path, monkeypatch, device, dtype):
         monkeypatch.setattr(O, fn, wrong)
         bad = O.forward(toks, cfg, c.w64)
         monkeypatch.undo()
-        assert K.error(bad[rows], want[rows]) > 3 * tol, name
+        assert K.error(bad[rows], want[rows]) > (1.5 if dtype == "bf16" else 100) * tol, name
     for cuts in ([70], [1], [29, 2]):
         assert K.error(K.run_cut(c.engine(device, dtype), toks, cuts), want) < tol
 
