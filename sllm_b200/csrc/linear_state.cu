@@ -214,7 +214,7 @@ __host__ __device__ constexpr int rank_pad(int r) { return (r + 7) & ~7; }
 
 // grid (heads, sequences), 256 threads; warps sweep the head's column tiles.
 template <typename T, int kKL, int kForm>
-__global__ void __launch_bounds__(kLsDecodeThreads) linear_decode_kernel(const LinearStateParams<T> p) {
+__global__ void __launch_bounds__(kLsDecodeThreads, 2) linear_decode_kernel(const LinearStateParams<T> p) {
   pdl_wait();
   pdl_trigger();
   constexpr bool kDelta = kForm == kChannelDelta;
