@@ -116,7 +116,7 @@ def test_engine_loop_queue_full_cancel_timeout_and_sampling():
         assert d2.wait(30) and why2 == ["length"] and len(t2) == 5
         loop.cancel(blocker.rid)
         # timeout and stop token
-        r4, t4, d4, why4 = _collect(loop, [9, 9, 9], 10_000, deadline=time.monotonic() + 0.3)
+        r4, t4, d4, why4 = _collect(loop, [9, 9, 9], 10_000, deadline=time.monotonic() + 0.05)
         assert d4.wait(30) and why4 == ["timeout"]
         # seeded sampling is reproducible and differs from greedy somewhere
         outs = []
