@@ -67,7 +67,8 @@ int sllm_paged_attention(const void* q, int q_ld, const void* k_pages, const voi
                          int page_size, int window, float sm_scale, int kv_fp8, void* out_bf16, void* out_fp8,
                          float* out_scale, int ld_scale, const float* sinks, int splits, float* ws,
                          long long ws_floats, int* counters, int n_counters, const void* gate, long long ld_gate,
-                         int gate_heads, int keep_first, int chunk, const float* slopes, void* stream);
+                         int gate_heads, int keep_first, int chunk, const float* slopes, const float* dist, int n_dist,
+                         int ld_dist, void* stream);
 
 /* decode_attention_tc.cu */
 int sllm_decode_attention_tc(const void* q, int q_ld, const void* k_pages, const void* v_pages, const float* k_scale,

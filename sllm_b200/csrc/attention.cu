@@ -172,6 +172,11 @@ __global__ void __launch_bounds__(128) paged_attention_kernel(const PagedAttnPar
 #pragma unroll
       for (int g = 0; g < G; ++g) s[g] = fmaf(-p.slopes[kvh * G + g], static_cast<float>(kv_len - 1 - tok), s[g]);
     }
+    if (p.dist.table && valid) {
+      const int d = min(kv_len - 1 - tok, p.dist.n - 1);
+#pragma unroll
+      for (int g = 0; g < G; ++g) s[g] += p.dist.head(kvh * G + g)[d];
+    }
 #pragma unroll
     for (int g = 0; g < G; ++g) {
       const float sv = valid ? s[g] : -INFINITY;
@@ -318,7 +323,8 @@ SLLM_EXPORT int sllm_paged_attention(const void* q, int q_ld, const void* k_page
                                      void* out_fp8, float* out_scale, int ld_scale, const float* sinks, int splits,
                                      float* ws, long long ws_floats, int* counters, int n_counters, const void* gate,
                                      long long ld_gate, int gate_heads, int keep_first, int chunk, const float* slopes,
-                                     void* stream) {
+                                     const float* dist, int n_dist, int ld_dist, void* stream) {
+  if (dist && (n_dist < 1 || ld_dist < kDistFront + n_dist)) return SLLM_ERR_INVALID_ARGUMENT;
   if (keep_first < 0 || chunk < 0 || (keep_first > 0 && window <= 0) || (chunk > 0 && window > 0)) return SLLM_ERR_INVALID_ARGUMENT;
   if (!q || !k_pages || !v_pages || !block_table || !seq_index || !kv_lens || rows <= 0 || hkv <= 0 || hq % hkv)
     return SLLM_ERR_INVALID_ARGUMENT;
@@ -337,7 +343,7 @@ SLLM_EXPORT int sllm_paged_attention(const void* q, int q_ld, const void* k_page
   p.out_scale = out_scale; p.ld_scale = ld_scale; p.sinks = sinks;
   p.ws_o = nullptr; p.ws_ml = nullptr; p.counters = counters; p.status_word = nullptr;
   p.gate = static_cast<const __nv_bfloat16*>(gate); p.ld_gate = ld_gate;
-  p.gate_heads = gate_heads; p.keep_first = keep_first; p.chunk = chunk; p.slopes = slopes;
+  p.gate_heads = gate_heads; p.keep_first = keep_first; p.chunk = chunk; p.slopes = slopes; p.dist = {dist, n_dist, ld_dist};
   p.early_trigger = 0;
   if (splits > 1) {
     const long long units = static_cast<long long>(rows) * hkv;

@@ -23,6 +23,16 @@ struct VisibleKeys {
   __device__ __forceinline__ int position(int i) const { return i < keep ? i : i - keep + first; }
 };
 
+// What joins a score by its distance (keys back from the query): table[head][distance], the last entry for all distances
+// beyond.  Rows lie `ld` floats apart; kDistFront floats lie before a row's first entry and copies of its last one behind it, so
+// that a tile of 128 x 128 scores is indexed without looking at its edges.
+constexpr int kDistFront = 256, kDistBack = 256;
+struct DistanceBias {
+  const float* table;        // optional [heads, ld]: kDistFront, n entries, kDistBack copies of the last
+  int n, ld;
+  __device__ __forceinline__ const float* head(int h) const { return table + static_cast<size_t>(h) * ld + kDistFront; }
+};
+
 struct PagedAttnParams {
   const __nv_bfloat16* q;  // [rows, hq * hd] (row stride q_ld)
   int q_ld;
@@ -51,6 +61,7 @@ struct PagedAttnParams {
   // CUDA-core kernel only: see VisibleKeys; slopes (optional [hq]) are taken off a score per position of distance
   int keep_first, chunk;
   const float* slopes;
+  DistanceBias dist;        // CUDA-core kernel only
   int* status_word;         // device status word for bounded waits (tensor-core kernel)
   int early_trigger;        // tensor-core kernel: let dependent launches start once the CTA holds its TMEM
   STEP_TRACE_FIELD

@@ -81,13 +81,13 @@ __global__ void __launch_bounds__(kDrRowWarps * 32) delta_pre_kernel(const Delta
   }
   s1 = warp_sum(s1);
   s2 = warp_sum(s2);
-  float* dst = p.vec + (static_cast<size_t>(h) * p.tokens + t) * state_record(true, pad, D);
+  float* dst = p.vec + (static_cast<size_t>(h) * p.tokens + t) * state_record(kRemoval, pad, D);
   lane_store(dst + kVecWR * pad, d0, pad, r);
   lane_store(dst + kVecW * pad, d0, pad, w);
   lane_store(dst + kVecK * pad, d0, pad, k);
   lane_store(dst + kVecU * pad, d0, pad, u);
   lane_store(dst + kVecAU * pad, d0, pad, a);
-  dst += state_vecs(true) * pad;
+  dst += state_vecs(kRemoval) * pad;
   lane_store(dst, d0, state_vpad(D), v);
   if (lane == 0) *reinterpret_cast<float2*>(dst + state_vpad(D)) = make_float2(s1, s2);
 }
@@ -136,7 +136,7 @@ __global__ void __launch_bounds__(kDrDecodeThreads) delta_decode_kernel(const De
   pdl_trigger();
   constexpr int pad = kKL * kDrKeys;
   constexpr int kWarps = kDrDecodeThreads / 32;
-  __shared__ __align__(16) float vs[(state_vecs(true) + 1) * pad];
+  __shared__ __align__(16) float vs[(state_vecs(kRemoval) + 1) * pad];
   __shared__ float o_s[pad];
   __shared__ float red[kWarps];
   extern __shared__ float low[];                     // [rank] tanh of the low-rank decay input
@@ -198,7 +198,7 @@ __global__ void __launch_bounds__(kDrDecodeThreads) delta_decode_kernel(const De
     }
     float v[2] = {0.f, 0.f}, o[2];
     if (col < pad) { v[0] = vs[5 * pad + col]; v[1] = vs[5 * pad + col + 1]; }
-    state_token<kKL, 2, true>(S, vs, kl, v, s1, s2, o);
+    state_token<kKL, 2, kRemoval>(S, vs, kl, v, make_float4(s1, s2, 0.f, 0.f), o);
     state_io<kKL, 2, true>(S, st, D, D, kl, col);
     if (kl == 0 && col < pad) { o_s[col] = o[0]; o_s[col + 1] = o[1]; }
   }
@@ -246,7 +246,7 @@ static int delta_prompt_launch(DeltaParams<T> p, int sequences, cudaStream_t st)
   const int pad = state_pad(p.dim);
   if (delta_rows<T>(p, pad, true, st) != cudaSuccess) return SLLM_ERR_CUDA;
   const ScanParams sp{p.vec, p.state, p.slot_stride, p.row_off, p.slots, p.o_raw, p.heads, p.dim, p.dim, p.tokens};
-  const int rc = state_scan_launch(sp, true, sequences, st);
+  const int rc = state_scan_launch(sp, kRemoval, sequences, st);
   if (rc != SLLM_OK) return rc;
   return delta_rows<T>(p, pad, false, st) == cudaSuccess ? SLLM_OK : SLLM_ERR_CUDA;
 }
@@ -295,7 +295,7 @@ SLLM_EXPORT int sllm_general_delta(const SllmDeltaArgs* a, void* stream) {
     return SLLM_ERR_INVALID_ARGUMENT;
   if (a->dim > 512) return SLLM_ERR_UNSUPPORTED_SHAPE;
   const int pad = state_pad(a->dim);
-  const long long nv = static_cast<long long>(a->heads) * a->tokens * state_record(true, pad, a->dim);
+  const long long nv = static_cast<long long>(a->heads) * a->tokens * state_record(kRemoval, pad, a->dim);
   const long long no = static_cast<long long>(a->tokens) * a->heads * a->dim;
   if (a->decode) {
     if (!a->w2 || a->rank <= 0 || a->ld_w2 < a->rank || a->rank > 8192) return SLLM_ERR_INVALID_ARGUMENT;

@@ -11,6 +11,7 @@
 //   latent_prefill_kernel  see below; it also serves ordinary keys and values gathered from their pages (kv_attention.cu),
 //                          with fewer key / value heads than query heads, attention sinks and a gate per output channel
 #include "typed.cuh"
+#include "attention_common.cuh"
 #include "api.h"
 #include "tmap.h"
 
@@ -110,7 +111,7 @@ latent_pack_q_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, __nv_bf
 //   warps 4-11  softmax: two threads per query row, 64 keys each; row maxima meet in shared memory, P goes to shared
 //               memory as the bf16 K-major operand, each thread folds half of the value columns into registers
 // Causal with any offset between queries and context, optional sliding window (key tiles outside it are not visited).
-// kRich adds chunks of positions, distance slopes, and windows whose first `keep_first` positions stay visible: a tile that
+// kRich adds chunks of positions, distance slopes, distance biases (a head's table in shared memory where it fits), and windows whose first `keep_first` positions stay visible: a tile that
 // lies past those walks two runs of key tiles, the kept positions and the window.
 constexpr int kLpThreads = 384;
 constexpr int kLpTile = 128;
@@ -122,6 +123,8 @@ struct LatentPrefillParams {
   int heads, kv_heads, dim, vdim, dim_chunks, v_stages, window, keep_first, chunk;
   float scale_log2;
   const float* slopes;       // optional [heads]: taken off a score per position of distance
+  DistanceBias dist;         // what joins a score by its distance
+  int dist_smem;             // bytes of a head's table in shared memory (0: it is read where it is)
   const float* sinks;        // optional [heads]: scores that join the denominator only
   const __nv_bfloat16* gate; // optional logits [tokens, ld_gate], one per head or (gate_channels) per output channel
   long long ld_gate;
@@ -174,6 +177,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   uint8_t* k_s = p_s + 2 * kLpChunk;                 // [2][kNQ]
   uint8_t* v_s = k_s + 2 * kNQ * kLpChunk;           // [v_stages][kNV]
   LatentPrefillShared* sh = reinterpret_cast<LatentPrefillShared*>(v_s + p.v_stages * kNV * kLpChunk);
+  float* dist_s = reinterpret_cast<float*>(sh + 1);
   constexpr uint32_t kTmemCols = 512;                // S at columns 0 and 128, PV at 256
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int head = blockIdx.y, kvh = head / (p.heads / p.kv_heads);
@@ -210,6 +214,12 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   if (warp == 1) {
     tmem_alloc(&sh->tmem_base, kTmemCols);
     tmem_relinquish();
+  }
+  if constexpr (kRich) {
+    if (p.dist_smem > 0) {
+      const float* src = p.dist.head(head) - kDistFront;
+      for (int i = threadIdx.x; i < p.dist_smem / 4; i += kLpThreads) dist_s[i] = src[i];
+    }
   }
   tc_fence_before();
   __syncthreads();
@@ -298,7 +308,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
     float m = -INFINITY, l = 0.f, alpha_prev = 0.f;
     bool ok = true;
     const float slope = kRich && p.slopes ? p.slopes[head] * 1.4426950408889634f : 0.f;
-    const float mul = kRich && p.slopes ? 1.f : p.scale_log2;   // with slopes the scores are scaled before the mask
+    const float mul = kRich && (p.slopes || p.dist.table) ? 1.f : p.scale_log2;   // scores that something joins are scaled before the mask
+    const float* dist = !kRich || !p.dist.table ? nullptr : p.dist_smem > 0 ? dist_s + kDistFront : p.dist.head(head);
     auto fold = [&](int j) {                         // o <- o * alpha(j) + PV(j)
       if (ok) ok = mbar_wait(&sh->o_full[j & 1], (j >> 1) & 1, abort_flag, p.status, SLLM_DEV_TIMEOUT_TMEM_FULL);
       tc_fence_after();
@@ -331,6 +342,11 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
           const float d0 = static_cast<float>(k0 + half * 64 - qpos);
 #pragma unroll
           for (int i = 0; i < 64; ++i) s[i] = fmaf(s[i], p.scale_log2, slope * (d0 + static_cast<float>(i)));
+        }
+        if (dist) {                                  // entries outside the row belong to keys that are masked below
+          const float* b = dist + min(q0 - k0, p.dist.n - 1 + kLpTile) + r - half * 64;
+#pragma unroll
+          for (int i = 0; i < 64; ++i) s[i] = fmaf(s[i], p.scale_log2, b[-i] * 1.4426950408889634f);
         }
         // keys [lo, hi] of this thread's 64 are visible, and those before `head_keys`
         int hi = 64, lo = 0, head_keys = 0;
@@ -426,13 +442,21 @@ static int latent_prefill_go(const CUtensorMap& tq, const CUtensorMap& tkv, cons
   // two V stages where they fit; at least 120 KB, so that one CTA (which takes the whole TMEM) is on an SM at a time
   p.v_stages = (3 * kNQ + 2 + 2 * kNV) * kLpChunk <= 208 * 1024 ? 2 : 1;
   size_t smem = static_cast<size_t>(3 * kNQ + 2 + p.v_stages * kNV) * kLpChunk + sizeof(LatentPrefillShared) + 1024;
+  if (kRich && p.dist.table) {                       // distances up to the window's, and what a tile reads beyond
+    const int n = p.window > 0 && p.keep_first == 0 && p.window < p.dist.n ? p.window : p.dist.n;
+    const int bytes = (kDistFront + n + kDistBack) * 4;
+    if (smem + bytes <= 227 * 1024) {
+      p.dist_smem = bytes;
+      smem += bytes;
+    }
+  }
   if (smem < 120 * 1024) smem = 120 * 1024;
-  static bool cfg = false;
-  if (!cfg) {
+  static size_t configured = 0;
+  if (smem > configured) {
     if (cudaFuncSetAttribute(latent_prefill_kernel<kNQ, kNV, kRich>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) !=
         cudaSuccess)
       return SLLM_ERR_CUDA;
-    cfg = true;
+    configured = smem;
   }
   return launch_kernel(latent_prefill_kernel<kNQ, kNV, kRich>, dim3(tiles, p.heads), dim3(kLpThreads), smem, st, 1u, tq, tkv, tr, p) ==
                  cudaSuccess ? SLLM_OK : SLLM_ERR_CUDA;
@@ -441,7 +465,7 @@ static int latent_prefill_go(const CUtensorMap& tq, const CUtensorMap& tkv, cons
 template <int kNQ, int kNV>
 static int latent_prefill_launch(const CUtensorMap& tq, const CUtensorMap& tkv, const CUtensorMap& tr, const LatentPrefillParams& p,
                                  int tiles, cudaStream_t st) {
-  return p.keep_first > 0 || p.chunk > 0 || p.slopes ? latent_prefill_go<kNQ, kNV, true>(tq, tkv, tr, p, tiles, st)
+  return p.keep_first > 0 || p.chunk > 0 || p.slopes || p.dist.table ? latent_prefill_go<kNQ, kNV, true>(tq, tkv, tr, p, tiles, st)
                                                      : latent_prefill_go<kNQ, kNV, false>(tq, tkv, tr, p, tiles, st);
 }
 
@@ -514,21 +538,22 @@ SLLM_EXPORT int sllm_latent_prefill(const void* q, int tokens, const void* kv, c
 }
 
 // The same kernel over ordinary keys and values: q [tokens, heads, dim padded to 64 with zeros]; kv [context rows, kv_heads *
-// (dim + vdim)]; sinks, slopes: optional [heads]; gate: optional logits [tokens, ld_gate], one per output channel
+// (dim + vdim)]; sinks, slopes: optional [heads]; dist: see DistanceBias, its back part included; gate: optional logits [tokens, ld_gate], one per output channel
 // (gate_heads: per head).
 SLLM_EXPORT int sllm_kv_prefill(const void* q, int tokens, const void* kv, int context, const int* tiles, int num_tiles, int heads,
-                                int kv_heads, int dim, int vdim, int window, int keep_first, int chunk, const float* slopes, float scale,
-                                const float* sinks, const void* gate, long long ld_gate, int gate_heads, void* out, int* status,
-                                void* stream) {
+                                int kv_heads, int dim, int vdim, int window, int keep_first, int chunk, const float* slopes,
+                                const float* dist, int n_dist, int ld_dist, float scale, const float* sinks, const void* gate,
+                                long long ld_gate, int gate_heads, void* out, int* status, void* stream) {
   if (!q || !kv || !tiles || !out || tokens <= 0 || context <= 0 || num_tiles <= 0 || heads <= 0 || heads > 65535 || kv_heads <= 0 ||
       heads % kv_heads || dim <= 0 || vdim <= 0 || window < 0 || keep_first < 0 || chunk < 0 || (keep_first > 0 && window == 0) ||
       (chunk > 0 && window > 0))
     return SLLM_ERR_INVALID_ARGUMENT;
+  if (dist && (slopes || n_dist < 1 || ld_dist < kDistFront + n_dist + kDistBack)) return SLLM_ERR_INVALID_ARGUMENT;
   if (gate && !gate_heads && ((ld_gate & 7) || (reinterpret_cast<uintptr_t>(gate) & 15))) return SLLM_ERR_ALIGNMENT;
   LatentPrefillParams p = {};
   p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim; p.window = window; p.scale_log2 = scale * 1.4426950408889634f;
   p.sinks = sinks; p.gate = static_cast<const __nv_bfloat16*>(gate); p.ld_gate = ld_gate; p.gate_channels = !gate_heads;
-  p.keep_first = keep_first; p.chunk = chunk; p.slopes = slopes;
+  p.keep_first = keep_first; p.chunk = chunk; p.slopes = slopes; p.dist = {dist, n_dist, ld_dist};
   p.out = static_cast<__nv_bfloat16*>(out); p.status = status;
   return latent_prefill_impl(q, tokens, kv, nullptr, context, tiles, num_tiles, 0, p, static_cast<cudaStream_t>(stream));
 }

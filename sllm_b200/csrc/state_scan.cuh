@@ -1,11 +1,13 @@
 // One step of a matrix-valued recurrent state, per head, S [dim keys, vdim values] in fp32:
-//   S <- diag(w) S - au (u^T S) + k v^T,   o = S^T r          (delta: with the removal term, else without it)
+//   S <- diag(w) S - au (u^T S) + k v^T,   o = S^T r          (kRemoval: with the removal term, kPlain: without it)
+//   S <- g S;  S <- S + k (beta (v - S^T k))^T,   o = S^T q   (kGatedDelta: one decay g per head, beta v in place of v)
 // Columns of S (value channels) never meet, so heads are cut into column tiles.  A thread keeps 16 keys x 2 or 4 columns of S
 // in registers; kKL = 1 .. 32 lanes share a column.  All dot products of a token are taken from the OLD state in one sweep,
-//   o = (w r)^T S - (u^T S) (au^T r) + v k^T r
+//   o = (w r)^T S - (u^T S) (au^T r) + v k^T r,     o = g q^T S + (k^T q) (beta v - beta g k^T S)
 // so a token costs one shuffle reduction and no barrier.
 #pragma once
 #include "typed.cuh"
+#include "state_scan.h"
 
 namespace sllm {
 
@@ -17,13 +19,14 @@ __host__ __device__ constexpr int state_pad(int dim) {   // padded head size: 16
   return kl * kDrKeys;
 }
 
-// What the scan reads per (head, token): the vectors [pad] in this order (the last two with delta only), v [value pad], and
-// the pair au^T r, k^T r.
+// What the scan reads per (head, token): the vectors [pad] in this order (the last two with kRemoval only; kGatedDelta: q, k),
+// v [value pad], and four scalars: au^T r, k^T r, -, - (kGatedDelta: g, beta g, k^T q, -).
 enum StateVec { kVecWR = 0, kVecW = 1, kVecK = 2, kVecU = 3, kVecAU = 4 };
-__host__ __device__ constexpr int state_vecs(bool delta) { return delta ? 5 : 3; }
+enum GatedVec { kVecGQ = 0, kVecGK = 1 };
+__host__ __device__ constexpr int state_vecs(int step) { return step == kGatedDelta ? 2 : step == kRemoval ? 5 : 3; }
 __host__ __device__ constexpr int state_vpad(int vdim) { return (vdim + 3) & ~3; }
-__host__ __device__ constexpr int state_record(bool delta, int pad, int vdim) {   // floats
-  return state_vecs(delta) * pad + state_vpad(vdim) + 4;
+__host__ __device__ constexpr int state_record(int step, int pad, int vdim) {   // floats
+  return state_vecs(step) * pad + state_vpad(vdim) + 4;
 }
 
 // Lane l of a warp loads channels d0 = l kN .. + kN - 1 of a head; vec: widths and offsets allow 4-channel accesses.
@@ -59,12 +62,65 @@ __device__ __forceinline__ void lane_store(float* dst, int d0, int limit, const 
   }
 }
 
-// One token on a thread's 16 keys x kC columns: S is updated, o holds the outputs on every lane of the columns.
-// vs: the token's vectors in shared memory.  Key of S[j * 4 + e]: (j * kKL + kl) * 4 + e.
-template <int kKL, int kC, bool kDelta>
-__device__ __forceinline__ void state_token(float (&S)[kDrKeys][kC], const float* vs, int kl, const float (&v)[kC], float s1, float s2,
+// The step with one decay per head: two vectors and three scalars.
+template <int kKL, int kC>
+__device__ __forceinline__ void gated_token(float (&S)[kDrKeys][kC], const float* vs, int kl, const float (&v)[kC], const float4& sc,
                                             float (&o)[kC]) {
   constexpr int pad = kKL * kDrKeys;
+  float pc[2][kC], qc[2][kC];                        // two chains per column
+#pragma unroll
+  for (int c = 0; c < kC; ++c) pc[0][c] = pc[1][c] = qc[0][c] = qc[1][c] = 0.f;
+  float ka[kDrKeys];
+#pragma unroll
+  for (int j = 0; j < kDrKeys / 4; ++j) {
+    float qa[4], kv[4];
+    ld_vec<4>(vs + kVecGQ * pad + (j * kKL + kl) * 4, qa);
+    ld_vec<4>(vs + kVecGK * pad + (j * kKL + kl) * 4, kv);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      ka[j * 4 + e] = kv[e];
+#pragma unroll
+      for (int c = 0; c < kC; ++c) {
+        pc[e & 1][c] = fmaf(kv[e], S[j * 4 + e][c], pc[e & 1][c]);
+        qc[e & 1][c] = fmaf(qa[e], S[j * 4 + e][c], qc[e & 1][c]);
+      }
+    }
+  }
+  float p[kC], q[kC];
+#pragma unroll
+  for (int c = 0; c < kC; ++c) {
+    p[c] = pc[0][c] + pc[1][c];
+    q[c] = qc[0][c] + qc[1][c];
+  }
+#pragma unroll
+  for (int x = kKL / 2; x > 0; x >>= 1)
+#pragma unroll
+    for (int c = 0; c < kC; ++c) {
+      p[c] += __shfl_xor_sync(0xffffffffu, p[c], x);
+      q[c] += __shfl_xor_sync(0xffffffffu, q[c], x);
+    }
+#pragma unroll
+  for (int c = 0; c < kC; ++c) {
+    p[c] = fmaf(-sc.y, p[c], v[c]);                  // what is written along k
+    o[c] = fmaf(sc.x, q[c], sc.z * p[c]);
+  }
+#pragma unroll
+  for (int e = 0; e < kDrKeys; ++e)
+#pragma unroll
+    for (int c = 0; c < kC; ++c) S[e][c] = fmaf(ka[e], p[c], sc.x * S[e][c]);
+}
+
+// One token on a thread's 16 keys x kC columns: S is updated, o holds the outputs on every lane of the columns.
+// vs: the token's vectors in shared memory; sc: its scalars.  Key of S[j * 4 + e]: (j * kKL + kl) * 4 + e.
+template <int kKL, int kC, int kStep>
+__device__ __forceinline__ void state_token(float (&S)[kDrKeys][kC], const float* vs, int kl, const float (&v)[kC], const float4& sc,
+                                            float (&o)[kC]) {
+  constexpr int pad = kKL * kDrKeys;
+  if constexpr (kStep == kGatedDelta) {
+    gated_token<kKL, kC>(S, vs, kl, v, sc, o);
+    return;
+  }
+  constexpr bool kDelta = kStep == kRemoval;
   float pc[2][kC], qc[2][kC];                        // two chains per column
 #pragma unroll
   for (int c = 0; c < kC; ++c) pc[0][c] = pc[1][c] = qc[0][c] = qc[1][c] = 0.f;
@@ -111,7 +167,7 @@ __device__ __forceinline__ void state_token(float (&S)[kDrKeys][kC], const float
       }
   }
 #pragma unroll
-  for (int c = 0; c < kC; ++c) o[c] = kDelta ? q[c] - p[c] * s1 + v[c] * s2 : fmaf(v[c], s2, q[c]);
+  for (int c = 0; c < kC; ++c) o[c] = kDelta ? q[c] - p[c] * sc.x + v[c] * sc.y : fmaf(v[c], sc.y, q[c]);
 }
 
 template <int kKL, int kC, bool kStore>

@@ -4,6 +4,9 @@
 
 namespace sllm {
 
+// What one token does to a state, see state_scan.cuh.
+enum StateStep { kPlain = 0, kRemoval = 1, kGatedDelta = 2 };
+
 // vec: [heads][tokens] records, see state_record in state_scan.cuh.  State of slot s, head h: state + s * slot_stride +
 // h * dim * vdim, [dim keys][vdim values].  o_raw: [tokens, heads * vdim].
 struct ScanParams {
@@ -15,7 +18,7 @@ struct ScanParams {
   int heads, dim, vdim, tokens;
 };
 
-// delta: records carry the removal vectors.  Returns an SllmStatus.
-int state_scan_launch(const ScanParams& p, bool delta, int sequences, cudaStream_t stream);
+// step: a StateStep, which the records are made for.  Returns an SllmStatus.
+int state_scan_launch(const ScanParams& p, int step, int sequences, cudaStream_t stream);
 
 }  // namespace sllm

@@ -1,6 +1,6 @@
 """Op layer: hand-written sm_100a kernels for CUDA tensors, PyTorch restatements for CPU tensors."""
 from .core import (Again, KVLayer, LinearWeight, QTensor, Workspace, add_group_norm, argmax, device_status, elementwise,
-                   embed_group_norm, embedding, gated_act, gemm_raw, group_norm, linear, paged_attention, quant_fp8, rmsnorm, rope_kv_append, workspace)
+                   embed_group_norm, embedding, gated_act, gemm_raw, group_norm, linear, paged_attention, poly_norm, quant_fp8, rmsnorm, rope_kv_append, workspace)
 from ._lib import KernelError, kernels_available
 
 

@@ -174,6 +174,7 @@ _KERNEL_SIGNATURES = {
     "sllm_rmsnorm": (I, [P, P, P, P, P, I, I, I, F, I, P]),
     "sllm_gated_act": (I, [P, P, P, P, I, I, I, I, P]),
     "sllm_gated_act_any": (I, [P, P, I, I, I, I, I, P]),
+    "sllm_poly_norm": (I, [P, L, P, I, I, P, F, I, P]),
     "sllm_quant_fp8_1x128": (I, [P, P, P, I, I, I, P]),
     "sllm_rope_kv_append": (I, [P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, F, F, P, P]),
     "sllm_rope_kv_append_paired": (I, [P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, F, F, P, I, P]),
@@ -187,7 +188,7 @@ _KERNEL_SIGNATURES = {
     "sllm_prefill_attention": (I, [P, I, I, P, I, I, I, I, F, P, P, P, I, P, P]),
     "sllm_paged_attention_workspace_floats": (L, [I, I, I, I, I]),
     "sllm_paged_attention": (I, [P, I, P, P, P, P, F, F, P, I, P, P, I, I, I, I, I, I, F, I, P, P, P, I, P, I, P, L,
-                                  P, I, P, L, I, I, I, P, P]),
+                                  P, I, P, L, I, I, I, P, P, I, I, P]),
 }
 
 # Entry points added by later translation units register themselves here (name -> (restype, argtypes)).

@@ -400,6 +400,19 @@ def gated_act(x: torch.Tensor, act: str = "silu", quant: bool = False):
     return y
 
 
+def poly_norm(x: torch.Tensor, coef: torch.Tensor, eps: float) -> torch.Tensor:
+    """a N(x) + b N(x^2) + c N(x^3) + e of each row [M, n] (row stride allowed), coef fp32 {a, b, c, e}, N(v) = v / rms(v)."""
+    if _lib.on_cpu(x):
+        z = x.float()
+        n = lambda v: v / torch.sqrt((v * v).mean(-1, keepdim=True) + eps)
+        return (coef[0] * n(z) + coef[1] * n(z * z) + coef[2] * n(z * z * z) + coef[3]).to(x.dtype)
+    m, n = x.shape
+    y = torch.empty((m, n), dtype=x.dtype, device=x.device)
+    rc = _lib.kernels().sllm_poly_norm(_p(x), x.stride(0), _p(y), m, n, _p(coef), eps, int(x.dtype == torch.float32), _stream())
+    _lib.check(rc, "poly_norm")
+    return y
+
+
 def embedding(table: torch.Tensor, ids: torch.Tensor, scale: float = 1.0) -> torch.Tensor:
     if _lib.on_cpu(table):
         y = table[ids.long()]
@@ -544,6 +557,11 @@ def rope_kv_append(qkv: torch.Tensor, positions: torch.Tensor, seq_index: torch.
     return qkv[:, :hq * hd]
 
 
+def dist_args(dist) -> tuple:
+    """Kernel arguments of an optional distance bias."""
+    return (None, 0, 0) if dist is None else (_p(dist.table), dist.n, dist.table.stride(0))
+
+
 def _attn_splits(rows: int, hkv: int, max_kv: int) -> int:
     """KV splits so that about 8 CTAs (32 warps) per SM are in flight: the kernel hides its
     load -> compute -> load chains with occupancy, and each split keeps >= 128 keys."""
@@ -559,14 +577,14 @@ def paged_attention(q: torch.Tensor, kv: KVLayer, block_table: torch.Tensor, seq
                     sm_scale: Optional[float] = None, max_kv: int = 0, quant_out: bool = False,
                     sinks: Optional[torch.Tensor] = None, impl: Optional[str] = None, out: Optional[QTensor] = None,
                     gate: Optional[torch.Tensor] = None, gate_heads: bool = False, keep_first: int = 0, chunk: int = 0,
-                    slopes: Optional[torch.Tensor] = None):
+                    slopes: Optional[torch.Tensor] = None, dist=None):
     """Attention of each query row over its sequence's pages. q: [R, hq*hd] (row stride allowed).
     Returns [R, hq*hd] (bf16) or a QTensor when quant_out (head_dim 128); ``out`` supplies the QTensor to fill
     (its scale plane may have a leading dimension larger than R), or the bf16 rows.  ``gate``: logits [R, hq*hd] (row stride
     allowed) whose sigmoid multiplies the output, with ``gate_heads`` one per head.  ``keep_first`` positions stay visible
     behind a window; ``chunk`` limits a row to the keys of its own chunk of positions; ``slopes`` (fp32 [hq]) are taken off
-    the scores per position of distance.  None of these five is on the tensor-core kernel, and the CPU form has ``gate``
-    only (ops.kv_attention states the others)."""
+    the scores per position of distance; ``dist`` (ops.kv_attention.DistanceBias) joins them by distance.  None of these six
+    is on the tensor-core kernel, and the CPU form has ``gate`` only (ops.kv_attention states the others)."""
     scale = sm_scale if sm_scale is not None else 1.0 / math.sqrt(hd)
     r = q.shape[0]
     if _lib.on_cpu(q):
@@ -592,7 +610,7 @@ def paged_attention(q: torch.Tensor, kv: KVLayer, block_table: torch.Tensor, seq
                 vv = kv.v[blks].transpose(1, 2).reshape(-1, hkv, hd).to(torch.float32)
             out[i] = ref.attention_rows(q[i].view(hq, hd), kk, vv, n, window, scale, sinks)
         out = out.view(r, hq * hd)
-        if keep_first or chunk or slopes is not None or gate_heads:
+        if keep_first or chunk or slopes is not None or gate_heads or dist is not None:
             raise ValueError("ops.kv_attention states these masks for CPU tensors")
         if gate is not None:
             out = out * torch.sigmoid(gate.float())
@@ -614,7 +632,7 @@ def paged_attention(q: torch.Tensor, kv: KVLayer, block_table: torch.Tensor, seq
         out_b, out_q, out_s, ld = ob, None, None, 0
     use_tc = (kv.fp8 and hd == 128 and (hq // hkv) in (1, 2, 4, 8, 16) and 128 % kv.page_size == 0
               and kv.page_size >= 8 and impl != "cuda_core" and gate is None
-              and not (keep_first or chunk or slopes is not None))
+              and not (keep_first or chunk or slopes is not None or dist is not None))
     if impl == "tensor_core" and not use_tc:
         raise ValueError("tensor-core decode attention needs FP8 pages, head_dim 128 and a GQA group <= 16")
     if use_tc:
@@ -642,6 +660,6 @@ def paged_attention(q: torch.Tensor, kv: KVLayer, block_table: torch.Tensor, seq
         _p(block_table), block_table.stride(0), _p(seq_index), _p(kv_lens), r, hq, hkv, hd, kv.page_size, window,
         scale, kv.mode, _p(out_b), _p(out_q), _p(out_s), ld, _p(sinks), splits, _p(wsp.ws), wsp.ws.numel(),
         _p(wsp.counters), wsp.counters.numel(), _p(gate), gate.stride(0) if gate is not None else 0,
-        int(gate_heads), keep_first, chunk, _p(slopes), _stream())
+        int(gate_heads), keep_first, chunk, _p(slopes), *dist_args(dist), _stream())
     _lib.check(rc, "paged_attention")
     return oq if quant_out else ob

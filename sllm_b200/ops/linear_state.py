@@ -1,5 +1,5 @@
 """Linear attention with a matrix-valued fp32 state per head: gated linear attention, retention, and a delta rule with a decay
-per key channel (kernels in csrc/linear_state.cu; the PyTorch branch restates them for CPU tensors)."""
+per key channel or per head (kernels in csrc/linear_state.cu; the PyTorch branch restates them for CPU tensors)."""
 from __future__ import annotations
 
 import ctypes as C
@@ -13,8 +13,8 @@ from . import _lib
 from .short_conv import causal_conv
 
 P, I, F, L = C.c_void_p, C.c_int, C.c_float, C.c_longlong
-GATED, FIXED, DELTA = 0, 1, 2
-UNIT_EPS = 1e-6              # of the delta form's unit vectors x / sqrt(sum x^2 + UNIT_EPS)
+GATED, FIXED, DELTA, HEAD_DELTA = 0, 1, 2, 3
+UNIT_EPS = 1e-6              # of the delta forms' unit vectors x / sqrt(sum x^2 + UNIT_EPS)
 
 
 class LinearStateArgs(C.Structure):
@@ -42,9 +42,11 @@ def _k():
 @dataclass
 class StateSpec:
     """Sizes and constants of one layer.  ``form``: GATED (decay sigmoid(z)^(1 / tau) per key channel, z low-rank), FIXED (one
-    decay per head) or DELTA (delta rule with a decay exp(-rate softplus(z)) per key channel, short convolutions with SiLU on q,
-    k and v, unit query and key).  ``columns``: where the parts of the packed input projection start: q, k, v, g, a (low-rank
-    decay input), b (write strengths); in the delta form q, k and v are consecutive and g is the gate's low-rank input."""
+    decay per head), DELTA (delta rule with a decay exp(-rate softplus(z)) per key channel, short convolutions with SiLU on q,
+    k and v, unit query and key) or HEAD_DELTA (the same with one decay per head, z a column of the projection plus a bias, and
+    an output gate as in the first two).  ``columns``: where the parts of the packed input projection start: q, k, v, g, a
+    (low-rank decay input, in the head form z), b (write strengths); in the delta forms q, k and v are consecutive, and in the
+    channel form g is the gate's low-rank input."""
     form: int
     heads: int
     kv_heads: int            # query / key heads (value heads are a multiple)
@@ -57,6 +59,10 @@ class StateSpec:
     taps: int = 1
     rank_a: int = 0
     rank_g: int = 0
+
+    @property
+    def delta(self) -> bool:
+        return self.form in (DELTA, HEAD_DELTA)
 
     @property
     def channels(self) -> int:
@@ -73,8 +79,8 @@ class StateWeights:
     """Vectors are fp32; the low-rank second factors [*, rank padded to 8] are in the model's type."""
     w_a: Optional[object] = None                # LinearWeight [heads * dim, rank_a padded]
     w_g: Optional[object] = None                # LinearWeight [heads * vdim, rank_g padded]
-    bias: Optional[torch.Tensor] = None         # [heads * dim], of z
-    rate: Optional[torch.Tensor] = None         # [heads]: the decay itself (FIXED), exp(A_log) (DELTA)
+    bias: Optional[torch.Tensor] = None         # [heads * dim], of z (HEAD_DELTA: [heads])
+    rate: Optional[torch.Tensor] = None         # [heads]: the decay itself (FIXED), exp(A_log) (the delta forms)
     conv_w: Optional[torch.Tensor] = None       # [taps, channels], last row: the current token
     norm: Optional[torch.Tensor] = None         # [vdim]
 
@@ -98,19 +104,21 @@ def _cpu(proj, spec: StateSpec, w: StateWeights, eps, state, ring, b) -> torch.T
     t, H, G, D, V, col = proj.shape[0], spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.columns
     f = lambda name, n: proj[:, col[name]:col[name] + n].float()
     low = lambda name, r, m: f(name, r) @ m.w[:, :r].float().t()
-    if spec.form == DELTA:
+    if spec.delta:
         x = F_.silu(causal_conv(f("q", spec.channels), w.conv_w, ring, b.row_off, b.slots, b.positions))
         q, k, v = x.split([G * D, G * D, H * V], dim=1)
     else:
         q, k, v = f("q", G * D), f("k", G * D), f("v", H * V)
     q, k, v = q.reshape(t, G, D), k.reshape(t, G, D), v.reshape(t, H, V)
     beta = None
-    if spec.form == DELTA:
+    if spec.delta:
         q, k = (y / torch.sqrt((y * y).sum(-1, keepdim=True) + UNIT_EPS) for y in (q, k))
         beta = torch.sigmoid(f("b", H))
     q, k = ((y * s).repeat_interleave(H // G, dim=1) for y, s in ((q, spec.q_scale), (k, spec.k_scale)))
     if spec.form == FIXED:
         g = w.rate.view(1, H, 1).expand(t, H, D)
+    elif spec.form == HEAD_DELTA:
+        g = torch.exp(-w.rate * F_.softplus(f("a", H) + w.bias)).unsqueeze(-1).expand(t, H, D)
     else:
         z = (low("a", spec.rank_a, w.w_a) + w.bias).view(t, H, D)
         g = torch.exp(-F_.softplus(-z) / spec.tau) if spec.form == GATED else torch.exp(-w.rate.view(1, H, 1) * F_.softplus(z))
@@ -125,7 +133,7 @@ def _cpu(proj, spec: StateSpec, w: StateWeights, eps, state, ring, b) -> torch.T
 def linear_state(proj: torch.Tensor, spec: StateSpec, w: StateWeights, eps: float, state: torch.Tensor, ring: Optional[torch.Tensor],
                  b) -> torch.Tensor:
     """proj [T, *] packed projections of a ForwardBatch's rows; state [slots, heads, dim, vdim] and ring [slots, taps, channels]
-    (delta form) are fp32 views with a common slot stride, updated in place.  Returns [T, heads * vdim], normed and gated."""
+    (delta forms) are fp32 views with a common slot stride, updated in place.  Returns [T, heads * vdim], normed and gated."""
     t, H, D, V, col = proj.shape[0], spec.heads, spec.dim, spec.vdim, spec.columns
     if _lib.on_cpu(proj):
         return _cpu(proj, spec, w, eps, state, ring, b)
@@ -134,7 +142,7 @@ def linear_state(proj: torch.Tensor, spec: StateSpec, w: StateWeights, eps: floa
     out = torch.empty((t, spec.out_cols), dtype=proj.dtype, device=proj.device)
     decay = gate = scratch = None
     if not decode:
-        if spec.form != FIXED:
+        if spec.form in (GATED, DELTA):
             decay = linear(proj[:, col["a"]:col["a"] + w.w_a.in_features], w.w_a, out_fp32=True)
         if spec.form == DELTA:
             gate = linear(proj[:, col["g"]:col["g"] + w.w_g.in_features], w.w_g)

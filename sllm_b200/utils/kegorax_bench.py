@@ -90,7 +90,7 @@ def attention(tab: _Table, heads: int, batch: int, ctx: int, seqs: int, n: int) 
                 append, nbytes=T * 2 * cols * 2, like_bytes=T * old)
         pt = A.plan_portions(b.row_off_host, b.starts_host, spec.window, "cuda", spec.keep_first, spec.chunk)[0]
         run = lambda: k.sllm_kv_prefill(_p(q), T, _p(rows), T, _p(pt.tiles), pt.tiles.shape[0], heads, hkv, HD, HD, spec.window, spec.keep_first,
-                                        spec.chunk, _p(sl), spec.scale, _p(sinks), _p(g), g.stride(0) if g is not None else 0, 1, _p(out),
+                                        spec.chunk, _p(sl), None, 0, 0, spec.scale, _p(sinks), _p(g), g.stride(0) if g is not None else 0, 1, _p(out),
                                         _p(status), _stream())
         paged = _us([lambda: ops.paged_attention(q.view(T, -1), kl, table, b.seq_index, b.kv_lens, heads, hkv, HD, window=spec.window, max_kv=n)] * 2)
         w = spec.window

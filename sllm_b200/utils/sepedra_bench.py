@@ -89,7 +89,7 @@ def attention(tab: _Table, heads: int, batch: int, ctx: int, seqs: int, n: int) 
     tab.add("kv_gather", _us([lambda: k.sllm_kv_gather(_p(pages.k), _p(pages.v), PAGE, _p(table), table.stride(0), _p(pt.spans), seqs, n,
                                                        _p(rows), hkv, HD, HD, _stream())] * 3),
             "rope_kv_append", append, nbytes=T * 2 * hkv * 2 * HD * 2, like_bytes=T * old)
-    attn = _us([lambda: k.sllm_kv_prefill(_p(q), T, _p(rows), T, _p(pt.tiles), pt.tiles.shape[0], heads, hkv, HD, HD, 0, 0, 0, None, spec.scale,
+    attn = _us([lambda: k.sllm_kv_prefill(_p(q), T, _p(rows), T, _p(pt.tiles), pt.tiles.shape[0], heads, hkv, HD, HD, 0, 0, 0, None, None, 0, 0, spec.scale,
                                           _p(sinks), _p(gate), gate.stride(0), 0, _p(out), _p(status), _stream())] * 3)
     paged = _us([lambda: ops.paged_attention(q.view(T, -1), kl, table, b.seq_index, b.kv_lens, heads, hkv, HD, max_kv=n)] * 2)
     dense = _us([lambda: PF.prefill_attention(qkv, b, heads, hkv, HD)] * 3)
