@@ -14,7 +14,7 @@ Kinds:
                  `qwen3_5_moe_text` with routed MXFP4 experts stored as packed U8 values plus E8M0 `weight_scale`
                  planes and a gated shared expert); the decoder tensors under `model.language_model.` are consumed,
                  `model.visual.*` and `mtp.*` are recorded as known-unconsumed; same lock verification
-  zokuvik, sepedra, kegorax
+  zokuvik, sepedra, kegorax, fekolorn
                  a folder of that design (config.json with `architecture`, model.safetensors); same lock verification.
                  The seeded shapes of these families (`zokuvik`, `tiny-zokuvik`, ...) are written by random-llama
 `--weight-format bf16|fp8` selects the resident encoding (fp8 = E4M3FN with FP32 scales per 1x128 block).
@@ -30,7 +30,7 @@ import sys
 
 from .common import CliError, StrictParser, emit, run_main
 
-KINDS = ("random-llama", "hf-llama", "hf-qwen35", "mixed-precision", "zokuvik", "sepedra", "kegorax")
+KINDS = ("random-llama", "hf-llama", "hf-qwen35", "mixed-precision", "zokuvik", "sepedra", "kegorax", "fekolorn")
 
 
 def _hf_config(raw: dict, weight_format: str):
@@ -292,6 +292,7 @@ def main(argv=None) -> int:
                 raise CliError("--manifest must hold a JSON object")
         fps, tokenizer_json, chat_template = [], None, None
         named = dict(MC.NAMED)
+        from ..models import fekolorn as _fk
         from ..models import kegorax as _kg
         from ..models import moe as _moe
         from ..models import qwen35 as _q35
@@ -300,7 +301,7 @@ def main(argv=None) -> int:
         from ..models import zokuvik as _zk
         named.update({"tiny-moe": _moe.tiny_moe, "tiny-shared-moe": _moe.tiny_shared_moe, "tiny-qwen35": _q35.tiny_qwen35,
                       "tiny-qwen35-moe": _q35.tiny_qwen35_moe, "tiny-zokuvik": _zk.tiny_zokuvik, "tiny-sepedra": _sp.tiny_sepedra,
-                      "tiny-kegorax": _kg.tiny_kegorax})
+                      "tiny-kegorax": _kg.tiny_kegorax, "tiny-fekolorn": _fk.tiny_fekolorn})
         if a.kind == "random-llama":
             if a.artifact not in named:
                 raise CliError(f"--artifact must be one of {sorted(named)}")
@@ -309,8 +310,8 @@ def main(argv=None) -> int:
                 ok = ("bf16", "fp32", "fp8") if cfg.family == "qwen35" else ("bf16", "fp32")
                 if a.weight_format not in ok:
                     raise CliError("the mixture-of-experts family keeps bf16 attention (experts are MXFP4); the hybrid "
-                                   "family takes bf16, fp32 or fp8 projections; the zokuvik, sepedra and kegorax families bf16 "
-                                   "or fp32")
+                                   "family takes bf16, fp32 or fp8 projections; the zokuvik, sepedra, kegorax and "
+                                   "fekolorn families bf16 or fp32")
                 if a.with_vision or a.with_mtp:
                     raise CliError("--with-vision / --with-mtp apply to the dense decoder family")
             cfg.weight_format = a.weight_format

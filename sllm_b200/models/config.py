@@ -13,7 +13,7 @@ from typing import Optional
 @dataclass
 class ModelConfig:
     name: str = "tiny-llama"
-    family: str = "llama"            # llama | moe | qwen35 | gemma4 | zokuvik | sepedra | kegorax
+    family: str = "llama"            # llama | moe | qwen35 | gemma4 | zokuvik | sepedra | kegorax | fekolorn
     n_layers: int = 2
     d_model: int = 256
     n_heads: int = 4
@@ -66,6 +66,8 @@ class ModelConfig:
     layer_specs: Optional[list] = None
     layer_loop: Optional[dict] = None        # {"start", "stop", "times"}: layers that run several times in a row, same weights
     norm_groups: int = 1
+    streams: int = 1                         # parallel residual streams (hyper-connections)
+    bigram: Optional[dict] = None            # {"buckets", "mul_prev", "mul_cur"}: embedding of (previous token, token)
     # vision-language models: rotary pairs [0, t) follow the temporal index, [t, t + h) the height index and the rest
     # the width index of a token's 3-axis position (text tokens carry the same value on all three)
     mrope_sections: Optional[list] = None
@@ -182,7 +184,13 @@ def _kegorax():
     return kegorax_shape()
 
 
+def _fekolorn():
+    from .fekolorn import fekolorn_shape
+    return fekolorn_shape()
+
+
 NAMED = {
+    "fekolorn": _fekolorn,
     "kegorax": _kegorax,
     "sepedra": _sepedra,
     "zokuvik": _zokuvik,

@@ -11,8 +11,8 @@ ffn_gate_inp (router; rows past n_experts: the shared-expert gate and zero paddi
 ffn_gate_up_shexp | ffn_down_shexp.  Hybrid layer i: blk.i.attn_norm | ffn_norm | ffn_gate | ffn_up | ffn_down (or, with
 a sparse MLP, the ffn_gate_inp / ffn_*_exps / ffn_*_shexp tensors of the MoE layer) and either
 attn_q | attn_k | attn_v | attn_gate | attn_output | attn_q_norm | attn_k_norm (full attention) or ssm_in | ssm_conv1d |
-ssm_a | ssm_dt | ssm_norm | ssm_out (gated delta net).  A `zokuvik`, `sepedra` or `kegorax` file keeps the design's own names
-(source_shapes of its module): its layers differ in kind and size, and the configuration in the metadata lists them.
+ssm_a | ssm_dt | ssm_norm | ssm_out (gated delta net).  A `zokuvik`, `sepedra`, `kegorax` or `fekolorn` file keeps the design's
+own names (source_shapes of its module): its layers differ in kind and size, and the configuration in the metadata lists them.
 
 Reference: the per-family conversion plans of crates/sllm-core/src/gguf_convert.rs:145-704 (Qwen3.5 BF16 / FP8 /
 MoE-MXFP4 plans) and the expert tensor contract of crates/sllm-core/src/qwen35_moe.rs:1277-1600.

@@ -28,6 +28,7 @@ from ..ops import moe as M
 from ..ops.core import LinearWeight
 from .config import ModelConfig
 from .llama import NoTP
+from .packing import SourceTensors
 
 ARCHITECTURE = "Kegorax"
 MIXERS = ("parallel", "parallel_2", "channel_delta")
@@ -235,54 +236,11 @@ class KegoraxWeights:
     vocab_offset: int = 0
 
 
-def _pad(n: int) -> int:
-    return (n + 7) // 8 * 8
-
-
 def pack_weights(cfg: ModelConfig, get: Callable, device) -> KegoraxWeights:
     """``get(name)`` returns a source tensor (any float type, any device)."""
     device = torch.device(device)
-    dt = torch.float32 if cfg.weight_format == "fp32" else torch.bfloat16
-    shapes = source_shapes(cfg, lambda n: int(get(n).shape[0]))
-
-    def fetch(name: str) -> torch.Tensor:
-        t = get(name)
-        if tuple(t.shape) != shapes[name]:
-            raise ValueError(f"{name}: shape {tuple(t.shape)}, expected {shapes[name]}")
-        return t
-
-    def raw(name):
-        return fetch(name).to(device=device, dtype=dt)
-
-    def mat(*names) -> LinearWeight:
-        return LinearWeight("dense", torch.cat([raw(n) for n in names], dim=0).contiguous())
-
-    def vec(*names):
-        return torch.cat([fetch(n).to(device=device, dtype=torch.float32).reshape(-1) for n in names]).contiguous()
-
-    def taps(*names):
-        return torch.cat([fetch(n).to(device=device, dtype=torch.float32) for n in names]).t().contiguous()
-
-    def second_factor(name) -> LinearWeight:
-        w = raw(name)
-        out = w.new_zeros((w.shape[0], _pad(w.shape[1])))
-        out[:, :w.shape[1]] = w
-        return LinearWeight("dense", out)
-
-    def packed(q: str, parts: list):
-        """parts: lists of names whose rows follow each other; every list starts at a multiple of 8 rows."""
-        rows, blocks, at = [], [], 0
-        for names in parts:
-            for n in names:
-                w = raw(q + n)
-                rows.append((n, at, w.shape[0]))
-                blocks.append(w)
-                at += w.shape[0]
-            if at % 8:
-                blocks.append(blocks[-1].new_zeros((8 - at % 8, blocks[-1].shape[1])))
-                at = _pad(at)
-        return LinearWeight("dense", torch.cat(blocks).contiguous()), rows
-
+    src = SourceTensors(cfg, get, source_shapes(cfg, lambda n: int(get(n).shape[0])), device)
+    shapes, fetch, raw, mat, vec, taps = src.shapes, src.fetch, src.raw, src.mat, src.vec, src.taps
     layers = []
     for i, e in enumerate(cfg.layer_specs):
         p, q = f"l{i}.", f"l{i}.mix."
@@ -290,10 +248,10 @@ def pack_weights(cfg: ModelConfig, get: Callable, device) -> KegoraxWeights:
         m = _state_mixer(e)
         kw: dict = dict(norm1=vec(p + "norm1"))
         if e["type"] == "channel_delta":
-            in_proj, rows = packed(q, [["q", "k", "v"], ["b"], ["a1"], ["g1"]])
+            in_proj, rows = src.packed(q, [["q", "k", "v"], ["b"], ["a1"], ["g1"]])
             r, at = "", {n: a for n, a, _ in rows}
             kw["a_log"] = vec(q + "A_log")
-            sw = S.StateWeights(w_a=second_factor(q + "a2"), w_g=second_factor(q + "g2"), bias=vec(q + "dt_bias"),
+            sw = S.StateWeights(w_a=src.second_factor(q + "a2"), w_g=src.second_factor(q + "g2"), bias=vec(q + "dt_bias"),
                                 rate=torch.exp(kw["a_log"].double()).float(), conv_w=taps(*(f"{q}{x}.conv" for x in ("q", "k", "v"))),
                                 norm=vec(q + "norm"))
             st = S.StateSpec(S.DELTA, H, G, D, V, {"q": at["q"], "k": at["k"], "v": at["v"], "g": at["g1"], "a": at["a1"], "b": at["b"]},
@@ -301,13 +259,13 @@ def pack_weights(cfg: ModelConfig, get: Callable, device) -> KegoraxWeights:
         else:
             chunked, r = e["type"] == "parallel", "right."
             parts = [["left.q", "left.k", "left.v"]] + ([["left.g"]] if chunked else []) + [[r + x] for x in ("q", "k", "v", "g")]
-            in_proj, rows = packed(q, parts + ([[r + "a1"]] if chunked else []))
+            in_proj, rows = src.packed(q, parts + ([[r + "a1"]] if chunked else []))
             at = {n: a for n, a, _ in rows}
             cols = {x: at[r + x] for x in ("q", "k", "v", "g")}
             s = attention_spec(e)
             kw.update(attn=s, o_attn=mat(q + "left.o"))
             if chunked:
-                sw = S.StateWeights(w_a=second_factor(q + r + "a2"), bias=vec(q + r + "a2.b"), norm=vec(q + r + "norm"))
+                sw = S.StateWeights(w_a=src.second_factor(q + r + "a2"), bias=vec(q + r + "a2.b"), norm=vec(q + r + "norm"))
                 st = S.StateSpec(S.GATED, H, H, D, V, dict(cols, a=at[r + "a1"]), q_scale=D ** -0.5, tau=float(m["tau"]),
                                  rank_a=shapes[q + r + "a1"][0])
                 kw.update(gate_col=at["left.g"], inv_freq=s.inv_freq(device), sinks=vec(q + "left.sink"), attn_out=vec(q + "left.out"),

@@ -300,7 +300,7 @@ def load_llama_gguf(g: G.GgufFile, device, tp_size: int = 1, tp_rank: int = 0, k
 def load_model_gguf(g: G.GgufFile, device, tp_size: int = 1, tp_rank: int = 0, ep_size: int = 1, ep_rank: int = 0,
                     kv_format: Optional[str] = None):
     """(cfg, weights, family) of this rank for any model family a file can carry: the dense decoder (`llama`,
-    `gemma4`) through load_llama_gguf, `moe`, `qwen35`, `zokuvik`, `sepedra` and `kegorax` through models.family_io."""
+    `gemma4`) through load_llama_gguf, `moe`, `qwen35`, `zokuvik`, `sepedra`, `kegorax` and `fekolorn` through models.family_io."""
     cfg = config_from_gguf(g)
     if cfg.family in ("moe", "qwen35", *LAYERED):
         from . import family_io

@@ -19,11 +19,13 @@ KERNEL_UNITS = {
                 "moe_dense"),
     "kegorax": ("elementwise", "gemm_tcgen05", "gemm_simt", "group_norm", "attention", "kv_attention", "short_conv", "latent_prefill",
                 "linear_state", "state_scan", "moe", "moe_dense"),
+    "fekolorn": ("elementwise", "gemm_tcgen05", "gemm_simt", "hyper_streams", "poly_norm", "attention", "kv_attention", "short_conv",
+                 "latent_prefill", "linear_state", "state_scan"),
 }
 
 # families whose configuration lists its layers (ModelConfig.layer_specs): modules with ARCHITECTURE, config_from_source,
 # pack_weights, named_tensors and make_cache.  They run on one GPU, in bf16 or fp32
-LAYERED = ("zokuvik", "sepedra", "kegorax")
+LAYERED = ("zokuvik", "sepedra", "kegorax", "fekolorn")
 
 
 def layered(family: str):
@@ -48,6 +50,9 @@ def make_model(cfg: ModelConfig, weights, tp=None, ep=None):
     if cfg.family == "kegorax":
         from .kegorax import KegoraxModel
         return KegoraxModel(cfg, weights, tp)
+    if cfg.family == "fekolorn":
+        from .fekolorn import FekolornModel
+        return FekolornModel(cfg, weights, tp)
     from .llama import LlamaModel
     return LlamaModel(cfg, weights, tp)
 
@@ -80,6 +85,9 @@ def init_random_weights(cfg: ModelConfig, device, seed: int = 0, tp_size: int = 
     if cfg.family == "kegorax":
         from .kegorax import init_random_kegorax_weights
         return init_random_kegorax_weights(cfg, device, seed)
+    if cfg.family == "fekolorn":
+        from .fekolorn import init_random_fekolorn_weights
+        return init_random_fekolorn_weights(cfg, device, seed)
     from .llama import init_random_weights as init
     return init(cfg, device, seed, tp_size, tp_rank)
 
