@@ -59,7 +59,7 @@ def parse_args():
                     help="4-bit-weight models: quantise activations to the weights' 4-bit format and run the GEMMs on the "
                          "block-scaled tensor-core kernel (W4A4) instead of W4A16")
     ap.add_argument("--layers", type=int, default=0, help="profiling only: override the layer count")
-    ap.add_argument("--compare", default=None, choices=["zokuvik", "sepedra", "kegorax"],
+    ap.add_argument("--compare", default=None, choices=["zokuvik", "sepedra", "kegorax", "fekolorn"],
                     help="instead of the headline workload: prompt and decode throughput and per-kernel roofline fractions of "
                          "a design beside the framework's closest model at equal sizes (one GPU)")
     ap.add_argument("--no-batch1", action="store_true", help="skip the extra batch-1 measurement")
@@ -337,7 +337,8 @@ def main():
 
     if args.compare:
         import importlib
-        module = {"zokuvik": "family_bench", "sepedra": "sepedra_bench", "kegorax": "kegorax_bench"}[args.compare]
+        module = {"zokuvik": "family_bench", "sepedra": "sepedra_bench", "kegorax": "kegorax_bench",
+                  "fekolorn": "fekolorn_bench"}[args.compare]
         return importlib.import_module(f"sllm_b200.utils.{module}").main(args)
     if args.act4:
         from sllm_b200.ops import w4 as _w4

@@ -8,6 +8,8 @@
 // once per group.  Inside a warp, keys are handled 32 at a time: lane <-> key for Q.K (no shuffles in
 // the inner product), then lane <-> channel for P.V.  Per-(token, head) FP8 scales are folded into
 // the score (K) and into the probability (V), so pages are consumed in their stored encoding.
+// The any-size form (bf16 pages whose rows are padded to 16 bytes with zeros) takes heads of any widths up to HD and any GQA
+// group: a CTA then owns G of a kv head's query heads.
 // Partial (max, sum, acc) triples of the splits are merged by the last CTA to arrive (counter per
 // (row, kv head)); nobody waits.
 //
@@ -24,7 +26,7 @@ namespace sllm {
 
 // kFmt: 0 bf16 pages, 1 E4M3 pages (scale per token and head, or static), 2 NVFP4 rows (E2M1 codes, E4M3 scale per 16
 // channels inside the row, fp32 outer scale per token and head in the scale plane; see nvfp4_row_bytes).
-template <int HD, int G, int kFmt>
+template <int HD, int G, int kFmt, bool kAny>
 __global__ void __launch_bounds__(128) paged_attention_kernel(const PagedAttnParams p) {
   pdl_wait();
   pdl_trigger();
@@ -40,9 +42,9 @@ __global__ void __launch_bounds__(128) paged_attention_kernel(const PagedAttnPar
   __shared__ int s_is_last;
   __shared__ float s_red[4];
 
-  const int r = blockIdx.x, kvh = blockIdx.y, split = blockIdx.z, splits = gridDim.z;
+  // kvh: number of the CTA's group of G query heads, page_head: the kv head that it reads
+  const int r = blockIdx.x, kvh = blockIdx.y, split = blockIdx.z, splits = gridDim.z, page_head = kAny ? kvh / p.subs : kvh;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int hq = p.hkv * G;
   const int seq = p.seq_index[r];
   const int kv_len = p.kv_lens[r];
   const VisibleKeys keys(kv_len, p.window, p.keep_first, p.chunk);
@@ -55,8 +57,9 @@ __global__ void __launch_bounds__(128) paged_attention_kernel(const PagedAttnPar
   for (int e = threadIdx.x; e < G * HD; e += blockDim.x) {
     const int g = e / HD, d = e % HD;
     // FP8 pages decode to value * 2^-120; half of the compensation (2^60) rides on q, half on the scale.
-    q_s[e] = __bfloat162float(p.q[static_cast<size_t>(r) * p.q_ld + (kvh * G + g) * HD + d]) * p.sm_scale *
-             (kFp8 ? kPow60 : 1.f);
+    const __nv_bfloat16* qr = p.q + static_cast<size_t>(r) * p.q_ld;
+    if constexpr (kAny) q_s[e] = d < p.dim ? __bfloat162float(qr[(kvh * G + g) * p.q_head + d]) * p.sm_scale : 0.f;
+    else q_s[e] = __bfloat162float(qr[(kvh * G + g) * HD + d]) * p.sm_scale * (kFp8 ? kPow60 : 1.f);
   }
   __syncthreads();
 
@@ -81,7 +84,7 @@ __global__ void __launch_bounds__(128) paged_attention_kernel(const PagedAttnPar
     float vsc = 0.f;
     if (valid) {
       const int blk = bt[tok / p.page_size];
-      slot = (static_cast<size_t>(blk) * p.hkv + kvh) * p.page_size + tok % p.page_size;   // head-major pages
+      slot = (static_cast<size_t>(blk) * p.hkv + page_head) * p.page_size + tok % p.page_size;   // head-major pages
     }
     if (kNv4 && valid) {
       // the whole row (code words, then the block-scale words) is requested before any of it is used
@@ -123,14 +126,15 @@ __global__ void __launch_bounds__(128) paged_attention_kernel(const PagedAttnPar
       constexpr int kBatch = kVecs < 8 ? kVecs : 8;
       constexpr int kElemsPerVec = kFp8 ? 16 : 8;
       const uint4* krow = reinterpret_cast<const uint4*>(static_cast<const uint8_t*>(p.k_pages) +
-                                                         slot * HD * (kFp8 ? 1 : 2));
+                                                         slot * (kAny ? p.ld_k : HD) * (kFp8 ? 1 : 2));
 #pragma unroll
       for (int b0 = 0; b0 < kVecs; b0 += kBatch) {
         uint4 raw[kBatch];
 #pragma unroll
-        for (int u = 0; u < kBatch; ++u) raw[u] = krow[b0 + u];
+        for (int u = 0; u < kBatch; ++u) raw[u] = !kAny || (b0 + u) * 8 < p.ld_k ? krow[b0 + u] : make_uint4(0, 0, 0, 0);
 #pragma unroll
         for (int u = 0; u < kBatch; ++u) {
+          if (kAny && (b0 + u) * 8 >= p.dim) break;
           float kf[kElemsPerVec];
           if (kFp8) {
             const uint32_t* w32 = reinterpret_cast<const uint32_t*>(&raw[u]);
@@ -234,12 +238,13 @@ __global__ void __launch_bounds__(128) paged_attention_kernel(const PagedAttnPar
             for (int e = 0; e < 4; ++e) vf[u][(4 + e) % EPL] = f4[e];
           }
         } else {
-          const __nv_bfloat16* vp = static_cast<const __nv_bfloat16*>(p.v_pages) + vslot * HD + lane * EPL;
+          const __nv_bfloat16* vp = static_cast<const __nv_bfloat16*>(p.v_pages) + vslot * (kAny ? p.ld_v : HD) + lane * EPL;
 #pragma unroll
           for (int e = 0; e < EPL; e += 2) {
-            const __nv_bfloat162 h = live ? *reinterpret_cast<const __nv_bfloat162*>(vp + e) : __nv_bfloat162();
-            vf[u][e] = live ? __bfloat162float(h.x) : 0.f;
-            vf[u][(e + 1) % EPL] = live ? __bfloat162float(h.y) : 0.f;
+            const bool in = live && (!kAny || lane * EPL + e < p.ld_v);
+            const __nv_bfloat162 h = in ? *reinterpret_cast<const __nv_bfloat162*>(vp + e) : __nv_bfloat162();
+            vf[u][e] = in ? __bfloat162float(h.x) : 0.f;
+            vf[u][(e + 1) % EPL] = in ? __bfloat162float(h.y) : 0.f;
           }
         }
       }
@@ -276,21 +281,22 @@ __global__ void __launch_bounds__(128) paged_attention_kernel(const PagedAttnPar
   }
   __syncthreads();
 
-  attention_tail<HD, G, 4, SyncCta>(p, r, kvh, split, splits, threadIdx.x, m_s, l_s, o_s, &s_is_last, s_red);
+  attention_tail<HD, G, 4, SyncCta>(p, r, kvh, split, splits, threadIdx.x, m_s, l_s, o_s, &s_is_last, s_red,
+                                     kAny ? p.vdim : HD);
 }
 
-template <int HD, int G, int kFp8>
+template <int HD, int G, int kFmt, bool kAny = false>
 static int launch_paged(const PagedAttnParams& p, int rows, int splits, cudaStream_t st) {
   const size_t smem = sizeof(float) * (G * HD + 4 * 32 * G + 8 * G + 4 * G * HD);
   static bool cfg = false;
   if (!cfg) {
     if (smem > 48 * 1024)
-      cudaFuncSetAttribute(paged_attention_kernel<HD, G, kFp8>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+      cudaFuncSetAttribute(paged_attention_kernel<HD, G, kFmt, kAny>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                            static_cast<int>(smem));
     cfg = true;
   }
-  dim3 grid(rows, p.hkv, splits);
-  launch_kernel(paged_attention_kernel<HD, G, kFp8>, dim3(grid), dim3(128), smem, st, 1u, p);
+  dim3 grid(rows, kAny ? p.hkv * p.subs : p.hkv, splits);
+  launch_kernel(paged_attention_kernel<HD, G, kFmt, kAny>, dim3(grid), dim3(128), smem, st, 1u, p);
   return cudaGetLastError() == cudaSuccess ? SLLM_OK : SLLM_ERR_CUDA;
 }
 
@@ -305,9 +311,58 @@ static int dispatch_g(const PagedAttnParams& p, int rows, int g, int splits, cud
   }
 }
 
+template <int HD>
+static int dispatch_any(const PagedAttnParams& p, int rows, int g, int splits, cudaStream_t st) {
+  switch (g) {
+    case 1: return launch_paged<HD, 1, 0, true>(p, rows, splits, st);
+    case 2: return launch_paged<HD, 2, 0, true>(p, rows, splits, st);
+    case 4: return launch_paged<HD, 4, 0, true>(p, rows, splits, st);
+    default: return launch_paged<HD, 8, 0, true>(p, rows, splits, st);
+  }
+}
+
 }  // namespace sllm
 
 using namespace sllm;
+
+// Query heads of a CTA in the any-size form: the largest of 8, 4, 2, 1 that divides the GQA group.
+static int any_group(int g) { return g % 8 == 0 ? 8 : g % 4 == 0 ? 4 : g % 2 == 0 ? 2 : 1; }
+static int any_width(int dim, int vdim) { return dim <= 64 && vdim <= 64 ? 64 : dim <= 128 && vdim <= 128 ? 128 : 256; }
+
+// q [rows, hq, q_head]; pages bf16, rows of ld_k / ld_v elements (multiples of 8) whose padding is zero; gate: optional logits,
+// one per output channel or (gate_heads) per head; out [rows, hq * vdim].
+SLLM_EXPORT int sllm_paged_attention_any(const void* q, int q_head, const void* k_pages, const void* v_pages, int ld_k, int ld_v,
+                                         const int* block_table, int max_blocks, const int* seq_index, const int* kv_lens, int rows,
+                                         int hq, int hkv, int dim, int vdim, int page_size, int window, int keep_first, int chunk,
+                                         float sm_scale, const float* sinks, const float* slopes, const float* dist, int n_dist,
+                                         int ld_dist, const void* gate, long long ld_gate, int gate_heads, void* out, int splits,
+                                         float* ws, long long ws_floats, int* counters, int n_counters, void* stream) {
+  if (!q || !k_pages || !v_pages || !block_table || !seq_index || !kv_lens || !out || rows <= 0 || hkv <= 0 || hq <= 0 || hq % hkv ||
+      dim <= 0 || vdim <= 0 || q_head < dim || ld_k < dim || ld_v < vdim || page_size <= 0 || splits < 1 || splits > 65535 || hq > 65535 ||
+      window < 0 || keep_first < 0 || chunk < 0 || (keep_first > 0 && window == 0) || (chunk > 0 && window > 0) ||
+      (dist && (n_dist < 1 || ld_dist < kDistFront + n_dist)))
+    return SLLM_ERR_INVALID_ARGUMENT;
+  if (dim > 256 || vdim > 256) return SLLM_ERR_UNSUPPORTED_SHAPE;
+  if ((ld_k & 7) || (ld_v & 7) || ((reinterpret_cast<uintptr_t>(k_pages) | reinterpret_cast<uintptr_t>(v_pages)) & 15))
+    return SLLM_ERR_ALIGNMENT;
+  const int g = any_group(hq / hkv), width = any_width(dim, vdim);
+  PagedAttnParams p = {};
+  p.q = static_cast<const __nv_bfloat16*>(q); p.q_ld = hq * q_head; p.q_head = q_head; p.k_pages = k_pages; p.v_pages = v_pages;
+  p.ld_k = ld_k; p.ld_v = ld_v; p.dim = dim; p.vdim = vdim; p.subs = hq / hkv / g; p.block_table = block_table; p.max_blocks = max_blocks;
+  p.seq_index = seq_index; p.kv_lens = kv_lens; p.hkv = hkv; p.page_size = page_size; p.window = window; p.keep_first = keep_first;
+  p.chunk = chunk; p.sm_scale = sm_scale; p.out_bf16 = static_cast<__nv_bfloat16*>(out); p.sinks = sinks; p.slopes = slopes;
+  p.dist = {dist, n_dist, ld_dist}; p.gate = static_cast<const __nv_bfloat16*>(gate); p.ld_gate = ld_gate; p.gate_heads = gate_heads;
+  p.counters = counters;
+  if (splits > 1) {
+    const long long units = static_cast<long long>(rows) * (hq / g);
+    if (!ws || !counters || ws_floats < units * splits * g * (width + 2) || n_counters < units) return SLLM_ERR_WORKSPACE_TOO_SMALL;
+    p.ws_o = ws;
+    p.ws_ml = ws + units * splits * g * width;
+  }
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return width == 64 ? dispatch_any<64>(p, rows, g, splits, st)
+                     : width == 128 ? dispatch_any<128>(p, rows, g, splits, st) : dispatch_any<256>(p, rows, g, splits, st);
+}
 
 SLLM_EXPORT long long sllm_paged_attention_workspace_floats(int rows, int hq, int hd, int hkv, int splits) {
   if (splits <= 1) return 0;

@@ -62,6 +62,7 @@ struct PagedAttnParams {
   int keep_first, chunk;
   const float* slopes;
   DistanceBias dist;        // CUDA-core kernel only
+  int q_head, dim, vdim, ld_k, ld_v, subs;   // CUDA-core kernel for any sizes
   int* status_word;         // device status word for bounded waits (tensor-core kernel)
   int early_trigger;        // tensor-core kernel: let dependent launches start once the CTA holds its TMEM
   STEP_TRACE_FIELD
@@ -76,15 +77,16 @@ struct SyncBar1x128 {  // the 128 softmax threads of a warp-specialised CTA
 };
 
 // Tail run by 128 threads (tid 0..127).  m_s / l_s: [W][G], o_s: [W][G][HD] partial softmax states of W
-// producers inside the CTA (maxima in natural-log units); s_is_last / s_red: shared scratch.
+// producers inside the CTA (maxima in natural-log units); s_is_last / s_red: shared scratch.  The row's heads are gridDim.y groups
+// of G; vd: channels of a head in the output (HD or less).
 template <int HD, int G, int W, class Sync>
 __device__ __forceinline__ void attention_tail(const PagedAttnParams& p, int r, int kvh, int split, int splits,
                                                int tid, const float* m_s, const float* l_s, const float* o_s,
-                                               int* s_is_last_p, float* s_red) {
+                                               int* s_is_last_p, float* s_red, int vd = HD) {
   const int warp = tid >> 5, lane = tid & 31;
-  const int hq = p.hkv * G;
+  const int hq = gridDim.y * G;
   int& s_is_last = *s_is_last_p;
-  const size_t unit = static_cast<size_t>(r) * p.hkv + kvh;
+  const size_t unit = static_cast<size_t>(r) * gridDim.y + kvh;
   bool finalize = true;
   if (splits > 1) {
     float* wo = p.ws_o + (unit * splits + split) * (G * HD);
@@ -126,7 +128,7 @@ __device__ __forceinline__ void attention_tail(const PagedAttnParams& p, int r, 
   // ---- final normalisation (+ optional FP8 1x128 quantisation: one block per head when HD == 128)
   for (int e0 = 0; e0 < G * HD; e0 += 128) {
     const int e = e0 + tid;
-    const bool in = e < G * HD;
+    const bool in = e < G * HD && e % HD < vd;
     const int g = in ? e / HD : 0, d = in ? e % HD : 0;
     float M = -INFINITY, L = 0.f, O = 0.f;
     if (in) {
@@ -165,9 +167,9 @@ __device__ __forceinline__ void attention_tail(const PagedAttnParams& p, int r, 
     }
     float val = (L > 0.f) ? O / L : 0.f;
     if (p.gate && in)
-      val /= 1.f + __expf(-__bfloat162float(p.gate[static_cast<size_t>(r) * p.ld_gate + (p.gate_heads ? kvh * G + g : (kvh * G + g) * HD + d)]));
+      val /= 1.f + __expf(-__bfloat162float(p.gate[static_cast<size_t>(r) * p.ld_gate + (p.gate_heads ? kvh * G + g : (kvh * G + g) * vd + d)]));
     val = __bfloat162float(__float2bfloat16_rn(val));
-    const size_t oidx = static_cast<size_t>(r) * hq * HD + (kvh * G + g) * HD + d;
+    const size_t oidx = static_cast<size_t>(r) * hq * vd + (kvh * G + g) * vd + d;
     if (p.out_fp8) {
       // HD == 128 == blockDim: this iteration is exactly head g.
       float a = fabsf(val);

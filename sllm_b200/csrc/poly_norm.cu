@@ -80,8 +80,9 @@ template <typename T>
 static int poly_norm_launch(const void* x, long long ldx, void* y, int rows, int n, const float* coef, float eps, cudaStream_t st) {
   const bool vec = n % kVec16<T> == 0 && ldx % kVec16<T> == 0 && !((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(y)) & 15);
   const int pieces = (n + kPnThreads * kVec16<T> - 1) / (kPnThreads * kVec16<T>);
-  auto* kernel = !vec || pieces > 8 ? poly_norm_kernel<T, 0> : pieces > 4 ? poly_norm_kernel<T, 8> : pieces > 3 ? poly_norm_kernel<T, 4>
-               : pieces > 2 ? poly_norm_kernel<T, 3> : pieces > 1 ? poly_norm_kernel<T, 2> : poly_norm_kernel<T, 1>;
+  auto* kernel = !vec || pieces > 8 ? poly_norm_kernel<T, 0> : pieces > 6 ? poly_norm_kernel<T, 8> : pieces > 5 ? poly_norm_kernel<T, 6>
+               : pieces > 4 ? poly_norm_kernel<T, 5> : pieces > 3 ? poly_norm_kernel<T, 4> : pieces > 2 ? poly_norm_kernel<T, 3>
+               : pieces > 1 ? poly_norm_kernel<T, 2> : poly_norm_kernel<T, 1>;
   return launch_kernel(kernel, dim3(rows), dim3(kPnThreads), 0, st, 1u, static_cast<const T*>(x), ldx, static_cast<T*>(y), n, coef, eps) ==
                  cudaSuccess ? SLLM_OK : SLLM_ERR_CUDA;
 }

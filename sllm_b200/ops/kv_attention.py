@@ -33,6 +33,7 @@ class KvPrepareArgs(C.Structure):
 _SIGS = {
     "sllm_kv_prepare": (I, [P, P]),
     "sllm_kv_abi": (I, [P, I]),
+    "sllm_paged_attention_any": (I, [P, I, P, P, I, I, P, I, P, P] + [I] * 9 + [F, P, P, P, I, I, P, L, I, P, I, P, L, P, I, P]),
     "sllm_kv_gather": (I, [P, P, I, P, I, P, I, I, P, I, I, I, P]),
     "sllm_kv_attention": (I, [P, P, P, P, L, P, P, I, P, P, I, I, I, I, I, I, I, I, I, I, I, I, P, P, I, I, I, F, P, I, P]),
     "sllm_kv_prefill": (I, [P, I, P, I, P, I, I, I, I, I, I, I, I, P, P, I, I, F, P, P, L, I, P, P, P]),
@@ -253,6 +254,21 @@ def paged_rows(q: torch.Tensor, gate: Optional[torch.Tensor], spec: KVSpec, kv: 
                                     sm_scale=spec.scale, max_kv=max_kv, sinks=sinks, gate=gate, out=out, gate_heads=spec.gate_heads,
                                     keep_first=spec.keep_first, chunk=spec.chunk, slopes=slopes, dist=dist)
     out = torch.empty((r, H * V), dtype=q.dtype, device=q.device) if out is None else out
+    if q.dtype == torch.bfloat16 and max(D, V) <= 256 and kv.k.shape[3] % 8 == 0 and kv.v.shape[3] % 8 == 0 and impl != "cuda_core_any":
+        ws = core.workspace(q.device)
+        mk = max_kv if max_kv > 0 else block_table.shape[1] * kv.page_size
+        mk = min(mk, spec.window + spec.keep_first) if spec.window else min(mk, spec.chunk) if spec.chunk else mk
+        splits = core._attn_splits(r, H // math.gcd(H // G, 8), mk)
+        if _lib.audit_enabled():
+            _lib.record_dispatch("paged_attention", "paged_attention_kernel", rows=r, hq=H, hkv=G, hd=D, window=spec.window, splits=splits)
+        rc = _k().sllm_paged_attention_any(core._p(q), spec.q_pad, core._p(kv.k), core._p(kv.v), kv.k.shape[3], kv.v.shape[3],
+                                           core._p(block_table), block_table.stride(0), core._p(seq_index), core._p(kv_lens), r, H, G, D, V,
+                                           kv.page_size, spec.window, spec.keep_first, spec.chunk, spec.scale, core._p(sinks),
+                                           core._p(slopes), *core.dist_args(dist), core._p(gate), gate.stride(0) if gate is not None else 0,
+                                           int(spec.gate_heads), core._p(out), splits, core._p(ws.ws), ws.ws.numel(), core._p(ws.counters),
+                                           ws.counters.numel(), core._stream())
+        _lib.check(rc, "paged_attention_any")
+        return out
     rc = _k().sllm_kv_attention(core._p(q), core._p(kv.k), core._p(kv.v), core._p(gate), gate.stride(0) if gate is not None else 0,
                                 core._p(sinks), core._p(block_table), block_table.stride(0), core._p(seq_index), core._p(kv_lens), r, H,
                                 G, D, V, spec.q_pad, kv.k.shape[3], kv.v.shape[3], kv.page_size, spec.window, spec.keep_first, spec.chunk,
