@@ -22,7 +22,7 @@ PAD = 8                                             # elements: 16 bytes of bf16
 
 class LayeredCache(StateSlots, PagedKVCache):
     def __init__(self, cfg: ModelConfig, num_pages: int, device, max_seqs: int, planes: dict, states: dict):
-        """planes: layer -> [(heads, width)]; states: layer -> [shape]."""
+        """planes: layer -> [(heads, width)]; states: layer, or a key of a state that is no layer's -> [shape]."""
         fmt = cfg.kv_format
         if fmt not in ("fp32", "bf16"):
             raise ValueError(f"pages of this cache are stored as bf16 or fp32, not {fmt!r}")
@@ -61,7 +61,7 @@ class LayeredCache(StateSlots, PagedKVCache):
     def layer(self, i: int):
         return self._layers.get(i)
 
-    def state(self, i: int, part: int = 0) -> torch.Tensor:
+    def state(self, i, part: int = 0) -> torch.Tensor:
         """[slots, *shape] view of one of a layer's state arrays (the slot stride is the whole state row)."""
         return self._states[i][part]
 

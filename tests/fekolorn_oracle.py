@@ -86,15 +86,22 @@ def softmax_sink(s: torch.Tensor, sink: float) -> torch.Tensor:
     return e / (torch.exp(float(sink) - top) + e.sum(-1, keepdim=True))
 
 
+def distance_bias(rel: torch.Tensor, far: float, t: int) -> torch.Tensor:
+    """[H, t, t]: rel[bucket(i - j), h] for j <= i."""
+    rows = torch.tensor([bucket(n, rel.shape[0], far) for n in range(t)])
+    gap = (torch.arange(t)[:, None] - torch.arange(t)[None, :]).clamp(min=0)
+    return rel[rows[gap]].permute(2, 0, 1)
+
+
 def attend(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, scale: float, seen: torch.Tensor, sinks, bias=None) -> torch.Tensor:
-    """q [T, H, dim], k [T, G, dim], v [T, G, vdim]; bias: (i, j, h) -> what joins the scaled score."""
+    """q [T, H, dim], k [T, G, dim], v [T, G, vdim]; bias [H, T, T] joins the scaled scores."""
     t, H, G = q.shape[0], q.shape[1], k.shape[1]
     o = torch.empty(t, H, v.shape[2], dtype=q.dtype)
     for h in range(H):
         g = h // (H // G)
         s = (q[:, h] @ k[:, g].T) * scale
         if bias is not None:
-            s = s + torch.tensor([[bias(i, j, h) if j <= i else 0.0 for j in range(t)] for i in range(t)], dtype=q.dtype)
+            s = s + bias[h]
         o[:, h] = softmax_sink(s.masked_fill(~seen, float("-inf")), sinks[h]) @ v[:, g]
     return o
 
@@ -111,11 +118,8 @@ def window_attention(h: torch.Tensor, w: dict, p: str, m: dict, eps: float, firs
     k = (rms(h @ w[p + "k"].T, eps) * w[p + "k.norm"]).view(t, G, m["dim"])
     own = h @ w[p + "v"].T
     v = mixed_values(own, first, w.get(p + "vmix")).view(t, G, m["vdim"])
-    rel = w[p + "rel"]
-    rows = [bucket(n, rel.shape[0], m["bias_max"]) for n in range(t)]
-    table = rel.tolist()
     seen = visible(t, lambda i, j: sees_window(i, j, m["mask"]["size"]))
-    o = attend(q, k, v, m["scale"], seen, w[p + "sink"], lambda i, j, x: table[rows[i - j]][x])
+    o = attend(q, k, v, m["scale"], seen, w[p + "sink"], distance_bias(w[p + "rel"], m["bias_max"], t))
     return o.reshape(t, -1) @ w[p + "o"].T, own
 
 
