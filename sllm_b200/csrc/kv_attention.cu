@@ -38,16 +38,16 @@ struct KvPrepareParams {
   const int *row_off, *slots, *positions, *seq_index, *block_table;
   T *q, *k_pages, *v_pages;
   long long ring_stride;
-  int ldp, max_blocks, heads, kv_heads, dim, vdim, q_pad, ld_k, ld_v, rot_dims, taps, page_size, tokens, run, norm, decode, vec,
+  int ldp, max_blocks, heads, kv_heads, dim, vdim, q_pad, ld_k, ld_v, rot_dims, taps, page_size, tokens, run, norm, decode,
       interleaved;
   float eps;
 };
 
 enum KvNorm { kNormNone = 0, kNormHead = 1, kNormAll = 2 };   // of q and k: per head, over all heads at once
 
-// kNP: channel pairs per lane; kTaps: filter length after padding.  grid (ceil(T / run), <= ceil(all heads / 8)); a warp takes
+// kNP: channel pairs per lane; kTaps: filter length after padding; kVec: every pair is one aligned access.  grid (ceil(T / run), <= ceil(all heads / 8)); a warp takes
 // every (8 gridDim.y)-th head.
-template <typename T, int kNP, int kTaps>
+template <typename T, int kNP, int kTaps, bool kVec>
 __global__ void __launch_bounds__(kKpThreads) kv_prepare_kernel(const KvPrepareParams<T> p) {
   pdl_wait();
   pdl_trigger();
@@ -80,7 +80,7 @@ __global__ void __launch_bounds__(kKpThreads) kv_prepare_kernel(const KvPrepareP
 #pragma unroll
       for (int m = 0; m < 2; ++m) {
         const int c0 = m ? p.heads * p.dim : 0, c1 = c0 + (m ? p.kv_heads : p.heads) * p.dim;
-        if (p.vec) {
+        if constexpr (kVec) {
 #pragma unroll 4
           for (int c = c0 + 2 * (pt * 32 + lane); c < c1; c += 64 * parts) {
             float x[2];
@@ -120,16 +120,17 @@ __global__ void __launch_bounds__(kKpThreads) kv_prepare_kernel(const KvPrepareP
     const int col = is_v ? (p.heads + p.kv_heads) * p.dim + kvh * p.vdim : head * p.dim;
     const int channels = (p.heads + p.kv_heads) * p.dim + p.kv_heads * p.vdim;
     auto ld2 = [&](const auto* src, int c, float (&v)[2]) {
-      if (p.vec && c + 1 < width) {
-        ld_vec<2>(src + c, v);
+      if constexpr (kVec) {
+        v[0] = v[1] = 0.f;
+        if (c < width) ld_vec<2>(src + c, v);
       } else {
         v[0] = c < width ? ld_f(src + c) : 0.f;
         v[1] = c + 1 < width ? ld_f(src + c + 1) : 0.f;
       }
     };
     auto st2 = [&](auto* dst, int c, int w, const float (&v)[2]) {
-      if (p.vec && c + 1 < w) {
-        st_vec<2>(dst + c, v);
+      if constexpr (kVec) {
+        if (c < w) st_vec<2>(dst + c, v);
       } else {
         if (c < w) st_f(dst + c, v[0]);
         if (c + 1 < w) st_f(dst + c + 1, v[1]);
@@ -156,6 +157,18 @@ __global__ void __launch_bounds__(kKpThreads) kv_prepare_kernel(const KvPrepareP
       if (p.bias) ld2(p.bias + col, 2 * (lane + 32 * s), bias[s]);
     }
     float win[kTaps > 1 ? kTaps - 1 : 1][kNP][2];         // win[b - 1]: the input b positions back
+    // the next token's inputs are requested a token early, and kept as they come until they are used
+    constexpr bool kAhead = kVec && kTaps == 1;
+    using Pair = std::conditional_t<std::is_same_v<T, float>, float2, __nv_bfloat162>;
+    Pair ahead[kNP];
+    auto request = [&](const T* src) {
+#pragma unroll
+      for (int s = 0; s < kNP; ++s) {
+        const int c = 2 * (lane + 32 * s);
+        ahead[s] = c < width ? *reinterpret_cast<const Pair*>(src + c) : Pair();
+      }
+    };
+    if constexpr (kAhead) request(p.proj + static_cast<size_t>(r0) * p.ldp + col);
     int prev = -1;
     for (int i = 0; i < n; ++i) {
       const int row = r0 + i, pos = m_pos[i], seq = m_seq[i];
@@ -176,11 +189,22 @@ __global__ void __launch_bounds__(kKpThreads) kv_prepare_kernel(const KvPrepareP
       }
       float y[kNP][2];
       float ss = 0.f;
+      Pair now[kNP];
+      if constexpr (kAhead) {
+#pragma unroll
+        for (int s = 0; s < kNP; ++s) now[s] = ahead[s];
+        if (i + 1 < n) request(src + p.ldp);
+      }
 #pragma unroll
       for (int s = 0; s < kNP; ++s) {
         const int c = 2 * (lane + 32 * s);
         float x[2];
-        ld2(src, c, x);
+        if constexpr (kAhead) {
+          x[0] = static_cast<float>(now[s].x);
+          x[1] = static_cast<float>(now[s].y);
+        } else {
+          ld2(src, c, x);
+        }
         x[0] += bias[s][0];
         x[1] += bias[s][1];
         if (p.decode && p.ring) st2(ring + static_cast<size_t>(pos % p.taps) * channels, c, width, x);
@@ -390,9 +414,12 @@ SLLM_EXPORT int sllm_kv_abi(int* out, int n) {
   return 2;
 }
 
-template <typename T, int kNP, int kTaps>
+template <typename T, int kTaps, bool kVec>
 static cudaError_t kv_prepare_go(const KvPrepareParams<T>& p, int by, size_t smem, cudaStream_t st) {
-  return launch_kernel(kv_prepare_kernel<T, kNP, kTaps>, dim3((p.tokens + p.run - 1) / p.run, by), dim3(kKpThreads), smem, st, 1u, p);
+  const int wide = p.q_pad > p.vdim ? p.q_pad : p.vdim;
+  auto* kernel = wide <= 64 ? kv_prepare_kernel<T, 1, kTaps, kVec> : wide <= 128 ? kv_prepare_kernel<T, 2, kTaps, kVec>
+                                                                                  : kv_prepare_kernel<T, 4, kTaps, kVec>;
+  return launch_kernel(kernel, dim3((p.tokens + p.run - 1) / p.run, by), dim3(kKpThreads), smem, st, 1u, p);
 }
 
 template <typename T>
@@ -410,7 +437,7 @@ static int kv_prepare_launch(const SllmKvPrepare* a, cudaStream_t st) {
   p.q_pad = a->q_pad; p.ld_k = a->ld_k; p.ld_v = a->ld_v; p.rot_dims = a->rot_dims; p.taps = a->taps; p.page_size = a->page_size;
   p.v_other = t(a->v_other); p.v_mix = a->v_mix; p.ld_other = a->ld_other; p.v_norm = a->v_norm;
   p.tokens = a->tokens; p.norm = a->norm; p.decode = a->decode; p.eps = a->eps;
-  p.vec = !((p.ldp | p.dim | p.vdim | p.q_pad | p.ld_k | p.ld_v) & 1) && !(a->ring_stride & 1) &&
+  const bool vec = !((p.ldp | p.dim | p.vdim | p.q_pad | p.ld_k | p.ld_v) & 1) && !(a->ring_stride & 1) &&
           !((reinterpret_cast<uintptr_t>(a->proj) | reinterpret_cast<uintptr_t>(a->q) | reinterpret_cast<uintptr_t>(a->v_other)) & 7) &&
           !(p.ld_other & 1);
   int by = (p.heads + 2 * p.kv_heads + 7) / 8;
@@ -418,18 +445,10 @@ static int kv_prepare_launch(const SllmKvPrepare* a, cudaStream_t st) {
   p.run = kKpRun;
   while (p.run > 1 && (p.decode || static_cast<long long>((p.tokens + p.run - 1) / p.run) * by < 296)) p.run >>= 1;
   const size_t smem = sizeof(float2) * p.run * (p.rot_dims / 2 + 1);
-  const int wide = p.q_pad > p.vdim ? p.q_pad : p.vdim;
   cudaError_t e;
-  if (p.taps == 1) {
-    e = wide <= 64 ? kv_prepare_go<T, 1, 1>(p, by, smem, st) : wide <= 128 ? kv_prepare_go<T, 2, 1>(p, by, smem, st)
-                                                                            : kv_prepare_go<T, 4, 1>(p, by, smem, st);
-  } else if (p.taps <= 4) {
-    e = wide <= 64 ? kv_prepare_go<T, 1, 4>(p, by, smem, st) : wide <= 128 ? kv_prepare_go<T, 2, 4>(p, by, smem, st)
-                                                                            : kv_prepare_go<T, 4, 4>(p, by, smem, st);
-  } else {
-    e = wide <= 64 ? kv_prepare_go<T, 1, 8>(p, by, smem, st) : wide <= 128 ? kv_prepare_go<T, 2, 8>(p, by, smem, st)
-                                                                            : kv_prepare_go<T, 4, 8>(p, by, smem, st);
-  }
+  if (p.taps == 1) e = vec ? kv_prepare_go<T, 1, true>(p, by, smem, st) : kv_prepare_go<T, 1, false>(p, by, smem, st);
+  else if (p.taps <= 4) e = vec ? kv_prepare_go<T, 4, true>(p, by, smem, st) : kv_prepare_go<T, 4, false>(p, by, smem, st);
+  else e = vec ? kv_prepare_go<T, 8, true>(p, by, smem, st) : kv_prepare_go<T, 8, false>(p, by, smem, st);
   if (e != cudaSuccess) return SLLM_ERR_CUDA;
   if (p.decode || p.taps < 2 || !p.conv_w) return SLLM_OK;
   const int channels = (p.heads + p.kv_heads) * p.dim + p.kv_heads * p.vdim;
